@@ -654,3 +654,105 @@ class GalupelConfig(ModelConfig):
         if self.logit_softcap is not None:
             d["logit_softcap"] = self.logit_softcap
         return d
+
+
+@dataclass
+class TidenexConfig(ModelConfig):
+    """Tidenex: a pre-norm decoder (layer norms with weight and bias) whose layers are differential attention or two mixers side by
+    side (biased grouped-query attention with a bias by distance, and the HGRN2 recurrence), with dense gelu feed-forwards; a range
+    of layers may run several times in a row with the same weights, and the embedding output joins the stream again in front
+    of every pass but the first.  The embedding is also the output matrix.  config.json keys: ``vocab``, ``width``,
+    ``norm.eps``, ``loop`` {start, stop, times} (absent: every layer once) and ``layers``: a list of ``{"type", "mixer", "mlp"}`` with
+
+    * type ``attention``: mixer {heads, kv_heads, dim, vdim, scale, diff, rot {base, dims}} (``dim`` is the size of one of a head's two
+      maps; ``rot`` may be absent);
+    * type ``parallel``: mixer {left {heads, kv_heads, dim, vdim, scale, q_temp {coef, every}}, right {heads, dim, vdim}, left_scale,
+      right_scale} (``q_temp`` may be absent);
+    * mlp: null or dense {ff}.
+
+    The design has no limit on positions; ``max_position_embeddings`` is what an int32 position allows the engine."""
+
+    norm_eps: float = 0.0
+    loop: dict[str, int] | None = None
+    layers: list[dict[str, Any]] = field(default_factory=list)
+
+    @classmethod
+    def from_dict(cls, raw: dict[str, Any]) -> "TidenexConfig":
+        def attention_sizes(m: dict, where: str) -> dict[str, Any]:
+            out: dict[str, Any] = _positive_ints(m, ("heads", "kv_heads", "dim", "vdim"), where)
+            if out["heads"] % out["kv_heads"]:
+                raise ConfigError(f"{where}: heads must be a multiple of kv_heads: {out}")
+            out["scale"] = _need(m, "scale", float)
+            return out
+
+        def sub(m: dict, key: str, where: str) -> dict:
+            v = m.get(key)
+            if not isinstance(v, dict):
+                raise ConfigError(f"{where}: lacks the object {key!r}")
+            return v
+        layers = _need(raw, "layers", list)
+        if not isinstance(layers, list) or not layers:
+            raise ConfigError("config.json key 'layers' must be a list with at least one layer")
+        checked = []
+        for i, layer in enumerate(layers):
+            where = f"layer {i}"
+            kind = layer.get("type") if isinstance(layer, dict) else None
+            if kind not in ("attention", "parallel"):
+                raise ConfigError(f"{where}: 'type' must be 'attention' or 'parallel', got {kind!r}")
+            mixer = sub(layer, "mixer", where)
+            if kind == "attention":
+                m = attention_sizes(mixer, where)
+                m["diff"] = _need(mixer, "diff", float)
+                rot = _opt_object(mixer, "rot", where)
+                if rot is not None:
+                    m["rot"] = {"base": _need(rot, "base", float), "dims": _need(rot, "dims", int)}
+                    if m["rot"]["dims"] % 2 or not 0 <= m["rot"]["dims"] <= m["dim"] or not m["rot"]["base"] > 0:
+                        raise ConfigError(f"{where}: rot.dims must be even and at most dim, rot.base positive: {m['rot']}")
+            else:
+                left = sub(mixer, "left", where)
+                m = {"left": attention_sizes(left, where + " left"),
+                     "right": _positive_ints(sub(mixer, "right", where), ("heads", "dim", "vdim"), where + " right"),
+                     "left_scale": _need(mixer, "left_scale", float), "right_scale": _need(mixer, "right_scale", float)}
+                temp = _opt_object(left, "q_temp", where + " left")
+                if temp is not None:
+                    m["left"]["q_temp"] = {"coef": _need(temp, "coef", float), "every": _need(temp, "every", float)}
+                    if not m["left"]["q_temp"]["every"] > 0:
+                        raise ConfigError(f"{where} left: q_temp.every must be positive")
+            mlp = layer.get("mlp")
+            if mlp is not None:
+                if not isinstance(mlp, dict) or mlp.get("kind") != "dense":
+                    raise ConfigError(f"{where}: 'mlp' must be null or of kind 'dense', got {mlp!r}")
+                mlp = {"kind": "dense", **_positive_ints(mlp, ("ff",), where + " mlp")}
+            checked.append({"type": kind, "mixer": m, "mlp": mlp})
+        loop = _opt_object(raw, "loop", "config.json")
+        if loop is not None:
+            loop = {k: _need(loop, k, int) for k in ("start", "stop", "times")}
+            if not 0 <= loop["start"] <= loop["stop"] <= len(checked) or loop["times"] < 1:
+                raise ConfigError(f"loop must name a range of layers and a positive number of passes: {loop}")
+            if loop["start"] == loop["stop"]:
+                loop = None
+        eos = raw.get("eos_token_id", -1)
+        cfg = cls(architecture=architecture_name(raw), vocab_size=_need(raw, "vocab", int), hidden_size=_need(raw, "width", int),
+                  num_hidden_layers=len(checked), max_position_embeddings=int(raw.get("max_position_embeddings", 1 << 30)),
+                  eos_token_id=-1 if eos is None else int(eos), norm_eps=_need(sub(raw, "norm", "config.json"), "eps", float),
+                  loop=loop, layers=checked)
+        if cfg.vocab_size < 1 or cfg.hidden_size < 1:
+            raise ConfigError("vocab and width must be positive")
+        if not cfg.norm_eps > 0:
+            raise ConfigError("norm.eps must be positive")
+        return cfg
+
+    def layer_runs(self) -> list[tuple[int, bool]]:
+        """The order in which layers run as (layer, rejoin) pairs; ``rejoin``: the embedding output joins the stream right before
+        the layer (the first layer of every pass over the looped range but the first pass)."""
+        n = len(self.layers)
+        a, b, times = (self.loop["start"], self.loop["stop"], self.loop["times"]) if self.loop else (0, 0, 0)
+        passes = [(i, t > 0 and i == a) for t in range(times) for i in range(a, b)]
+        return [(i, False) for i in range(a)] + passes + [(i, False) for i in range(b, n)]
+
+    def to_json_dict(self) -> dict[str, Any]:
+        d = {"architecture": self.architecture, "vocab": self.vocab_size, "width": self.hidden_size, "norm": {"eps": self.norm_eps},
+             "layers": self.layers}
+        if self.loop:
+            d["loop"] = self.loop
+        return d

@@ -456,6 +456,9 @@ struct DecodePrep {
   // max(0, context - pool_window) / pool_p rows, all of them, and nothing of this step is among them (0: an ordinary cache)
   int pool_p;
   int pool_window;
+  // a distance bias (not FUSED only): r1 ln(1 + r2 (position - j)) of the head is taken off the scaled score (null: none)
+  const float* bias_r1;
+  const float* bias_r2;
 };
 
 // The two products are mma.sync m16n8k16 with ldmatrix.
@@ -688,9 +691,20 @@ decode_partition_tma_mma_kernel(const __grid_constant__ CUtensorMap kv_map, cons
     }
   };
   const float cap = prep.softcap;
-  const float sl2 = cap > 0.f ? 1.4426950408889634f : scale * 1.4426950408889634f;
+  // (with a distance bias the scores are brought to units of log 2 first, and exponents take them as they are)
+  const bool biased = !FUSED && prep.bias_r1 != nullptr;
+  const float sl2 = biased ? 1.0f : (cap > 0.f ? 1.4426950408889634f : scale * 1.4426950408889634f);
   const float cap_in = cap > 0.f ? scale * 1.4426950408889634f * (2.0f / cap) : 0.f;
-  const float scale_m = cap > 0.f ? 1.0f : scale;         // what brings a maximum to natural-log units
+  const float scale_m = biased ? 0.6931471805599453f : (cap > 0.f ? 1.0f : scale);         // what brings a maximum to natural-log units
+  float r1[2] = {0.f, 0.f}, r2[2] = {0.f, 0.f};            // of the strip's rows lane / 4 and lane / 4 + 8
+  if (biased) {
+#pragma unroll
+    for (int e = 0; e < 2; ++e) {
+      const int row = min((lane >> 2) + 8 * e, n_g - 1);
+      r1[e] = prep.bias_r1[kvh * G + g0 + row];
+      r2[e] = prep.bias_r2[kvh * G + g0 + row];
+    }
+  }
   const int mi = lane >> 3;
   // Each warp keeps the running maximum, sum and output of its 32 keys of every tile (rows g and g + 8 of the strip);
   // the sums stay per thread until the end (the factor a new maximum brings is the same for the four threads of a row).
@@ -750,6 +764,11 @@ decode_partition_tma_mma_kernel(const __grid_constant__ CUtensorMap kv_map, cons
         if (cap > 0.f) {                               // c tanh(x) = c (1 - 2 / (1 + 2^(2 log2(e) x)))
           s[i][e] = cap - 2.0f * cap * __frcp_rn(1.0f + exp2f(s[i][e] * cap_in));
           s[i][e + 2] = cap - 2.0f * cap * __frcp_rn(1.0f + exp2f(s[i][e + 2] * cap_in));
+        }
+        if (biased) {                                  // (j beyond the newest key: masked below)
+          const float dist = (float)max(L - 1 - j, 0);
+          s[i][e] = fmaf(-r1[0], __log2f(fmaf(r2[0], dist, 1.0f)), s[i][e] * (scale * 1.4426950408889634f));
+          s[i][e + 2] = fmaf(-r1[1], __log2f(fmaf(r2[1], dist, 1.0f)), s[i][e + 2] * (scale * 1.4426950408889634f));
         }
         if (j >= tile_hi || (j < lo_w && j >= keep)) s[i][e] = s[i][e + 2] = -INFINITY;
       }
@@ -853,7 +872,8 @@ __global__ void decode_merge_kernel(T* __restrict__ out, int64_t out_row_stride,
                                     const float* __restrict__ tmp_out, const float* __restrict__ tmp_m,
                                     const float* __restrict__ tmp_l, int nh, int hd, int max_parts, int part_keys,
                                     int sink, const float* __restrict__ gate, int64_t gate_stride,
-                                    const float* __restrict__ sinks, int pool_base, int pool_parts, int pool_p, int pool_window) {
+                                    const float* __restrict__ sinks, int pool_base, int pool_parts, int pool_p, int pool_window,
+                                    int out_hd) {
   constexpr int CHUNK = 128;                         // partitions whose factors are held in shared memory at a time
   __shared__ float f_s[CHUNK], red[32];
   const int b = blockIdx.x, h = blockIdx.y;
@@ -891,10 +911,10 @@ __global__ void decode_merge_kernel(T* __restrict__ out, int64_t out_row_stride,
       lt += f * lv[p];
       acc += f * ov[p];
     }
-    if (tid < hd) {
+    if (tid < out_hd) {
       float v = lt > 0.f ? acc / lt : 0.f;
       if (gate) v = v / (1.f + expf(-gate[tok * gate_stride + (int64_t)h * hd + tid]));
-      out[tok * out_row_stride + (int64_t)h * hd + tid] = from_f<T>(v);
+      out[tok * out_row_stride + (int64_t)h * out_hd + tid] = from_f<T>(v);
     }
     return;
   }
@@ -960,16 +980,67 @@ __global__ void decode_merge_kernel(T* __restrict__ out, int64_t out_row_stride,
       }
     }
   }
-  T* o = out + tok * out_row_stride + (int64_t)h * hd;
+  T* o = out + tok * out_row_stride + (int64_t)h * out_hd;
 #pragma unroll
   for (int c = 0; c < 4; ++c) {
     const int d = tid + c * (int)blockDim.x;
-    if (d < hd) {
+    if (d < out_hd) {
       float v = lt > 0.f ? acc[c] / lt : 0.f;
       if (gate) v = v / (1.f + expf(-gate[tok * gate_stride + (int64_t)h * hd + d]));
       o[d] = from_f<T>(v);
     }
   }
+}
+
+// The merge of heads that come in pairs (two maps over the same values): head h of the output is the difference of query heads
+// 2h and 2h + 1, a = a_0 - lambda a_1, divided by its root mean square over the head's values and times ``gain``.  One block =
+// one (request, pair); the thread (map, column) merges its column in index order, sixteen partitions' loads at a time.
+template <typename T>
+__global__ void __launch_bounds__(256)
+decode_merge_pairs_kernel(T* __restrict__ out, int64_t out_row_stride, const int* __restrict__ cu_seqlens,
+                          const int* __restrict__ context_lens, const float* __restrict__ tmp_out, const float* __restrict__ tmp_m,
+                          const float* __restrict__ tmp_l, int nh, int hd, int max_parts, int part_keys, int out_hd, float lambda,
+                          float gain, float eps) {
+  __shared__ float second[128], red[32];
+  const int b = blockIdx.x, h = blockIdx.y;
+  const int map = threadIdx.x / hd, d = threadIdx.x - map * hd;       // blockDim.x = 2 hd
+  const int L = context_lens[b];                     // written by the host, not by a kernel of this step
+  const int64_t tok = cu_seqlens[b];
+  pdl_wait();
+  pdl_launch_dependents();
+  const int P = max(1, min(max_parts, (L + part_keys - 1) / part_keys));
+  const int64_t row0 = ((int64_t)b * nh + 2 * h + map) * max_parts;
+  float M = -INFINITY, lt = 0.f, acc = 0.f;
+  for (int p0 = 0; p0 < P; p0 += 16) {
+    float mv[16], lv[16], ov[16];
+#pragma unroll
+    for (int i = 0; i < 16; ++i) {
+      mv[i] = p0 + i < P ? tmp_m[row0 + p0 + i] : -INFINITY;
+      lv[i] = p0 + i < P ? tmp_l[row0 + p0 + i] : 0.f;
+      ov[i] = p0 + i < P ? tmp_out[(row0 + p0 + i) * hd + d] : 0.f;        // (never written where mv is -inf: not used then)
+    }
+    float Mn = M;
+#pragma unroll
+    for (int i = 0; i < 16; ++i) Mn = fmaxf(Mn, mv[i]);
+    if (Mn == -INFINITY) continue;
+    const float a = expf(M - Mn);
+    M = Mn;
+    lt *= a;
+    acc *= a;
+#pragma unroll
+    for (int i = 0; i < 16; ++i) {
+      if (mv[i] == -INFINITY) continue;
+      const float f = expf(mv[i] - Mn);
+      lt += f * lv[i];
+      acc += f * ov[i];
+    }
+  }
+  float v = lt > 0.f ? acc / lt : 0.f;
+  if (map == 1) second[d] = v;
+  __syncthreads();
+  v = map == 0 && d < out_hd ? v - lambda * second[d] : 0.f;
+  const float ss = block_sum(v * v, red);
+  if (map == 0 && d < out_hd) out[tok * out_row_stride + (int64_t)h * out_hd + d] = from_f<T>(v * (gain / sqrtf(ss / (float)out_hd + eps)));
 }
 
 ME_API int me_attn_decode_partition() { return DEC_PART; }
@@ -993,8 +1064,17 @@ ME_API int me_attn_decode(const void* qkv, int dtype, int64_t q_row_stride, void
                           int window, float* tmp_out, float* tmp_m, float* tmp_l, int max_parts,
                           int* err, int kind, const void* kv_map, int sink, const float* gate, int64_t gate_stride,
                           int keep_first, int chunk, float softcap, const float* sinks, const void* pool_map,
-                          const int* pooled_tables, int pbt_stride, int pool_p, int pool_parts, cudaStream_t stream) {
+                          const int* pooled_tables, int pbt_stride, int pool_p, int pool_parts, const float* bias_r1,
+                      const float* bias_r2, int out_hd, int pairs, float pair_lambda, float pair_gain, float pair_eps, cudaStream_t stream) {
   if (num_reqs == 0) return 0;
+  // out_hd: how many elements of a head leave (0: all; rows of the cache may be longer than the values).  bias_r1, bias_r2
+  // (float32 [nh], both or neither; the tensor-map kernel's alone): r1 ln(1 + r2 distance) is taken off the scaled scores.
+  // pairs: query heads come in pairs whose difference is normed and written (decode_merge_pairs_kernel).
+  if (out_hd == 0) out_hd = hd;
+  ME_REQUIRE(out_hd > 0 && out_hd <= hd && !(gate && out_hd != hd), "me_attn_decode: %d of %d output elements", out_hd, hd);
+  ME_REQUIRE((bias_r1 == nullptr) == (bias_r2 == nullptr) && !(bias_r1 && (softcap > 0.f || sinks || sink || pool_p > 0)),
+             "me_attn_decode: a distance bias has two numbers a head and goes without caps, sinks and pooled blocks");
+  ME_REQUIRE(!pairs || (nh % 2 == 0 && hd <= 128 && !gate && !sinks && !sink && pool_p == 0), "me_attn_decode: pairs of heads go without gates, sinks and pooled blocks");
   ME_REQUIRE(hd % 8 == 0 && hd >= 8 && hd <= 256, "me_attn_decode: head_dim %d is not a multiple of 8 up to 256", hd);
   ME_REQUIRE(nh > 0 && nkv > 0 && nh % nkv == 0, "me_attn_decode: %d heads, %d kv heads", nh, nkv);
   ME_REQUIRE(max_parts >= 1 && max_parts <= 65535, "me_attn_decode: max_parts %d", max_parts);
@@ -1021,8 +1101,8 @@ ME_API int me_attn_decode(const void* qkv, int dtype, int64_t q_row_stride, void
   // the extra term of the softmax is exp(sinks[head]) (added once, in the merge).
   ME_REQUIRE(keep_first >= 0 && chunk >= 0 && softcap >= 0.f && !(chunk > 0 && window > 0) && (keep_first == 0 || window > 0),
              "me_attn_decode: a window (with kept first keys) or chunks, not both");
-  ME_REQUIRE(tma_mma || (keep_first == 0 && chunk == 0 && softcap == 0.f),
-             "me_attn_decode: kept first keys, chunks and capped scores need the kernel fed by tensor-map loads");
+  ME_REQUIRE(tma_mma || (keep_first == 0 && chunk == 0 && softcap == 0.f && !bias_r1),
+             "me_attn_decode: kept first keys, chunks, capped scores and biases need the kernel fed by tensor-map loads");
   // Pooled blocks (pool_p > 0; the tensor-map kernel's alone, with a plain window): the last pool_parts of a head's max_parts slots
   // take the partitions of a second launch over the cache of pooled blocks, whose "context" is the number of blocks the
   // request sees; the merge joins both runs.
@@ -1035,6 +1115,8 @@ ME_API int me_attn_decode(const void* qkv, int dtype, int64_t q_row_stride, void
     none.keep_first = keep_first;
     none.chunk = chunk;
     none.softcap = softcap;
+    none.bias_r1 = bias_r1;
+    none.bias_r2 = bias_r2;
     int rc = hd == 64 ? launch_partition_tma_mma<64, false, 2, 16>(kv_map, num_reqs, max_parts, stream, qkv, q_row_stride, block_tables, bt_stride,
                                                             cu_seqlens, context_lens, nh, nkv, page_size, scale, window, tmp_out, tmp_m, tmp_l, 1, err, none, tok_parts)
                       : launch_partition_tma_mma<128, false, 2, 16>(kv_map, num_reqs, max_parts, stream, qkv, q_row_stride, block_tables, bt_stride,
@@ -1073,11 +1155,18 @@ ME_API int me_attn_decode(const void* qkv, int dtype, int64_t q_row_stride, void
   ME_DEC_CASE(1, 4) ME_DEC_CASE(2, 4)
 #undef ME_DEC_CASE
   ME_LAUNCH_CHECK("me_attn_decode (partitions)");
+  if (pairs) {
+    ME_DISPATCH_DTYPE(dtype, T, (me_launch(decode_merge_pairs_kernel<T>, dim3(num_reqs, nh / 2), dim3(2 * hd), 0, stream, (T*)out,
+        out_row_stride, cu_seqlens, context_lens, (const float*)tmp_out, (const float*)tmp_m, (const float*)tmp_l, nh, hd, max_parts, DEC_PART,
+        out_hd, pair_lambda, pair_gain, pair_eps)));
+    ME_LAUNCH_CHECK("me_attn_decode (merge of pairs)");
+    return 0;
+  }
   dim3 mgrid(num_reqs, nh);
   const int mthreads = hd >= 128 ? 128 : (hd >= 64 ? 64 : 32);
   ME_DISPATCH_DTYPE(dtype, T, (me_launch(decode_merge_kernel<T>, mgrid, dim3(mthreads), 0, stream,
       (T*)out, out_row_stride, cu_seqlens, context_lens, tmp_out, tmp_m, tmp_l, nh, hd, max_parts, DEC_PART, sink, gate,
-      gate_stride, sinks, tok_parts, pool_parts, pool_p, window)));
+      gate_stride, sinks, tok_parts, pool_parts, pool_p, window, out_hd)));
   ME_LAUNCH_CHECK("me_attn_decode (merge)");
   return 0;
 }
@@ -1147,7 +1236,7 @@ ME_API int me_attn_decode_fused(const void* qkv, int64_t q_row_stride, void* out
   dim3 mgrid(num_reqs, nh);
   me_launch(decode_merge_kernel<bf16>, mgrid, dim3(hd >= 128 ? 128 : 64), 0, stream, (bf16*)out, out_row_stride, cu_seqlens,
             context_lens, tmp_out, tmp_m, tmp_l, nh, hd, max_parts, DEC_PART * tiles, 0, (const float*)nullptr, (int64_t)0,
-            (const float*)nullptr, 0, 0, 0, 0);
+            (const float*)nullptr, 0, 0, 0, 0, hd);
   ME_LAUNCH_CHECK("me_attn_decode_fused (merge)");
   return 0;
 }

@@ -37,6 +37,11 @@ __device__ __forceinline__ float ex2(float x) {
   asm("ex2.approx.ftz.f32 %0, %1;\n" : "=f"(y) : "f"(x));
   return y;
 }
+__device__ __forceinline__ float lg2(float x) {
+  float y;
+  asm("lg2.approx.ftz.f32 %0, %1;\n" : "=f"(y) : "f"(x));
+  return y;
+}
 __device__ __forceinline__ void mbar_arrive(unsigned long long* bar) {
   asm volatile("mbarrier.arrive.shared::cta.b64 _, [%0];\n" ::"r"(tma::smem_addr(bar)) : "memory");
 }
@@ -371,8 +376,9 @@ attn_prefill_tcgen05_kernel(const __grid_constant__ CUtensorMap q_map, const __g
 // are brought to the final reference and added at the end.
 // Parities: a wait names a phase of its barrier by parity, which is only right while the phase before it is
 // over.  Every wait below stands where that is known (the comment beside it says why).
-// EXTRA: kept first keys, chunks, capped scores and learned sinks are compiled in (the plain kernel keeps its registers).
-template <int HD, bool EXTRA>
+// EXTRA: kept first keys, chunks, capped scores, learned sinks and pooled blocks are compiled in (the plain kernel keeps its
+// registers).  BIASED (without EXTRA): a distance bias is.
+template <int HD, bool EXTRA, bool BIASED>
 __global__ void __launch_bounds__(TA_THREADS)
 attn_prefill_tcgen05_two_groups_kernel(const __grid_constant__ CUtensorMap q_map, const __grid_constant__ CUtensorMap kv_map,
                                        bf16* __restrict__ out, int64_t out_row_stride, const int* __restrict__ block_tables,
@@ -381,7 +387,8 @@ attn_prefill_tcgen05_two_groups_kernel(const __grid_constant__ CUtensorMap q_map
                                        int window, int sink, const float* __restrict__ gate, int64_t gate_stride,
                                        int* __restrict__ err, int keep_first_arg, int chunk_arg, float softcap_arg,
                                        const float* __restrict__ sinks_arg, const __grid_constant__ CUtensorMap pool_map,
-                                       const int* __restrict__ pooled_tables, int pbt_stride, int pool_p_arg) {
+                                       const int* __restrict__ pooled_tables, int pbt_stride, int pool_p_arg,
+                                       const float* __restrict__ bias_r1, const float* __restrict__ bias_r2, int out_hd) {
   const int keep_first = EXTRA ? keep_first_arg : 0, chunk = EXTRA ? chunk_arg : 0;
   const int pool_p = EXTRA ? pool_p_arg : 0;
   const float softcap = EXTRA ? softcap_arg : 0.f;
@@ -429,7 +436,8 @@ attn_prefill_tcgen05_two_groups_kernel(const __grid_constant__ CUtensorMap q_map
   };
   const int* pbt = (EXTRA && pool_p > 0) ? pooled_tables + (int64_t)b * pbt_stride : nullptr;
   // With a cap c the scores become c tanh(s * scale / c) before anything else; exponents then take log2(e) alone.
-  const float sl2 = softcap > 0.f ? 1.4426950408889634f : scale_log2;
+  // With a distance bias the scores become s * scale * log2(e) - r1 log2(1 + r2 (i - j)) first: exponents take them as they are.
+  const float sl2 = BIASED ? 1.0f : (softcap > 0.f ? 1.4426950408889634f : scale_log2);
   const float cap_in = softcap > 0.f ? scale_log2 * (2.0f / softcap) : 0.f;      // s -> 2 log2(e) s scale / c
   const int* bt = block_tables + (int64_t)b * bt_stride;
 
@@ -569,6 +577,7 @@ attn_prefill_tcgen05_two_groups_kernel(const __grid_constant__ CUtensorMap q_map
     const int j_min = window > 0 ? pos - window + 1 : (chunk > 0 ? (pos / chunk) * chunk : -(1 << 30));
     const int chunk_hi = chunk > 0 ? (p_hi / chunk) * chunk : 0;
     const int nb_row = (EXTRA && row_ok) ? blocks_seen(pos) : 0;     // the pooled blocks this row sees: [0, nb_row)
+    const float r1 = BIASED ? bias_r1[head0 + r / tq] : 0.f, r2 = BIASED ? bias_r2[head0 + r / tq] : 0.f;
     // Both groups run every named barrier of every tile, also after a wait has given up (ok == false): then only
     // the work is skipped, so no warp is left waiting for a partner that has gone.
     for (int it = g; it < n_tiles; it += 2) {
@@ -616,13 +625,21 @@ attn_prefill_tcgen05_two_groups_kernel(const __grid_constant__ CUtensorMap q_map
 #pragma unroll
           for (int jj = 0; jj < 64; ++jj) half[jj] = softcap - 2.0f * softcap * __frcp_rn(1.0f + ex2(half[jj] * cap_in));
         };
+        // (keys behind the query give the logarithm of anything: they are unseen, and replaced by -inf before use)
+        auto bias_half = [&](float (&half)[64], float dist) {
+#pragma unroll
+          for (int jj = 0; jj < 64; ++jj)
+            half[jj] = fmaf(-r1, lg2(fmaf(r2, dist - (float)jj, 1.0f)), half[jj] * scale_log2);
+        };
         tc5::ld_64cols(t_s, s_lo);
         tc5::wait_ld();
         tc5::ld_64cols(t_s + 64, s_hi);                      // on its way while the first half is worked on
+        if (BIASED) bias_half(s_lo, (float)(pos - kt));
         if (softcap > 0.f) cap_half(s_lo);
         piece_max(piece(s_lo, 0), 0);
         piece_max(piece(s_lo, 1), 32);
         tc5::wait_ld();
+        if (BIASED) bias_half(s_hi, (float)(pos - kt - 64));
         if (softcap > 0.f) cap_half(s_hi);
         piece_max(piece(s_hi, 0), 64);
         piece_max(piece(s_hi, 1), 96);
@@ -762,7 +779,7 @@ attn_prefill_tcgen05_two_groups_kernel(const __grid_constant__ CUtensorMap q_map
       const int piece = lane % PIECES;
       for (int row = (warp - 2) * 16 + lane / PIECES; row < (warp - 1) * 16; row += ROWS_AT_ONCE) {
         const int tok = row % tq;
-        if (tok < n_tok) {
+        if (tok < n_tok && piece * 8 < out_hd) {
           uint4 pk = *reinterpret_cast<const uint4*>(q_s + row * (HD * 2) + ((piece ^ (row & 7)) << 4));
           if (gate) {
             // The output times the sigmoid of the gate's pre-activation, here where the lanes of a row read the gate's row
@@ -775,7 +792,7 @@ attn_prefill_tcgen05_two_groups_kernel(const __grid_constant__ CUtensorMap q_map
               h2[jj] = __floats2bfloat162_rn(__fdividef(v.x, 1.f + __expf(-gr[2 * jj])), __fdividef(v.y, 1.f + __expf(-gr[2 * jj + 1])));
             }
           }
-          *reinterpret_cast<uint4*>(out + (int64_t)(tok0 + q0 + tok) * out_row_stride + (int64_t)(head0 + row / tq) * HD + piece * 8) = pk;
+          *reinterpret_cast<uint4*>(out + (int64_t)(tok0 + q0 + tok) * out_row_stride + (int64_t)(head0 + row / tq) * out_hd + piece * 8) = pk;
         }
       }
     }
@@ -792,15 +809,17 @@ int launch_ta(const void* q_map, const void* kv_map, void* out, int64_t out_row_
               const int* cu_seqlens, const int* context_lens, const int* tiles, int num_tiles, int nh, int nkv, int gp,
               int page_size, float scale, int window, int sink, const float* gate, int64_t gate_stride, int* err,
               int keep_first, int chunk, float softcap, const float* sinks, const void* pool_map, const int* pooled_tables,
-              int pbt_stride, int pool_p, cudaStream_t stream) {
+              int pbt_stride, int pool_p, const float* bias_r1, const float* bias_r2, int out_hd, cudaStream_t stream) {
   const size_t smem = TWO_GROUPS ? (size_t)TA_ROWS * HD * 2 + 6 * (size_t)KT * HD * 2 + 1024
                                  : (size_t)TA_ROWS * HD * 2 + 4 * (size_t)KT * HD * 2 + 2 * (size_t)TA_ROWS * KT * 2 + 1024;
   static bool attr_set = false;
   if (!attr_set) {
-    cudaError_t e = TWO_GROUPS ? cudaFuncSetAttribute(attn_prefill_tcgen05_two_groups_kernel<HD, false>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem)
+    cudaError_t e = TWO_GROUPS ? cudaFuncSetAttribute(attn_prefill_tcgen05_two_groups_kernel<HD, false, false>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem)
                                : cudaFuncSetAttribute(attn_prefill_tcgen05_kernel<HD, KT>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
     if (TWO_GROUPS && e == cudaSuccess)
-      e = cudaFuncSetAttribute(attn_prefill_tcgen05_two_groups_kernel<HD, true>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+      e = cudaFuncSetAttribute(attn_prefill_tcgen05_two_groups_kernel<HD, true, false>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+    if (TWO_GROUPS && e == cudaSuccess)
+      e = cudaFuncSetAttribute(attn_prefill_tcgen05_two_groups_kernel<HD, false, true>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
     ME_REQUIRE(e == cudaSuccess, "me_attn_prefill_tcgen05: cannot raise shared memory: %s", cudaGetErrorString(e));
     attr_set = true;
   }
@@ -809,13 +828,14 @@ int launch_ta(const void* q_map, const void* kv_map, void* out, int64_t out_row_
   // and 16% slower at 2,048, where the last round then holds long tiles.)
   dim3 grid(nkv * (nh / nkv / gp), num_tiles);
   if constexpr (TWO_GROUPS) {
-    auto kernel = (keep_first > 0 || chunk > 0 || softcap > 0.f || sinks || pool_p > 0) ? attn_prefill_tcgen05_two_groups_kernel<HD, true>
-                                                                          : attn_prefill_tcgen05_two_groups_kernel<HD, false>;
+    auto kernel = bias_r1 ? attn_prefill_tcgen05_two_groups_kernel<HD, false, true>
+                : (keep_first > 0 || chunk > 0 || softcap > 0.f || sinks || pool_p > 0) ? attn_prefill_tcgen05_two_groups_kernel<HD, true, false>
+                                                                                        : attn_prefill_tcgen05_two_groups_kernel<HD, false, false>;
     me_launch(kernel, grid, dim3(TA_THREADS), smem, stream, *reinterpret_cast<const CUtensorMap*>(q_map),
               *reinterpret_cast<const CUtensorMap*>(kv_map), (bf16*)out, out_row_stride, block_tables, bt_stride, cu_seqlens,
               context_lens, tiles, nh, nkv, gp, page_size, scale * 1.4426950408889634f, window, sink, gate, gate_stride, err,
               keep_first, chunk, softcap, sinks, *reinterpret_cast<const CUtensorMap*>(pool_p > 0 ? pool_map : kv_map), pooled_tables,
-              pbt_stride, pool_p);
+              pbt_stride, pool_p, bias_r1, bias_r2, out_hd);
   } else
     me_launch(attn_prefill_tcgen05_kernel<HD, KT>, grid, dim3(TA_THREADS), smem, stream, *reinterpret_cast<const CUtensorMap*>(q_map),
               *reinterpret_cast<const CUtensorMap*>(kv_map), (bf16*)out, out_row_stride, block_tables, bt_stride, cu_seqlens,
@@ -844,13 +864,16 @@ ME_API int me_attn_prefill_tcgen05_heads_per_block(int nh, int nkv, int hd, int 
 // ``softcap`` c: scores become c tanh(score * scale / c).  ``sinks``: float32 [nh], the extra term is exp(sinks[head]),
 // neither scaled nor capped.  ``pool_map``, ``pooled_tables``, ``pool_p``: a second cache of the same layout with one row per
 // block of pool_p tokens and its block tables; with a window a query at p also sees the blocks b with (b + 1) pool_p <=
-// p - window + 1 (0: none).  These five are the kernel with two groups' alone.
+// p - window + 1 (0: none).  ``bias_r1``, ``bias_r2`` (float32 [nh], both or neither): r1 ln(1 + r2 (p - j)) is taken off the
+// scaled score of a key at j.  ``out_hd``: how many elements of a head leave (a multiple of 8; the cache's rows may be longer than the values);
+// rows of ``out`` hold nh * out_hd of them.  These seven are the kernel with two groups' alone.
 ME_API int me_attn_prefill_tcgen05(const void* q_map, const void* kv_map, void* out, int64_t out_row_stride,
                                    const int* block_tables, int bt_stride, const int* cu_seqlens, const int* context_lens,
                                    const int* tiles, int num_tiles, int nh, int nkv, int hd, int page_size, float scale,
                                    int window, int key_tile, int sink, const float* gate, int64_t gate_stride, int* err,
                                    int keep_first, int chunk, float softcap, const float* sinks, const void* pool_map,
-                                   const int* pooled_tables, int pbt_stride, int pool_p, cudaStream_t stream) {
+                                   const int* pooled_tables, int pbt_stride, int pool_p, const float* bias_r1, const float* bias_r2,
+                                   int out_hd, cudaStream_t stream) {
   if (num_tiles == 0) return 0;
   const int gp = me_attn_prefill_tcgen05_heads_per_block(nh, nkv, hd, page_size);
   ME_REQUIRE(gp > 0, "me_attn_prefill_tcgen05: head_dim %d, %d/%d heads, pages of %d are not taken", hd, nh, nkv, page_size);
@@ -860,8 +883,12 @@ ME_API int me_attn_prefill_tcgen05(const void* q_map, const void* kv_map, void* 
   // key_tile: keys per step of the loop.  128 (and 0): the kernel with two softmax groups and P in tensor memory, the
   // faster one; 64: the kernel with one group and P in shared memory, which needs less of both memories.
   if (key_tile == 0) key_tile = 128;
-  ME_REQUIRE(key_tile == 128 || (keep_first == 0 && chunk == 0 && softcap == 0.f && sinks == nullptr && pool_p == 0),
-             "me_attn_prefill_tcgen05: kept first keys, chunks, capped scores, learned sinks and pooled blocks need the key tile of 128");
+  if (out_hd == 0) out_hd = hd;
+  ME_REQUIRE(key_tile == 128 || (keep_first == 0 && chunk == 0 && softcap == 0.f && sinks == nullptr && pool_p == 0 && !bias_r1 && out_hd == hd),
+             "me_attn_prefill_tcgen05: kept first keys, chunks, capped scores, learned sinks, pooled blocks, biases and short outputs need the key tile of 128");
+  ME_REQUIRE(out_hd > 0 && out_hd <= hd && out_hd % 8 == 0 && !(gate && out_hd != hd), "me_attn_prefill_tcgen05: %d of %d output elements", out_hd, hd);
+  ME_REQUIRE((bias_r1 == nullptr) == (bias_r2 == nullptr) && !(bias_r1 && (softcap > 0.f || sinks || sink || pool_p > 0 || keep_first > 0 || chunk > 0)),
+             "me_attn_prefill_tcgen05: a distance bias has two numbers a head and goes with a plain window at most");
   ME_REQUIRE(pool_p == 0 || (pool_p > 0 && pool_map && pooled_tables && window > 0 && keep_first == 0 && chunk == 0),
              "me_attn_prefill_tcgen05: pooled blocks of %d tokens need their cache and a plain window", pool_p);
   ME_REQUIRE(keep_first >= 0 && chunk >= 0 && softcap >= 0.f && !(chunk > 0 && window > 0) && (keep_first == 0 || window > 0),
@@ -871,7 +898,7 @@ ME_API int me_attn_prefill_tcgen05(const void* q_map, const void* kv_map, void* 
   int rc;
 #define ME_TA_ARGS q_map, kv_map, out, out_row_stride, block_tables, bt_stride, cu_seqlens, context_lens, tiles, num_tiles, nh, nkv, gp, \
                    page_size, scale, window, sink, gate, gate_stride, err, keep_first, chunk, softcap, sinks, pool_map, pooled_tables, \
-                   pbt_stride, pool_p, stream
+                   pbt_stride, pool_p, bias_r1, bias_r2, out_hd, stream
   if (hd == 64) rc = key_tile == 64 ? launch_ta<64, 64, false>(ME_TA_ARGS) : launch_ta<64, 128, true>(ME_TA_ARGS);
   else rc = key_tile == 64 ? launch_ta<128, 64, false>(ME_TA_ARGS) : launch_ta<128, 128, true>(ME_TA_ARGS);
 #undef ME_TA_ARGS

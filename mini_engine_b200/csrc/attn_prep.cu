@@ -1,133 +1,224 @@
 // Between the packed projection and the attention of a grouped-query mixer whose projections may have biases and whose
-// queries and keys may be normalised on either side of the rotation:
+// queries and keys may be normalised on either side of the rotation, or over the whole projection:
 //
 //   u = W h (+ bias)                                  per head of q (H heads of D), k (G heads of D), v (G heads of Dv)
 //   q, k: u <- u / rms(u) * w   (NORM_BEFORE, a weight of D values shared by the heads; q and k have one each)
+//   q, k: u <- u / rms(row) * w (NORM_ROW: the root mean square over all heads' values of the token's q, or of its k, and a
+//         weight for every one of them)
 //   q, k: rotary positions on the first ``rot`` elements of a head, element i paired with element i + rot/2:
 //         (a, b) -> (a cos t - b sin t, b cos t + a sin t), t = position * freq[i]; the angle is formed in double precision
 //         from the int32 position and a table of rot/2 frequencies (so any scaling of the frequencies is the table's
-//         business), brought into [-pi, pi] there, then float32 sine and cosine
+//         business), brought into [-pi, pi] there, then float32 sine and cosine (or both come from a table of the step's
+//         tokens, ``angles``)
 //   q, k: u <- u / rms(u)       (NORM_AFTER, no weight)
 //   q: u <- u * q_scale[head]   (a learned number per query head that multiplies the head's scores; optional)
-//   q -> q_out [T, H*D]; k, v -> the paged cache rows that slot_mapping names ([page][keys | values][kv head][offset][HD])
+//   q: u <- u * (1 + temp_coef ln(floor((position + 1) / temp_every) + 1))      (a temperature that grows with the position)
+//   v: u <- u * v_scale
+//   q -> q_out [T, heads, q_row]; k, v -> the paged cache rows that slot_mapping names ([page][keys | values][kv head][offset][HD])
+//
+// With ``maps`` M = 2 every head of q and k has two maps of D elements side by side (two sets of scores over the same values):
+// the columns are q (H heads of M x D), k (G heads of M x D), v (G heads of Dv), and each map is normalised and rotated by itself.
+// The cache row of a key holds its maps one after the other; every query map gets a row of q_out of its own, its values where
+// that map lies in a key's row and zeros elsewhere, so that its product with a whole key row is its map's score.  Rows of
+// q_out and of the cache that are longer than what they hold are filled with zeros.
 //
 // With ``own_kv`` 0 the rows hold queries only (a mixer that reads another layer's keys and values) and nothing is written
-// to the cache.  rms(u) = sqrt(mean(u^2) + eps).  Everything is float32 until the stores.  One warp = one head of one token.
+// to the cache.  rms(u) = sqrt(mean(u^2) + eps).  Everything is float32 until the stores.  One warp = one map of one head of
+// one token; with NORM_ROW a block takes a token, so that the sums over the whole projection are taken once.
 #include "common.cuh"
 
 constexpr int AP_MAX = 256;     // largest head
 
-enum { AP_NORM_NONE = 0, AP_NORM_BEFORE = 1, AP_NORM_AFTER = 2 };
+enum { AP_NORM_NONE = 0, AP_NORM_BEFORE = 1, AP_NORM_AFTER = 2, AP_NORM_ROW = 3 };
 
+struct PrepArgs {
+  const float* proj;
+  int64_t ld;
+  const float* bias;
+  const float *q_w, *k_w;
+  int norm_mode;
+  float eps;
+  const double* freq;
+  int rot;
+  const float* angles;        // [T, rot/2, 2] cosine and sine, or null: formed here
+  const int* positions;
+  const int* slot_mapping;
+  int HD, page_size, H, G, D, Dv, M, q_row, n_tok;
+  const float* q_scale;
+  int own_kv;
+  float temp_coef, temp_every, v_scale;
+};
+
+// One unit of a token's row: hs counts the query maps, then the key maps, then the value heads.  inv_q, inv_k: 1 / rms of the
+// token's whole q and k (NORM_ROW only).
 template <typename T>
-__global__ void __launch_bounds__(128)
-attn_prep_kernel(const float* __restrict__ proj, int64_t ld, const float* __restrict__ bias, const float* __restrict__ q_w,
-                 const float* __restrict__ k_w, int norm_mode, float eps, const double* __restrict__ freq, int rot,
-                 const int* __restrict__ positions, const int* __restrict__ slot_mapping, T* __restrict__ q_out,
-                 T* __restrict__ pool, int HD, int page_size, int H, int G, int D, int Dv, int n_tok,
-                 const float* __restrict__ q_scale, int own_kv) {
-  __shared__ float stage[4][AP_MAX];
-  pdl_wait();
-  pdl_launch_dependents();
-  const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
-  const int per_tok = own_kv ? H + 2 * G : H;
-  const int64_t unit = (int64_t)blockIdx.x * 4 + warp;
-  if (unit >= (int64_t)n_tok * per_tok) return;
-  const int t = (int)(unit / per_tok), hs = (int)(unit - (int64_t)t * per_tok);
-  const bool is_q = hs < H, is_k = !is_q && hs < H + G;
-  const int head = is_q ? hs : (is_k ? hs - H : hs - H - G);
-  const int n = (is_q || is_k) ? D : Dv;
-  const int col0 = is_q ? head * D : (is_k ? H * D + head * D : (H + G) * D + head * Dv);
-  const float* src = proj + (int64_t)t * ld + col0;
+__device__ __forceinline__ void prep_unit(const PrepArgs& a, T* __restrict__ q_out, T* __restrict__ pool, float* st, int t, int hs, int lane,
+                                          float inv_q, float inv_k) {
+  const int D = a.D, M = a.M, HM = a.H * M, GM = a.G * M;
+  const bool is_q = hs < HM, is_k = !is_q && hs < HM + GM;
+  const int unit = is_q ? hs : (is_k ? hs - HM : hs - HM - GM);        // (head, map), or the value head
+  const int head = (is_q || is_k) ? unit / M : unit, map = (is_q || is_k) ? unit - head * M : 0;
+  const int n = (is_q || is_k) ? D : a.Dv;
+  const int col0 = is_q ? unit * D : (is_k ? HM * D + unit * D : (HM + GM) * D + unit * a.Dv);
+  const float* src = a.proj + (int64_t)t * a.ld + col0;
   float u[AP_MAX / 32];
   float ss = 0.f;
 #pragma unroll
   for (int i = 0; i < AP_MAX / 32; ++i) {
     const int d = lane + 32 * i;
-    u[i] = d < n ? src[d] + (bias ? bias[col0 + d] : 0.f) : 0.f;
+    u[i] = d < n ? src[d] + (a.bias ? a.bias[col0 + d] : 0.f) : 0.f;
     ss = fmaf(u[i], u[i], ss);
   }
   if (is_q || is_k) {
-    if (norm_mode == AP_NORM_BEFORE) {
-      const float r = 1.0f / sqrtf(warp_sum(ss) / (float)D + eps);
-      const float* w = is_q ? q_w : k_w;
+    if (a.norm_mode == AP_NORM_BEFORE || a.norm_mode == AP_NORM_ROW) {
+      const bool whole = a.norm_mode == AP_NORM_ROW;
+      const float r = whole ? (is_q ? inv_q : inv_k) : 1.0f / sqrtf(warp_sum(ss) / (float)D + a.eps);
+      const float* w = (is_q ? a.q_w : a.k_w) + (whole ? unit * D : 0);
 #pragma unroll
       for (int i = 0; i < AP_MAX / 32; ++i) {
         const int d = lane + 32 * i;
         if (d < D) u[i] = u[i] * r * w[d];
       }
     }
-    if (rot > 0) {
-      float* st = stage[warp];
+    if (a.rot > 0) {
 #pragma unroll
       for (int i = 0; i < AP_MAX / 32; ++i) {
         const int d = lane + 32 * i;
         if (d < D) st[d] = u[i];
       }
       __syncwarp();
-      const int half = rot / 2;
-      const double pos = (double)positions[t];
+      const int half = a.rot / 2;
+      const double pos = (double)a.positions[t];
 #pragma unroll
       for (int i = 0; i < AP_MAX / 32; ++i) {
         const int d = lane + 32 * i;
-        if (d < rot) {
+        if (d < a.rot) {
           const int f = d < half ? d : d - half;
-          double a = pos * freq[f];
-          a -= 6.283185307179586476925 * rint(a * 0.15915494309189533577);
           float sn, cs;
-          sincosf((float)a, &sn, &cs);
+          if (a.angles) {
+            const float2 c2 = *reinterpret_cast<const float2*>(a.angles + ((int64_t)t * half + f) * 2);
+            cs = c2.x;
+            sn = c2.y;
+          } else {
+            double x = pos * a.freq[f];
+            x -= 6.283185307179586476925 * rint(x * 0.15915494309189533577);
+            sincosf((float)x, &sn, &cs);
+          }
           u[i] = d < half ? st[d] * cs - st[d + half] * sn : st[d] * cs + st[d - half] * sn;
         }
       }
+      __syncwarp();                                    // (the warp may take another unit)
     }
-    if (norm_mode == AP_NORM_AFTER) {
+    if (a.norm_mode == AP_NORM_AFTER) {
       ss = 0.f;
 #pragma unroll
       for (int i = 0; i < AP_MAX / 32; ++i) ss = fmaf(u[i], u[i], ss);
-      const float r = 1.0f / sqrtf(warp_sum(ss) / (float)D + eps);
+      const float r = 1.0f / sqrtf(warp_sum(ss) / (float)D + a.eps);
 #pragma unroll
       for (int i = 0; i < AP_MAX / 32; ++i) u[i] *= r;
     }
-    if (is_q && q_scale) {
-      const float f = q_scale[head];
+    if (is_q && a.q_scale) {
+      const float f = a.q_scale[head];
 #pragma unroll
       for (int i = 0; i < AP_MAX / 32; ++i) u[i] *= f;
     }
-  }
-  T* dst;
-  if (is_q) {
-    dst = q_out + (int64_t)t * H * D + (int64_t)head * D;
+    if (is_q && a.temp_every > 0.f) {
+      const float f = fmaf(a.temp_coef, logf(floorf((float)(a.positions[t] + 1) / a.temp_every) + 1.0f), 1.0f);
+#pragma unroll
+      for (int i = 0; i < AP_MAX / 32; ++i) u[i] *= f;
+    }
   } else {
-    const int slot = slot_mapping ? slot_mapping[t] : -1;
+#pragma unroll
+    for (int i = 0; i < AP_MAX / 32; ++i) u[i] *= a.v_scale;
+  }
+  // the row that takes the unit, where in it the unit's values start, and which of its elements this warp fills with zeros
+  T* dst;
+  int base = map * D, zero_lo, zero_hi;
+  if (is_q) {
+    dst = q_out + ((int64_t)t * HM + unit) * a.q_row;
+    zero_lo = 0;
+    zero_hi = a.q_row;
+  } else {
+    const int slot = a.slot_mapping ? a.slot_mapping[t] : -1;
     if (slot < 0) return;
-    const int page = slot / page_size, off = slot - page * page_size;
-    dst = pool + ((((int64_t)page * 2 + (is_k ? 0 : 1)) * G + head) * page_size + off) * HD;
+    const int page = slot / a.page_size, off = slot - page * a.page_size;
+    dst = pool + ((((int64_t)page * 2 + (is_k ? 0 : 1)) * a.G + head) * a.page_size + off) * a.HD;
+    zero_lo = base;                                    // what lies behind the last map (or the value)
+    zero_hi = map == (is_k ? M - 1 : 0) ? a.HD : 0;
   }
 #pragma unroll
   for (int i = 0; i < AP_MAX / 32; ++i) {
     const int d = lane + 32 * i;
-    if (d < n) dst[d] = from_f<T>(u[i]);
+    if (d < n) dst[base + d] = from_f<T>(u[i]);
   }
+  for (int d = zero_lo + lane; d < zero_hi; d += 32)
+    if (d < base || d >= base + n) dst[d] = from_f<T>(0.f);
 }
 
-// proj: [T, ld] float32 rows holding q (H*D), k (G*D), v (G*Dv) in their first columns.  bias: [H*D + G*D + G*Dv] float32 or
-// null.  q_w, k_w: [D] float32 (NORM_BEFORE only).  freq: [rot/2] float64 or null with rot 0.  slot_mapping: [T] int32 cache
-// rows (page * page_size + offset; negative: not written) or null (no keys and values are written).  q_scale: [H] float32 or
-// null.  own_kv 0: the rows hold H*D query columns only.
+template <typename T>
+__global__ void __launch_bounds__(128) attn_prep_kernel(PrepArgs a, T* __restrict__ q_out, T* __restrict__ pool) {
+  __shared__ float stage[4][AP_MAX];
+  pdl_wait();
+  pdl_launch_dependents();
+  const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
+  const int per_tok = a.H * a.M + (a.own_kv ? a.G * (a.M + 1) : 0);
+  const int64_t unit = (int64_t)blockIdx.x * 4 + warp;
+  if (unit >= (int64_t)a.n_tok * per_tok) return;
+  const int t = (int)(unit / per_tok);
+  prep_unit<T>(a, q_out, pool, stage[warp], t, (int)(unit - (int64_t)t * per_tok), lane, 1.f, 1.f);
+}
+
+// A token a block: the sums over the whole q and the whole k first, then the units.
+template <typename T>
+__global__ void __launch_bounds__(256) attn_prep_row_kernel(PrepArgs a, T* __restrict__ q_out, T* __restrict__ pool) {
+  __shared__ float stage[8][AP_MAX];
+  __shared__ float red[32];
+  pdl_wait();
+  pdl_launch_dependents();
+  const int t = blockIdx.x, lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
+  const int nq = a.H * a.M * a.D, nk = a.own_kv ? a.G * a.M * a.D : 0;
+  const float* row = a.proj + (int64_t)t * a.ld;
+  float sq = 0.f, sk = 0.f;
+#pragma unroll 4
+  for (int c = threadIdx.x; c < nq; c += 256) {
+    const float u = row[c] + (a.bias ? a.bias[c] : 0.f);
+    sq = fmaf(u, u, sq);
+  }
+#pragma unroll 4
+  for (int c = nq + threadIdx.x; c < nq + nk; c += 256) {
+    const float u = row[c] + (a.bias ? a.bias[c] : 0.f);
+    sk = fmaf(u, u, sk);
+  }
+  const float inv_q = 1.0f / sqrtf(block_sum(sq, red) / (float)nq + a.eps);
+  const float inv_k = nk ? 1.0f / sqrtf(block_sum(sk, red) / (float)nk + a.eps) : 0.f;
+  const int per_tok = a.H * a.M + (a.own_kv ? a.G * (a.M + 1) : 0);
+  for (int hs = warp; hs < per_tok; hs += 8) prep_unit<T>(a, q_out, pool, stage[warp], t, hs, lane, inv_q, inv_k);
+}
+
+// proj: [T, ld] float32 rows holding q (H*M*D), k (G*M*D), v (G*Dv) in their first columns, M = maps.  bias: a float32 value for
+// each of these columns or null.  q_w, k_w: [D] float32 (NORM_BEFORE), [H*M*D] and [G*M*D] (NORM_ROW).  freq: [rot/2] float64 or
+// null with rot 0; angles: [T, rot/2, 2] float32 or null.  slot_mapping: [T] int32 cache rows (page * page_size + offset;
+// negative: not written) or null (no keys and values are written).  q_scale: [H] float32 or null.  own_kv 0: the rows hold the
+// query columns only.  q_out: [T, H*M, q_row].  temp_every 0: no temperature.
 ME_API int me_attn_prep(const float* proj, int64_t ld, const float* bias, const float* q_w, const float* k_w, int norm_mode,
-                        float eps, const double* freq, int rot, const int* positions, const int* slot_mapping, void* q_out,
-                        void* pool, int dtype, int HD, int page_size, int H, int G, int D, int Dv, int T, const float* q_scale,
-                        int own_kv, cudaStream_t stream) {
+                        float eps, const double* freq, int rot, const float* angles, const int* positions, const int* slot_mapping,
+                        void* q_out, int q_row, void* pool, int dtype, int HD, int page_size, int H, int G, int D, int Dv, int maps, int T,
+                        const float* q_scale, int own_kv, float temp_coef, float temp_every, float v_scale, cudaStream_t stream) {
   if (T == 0) return 0;
-  ME_REQUIRE(T > 0 && H > 0 && G > 0 && D >= 1 && D <= AP_MAX && Dv >= 1 && Dv <= AP_MAX, "me_attn_prep: bad sizes H=%d G=%d D=%d Dv=%d", H, G,
-             D, Dv);
+  ME_REQUIRE(T > 0 && H > 0 && G > 0 && D >= 1 && D <= AP_MAX && Dv >= 1 && Dv <= AP_MAX && (maps == 1 || maps == 2),
+             "me_attn_prep: bad sizes H=%d G=%d D=%d Dv=%d maps=%d", H, G, D, Dv, maps);
   ME_REQUIRE(rot >= 0 && rot <= D && rot % 2 == 0 && (rot == 0 || freq), "me_attn_prep: %d of %d elements cannot be rotated", rot, D);
-  ME_REQUIRE(norm_mode != AP_NORM_BEFORE || (q_w && (k_w || !own_kv)), "me_attn_prep: the norm in front of the rotation needs its weights");
-  ME_REQUIRE(!slot_mapping || (pool && HD >= D && HD >= Dv), "me_attn_prep: cache rows of %d elements are too short", HD);
-  const int64_t units = (int64_t)T * (own_kv ? H + 2 * G : H);
-  ME_DISPATCH_DTYPE(dtype, TT,
-      me_launch(attn_prep_kernel<TT>, dim3((unsigned)((units + 3) / 4)), dim3(128), 0, stream, proj, ld, bias, q_w, k_w, norm_mode, eps, freq,
-                rot, positions, slot_mapping, (TT*)q_out, (TT*)pool, HD, page_size, H, G, D, Dv, T, q_scale, own_kv));
+  ME_REQUIRE((norm_mode != AP_NORM_BEFORE && norm_mode != AP_NORM_ROW) || (q_w && (k_w || !own_kv)), "me_attn_prep: a weighted norm needs its weights");
+  ME_REQUIRE(q_row >= maps * D, "me_attn_prep: query rows of %d elements are too short", q_row);
+  ME_REQUIRE(!slot_mapping || (pool && HD >= maps * D && HD >= Dv), "me_attn_prep: cache rows of %d elements are too short", HD);
+  ME_REQUIRE(temp_every >= 0.f, "me_attn_prep: the temperature's step must not be negative");
+  const PrepArgs a = {proj, ld, bias, q_w, k_w, norm_mode, eps, freq, rot, angles, positions, slot_mapping, HD, page_size, H, G, D, Dv, maps,
+                      q_row, T, q_scale, own_kv, temp_coef, temp_every, v_scale};
+  const int64_t units = (int64_t)T * (H * maps + (own_kv ? G * (maps + 1) : 0));
+  ME_DISPATCH_DTYPE(dtype, TT, {
+    if (norm_mode == AP_NORM_ROW) me_launch(attn_prep_row_kernel<TT>, dim3(T), dim3(256), 0, stream, a, (TT*)q_out, (TT*)pool);
+    else me_launch(attn_prep_kernel<TT>, dim3((unsigned)((units + 3) / 4)), dim3(128), 0, stream, a, (TT*)q_out, (TT*)pool);
+  });
   ME_LAUNCH_CHECK("me_attn_prep");
   return 0;
 }

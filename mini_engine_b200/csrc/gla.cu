@@ -11,12 +11,33 @@
 //                 portion starts at position 0) and leaves the new state there; a token's result does not depend on where
 //                 the sequence was cut beyond the order of sums.  One block = one request x one head x GLA_VB columns of S.
 //                 Portions of prompts take GLA_LC tokens at a time (see gla_intra_kernel and the three kernels behind it).
+//
+// The recurrence in which ONE gate decides what is kept and what is written (HGRN2) is the same with k_t = 1 - a_t: instead of
+// keys and log decays the projection then holds the gate's pre-activation z per key channel,
+//   a = l + (1 - l) sigmoid(z + b),   k = (1 - l) sigmoid(-(z + b)) = 1 - a,   q <- q sigmoid(q)
+// with a lower bound l in [0, 1) and a bias b per channel (``ForgetGate``).  The kernels that read q and k first form all
+// three; the chunk kernels' first one leaves q and k in the projection's place for the others.
 #include "common.cuh"
 #include <type_traits>
 
 constexpr int GLA_VB = 16, GLA_DY = 16, GLA_THREADS = GLA_VB * GLA_DY;
 
 __device__ __forceinline__ float gla_log_sigmoid(float x) { return fminf(x, 0.f) - log1pf(expf(-fabsf(x))); }
+
+struct ForgetGate {
+  const float* bias;            // [H*D]
+  const float* lower;           // [H*D]
+};
+// From the pre-activation (with its bias) of a channel with lower bound l: the written share k = 1 - a and log a.  Where a is
+// close to 1 its logarithm comes from k, which is not rounded against 1; a gate that forgets everything (a < e^-40, four parts in
+// 10^18 of the state before it) counts as e^-40, so that sums of logarithms stay finite and keep their digits.
+__device__ __forceinline__ void forget_gate(float z, float l, float& k, float& log_a) {
+  const float e = expf(-fabsf(z)), s = 1.0f / (1.0f + e);
+  const float up = z >= 0.f ? s : e * s, down = z >= 0.f ? e * s : s;          // sigmoid(z), sigmoid(-z)
+  k = (1.0f - l) * down;
+  log_a = k < 0.5f ? log1pf(-k) : fmaxf(logf(fmaf(1.0f - l, up, l)), -40.0f);
+}
+__device__ __forceinline__ float gla_silu(float x) { return x / (1.0f + expf(-x)); }
 
 // la[t, c] = logsigmoid(b[c] + sum_r W2[c, r] a1[t, r]) * inv_tau.  One block = GLA_DT tokens x 128 channels: a thread
 // reads its channel's row of W2 once for all of the block's tokens.
@@ -50,10 +71,11 @@ gla_decay_kernel(const float* __restrict__ proj, int64_t ld, int off_a1, int ran
     if (t0 + t < T) la[(int64_t)(t0 + t) * C + c] = gla_log_sigmoid(z[t] + bc) * inv_tau;
 }
 
+template <bool GATED>
 __global__ void __launch_bounds__(GLA_THREADS)
 gla_scan_kernel(const float* __restrict__ proj, int64_t ld, int off_q, int off_k, int off_v, const float* __restrict__ la,
                 float* __restrict__ S_state, const int* __restrict__ cu_seqlens, const int* __restrict__ context_lens,
-                const int* __restrict__ state_slots, float* __restrict__ o, int H, int D, int V, float q_scale) {
+                const int* __restrict__ state_slots, float* __restrict__ o, int H, int D, int V, float q_scale, ForgetGate fg) {
   extern __shared__ __align__(16) float smem[];
   float* S = smem;                              // [D][GLA_VB + 1]
   float* q_s = S + D * (GLA_VB + 1);            // [D]
@@ -73,12 +95,22 @@ gla_scan_kernel(const float* __restrict__ proj, int64_t ld, int off_q, int off_k
   for (int d = dy; d < D; d += GLA_DY) S[d * (GLA_VB + 1) + vc] = (fresh || !v_ok) ? 0.f : Sg[(int64_t)d * V + v0 + vc];
   for (int i = 0; i < n_tok; ++i) {
     const float* row = proj + (int64_t)(tok0 + i) * ld;
-    const float* lar = la + (int64_t)(tok0 + i) * H * D + hd * D;
+    const float* lar = GATED ? nullptr : la + (int64_t)(tok0 + i) * H * D + hd * D;
     __syncthreads();                            // the token before is done with q_s, k_s, a_s, parts
     for (int d = tid; d < D; d += GLA_THREADS) {
-      q_s[d] = row[off_q + hd * D + d] * q_scale;
-      k_s[d] = row[off_k + hd * D + d];
-      a_s[d] = expf(lar[d]);
+      const float qv = row[off_q + hd * D + d];
+      if constexpr (GATED) {
+        const int c = hd * D + d;
+        float k, log_a;
+        forget_gate(row[off_k + c] + fg.bias[c], fg.lower[c], k, log_a);
+        q_s[d] = gla_silu(qv) * q_scale;
+        k_s[d] = k;
+        a_s[d] = expf(log_a);
+      } else {
+        q_s[d] = qv * q_scale;
+        k_s[d] = row[off_k + hd * D + d];
+        a_s[d] = expf(lar[d]);
+      }
     }
     const float vv = v_ok ? row[off_v + hd * V + v0 + vc] : 0.f;
     __syncthreads();
@@ -116,11 +148,13 @@ constexpr float GLA_LOG2E = 1.4426950408889634f;
 
 // tiles: (request, first token of the chunk within the request's tokens of this step) pairs.  la: in, the log decays
 // [T, H*D]; out, the chunk's inclusive sums B * log2(e).  A: [T, H, GLA_LC], row t holds A[t][s] for the chunk's tokens s
-// (zero for s > t).
+// (zero for s > t).  GATED: la is no input; q and k are formed from the projection (see the top of this file) and written back
+// to it, each by the one block that holds their chunk and head.
+template <bool GATED>
 __global__ void __launch_bounds__(256)
-gla_intra_kernel(const float* __restrict__ proj, int64_t ld, int off_q, int off_k, float* __restrict__ la,
+gla_intra_kernel(typename std::conditional<GATED, float, const float>::type* proj, int64_t ld, int off_q, int off_k, float* __restrict__ la,
                  const int* __restrict__ cu_seqlens, const int* __restrict__ tiles, float* __restrict__ A, int H, int D,
-                 float q_scale) {
+                 float q_scale, ForgetGate fg) {
   extern __shared__ __align__(16) float smem[];
   constexpr int LC = GLA_LC;
   const int ldq = D + 1;
@@ -138,9 +172,24 @@ gla_intra_kernel(const float* __restrict__ proj, int64_t ld, int off_q, int off_
 #pragma unroll 4
   for (int idx = tid; idx < LC * D; idx += 256) {
     const int t = idx / D, d = idx - t * D;
-    const float* row = proj + (int64_t)(tok0 + min(t, L - 1)) * ld;
-    const float qv = row[off_q + hd * D + d] * q_scale, kv = row[off_k + hd * D + d];
-    const float bv = la[(int64_t)(tok0 + min(t, L - 1)) * H * D + hd * D + d] * GLA_LOG2E;
+    auto* row = proj + (int64_t)(tok0 + min(t, L - 1)) * ld;
+    float qv = row[off_q + hd * D + d], kv = row[off_k + hd * D + d], bv;
+    if constexpr (GATED) {
+      if (t >= L) {
+        qv = kv = bv = 0.f;
+      } else {
+        const int c = hd * D + d;
+        float log_a;
+        forget_gate(kv + fg.bias[c], fg.lower[c], kv, log_a);
+        qv = gla_silu(qv);
+        bv = log_a * GLA_LOG2E;
+        row[off_q + c] = qv;
+        row[off_k + c] = kv;
+      }
+    } else {
+      bv = la[(int64_t)(tok0 + min(t, L - 1)) * H * D + hd * D + d] * GLA_LOG2E;
+    }
+    qv *= q_scale;
     Qc[t * ldq + d] = t < L ? qv : 0.f;
     Kc[t * ldq + d] = t < L ? kv : 0.f;
     Bc[t * ldq + d] = t < L ? bv : 0.f;
@@ -425,13 +474,18 @@ static int gla_raise_smem(K kernel, size_t smem, const char* what) {
 
 ME_API int me_gla_chunk_len() { return GLA_LC; }
 
-ME_API int me_gla_scan(const float* proj, int64_t ld, int off_q, int off_k, int off_v, float* la, float* S_state,
+// gate_bias, gate_lower: [H*D] float32 or null.  With them columns off_k hold the gate's pre-activations instead of keys, la is a
+// work buffer only, and q and k are written over their columns of ``proj`` where the chunk kernels run.
+ME_API int me_gla_scan(float* proj, int64_t ld, int off_q, int off_k, int off_v, float* la, float* S_state,
                        const int* cu_seqlens, const int* context_lens, const int* state_slots, float* o, int B, int H, int D, int V,
                        float q_scale, const int* tiles, int n_tiles, int num_decodes, float* A_ws, float* states_ws,
-                       cudaStream_t stream) {
+                       const float* gate_bias, const float* gate_lower, cudaStream_t stream) {
   if (B == 0) return 0;
   ME_REQUIRE(B > 0 && H > 0 && D > 0 && V > 0, "me_gla_scan: bad sizes B=%d H=%d D=%d V=%d", B, H, D, V);
   ME_REQUIRE(H <= 65535 && num_decodes >= 0 && num_decodes <= B, "me_gla_scan: too many heads, or %d single-token requests of %d", num_decodes, B);
+  ME_REQUIRE((gate_bias == nullptr) == (gate_lower == nullptr), "me_gla_scan: a gate needs its bias and its lower bound");
+  const ForgetGate fg = {gate_bias, gate_lower};
+  const bool gated = gate_bias != nullptr;
   const int Dp = (D + 63) / 64 * 64, v_tiles = (V + GLA_VT - 1) / GLA_VT;
   const size_t smem_intra = sizeof(float) * 3 * GLA_LC * ((size_t)D + 1);
   const int Dq = (D + 3) / 4 * 4;
@@ -444,18 +498,25 @@ ME_API int me_gla_scan(const float* proj, int64_t ld, int off_q, int off_k, int 
   if (n_scan > 0) {
     const size_t smem = sizeof(float) * ((size_t)D * (GLA_VB + 1) + 3 * (size_t)D + GLA_DY * GLA_VB);
     ME_REQUIRE(smem <= 200 * 1024, "me_gla_scan: head size %d is too large", D);
-    if (gla_raise_smem(gla_scan_kernel, smem, "me_gla_scan")) return 1;
-    me_launch(gla_scan_kernel, dim3(n_scan, H, (V + GLA_VB - 1) / GLA_VB), dim3(GLA_THREADS), smem, stream, proj, ld, off_q, off_k, off_v,
-              (const float*)la, S_state, cu_seqlens, context_lens, state_slots, o, H, D, V, q_scale);
+    auto scan = gated ? gla_scan_kernel<true> : gla_scan_kernel<false>;
+    if (gla_raise_smem(scan, smem, "me_gla_scan")) return 1;
+    me_launch(scan, dim3(n_scan, H, (V + GLA_VB - 1) / GLA_VB), dim3(GLA_THREADS), smem, stream, (const float*)proj, ld, off_q, off_k, off_v,
+              (const float*)la, S_state, cu_seqlens, context_lens, state_slots, o, H, D, V, q_scale, fg);
     ME_LAUNCH_CHECK("me_gla_scan");
   }
   if (chunks) {
-    if (gla_raise_smem(gla_intra_kernel, smem_intra, "me_gla_scan (intra)")) return 1;
-    me_launch(gla_intra_kernel, dim3(n_tiles, H), dim3(256), smem_intra, stream, proj, ld, off_q, off_k, la, cu_seqlens, tiles, A_ws, H,
-              D, q_scale);
+    if (gated) {
+      if (gla_raise_smem(gla_intra_kernel<true>, smem_intra, "me_gla_scan (intra)")) return 1;
+      me_launch(gla_intra_kernel<true>, dim3(n_tiles, H), dim3(256), smem_intra, stream, proj, ld, off_q, off_k, la, cu_seqlens, tiles,
+                A_ws, H, D, q_scale, fg);
+    } else {
+      if (gla_raise_smem(gla_intra_kernel<false>, smem_intra, "me_gla_scan (intra)")) return 1;
+      me_launch(gla_intra_kernel<false>, dim3(n_tiles, H), dim3(256), smem_intra, stream, (const float*)proj, ld, off_q, off_k, la, cu_seqlens,
+                tiles, A_ws, H, D, q_scale, fg);
+    }
     ME_LAUNCH_CHECK("me_gla_scan (intra)");
     if (gla_raise_smem(gla_chunk_state_kernel, smem_state, "me_gla_scan (chunk states)")) return 1;
-    me_launch(gla_chunk_state_kernel, dim3(n_tiles, H, v_tiles), dim3(256), smem_state, stream, proj, ld, off_k, off_v, (const float*)la,
+    me_launch(gla_chunk_state_kernel, dim3(n_tiles, H, v_tiles), dim3(256), smem_state, stream, (const float*)proj, ld, off_k, off_v, (const float*)la,
               cu_seqlens, tiles, states_ws, H, D, V);
     ME_LAUNCH_CHECK("me_gla_scan (chunk states)");
     const bool walk4 = V % 4 == 0 && ((uintptr_t)states_ws % 16) == 0 && ((uintptr_t)S_state % 16) == 0;
@@ -469,7 +530,7 @@ ME_API int me_gla_scan(const float* proj, int64_t ld, int off_q, int off_k, int 
                 context_lens, state_slots, tiles, n_tiles, num_decodes, H, D, V);
     ME_LAUNCH_CHECK("me_gla_scan (state walk)");
     if (gla_raise_smem(gla_chunk_out_kernel, smem_out, "me_gla_scan (chunk outputs)")) return 1;
-    me_launch(gla_chunk_out_kernel, dim3(n_tiles, H, v_tiles), dim3(256), smem_out, stream, proj, ld, off_q, off_v, (const float*)la,
+    me_launch(gla_chunk_out_kernel, dim3(n_tiles, H, v_tiles), dim3(256), smem_out, stream, (const float*)proj, ld, off_q, off_v, (const float*)la,
               (const float*)A_ws, (const float*)states_ws, cu_seqlens, tiles, o, H, D, V, q_scale);
     ME_LAUNCH_CHECK("me_gla_scan (chunk outputs)");
   }

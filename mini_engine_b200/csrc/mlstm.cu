@@ -283,11 +283,12 @@ mlstm_chunk_kernel(const float* __restrict__ proj, int64_t ld, int off_q, int of
 }
 
 // out[t, h*V + v] = o / sqrt(mean_v(o^2) + eps) * w[h*V + v] * sigmoid(g[t, h*V + v]); one warp a head.  ``w_shared``: the
-// weight has V values that all heads share (w[v]); ``gate_silu``: the gate is g * sigmoid(g) instead of sigmoid(g).
+// weight has V values that all heads share (w[v]); ``gate_mode`` 1: the gate is g * sigmoid(g) instead of sigmoid(g), 2: none.
+// Rows of ``out`` lie out_ld elements apart.
 template <typename TO>
 __global__ void __launch_bounds__(128)
 mlstm_out_kernel(const float* __restrict__ o, const float* __restrict__ proj, int64_t ld, int off_g,
-                 const float* __restrict__ w, float eps, TO* __restrict__ out, int H, int V, int w_shared, int gate_silu) {
+                 const float* __restrict__ w, float eps, TO* __restrict__ out, int64_t out_ld, int H, int V, int w_shared, int gate_mode) {
   pdl_wait();
   pdl_launch_dependents();
   const int t = blockIdx.x, lane = threadIdx.x & 31, warp = threadIdx.x >> 5, nw = blockDim.x >> 5;
@@ -297,9 +298,12 @@ mlstm_out_kernel(const float* __restrict__ o, const float* __restrict__ proj, in
     for (int v = lane; v < V; v += 32) ss = fmaf(oo[v], oo[v], ss);
     const float r = 1.0f / sqrtf(warp_sum(ss) / (float)V + eps);
     for (int v = lane; v < V; v += 32) {
-      const float g = proj[(int64_t)t * ld + off_g + hd * V + v];
-      const float gate = (gate_silu ? g : 1.0f) / (1.0f + expf(-g));
-      out[((int64_t)t * H + hd) * V + v] = from_f<TO>(oo[v] * r * w[w_shared ? v : hd * V + v] * gate);
+      float gate = 1.0f;
+      if (gate_mode != 2) {
+        const float g = proj[(int64_t)t * ld + off_g + hd * V + v];
+        gate = (gate_mode ? g : 1.0f) / (1.0f + expf(-g));
+      }
+      out[(int64_t)t * out_ld + hd * V + v] = from_f<TO>(oo[v] * r * w[w_shared ? v : hd * V + v] * gate);
     }
   }
 }
@@ -349,11 +353,12 @@ ME_API int me_mlstm_scan(const float* proj, int64_t ld, int off_q, int off_k, in
 }
 
 ME_API int me_mlstm_out(const float* o, const float* proj, int64_t ld, int off_g, const float* w, float eps, void* out,
-                        int out_dtype, int T, int H, int V, int w_shared, int gate_silu, cudaStream_t stream) {
+                        int out_dtype, int64_t out_ld, int T, int H, int V, int w_shared, int gate_mode, cudaStream_t stream) {
   if (T == 0) return 0;
-  ME_REQUIRE(T > 0 && H > 0 && V > 0, "me_mlstm_out: bad sizes T=%d H=%d V=%d", T, H, V);
+  ME_REQUIRE(T > 0 && H > 0 && V > 0 && out_ld >= (int64_t)H * V, "me_mlstm_out: bad sizes T=%d H=%d V=%d", T, H, V);
+  ME_REQUIRE(gate_mode >= 0 && gate_mode <= 2 && (gate_mode == 2 || proj), "me_mlstm_out: gate mode %d", gate_mode);
   ME_DISPATCH_DTYPE(out_dtype, TO, me_launch(mlstm_out_kernel<TO>, dim3(T), dim3(128), 0, stream, o, proj, ld, off_g, w, eps,
-                                             (TO*)out, H, V, w_shared, gate_silu));
+                                             (TO*)out, out_ld, H, V, w_shared, gate_mode));
   ME_LAUNCH_CHECK("me_mlstm_out");
   return 0;
 }

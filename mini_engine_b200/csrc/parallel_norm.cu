@@ -1,8 +1,9 @@
 // The norm kernel of blocks whose mixer and feed-forward read the same residual stream (parallel sub-layers), with
 // layer norms that have a weight and a bias:
 //
-//   x <- x + ya + yb + va + vb          (ya, yb: the outputs of the block before, [T, W]; va, vb: vectors of W values,
-//                                        e.g. a projection's bias or what a pass over looped layers adds; each may be absent)
+//   x <- x + ya + yb + va + vb + e      (ya, yb: the outputs of the block before, [T, W]; va, vb: vectors of W values,
+//                                        e.g. a projection's bias or what a pass over looped layers adds; e: the token's
+//                                        row of the embedding table times a scale; each may be absent)
 //   out1 = (x - mean) / sqrt(var + eps) * w1 + b1        (the norm in front of the mixer)
 //   out2 = (x - mean) / sqrt(var + eps) * w2 + b2        (the norm in front of the feed-forward; may be absent)
 //
@@ -31,6 +32,23 @@ __device__ __forceinline__ void pn_store4(bf16* p, const float (&v)[4]) {
   *reinterpret_cast<uint2*>(p) = t;
 }
 
+// The embedding's row of token t, added by a kernel that looks it up itself (a looped model joins the embedding to the stream
+// again in front of a pass): ids as the embedding kernel takes them (~j stands for feedback[j]; ids outside the vocabulary,
+// which that kernel has flagged, add nothing).
+struct TokenRows {
+  const int* ids;             // null: none
+  const void* table;
+  int dtype, V;
+  const int* feedback;
+  int n_feedback;
+  float scale;
+};
+__device__ __forceinline__ int pn_token(const TokenRows& e, int r) {
+  int id = e.ids[r];
+  if (id < 0 && e.feedback != nullptr && ~id < e.n_feedback) id = e.feedback[~id];
+  return id >= 0 && id < e.V ? id : -1;
+}
+
 // VEC = 4: W is a multiple of four and every pointer is 16-byte aligned (8 for bfloat16); a thread takes four neighbours a
 // turn, so all loads of a row are in flight at once.  VEC = 1: any W.  The sums of a row are taken in the same order by every
 // launch of one VEC, and the host chooses VEC from W and the pointers alone.
@@ -39,14 +57,15 @@ __global__ void __launch_bounds__(256)
 parallel_norm_kernel(float* __restrict__ x, const TY* __restrict__ ya, const TY* __restrict__ yb, const float* __restrict__ va,
                      const float* __restrict__ vb, const float* __restrict__ w1, const float* __restrict__ b1,
                      TO* __restrict__ out1, const float* __restrict__ w2, const float* __restrict__ b2, TO* __restrict__ out2,
-                     const int* __restrict__ rows, int W, float eps) {
+                     const int* __restrict__ rows, int W, float eps, TokenRows emb) {
   extern __shared__ __align__(16) float row[];
   __shared__ float red[32];
   pdl_wait();
   pdl_launch_dependents();
   const int r = rows ? rows[blockIdx.x] : blockIdx.x;
   float* xr = x + (int64_t)r * W;
-  const bool changed = ya || yb || va || vb;
+  const int tok = emb.ids ? pn_token(emb, r) : -1;
+  const bool changed = ya || yb || va || vb || tok >= 0;
   float s = 0.f;
   if constexpr (VEC == 4) {
     for (int i = 4 * threadIdx.x; i < W; i += 4 * blockDim.x) {
@@ -56,6 +75,11 @@ parallel_norm_kernel(float* __restrict__ x, const TY* __restrict__ ya, const TY*
       if (yb) { pn_load4(yb + (int64_t)r * W + i, t); for (int j = 0; j < 4; ++j) v[j] += t[j]; }
       if (va) { pn_load4(va + i, t); for (int j = 0; j < 4; ++j) v[j] += t[j]; }
       if (vb) { pn_load4(vb + i, t); for (int j = 0; j < 4; ++j) v[j] += t[j]; }
+      if (tok >= 0) {
+        if (emb.dtype == ME_BF16) pn_load4(reinterpret_cast<const bf16*>(emb.table) + (int64_t)tok * W + i, t);
+        else pn_load4(reinterpret_cast<const float*>(emb.table) + (int64_t)tok * W + i, t);
+        for (int j = 0; j < 4; ++j) v[j] = fmaf(t[j], emb.scale, v[j]);
+      }
       if (changed && !rows) pn_store4(xr + i, v);
       pn_store4(row + i, v);
       s += (v[0] + v[1]) + (v[2] + v[3]);
@@ -67,6 +91,9 @@ parallel_norm_kernel(float* __restrict__ x, const TY* __restrict__ ya, const TY*
       if (yb) v += to_f<TY>(yb[(int64_t)r * W + i]);
       if (va) v += va[i];
       if (vb) v += vb[i];
+      if (tok >= 0)
+        v = fmaf(emb.dtype == ME_BF16 ? to_f<bf16>(reinterpret_cast<const bf16*>(emb.table)[(int64_t)tok * W + i])
+                                      : reinterpret_cast<const float*>(emb.table)[(int64_t)tok * W + i], emb.scale, v);
       if (changed && !rows) xr[i] = v;
       row[i] = v;
       s += v;
@@ -112,17 +139,21 @@ parallel_norm_kernel(float* __restrict__ x, const TY* __restrict__ ya, const TY*
 
 // x: [T, W] float32.  ya, yb: [T, W] of y_dtype or null.  va, vb: [W] float32 or null.  w1, b1 (w2, b2): [W] float32, a bias
 // may be null.  out1, out2: [n, W] of out_dtype; out2 may be null.  rows: [n] int32 or null (then n == T).
+// emb_ids: [T] int32 or null; emb_table: [emb_V, W] of emb_dtype.
 ME_API int me_parallel_norm(float* x, const void* ya, const void* yb, int y_dtype, const float* va, const float* vb, const float* w1,
                             const float* b1, void* out1, const float* w2, const float* b2, void* out2, int out_dtype,
-                            const int* rows, int n, int W, float eps, cudaStream_t stream) {
+                            const int* rows, int n, int W, float eps, const int* emb_ids, const void* emb_table, int emb_dtype,
+                            int emb_V, const int* emb_feedback, int emb_n_feedback, float emb_scale, cudaStream_t stream) {
   if (n == 0) return 0;
   ME_REQUIRE(n > 0 && W > 0 && W <= 24576, "me_parallel_norm: bad sizes n=%d W=%d", n, W);
   ME_REQUIRE((!out1 || w1) && (!out2 || w2), "me_parallel_norm: a norm needs its weight");
+  ME_REQUIRE(!emb_ids || (emb_table && emb_V > 0 && (emb_dtype == ME_F32 || emb_dtype == ME_BF16)), "me_parallel_norm: the embedding needs its table");
+  const TokenRows emb = {emb_ids, emb_table, emb_dtype, emb_V, emb_feedback, emb_n_feedback, emb_scale};
   auto misaligned = [](const void* p, size_t to) { return p && ((uintptr_t)p % to) != 0; };
   const size_t y_al = y_dtype == ME_F32 ? 16 : 8, o_al = out_dtype == ME_F32 ? 16 : 8;
   const bool vec = W % 4 == 0 && !misaligned(x, 16) && !misaligned(ya, y_al) && !misaligned(yb, y_al) && !misaligned(va, 16) &&
                    !misaligned(vb, 16) && !misaligned(w1, 16) && !misaligned(b1, 16) && !misaligned(w2, 16) && !misaligned(b2, 16) &&
-                   !misaligned(out1, o_al) && !misaligned(out2, o_al);
+                   !misaligned(out1, o_al) && !misaligned(out2, o_al) && (!emb_ids || !misaligned(emb_table, emb_dtype == ME_F32 ? 16 : 8));
   const int per = vec ? 4 : 1;
   const int threads = W >= 256 * per ? 256 : (W >= 128 * per ? 128 : 64);
   const size_t smem = sizeof(float) * W;
@@ -135,7 +166,7 @@ ME_API int me_parallel_norm(float* x, const void* ya, const void* yb, int y_dtyp
       attr_set = true;                                                                                                          \
     }                                                                                                                           \
     me_launch(parallel_norm_kernel<TY, TO, VEC>, dim3(n), dim3(threads), smem, stream, x, (const TY*)ya, (const TY*)yb, va, vb, w1, b1, \
-              (TO*)out1, w2, b2, (TO*)out2, rows, W, eps);                                                                      \
+              (TO*)out1, w2, b2, (TO*)out2, rows, W, eps, emb);                                                                    \
   } while (0)
   ME_DISPATCH_DTYPE((ya || yb) ? y_dtype : ME_F32, TY, ME_DISPATCH_DTYPE(out_dtype, TO, {
     if (vec) PN_LAUNCH(4);

@@ -20,6 +20,8 @@
 // window, the rows of the blocks that lie wholly in front of the window, (b + 1) P <= p - w + 1, in the same softmax.  The
 // pooled rows are visited first, in tiles counted from block 0.
 //
+// A distance bias (``r1``, ``r2``: two numbers a head): r1 ln(1 + r2 (p - j)) is taken off the scaled score of key j.
+//
 // One block = 16 queries of one request x one query head; 128 threads; thread (r, c) owns row r = tid / 8, keys
 // c, c+8, c+16, c+24 of a tile and output elements c, c+8, ...
 #include "common.cuh"
@@ -33,7 +35,8 @@ sink_attn_kernel(const T* __restrict__ q, int64_t q_stride, const float* __restr
                  int bt_stride, const int* __restrict__ cu_seqlens, const int* __restrict__ context_lens,
                  const int* __restrict__ tiles, int nh, int nkv, int D, int Dv, int HD, int page_size, float scale, int window,
                  int sink, const float* __restrict__ sinks, float softcap, int keep_first, int chunk,
-                 const T* __restrict__ pooled, const int* __restrict__ pooled_tables, int pbt_stride, int pool_p) {
+                 const T* __restrict__ pooled, const int* __restrict__ pooled_tables, int pbt_stride, int pool_p,
+                 const float* __restrict__ r1, const float* __restrict__ r2) {
   extern __shared__ float smem[];
   pdl_wait();
   pdl_launch_dependents();
@@ -66,6 +69,7 @@ sink_attn_kernel(const T* __restrict__ q, int64_t q_stride, const float* __restr
   const int keep_hi = (window > 0 && keep_first > 0) ? min(lo, (min(keep_first, hi) + SA_BK - 1) / SA_BK * SA_BK) : 0;
 
   float m = sinks ? sinks[head] : (sink ? 0.f : -INFINITY), l = (sinks || sink) ? 1.f : 0.f;
+  const float bias_a = r1 ? r1[head] : 0.f, bias_b = r1 ? r2[head] : 0.f;
   float acc[SA_MAX / 8];
 #pragma unroll
   for (int k = 0; k < SA_MAX / 8; ++k) acc[k] = 0.f;
@@ -109,6 +113,7 @@ sink_attn_kernel(const T* __restrict__ q, int64_t q_stride, const float* __restr
       const bool seen = blocks ? (row_ok && j < nb_r) : (row_ok && j <= p_r && j < L && in_mask);
       dot *= scale;
       if (softcap > 0.f) dot = softcap * tanhf(dot / softcap);
+      if (r1 && seen) dot -= bias_a * log1pf(bias_b * (float)(p_r - j));
       s[mm] = seen ? dot : -INFINITY;
       tmax = fmaxf(tmax, s[mm]);
     }
@@ -167,17 +172,19 @@ ME_API int me_sink_attn_tile_q() { return SA_BQ; }
 // tiles: [num_tiles, 2] (request, first local query) for requests that bring several tokens; the first num_decodes
 // requests bring one token each and get one block per head.  sinks: [nh] float32 or null; softcap, keep_first, chunk: 0 = none.
 // pooled, pooled_tables: the cache of pooled blocks (same layout and dtype) and its block tables, with pool_p tokens a block; null and 0: none.
+// r1, r2: float32 [nh], both or neither.
 ME_API int me_sink_attn(const void* q, int dtype, int64_t q_stride, const float* gate, int64_t gate_stride, void* out,
                         int64_t out_stride, const void* pool, const int* block_tables, int bt_stride, const int* cu_seqlens,
                         const int* context_lens, const int* tiles, int num_tiles, int num_decodes, int nh, int nkv, int D, int Dv,
                         int HD, int page_size, float scale, int window, int sink, const float* sinks, float softcap,
                         int keep_first, int chunk, const void* pooled, const int* pooled_tables, int pbt_stride, int pool_p,
-                        cudaStream_t stream) {
+                        const float* r1, const float* r2, cudaStream_t stream) {
   ME_REQUIRE(D >= 1 && D <= SA_MAX && Dv >= 1 && Dv <= SA_MAX, "me_sink_attn: key size %d / value size %d beyond %d", D, Dv, SA_MAX);
   ME_REQUIRE(HD >= D && HD >= Dv, "me_sink_attn: cache rows of %d elements are too short", HD);
   ME_REQUIRE(nh > 0 && nkv > 0 && nh % nkv == 0 && nh <= 65535, "me_sink_attn: %d heads, %d kv heads", nh, nkv);
   ME_REQUIRE(pool_p == 0 || (pool_p > 0 && pooled && pooled_tables && window > 0 && chunk == 0 && keep_first == 0),
              "me_sink_attn: pooled blocks of %d tokens need their cache and a plain window", pool_p);
+  ME_REQUIRE((r1 == nullptr) == (r2 == nullptr) && !(r1 && (softcap > 0.f || pool_p > 0)), "me_sink_attn: a distance bias has two numbers a head and goes without caps and pooled blocks");
   const size_t smem = sizeof(float) * ((size_t)(SA_BQ + SA_BK) * (D + 1) + (size_t)SA_BK * (Dv + 1) + SA_BQ * (SA_BK + 1));
   ME_DISPATCH_DTYPE(dtype, T, {
     static bool attr_set = false;
@@ -189,11 +196,11 @@ ME_API int me_sink_attn(const void* q, int dtype, int64_t q_stride, const float*
     if (num_decodes > 0)
       me_launch(sink_attn_kernel<T>, dim3(num_decodes, nh), dim3(SA_THREADS), smem, stream, (const T*)q, q_stride, gate, gate_stride,
                 (T*)out, out_stride, (const T*)pool, block_tables, bt_stride, cu_seqlens, context_lens, (const int*)nullptr, nh, nkv,
-                D, Dv, HD, page_size, scale, window, sink, sinks, softcap, keep_first, chunk, (const T*)pooled, pooled_tables, pbt_stride, pool_p);
+                D, Dv, HD, page_size, scale, window, sink, sinks, softcap, keep_first, chunk, (const T*)pooled, pooled_tables, pbt_stride, pool_p, r1, r2);
     if (num_tiles > 0)
       me_launch(sink_attn_kernel<T>, dim3(num_tiles, nh), dim3(SA_THREADS), smem, stream, (const T*)q, q_stride, gate, gate_stride,
                 (T*)out, out_stride, (const T*)pool, block_tables, bt_stride, cu_seqlens, context_lens, tiles, nh, nkv, D, Dv,
-                HD, page_size, scale, window, sink, sinks, softcap, keep_first, chunk, (const T*)pooled, pooled_tables, pbt_stride, pool_p);
+                HD, page_size, scale, window, sink, sinks, softcap, keep_first, chunk, (const T*)pooled, pooled_tables, pbt_stride, pool_p, r1, r2);
   });
   ME_LAUNCH_CHECK("me_sink_attn");
   return 0;

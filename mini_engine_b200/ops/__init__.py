@@ -27,7 +27,7 @@ _PROTOS = {
     "me_short_conv": [_P, _P, _P, _P, _P, _P, _P, _P, _I, _I, _I, _I, _I, _I, _I, _P],
     "me_polynorm": [_P, _I, _L, _P, _F, _P, _I, _L, _I, _I, _P],
     "me_mlstm_scan": [_P, _L, _I, _I, _I, _I, _I, _P, _P, _F, _P, _P, _P, _P, _P, _P, _P, _I, _I, _I, _I, _F, _I, _P],
-    "me_mlstm_out": [_P, _P, _L, _I, _P, _F, _P, _I, _I, _I, _I, _I, _I, _P],
+    "me_mlstm_out": [_P, _P, _L, _I, _P, _F, _P, _I, _L, _I, _I, _I, _I, _I, _P],
     "me_latent_prep": [_P, _L, _I, _I, _I, _P, _F, _P, _I, _P, _P, _P, _P, _P, _P, _I, _I, _I, _I, _I, _I, _P],
     "me_latent_attention": [_P, _P, _I, _P, _P, _I, _P, _P, _P, _I, _I, _P, _P, _P, _I, _I, _I, _I, _I, _F, _I, _P],
     "me_heads_to_rows": [_P, _P, _I, _I, _I, _I, _P],
@@ -39,7 +39,7 @@ _PROTOS = {
     "me_gemm_simt": [_P, _I, _L, _P, _I, _P, _I, _L, _I, _I, _I, _I, _P],
     "me_qk_norm_rope_kv_write": [_P, _I, _L, _I, _I, _I, _I, _P, _P, _F, _P, _I, _P, _P, _P, _I, _P],
     "me_attn_chunk": [_P, _I, _L, _P, _L, _P, _P, _I, _P, _P, _P, _I, _I, _I, _I, _I, _F, _I, _P],
-    "me_attn_decode": [_P, _I, _L, _P, _L, _P, _P, _I, _P, _P, _I, _I, _I, _I, _I, _F, _I, _P, _P, _P, _I, _P, _I, _P, _I, _P, _L, _I, _I, _F, _P, _P, _P, _I, _I, _I, _P],
+    "me_attn_decode": [_P, _I, _L, _P, _L, _P, _P, _I, _P, _P, _I, _I, _I, _I, _I, _F, _I, _P, _P, _P, _I, _P, _I, _P, _I, _P, _L, _I, _I, _F, _P, _P, _P, _I, _I, _I, _P, _P, _I, _I, _F, _F, _F, _P],
     "me_attn_decode_fused": [_P, _L, _P, _L, _P, _P, _P, _I, _P, _P, _I, _I, _I, _I, _I, _F, _I, _P, _P, _F, _P, _P, _P, _P, _P,
                              _I, _I, _I, _P, _P],
     "me_gemm_decode": [_I, _P, _L, _P, _I, _F, _P, _P, _I, _L, _P, _P, _P, _P, _I, _I, _I, _P, ctypes.c_uint64, _F, _F, _F, _P],
@@ -47,7 +47,7 @@ _PROTOS = {
     "me_gemm_tcgen05": [_P, _P, _P, _I, _L, _I, _I, _I, _I, _I, _I, _L, _F, _F, _F, _P, _P],
     "me_gemm_tcgen05_persistent": [_P, _P, _P, _I, _L, _I, _I, _I, _I, _I, _F, _F, _F, _P, _P],
     "me_gemm_tcgen05_shared": [_P, _P, _P, _I, _L, _I, _I, _I, _I, _I, _P, _P, _P, _P],
-    "me_attn_prefill_tcgen05": [_P, _P, _P, _L, _P, _I, _P, _P, _P, _I, _I, _I, _I, _I, _F, _I, _I, _I, _P, _L, _P, _I, _I, _F, _P, _P, _P, _I, _I, _P],
+    "me_attn_prefill_tcgen05": [_P, _P, _P, _L, _P, _I, _P, _P, _P, _I, _I, _I, _I, _I, _F, _I, _I, _I, _P, _L, _P, _I, _I, _F, _P, _P, _P, _I, _I, _P, _P, _I, _P],
     "me_tma_encode_2d": [_P, _P, ctypes.c_uint64, ctypes.c_uint64, ctypes.c_uint64, ctypes.c_uint32, ctypes.c_uint32, _I],
     "me_attn_prefill": [_P, _L, _P, _L, _P, _P, _I, _P, _P, _P, _I, _I, _I, _I, _I, _F, _I, _P],
     "me_sample": [_P, _L, _P, _P, _P, _P, _I, _I, _P, _P, _P],
@@ -56,11 +56,12 @@ _PROTOS = {
     "me_clamped_glu": [_P, _I, _L, _P, _I, _L, _I, _I, _F, _F, _F, _P],
     "me_conv_rope_kv": [_P, _L, _P, _P, _P, _I, _P, _I, _P, _P, _P, _P, _P, _P, _P, _P, _I, _I, _I, _I, _I, _I, _I, _I, _I, _I, _I, _P, _P],
     "me_rope_table": [_P, _P, _I, _I, _P, _P],
-    "me_sink_attn": [_P, _I, _L, _P, _L, _P, _L, _P, _P, _I, _P, _P, _P, _I, _I, _I, _I, _I, _I, _I, _I, _F, _I, _I, _P, _F, _I, _I, _P, _P, _I, _I, _P],
-    "me_parallel_norm": [_P, _P, _P, _I, _P, _P, _P, _P, _P, _P, _P, _P, _I, _P, _I, _I, _F, _P],
-    "me_attn_prep": [_P, _L, _P, _P, _P, _I, _F, _P, _I, _P, _P, _P, _P, _I, _I, _I, _I, _I, _I, _I, _I, _P, _I, _P],
+    "me_sink_attn": [_P, _I, _L, _P, _L, _P, _L, _P, _P, _I, _P, _P, _P, _I, _I, _I, _I, _I, _I, _I, _I, _F, _I, _I, _P, _F, _I, _I, _P, _P, _I, _I, _P, _P, _P],
+    "me_parallel_norm": [_P, _P, _P, _I, _P, _P, _P, _P, _P, _P, _P, _P, _I, _P, _I, _I, _F, _P, _P, _I, _I, _P, _I, _F, _P],
+    "me_attn_prep": [_P, _L, _P, _P, _P, _I, _F, _P, _I, _P, _P, _P, _P, _I, _P, _I, _I, _I, _I, _I, _I, _I, _I, _I, _P, _I, _F, _F, _F, _P],
+    "me_diff_combine": [_P, _I, _L, _P, _I, _L, _I, _I, _I, _I, _F, _F, _F, _P],
     "me_gla_decay": [_P, _L, _I, _I, _P, _I, _P, _F, _P, _I, _I, _P],
-    "me_gla_scan": [_P, _L, _I, _I, _I, _P, _P, _P, _P, _P, _P, _I, _I, _I, _I, _F, _P, _I, _I, _P, _P, _P],
+    "me_gla_scan": [_P, _L, _I, _I, _I, _P, _P, _P, _P, _P, _P, _I, _I, _I, _I, _F, _P, _I, _I, _P, _P, _P, _P, _P],
     "me_activation": [_P, _I, _L, _P, _I, _L, _I, _I, _I, _P],
     "me_soft_cap": [_P, _L, _F, _F, _P],
     "me_add_row_vector": [_P, _I, _I, _I, _P, _P],
@@ -849,14 +850,17 @@ def prefill_tcgen05_heads_per_block(num_heads: int, num_kv_heads: int, head_dim:
 def attention_prefill_tcgen05(qkv, out, num_heads, num_kv_heads, head_dim, pool, page_size, block_tables, meta,
                               scale, window, tiles=None, num_tiles=None, key_tile: int = 0, sink: bool = False,
                               gate: Optional[torch.Tensor] = None, keep_first: int = 0, chunk: int = 0, softcap: float = 0.0,
-                              sinks: Optional[torch.Tensor] = None, pooled: Optional[tuple] = None) -> None:
+                              sinks: Optional[torch.Tensor] = None, pooled: Optional[tuple] = None, bias: Optional[tuple] = None,
+                              out_dim: int = 0) -> None:
     """The tcgen05 / tensor-memory prefill kernel (bfloat16, head_dim 64 or 128, page sizes dividing 128) over
     tiles of 128 / heads-per-block tokens; Q, K and V arrive by tensor-map loads.  ``sink``: one more term, exp(0), in
     the softmax's denominator; ``gate``: float32 rows of pre-activations whose sigmoid multiplies the output.
     ``keep_first``: the window also shows the keys j < keep_first; ``chunk`` (instead of a window): the keys of the query's
     own chunk; ``softcap`` c: scores become c tanh(s / c) after the scale; ``sinks`` (float32 [heads]): the extra term is
     exp(sinks[head]); ``pooled`` = (cache, block tables, P): the blocks of P tokens in front of the window, one row each in a
-    second cache of the same layout (the kernel with the key tile of 128 only)."""
+    second cache of the same layout; ``bias`` = (r1, r2), float32 [heads] each: r1 ln(1 + r2 (p - j)) is taken off the scaled score
+    of a key at distance p - j; ``out_dim`` (0: all): how many elements of every head leave, ``out`` then holds
+    heads * out_dim columns (all of these in the kernel with the key tile of 128 only)."""
     gp = prefill_tcgen05_heads_per_block(num_heads, num_kv_heads, head_dim, page_size)
     _need(gp > 0 and qkv.dtype == torch.bfloat16 and qkv.is_contiguous() and qkv.data_ptr() % 16 == 0,
           "attention_prefill_tcgen05: shape or dtype not taken by the kernel")
@@ -869,7 +873,8 @@ def attention_prefill_tcgen05(qkv, out, num_heads, num_kv_heads, head_dim, pool,
           float(scale), int(window or 0), key_tile, 1 if sink else 0, _ptr(gate), gate.stride(0) if gate is not None else 0,
           meta.error_flag.data_ptr(), int(keep_first or 0), int(chunk or 0), float(softcap or 0.0), _ptr(sinks),
           kv_tensor_map(pooled[0], page_size).ptr if pooled else 0, pooled[1].data_ptr() if pooled else 0,
-          pooled[1].stride(0) if pooled else 0, int(pooled[2]) if pooled else 0, _stream())
+          pooled[1].stride(0) if pooled else 0, int(pooled[2]) if pooled else 0, _ptr(bias[0]) if bias else 0, _ptr(bias[1]) if bias else 0,
+          int(out_dim), _stream())
 
 
 use_tcgen05_attention = True   # False: portions of prompts use the mma.sync kernel instead (a switch for comparisons)
@@ -878,11 +883,13 @@ use_tcgen05_attention = True   # False: portions of prompts use the mma.sync ker
 def attention_decode(qkv, out, num_heads, num_kv_heads, head_dim, pool, page_size, block_tables, meta,
                      scale, window, kind: str = "auto", sink: bool = False, gate: Optional[torch.Tensor] = None,
                      keep_first: int = 0, chunk: int = 0, softcap: float = 0.0, sinks: Optional[torch.Tensor] = None,
-                     pooled: Optional[tuple] = None) -> None:
+                     pooled: Optional[tuple] = None, bias: Optional[tuple] = None, out_dim: int = 0,
+                     pairs: Optional[tuple[float, float, float]] = None) -> None:
     """The split-K decode kernel and its merge over requests [0, meta.num_decodes).  ``sink``: one more term, exp(0), in
     the softmax's denominator (added once, in the merge); ``gate``: float32 rows of pre-activations whose sigmoid
     multiplies the output.  ``sinks`` (float32 [heads]): the term is exp(sinks[head]).  ``keep_first``, ``chunk`` and
-    ``softcap`` as for ``attention_prefill_tcgen05`` (the partition kernel fed by tensor-map loads only).
+    ``softcap``, ``bias`` and ``out_dim`` as for ``attention_prefill_tcgen05`` (the partition kernel fed by tensor-map loads only).
+    ``pairs`` = (lambda, gain, eps): the merge joins heads 2h and 2h + 1 as ``diff_combine`` does and ``out`` holds half as many heads.
 
     ``kind`` picks the partition kernel: "auto" (for bfloat16 with head_dim 64 or 128 the tensor cores, fed by
     tensor-map loads where the page size divides 128, else by cp.async; otherwise the CUDA cores), or one
@@ -906,7 +913,8 @@ def attention_decode(qkv, out, num_heads, num_kv_heads, head_dim, pool, page_siz
           _ptr(meta.error_flag), DECODE_KINDS[kind], tm.ptr if tm is not None else 0, 1 if sink else 0, _ptr(gate),
           gate.stride(0) if gate is not None else 0, int(keep_first or 0), int(chunk or 0), float(softcap or 0.0), _ptr(sinks),
           kv_tensor_map(pooled[0], page_size).ptr if pooled else 0, pooled[1].data_ptr() if pooled else 0,
-          pooled[1].stride(0) if pooled else 0, int(pooled[2]) if pooled else 0, pool_parts, _stream())
+          pooled[1].stride(0) if pooled else 0, int(pooled[2]) if pooled else 0, pool_parts, _ptr(bias[0]) if bias else 0,
+          _ptr(bias[1]) if bias else 0, int(out_dim), 1 if pairs else 0, *(float(v) for v in (pairs or (0.0, 0.0, 0.0))), _stream())
     global launches
     launches += 2 if pooled else 1          # partition kernel(s) + merge kernel
 
@@ -1133,16 +1141,17 @@ def mlstm_scan(proj: torch.Tensor, offsets: dict, bias_i: torch.Tensor, bias_f: 
 
 
 def mlstm_out(o: torch.Tensor, proj: torch.Tensor, off_g: int, weight: torch.Tensor, eps: float, out: torch.Tensor,
-              num_heads: int, vdim: int, shared_weight: bool = False, gate: str = "sigmoid") -> None:
+              num_heads: int, vdim: int, shared_weight: bool = False, gate: Optional[str] = "sigmoid") -> None:
     """Each head's ``o`` divided by its root mean square, times ``weight`` and the sigmoid of the gate columns of ``proj``.
-    ``shared_weight``: the weight has ``vdim`` values that every head uses; ``gate`` "silu": g sigmoid(g) instead of sigmoid(g)."""
+    ``shared_weight``: the weight has ``vdim`` values that every head uses; ``gate`` "silu": g sigmoid(g) instead of sigmoid(g), None: no gate.
+    ``out`` may be columns of a wider tensor."""
     T = o.shape[0]
-    _need(gate in ("sigmoid", "silu"), "mlstm_out: the gate is 'sigmoid' or 'silu'")
+    _need(gate in (None, "sigmoid", "silu"), "mlstm_out: the gate is 'sigmoid', 'silu' or None")
     _need(weight.dtype == torch.float32 and weight.numel() == (vdim if shared_weight else num_heads * vdim),
           "mlstm_out: weight must be float32 [heads * vdim] ([vdim] when the heads share it)")
-    _need(out.is_contiguous() and tuple(out.shape) == (T, num_heads * vdim), "mlstm_out: output shape")
+    _need(out.stride(1) == 1 and tuple(out.shape) == (T, num_heads * vdim), "mlstm_out: output shape")
     _call("me_mlstm_out", o.data_ptr(), proj.data_ptr(), proj.stride(0), off_g, weight.data_ptr(), float(eps), out.data_ptr(),
-          _dt(out), T, num_heads, vdim, 1 if shared_weight else 0, 1 if gate == "silu" else 0, _stream())
+          _dt(out), out.stride(0), T, num_heads, vdim, 1 if shared_weight else 0, {"sigmoid": 0, "silu": 1, None: 2}[gate], _stream())
 
 
 # ---- gated linear attention --------------------------------------------------------------------------
@@ -1166,13 +1175,19 @@ GLA_CHUNK = 64        # tokens that the chunk kernels of csrc/gla.cu take at a t
 
 def gla_scan(proj: torch.Tensor, offsets: dict, la: torch.Tensor, S: torch.Tensor, meta, state_slots: torch.Tensor, o: torch.Tensor,
              num_heads: int, dim: int, vdim: int, q_scale: float, scores: Optional[torch.Tensor] = None,
-             chunk_states: Optional[torch.Tensor] = None) -> None:
+             chunk_states: Optional[torch.Tensor] = None, gate: Optional[tuple] = None) -> None:
     """Walks every request's tokens of this step through S_t = diag(exp(la_t)) S_(t-1) + k_t v_t^T, o_t = S_t^T q_t from the
     state in its slot (see csrc/gla.cu).  ``proj`` [T, N] float32 holds q, k, v at the column ``offsets``; ``la`` [T, heads * dim]
     and ``o`` [T, heads * vdim] float32.  With the float32 workspaces ``scores`` ([T, heads, GLA_CHUNK]) and ``chunk_states``
     (heads * dim * vdim values for every run of GLA_CHUNK tokens: ``gla_chunk_count``) the requests that bring several tokens
-    take GLA_CHUNK tokens at a time, all runs of the step side by side (``gla_chunks``); ``la`` is overwritten on the way."""
+    take GLA_CHUNK tokens at a time, all runs of the step side by side (``gla_chunks``); ``la`` is overwritten on the way.
+
+    ``gate`` = (bias, lower), float32 [heads * dim] each: the recurrence whose forget gate also says what is written.  The columns
+    ``offsets["k"]`` then hold the gate's pre-activations z, and a = lower + (1 - lower) sigmoid(z + bias), k = 1 - a, q <- silu(q);
+    ``la`` is a work buffer, and the q and k columns of ``proj`` are written on the way."""
     T = proj.shape[0]
+    _need(gate is None or all(g.dtype == torch.float32 and g.is_contiguous() and g.numel() == num_heads * dim for g in gate),
+          "gla_scan: a gate's bias and lower bound are float32 [heads * dim]")
     _need(proj.dtype == torch.float32 and proj.stride(1) == 1, "gla_scan: projections must be float32 rows")
     _need(all(t.dtype == torch.float32 and t.is_contiguous() for t in (S, la, o)), "gla_scan: float32 state, decays and output")
     _need(tuple(S.shape[1:]) == (num_heads, dim, vdim) and tuple(la.shape) == (T, num_heads * dim)
@@ -1188,7 +1203,8 @@ def gla_scan(proj: torch.Tensor, offsets: dict, la: torch.Tensor, S: torch.Tenso
     _call("me_gla_scan", proj.data_ptr(), proj.stride(0), offsets["q"], offsets["k"], offsets["v"], la.data_ptr(), S.data_ptr(),
           meta.cu_seqlens.data_ptr(), meta.context_lens.data_ptr(), state_slots.data_ptr(), o.data_ptr(), meta.num_reqs,
           num_heads, dim, vdim, float(q_scale), tiles.data_ptr() if chunked else 0, n_tiles if chunked else 0, meta.num_decodes,
-          scores.data_ptr() if chunked else 0, chunk_states.data_ptr() if chunked else 0, _stream())
+          scores.data_ptr() if chunked else 0, chunk_states.data_ptr() if chunked else 0, _ptr(gate[0]) if gate else 0,
+          _ptr(gate[1]) if gate else 0, _stream())
 
 
 def gla_chunk_count(meta) -> int:
@@ -1347,10 +1363,12 @@ def sandwich_norm(residual: torch.Tensor, y: Optional[torch.Tensor], post_weight
 
 def parallel_norm(residual: torch.Tensor, adds: Sequence[torch.Tensor], vectors: Sequence[torch.Tensor], eps: float,
                   norm1: tuple, out1: torch.Tensor, norm2: Optional[tuple] = None, out2: Optional[torch.Tensor] = None,
-                  rows: Optional[torch.Tensor] = None) -> None:
+                  rows: Optional[torch.Tensor] = None, embedding: Optional[tuple] = None) -> None:
     """``residual += sum(adds) + sum(vectors)`` (float32, in place; up to two [T, W] tensors of one dtype and two float32 [W]
     vectors), then one or two layer norms of the new rows: ``out = (x - mean) / sqrt(var + eps) * weight + bias`` with
-    ``norm`` = (weight, bias or None).  With ``rows`` only those rows are computed and ``residual`` is not written."""
+    ``norm`` = (weight, bias or None).  With ``rows`` only those rows are computed and ``residual`` is not written.
+    ``embedding`` = (token ids, table, feedback or None, scale): the tokens' rows of the table times the scale join the sum (ids as
+    ``embed`` takes them)."""
     T, W = residual.shape
     adds, vectors = [a for a in adds if a is not None], [v for v in vectors if v is not None]
     _need(residual.dtype == torch.float32 and residual.is_contiguous(), "parallel_norm: the residual must be float32 [T, W]")
@@ -1366,12 +1384,17 @@ def parallel_norm(residual: torch.Tensor, adds: Sequence[torch.Tensor], vectors:
               "parallel_norm: weights and biases are float32 [W]")
         _need(out.is_contiguous() and tuple(out.shape) == (n, W) and out.dtype == out1.dtype, "parallel_norm: output shape")
     _need(rows is None or (rows.dtype == torch.int32 and rows.is_contiguous()), "parallel_norm: rows must be int32")
+    ids, table, feedback, scale = embedding if embedding is not None else (None, None, None, 1.0)
+    if embedding is not None:
+        _need(rows is None and ids.dtype == torch.int32 and ids.is_contiguous() and ids.numel() == T and table.is_contiguous()
+              and table.dim() == 2 and table.shape[1] == W, "parallel_norm: the embedding needs an int32 id a row and a table [vocabulary, W]")
     adds += [None] * (2 - len(adds))
     vectors += [None] * (2 - len(vectors))
     _call("me_parallel_norm", residual.data_ptr(), _ptr(adds[0]), _ptr(adds[1]), _dt(adds[0]) if adds[0] is not None else 0,
           _ptr(vectors[0]), _ptr(vectors[1]), norm1[0].data_ptr(), _ptr(norm1[1]), out1.data_ptr(),
           _ptr(norm2[0]) if out2 is not None else 0, _ptr(norm2[1]) if out2 is not None else 0, _ptr(out2), _dt(out1), _ptr(rows), n, W,
-          float(eps), _stream())
+          float(eps), _ptr(ids), _ptr(table), _dt(table) if table is not None else 0, table.shape[0] if table is not None else 0, _ptr(feedback),
+          feedback.numel() if feedback is not None else 0, float(scale), _stream())
 
 
 ACTIVATIONS = {"relu_squared": 0, "gelu_tanh": 1, "silu": 2, "gelu": 3}     # "gelu": the exact form, z Phi(z)
@@ -1402,33 +1425,61 @@ def attn_prep(proj: torch.Tensor, bias: Optional[torch.Tensor], q_norm: Optional
               norm: Optional[str], eps: float, freq: Optional[torch.Tensor], positions: torch.Tensor,
               slot_mapping: Optional[torch.Tensor], q_out: torch.Tensor, pool: Optional[torch.Tensor], page_size: int,
               num_heads: int, num_kv_heads: int, dim: int, vdim: int, q_scale: Optional[torch.Tensor] = None,
-              own_kv: bool = True) -> None:
+              own_kv: bool = True, maps: int = 1, angles: Optional[torch.Tensor] = None,
+              temperature: Optional[tuple[float, float]] = None, v_scale: float = 1.0) -> None:
     """From the packed float32 projections q|k|v (the leading columns of ``proj``; q alone with ``own_kv`` False): bias, a weighted RMS norm of every q and k
-    head in front of the rotation (``norm`` "before") or a plain one behind it ("after"), the rotation of element i with
-    element i + len(freq) by position x ``freq`` (float64 frequencies), queries to ``q_out`` and keys and values into the
+    head in front of the rotation (``norm`` "before"), one over the whole q and the whole k of a token ("row", with a weight for every value)
+    or a plain one behind it ("after"), the rotation of element i with
+    element i + len(freq) by position x ``freq`` (float64 frequencies; ``angles``: the step's cosines and sines, ``rope_table``), queries to ``q_out`` and keys and values into the
     cache rows that ``slot_mapping`` names (see csrc/attn_prep.cu).  ``q_scale`` (float32 [heads]): every query head is
-    multiplied by its number at the end."""
+    multiplied by its number at the end.  ``temperature`` = (coef, every): q is multiplied by 1 + coef ln(floor((p + 1) / every) + 1).
+    ``v_scale`` multiplies the values.  ``maps`` 2: every q and k head has two maps of ``dim`` elements; ``q_out`` then has a row for
+    every map of every head.  ``q_out`` [T, rows * width]: rows wider than what they hold are filled with zeros (cache rows too)."""
     T = proj.shape[0]
-    C = num_heads * dim + (num_kv_heads * (dim + vdim) if own_kv else 0)
+    C = num_heads * maps * dim + (num_kv_heads * (maps * dim + vdim) if own_kv else 0)
     _need(own_kv or slot_mapping is None, "attn_prep: a mixer without keys and values of its own writes no cache rows")
     _need(q_scale is None or (q_scale.dtype == torch.float32 and q_scale.numel() == num_heads and q_scale.is_contiguous()),
           "attn_prep: q_scale must be float32 [heads]")
-    _need(norm in (None, "before", "after"), "attn_prep: norm is None, 'before' or 'after'")
+    _need(norm in (None, "before", "after", "row"), "attn_prep: norm is None, 'before', 'row' or 'after'")
     _need(proj.dtype == torch.float32 and proj.stride(1) == 1 and proj.shape[1] >= C, "attn_prep: projections must be float32 rows")
     _need(bias is None or (bias.dtype == torch.float32 and bias.numel() == C), "attn_prep: bias must be float32 [channels]")
-    _need(norm != "before" or all(w is not None and w.dtype == torch.float32 and w.numel() == dim
-                                  for w in ((q_norm, k_norm) if own_kv else (q_norm,))),
-          "attn_prep: the norm in front of the rotation needs float32 weights [dim]")
+    if norm in ("before", "row"):
+        sizes = (dim, dim) if norm == "before" else (num_heads * maps * dim, num_kv_heads * maps * dim)
+        _need(all(w is not None and w.dtype == torch.float32 and w.is_contiguous() and w.numel() == n
+                  for w, n in list(zip((q_norm, k_norm), sizes))[:2 if own_kv else 1]),
+              "attn_prep: a weighted norm needs float32 weights, [dim] in front of the rotation or one for every value of the row")
     _need(freq is None or (freq.dtype == torch.float64 and freq.is_contiguous() and 2 * freq.numel() <= dim), "attn_prep: freq must be float64 [<= dim / 2]")
-    _need(q_out.is_contiguous() and tuple(q_out.shape) == (T, num_heads * dim), "attn_prep: query output shape")
+    _need(angles is None or (freq is not None and angles.dtype == torch.float32 and angles.is_contiguous() and angles.numel() == 2 * T * freq.numel()),
+          "attn_prep: angles must be float32 [T, len(freq), 2]")
+    rows = num_heads * maps
+    _need(q_out.is_contiguous() and q_out.shape[0] == T and q_out.shape[1] % rows == 0 and q_out.shape[1] // rows >= maps * dim,
+          "attn_prep: query output shape")
     _need(slot_mapping is None or (pool is not None and pool.is_contiguous() and pool.dim() == 5 and pool.shape[1] == 2
-                                   and pool.shape[-1] >= max(dim, vdim) and pool.dtype == q_out.dtype),
-          "attn_prep: the cache must be [pages, 2, kv heads, page, >= max(dim, vdim)] of the activations' dtype")
+                                   and pool.shape[-1] >= max(maps * dim, vdim) and pool.dtype == q_out.dtype),
+          "attn_prep: the cache must be [pages, 2, kv heads, page, >= max(maps * dim, vdim)] of the activations' dtype")
+    _need(temperature is None or temperature[1] > 0, "attn_prep: the temperature's step must be positive")
     rot = 2 * freq.numel() if freq is not None else 0
-    _call("me_attn_prep", proj.data_ptr(), proj.stride(0), _ptr(bias), _ptr(q_norm), _ptr(k_norm), {None: 0, "before": 1, "after": 2}[norm],
-          float(eps), _ptr(freq) if rot else 0, rot, positions.data_ptr(), _ptr(slot_mapping), q_out.data_ptr(), _ptr(pool), _dt(q_out),
-          pool.shape[-1] if pool is not None else 0, page_size, num_heads, num_kv_heads, dim, vdim, T, _ptr(q_scale), 1 if own_kv else 0,
-          _stream())
+    coef, every = temperature if temperature is not None else (0.0, 0.0)
+    _call("me_attn_prep", proj.data_ptr(), proj.stride(0), _ptr(bias), _ptr(q_norm), _ptr(k_norm), {None: 0, "before": 1, "after": 2, "row": 3}[norm],
+          float(eps), _ptr(freq) if rot else 0, rot, _ptr(angles) if rot else 0, positions.data_ptr(), _ptr(slot_mapping), q_out.data_ptr(),
+          q_out.shape[1] // rows, _ptr(pool), _dt(q_out), pool.shape[-1] if pool is not None else 0, page_size, num_heads, num_kv_heads, dim, vdim,
+          maps, T, _ptr(q_scale), 1 if own_kv else 0, float(coef), float(every), float(v_scale), _stream())
+
+
+def padded_head(width: int) -> int:
+    """The row width at which heads of ``width`` elements run the tensor-core attention kernels: 64 or 128 (the rest of a row is
+    zeros); wider heads keep their width."""
+    return 64 if width <= 64 else (128 if width <= 128 else width)
+
+
+def diff_combine(maps: torch.Tensor, out: torch.Tensor, num_heads: int, vdim: int, lam: float, gain: float, eps: float, first: int = 0) -> None:
+    """``maps`` [T, 2 * heads * vdim] holds two results a head; ``out`` [T, heads * vdim] = d / sqrt(mean(d^2) + eps) * gain per head with
+    d = first - lam * second, for the rows from ``first`` on."""
+    T = maps.shape[0]
+    _need(maps.stride(1) == 1 and out.stride(1) == 1 and maps.shape[1] == 2 * num_heads * vdim and tuple(out.shape) == (T, num_heads * vdim),
+          "diff_combine: shapes")
+    _call("me_diff_combine", maps.data_ptr(), _dt(maps), maps.stride(0), out.data_ptr(), _dt(out), out.stride(0), first, T - first, num_heads, vdim,
+          float(lam), float(gain), float(eps), _stream())
 
 
 def clamped_glu(x: torch.Tensor, out: torch.Tensor, limit: float, alpha: float, shift: float = 1.0) -> None:
@@ -1488,7 +1539,8 @@ use_sink_attention_mma = True     # bfloat16 attention with a sink on the tensor
 def sink_attention(q: torch.Tensor, gate: Optional[torch.Tensor], out: torch.Tensor, pool: torch.Tensor, page_size: int,
                    block_tables: torch.Tensor, meta, num_heads: int, num_kv_heads: int, dim: int, vdim: int, scale: float,
                    window: Optional[int], sink: bool, sinks: Optional[torch.Tensor] = None, softcap: Optional[float] = None,
-                   keep_first: int = 0, chunk: Optional[int] = None, pooled: Optional[tuple] = None) -> None:
+                   keep_first: int = 0, chunk: Optional[int] = None, pooled: Optional[tuple] = None, bias: Optional[tuple] = None,
+                   pairs: Optional[tuple[float, float, float]] = None, padded: bool = False) -> None:
     """Attention over the paged cache with keys of ``dim`` and values of ``vdim`` elements: ``q`` [T, heads * dim] -> ``out``
     [T, heads * vdim]; a query at position p sees keys p - window < j <= p; with ``sink`` the softmax's denominator has one
     more term, exp(0); ``gate`` (float32 rows of pre-activations, heads * vdim wide) multiplies the output by its sigmoid.
@@ -1498,13 +1550,23 @@ def sink_attention(q: torch.Tensor, gate: Optional[torch.Tensor], out: torch.Ten
     with one row per block of P tokens (``pool_kv``); beside its window a query sees the rows of the blocks that lie wholly in
     front of the window, (b + 1) P <= p - window + 1, in the same softmax.
 
+    ``bias`` = (r1, r2), float32 [heads] each: r1 ln(1 + r2 (p - j)) is taken off the scaled score of a key at distance p - j.
+    ``pairs`` = (lambda, gain, eps): heads 2h and 2h + 1 are two maps over the same values, and ``out`` [T, heads / 2 * vdim] is what
+    ``diff_combine`` makes of them.  ``padded``: the rows of q and of the cached keys are filled with zeros up to the cache's row
+    size (``dim`` is that size), so that heads of any size up to it run the tensor-core kernels.
+
     bfloat16 with keys and values of 64 or 128 elements (the cache row's size) runs the engine's tensor-core kernels, the
     tcgen05 one for portions of prompts and the split-K one for single tokens; everything else the CUDA-core kernel of
     csrc/sink_attention.cu."""
     T = q.shape[0]
     HD = pool.shape[-1]
-    _need(q.stride(1) == 1 and out.stride(1) == 1 and q.shape[1] == num_heads * dim and tuple(out.shape) == (T, num_heads * vdim),
-          "sink_attention: shapes")
+    _need(q.stride(1) == 1 and out.stride(1) == 1 and q.shape[1] == num_heads * dim
+          and tuple(out.shape) == (T, num_heads // (2 if pairs else 1) * vdim) and (not pairs or num_heads % 2 == 0), "sink_attention: shapes")
+    _need(not padded or (dim == HD and gate is None), "sink_attention: padded rows of q are as wide as the cache's, and go without a gate")
+    _need(bias is None or (all(b.dtype == torch.float32 and b.numel() == num_heads and b.is_contiguous() for b in bias)
+                           and not (softcap or sink or sinks is not None or pooled or keep_first or chunk)),
+          "sink_attention: a distance bias is two float32 numbers a head and goes with a plain window at most")
+    _need(pairs is None or not (gate is not None or sink or sinks is not None or pooled), "sink_attention: pairs go without gates, sinks and pooled blocks")
     _need(pool.dtype == q.dtype == out.dtype and pool.is_contiguous() and pool.dim() == 5 and pool.shape[1] == 2 and HD >= max(dim, vdim),
           "sink_attention: the cache must be [pages, 2, kv heads, page, >= max(dim, vdim)] of the activations' dtype")
     _need(gate is None or (gate.dtype == torch.float32 and gate.stride(1) == 1 and gate.shape[1] == num_heads * vdim),
@@ -1513,7 +1575,7 @@ def sink_attention(q: torch.Tensor, gate: Optional[torch.Tensor], out: torch.Ten
     _need(sinks is None or (sinks.dtype == torch.float32 and sinks.numel() == num_heads and sinks.is_contiguous()),
           "sink_attention: learned sinks are float32 [heads]")
     _need(not (chunk and window), "sink_attention: a window or chunks, not both")
-    masked = bool(softcap or keep_first or chunk)      # what only the kernels fed by tensor-map loads know
+    masked = bool(softcap or keep_first or chunk or bias)      # what only the kernels fed by tensor-map loads know
     pool_p = 0
     if pooled is not None:
         _need(window and not chunk and not keep_first, "sink_attention: pooled blocks go with a plain window")
@@ -1522,14 +1584,19 @@ def sink_attention(q: torch.Tensor, gate: Optional[torch.Tensor], out: torch.Ten
               "sink_attention: the pooled cache has the layout and dtype of the cache, int32 tables and a block size")
         pool_p = int(pooled[2])
     decodes, tiles_left = meta.num_decodes, True
-    fast = (use_sink_attention_mma and q.dtype == torch.bfloat16 and dim == vdim == HD and HD in (64, 128)
+    fast = (use_sink_attention_mma and q.dtype == torch.bfloat16 and (dim == vdim == HD or padded) and HD in (64, 128)
             and meta.error_flag is not None and q.is_contiguous() and q.data_ptr() % 16 == 0)
-    extras = dict(keep_first=keep_first, chunk=chunk or 0, softcap=softcap or 0.0, sinks=sinks)
+    extras = dict(keep_first=keep_first, chunk=chunk or 0, softcap=softcap or 0.0, sinks=sinks, bias=bias, out_dim=vdim)
+    joined = out                                        # with pairs: what the two maps are joined into, from row joined_from on
+    joined_from = 0
     if fast and decodes and (not (masked or pooled) or (page_size >= 8 and DECODE_PARTITION % page_size == 0)):
         attention_decode(q, out, num_heads, num_kv_heads, HD, pool, page_size, block_tables, meta, scale, window, sink=sink, gate=gate,
-                         pooled=pooled, **extras)
-        decodes = 0
-    if fast and meta.num_tiles > 0 and use_tcgen05_attention and prefill_tcgen05_heads_per_block(num_heads, num_kv_heads, HD, page_size) > 0:
+                         pooled=pooled, pairs=pairs, **extras)
+        joined_from, decodes = decodes, 0
+    if pairs and (decodes or meta.num_tiles > 0):
+        out = meta.workspace("attn_maps", (T, num_heads * vdim), q.dtype)
+    if (fast and meta.num_tiles > 0 and use_tcgen05_attention and prefill_tcgen05_heads_per_block(num_heads, num_kv_heads, HD, page_size) > 0
+            and vdim % 8 == 0 and out.stride(0) % 8 == 0 and out.data_ptr() % 16 == 0):
         attention_prefill_tcgen05(q, out, num_heads, num_kv_heads, HD, pool, page_size, block_tables, meta, scale, window,
                                   sink=sink, gate=gate, pooled=pooled, **extras)
         tiles_left = False
@@ -1542,7 +1609,9 @@ def sink_attention(q: torch.Tensor, gate: Optional[torch.Tensor], out: torch.Ten
               meta.context_lens.data_ptr(), tiles.data_ptr(), n_tiles, decodes, num_heads, num_kv_heads, dim, vdim, HD, page_size,
               float(scale), int(window or 0), 1 if sink else 0, _ptr(sinks), float(softcap or 0.0), int(keep_first or 0),
               int(chunk or 0), pooled[0].data_ptr() if pool_p else 0, pooled[1].data_ptr() if pool_p else 0,
-              pooled[1].stride(0) if pool_p else 0, pool_p, _stream())
+              pooled[1].stride(0) if pool_p else 0, pool_p, _ptr(bias[0]) if bias else 0, _ptr(bias[1]) if bias else 0, _stream())
+    if pairs and out is not joined:
+        diff_combine(out, joined, num_heads // 2, vdim, *pairs, first=joined_from)
 
 
 def moe_route(logits: torch.Tensor, bias: Optional[torch.Tensor], top: int, idx: torch.Tensor, weights: torch.Tensor) -> None:

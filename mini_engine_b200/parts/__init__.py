@@ -11,8 +11,10 @@ from .conv import CausalShortConv
 from .polynorm_mlp import PolyNormMLP
 from .latent_attention import LatentAttention
 from .mlstm import MLSTM
-from .gla import GatedLinearAttention
+from .gla import GatedLinearAttention, HGRN2
 from .masked_attention import MaskedSinkAttention
+from .differential_attention import DifferentialAttention
+from .side_by_side import SideBySide
 from .sink_attention import SinkAttention
 from .pooled_attention import PooledWindowAttention
 from .glu_mlp import ClampedGLU, RoutedExperts

@@ -26,10 +26,13 @@ import torch
 
 @dataclass
 class DiskSource:
-    """Rows ``[row_start, row_start+rows)`` of a parameter come from one tensor on disk."""
+    """Rows ``[row_start, row_start+rows)`` of a parameter come from one tensor on disk; with ``cols`` the columns
+    ``[col_start, col_start+cols)`` of those rows (a parameter packed from several tensors side by side)."""
     disk_name: str
     row_start: int
     rows: int
+    col_start: int = 0
+    cols: Optional[int] = None
 
 
 @dataclass

@@ -78,6 +78,16 @@ class Block(Part):
             parts += [(s.feed_forward_norm_prefix, self.feed_forward_norm), (s.feed_forward_prefix, self.feed_forward)]
         return parts
 
+    def _unused_second_norm(self) -> list:
+        """A layer without a feed-forward has no use for the second norm; files that hold one all the same are accepted."""
+        if self.feed_forward is not None:
+            return []
+        spec = self.spec.feed_forward_norm or self.spec.norm
+        if spec is None or "size" not in spec.args or "param" not in spec.args:
+            return []
+        names = [spec.args["param"]] + ([spec.args["bias"]] if spec.args.get("bias") else [])
+        return [ParamDecl(self.spec.feed_forward_norm_prefix + n, (spec.args["size"],), role="vector", optional=True) for n in names]
+
     def cache_needs(self):
         """What one call of this block needs of the cache: the mixer's needs, and the block's own if it has any."""
         return self.mixer.cache_needs()
@@ -91,8 +101,23 @@ class Block(Part):
 
 class PreNormBlock(Block):
     """``r += mixer(norm(r)); r += feed_forward(norm(r))`` with each sum deferred into the norm that follows
-    (models/qwen3.py:65-74 in the reference)."""
+    (models/qwen3.py:65-74 in the reference).  The feed-forward may be absent.  With norms that can add a pending sum (kind
+    ``layernorm`` with a bias) a mixer's output bias (``output_bias()``) is deferred into that norm as well, and a
+    ``LayerCall`` may have the step's embedding rows join the stream right before the block (``add_embedding``)."""
     capturable = True
+    feed_forward_optional = True
+
+    def __init__(self, spec: BlockSpec, shared: Optional[dict] = None):
+        super().__init__(spec, shared)
+        self.embedding = (shared or {}).get("embedding")
+        # (the norm behind this block's last sub-layer, the next block's or the model's, is taken to be of the same kind)
+        self.sums_pending = all(getattr(n, "bias", None) is not None for n in (self.mixer_norm, self.feed_forward_norm) if n is not None)
+        self.takes_embedding = self.sums_pending and self.embedding is not None
+        if self.sums_pending and hasattr(self.mixer, "defer_output_bias"):
+            self.mixer.defer_output_bias = True
+
+    def param_decls(self):
+        return self._unused_second_norm()
 
     def upcoming(self) -> Upcoming:
         """What this block starts with, for the block that runs before it."""
@@ -103,12 +128,20 @@ class PreNormBlock(Block):
         that it has been).  Returns this block's last output the same way.  ``upcoming``: what runs after this
         block (``Upcoming``), if the caller knows it."""
         mixer, ffn = self.mixer, self.feed_forward
-        x = self.mixer_norm.forward(residual, delta, ctx, lazy=mixer.takes_pending_norm)
+        if call.add_embedding:
+            x = self.mixer_norm._sum_and_norm(residual, delta, ctx, None, "norm_out", None, embedding=self.embedding)
+        else:
+            x = self.mixer_norm.forward(residual, delta, ctx, lazy=mixer.takes_pending_norm)
         if mixer.adds_to_residual:
             mixed = mixer.forward(x, ctx, call, residual=residual,
-                                  upcoming=Upcoming(self.feed_forward_norm, ffn.first_weight()))
+                                  upcoming=Upcoming(self.feed_forward_norm, ffn.first_weight()) if ffn is not None else upcoming)
         else:
             mixed = mixer.forward(x, ctx, call)
+        bias = mixer.output_bias() if self.sums_pending and hasattr(mixer, "output_bias") else None
+        if bias is not None:
+            mixed = PendingSum([mixed], [bias])
+        if ffn is None:
+            return mixed
         x = self.feed_forward_norm.forward(residual, mixed, ctx, lazy=ffn.takes_pending_norm)
         if ffn.adds_to_residual:
             return ffn.forward(x, ctx, residual=residual, upcoming=upcoming)
@@ -254,14 +287,7 @@ class ParallelBlock(Block):
             self.mixer.defer_output_bias = True
 
     def param_decls(self):
-        """A layer without a feed-forward has no use for the second norm; files that hold one all the same are accepted."""
-        if self.feed_forward is not None:
-            return []
-        spec = self.spec.feed_forward_norm or self.spec.norm
-        if spec is None or "size" not in spec.args:
-            return []
-        names = [spec.args.get("param", "weight")] + ([spec.args["bias"]] if spec.args.get("bias") else [])
-        return [ParamDecl(self.spec.feed_forward_norm_prefix + n, (spec.args["size"],), role="vector", optional=True) for n in names]
+        return self._unused_second_norm()
 
     def forward(self, residual, delta, ctx, call, upcoming=None):
         vectors = []
@@ -294,14 +320,7 @@ class PostNormBlock(Block):
                 raise ValueError("a 'post_norm' block needs norms that can add a normalised output to the stream (kind 'group_rmsnorm')")
 
     def param_decls(self):
-        """A layer without a feed-forward has no use for the second norm; files that hold one all the same are accepted."""
-        if self.feed_forward is not None:
-            return []
-        spec = self.spec.feed_forward_norm or self.spec.norm
-        if spec is None or "size" not in spec.args:
-            return []
-        return [ParamDecl(self.spec.feed_forward_norm_prefix + spec.args.get("param", "weight"), (spec.args["size"],), role="vector",
-                          optional=True)]
+        return self._unused_second_norm()
 
     def forward(self, residual, delta, ctx, call, upcoming=None):
         if isinstance(delta, StreamCopy):

@@ -34,6 +34,11 @@ class TokenEmbedding(Part):
         return out
 
 
+    def rows_of_step(self, ctx) -> tuple:
+        """(token ids, table, feedback, scale): what a kernel needs to look the step's rows up again by itself."""
+        return ctx.token_ids, self.p(self.param), getattr(ctx, "token_feedback", None), self.scale
+
+
 class LMHead(Part):
     capturable = True
 

@@ -13,19 +13,30 @@ from .base import AddedToResidual, DiskSource, ParamDecl, Part, PendingNorm
 
 
 class Linear(Part):
-    """``pieces``: (disk name relative to the owner, rows) for every packed piece."""
+    """``pieces``: (disk name relative to the owner, rows) for every packed piece.  ``input_pieces`` (instead): (disk name,
+    columns) for maps of the same rows whose results are added: their matrices lie side by side in one weight, whose input is
+    their inputs side by side (``in_features`` is the sum of the columns, ``out_features`` the rows)."""
 
     capturable = True
 
-    def __init__(self, in_features: int, pieces: Sequence[tuple[str, int]], name: str = "weight"):
+    def __init__(self, in_features: int, pieces: Sequence[tuple[str, int]] = (), name: str = "weight",
+                 input_pieces: Optional[Sequence[tuple[str, int]]] = None, out_features: Optional[int] = None):
         super().__init__()
         self.in_features = in_features
         self.pieces = list(pieces)
-        self.out_features = sum(r for _, r in self.pieces)
+        self.input_pieces = list(input_pieces) if input_pieces is not None else None
+        self.out_features = sum(r for _, r in self.pieces) if self.input_pieces is None else int(out_features)
+        if self.input_pieces is not None and sum(c for _, c in self.input_pieces) != in_features:
+            raise ValueError("Linear: the input pieces do not add up to the input's size")
         self.name = name
 
     def param_decls(self):
         sources, start = [], 0
+        if self.input_pieces is not None:
+            for disk, cols in self.input_pieces:
+                sources.append(DiskSource(disk, 0, self.out_features, start, cols))
+                start += cols
+            return [ParamDecl(self.name, (self.out_features, self.in_features), sources=sources)]
         for disk, rows in self.pieces:
             sources.append(DiskSource(disk, start, rows))
             start += rows

@@ -28,6 +28,7 @@ class LayerCall:
     writes_cache: bool = True
     kv_slot: "Optional[int]" = None    # a mixer that reads ANOTHER call's keys and values: the cache slot that holds them
     add_row: "Optional[int]" = None    # the row of the model's pass vectors that joins the stream right before this call
+    add_embedding: bool = False        # the step's embedding rows join the stream once more right before this call
 
 
 @dataclass
@@ -89,6 +90,7 @@ class DecoderModel(Part):
             raise ValueError(f"norm kind {plan.embed_norm.kind!r} cannot normalise the stream in place (ModelPlan.embed_norm)")
         self.tables = {k: TokenEmbedding(rows, cols, param=name) for k, (name, rows, cols) in plan.tables.items()}
         self.shared.update(self.tables)
+        self.shared["embedding"] = self.embed
         self.pass_vectors = None
         if plan.pass_vectors is not None:
             self.pass_vectors = self.shared["pass_vectors"] = PassVectors(plan.pass_vectors[0], plan.pass_vectors[1], plan.hidden_size)
@@ -111,6 +113,8 @@ class DecoderModel(Part):
                 if self.pass_vectors is None or not 0 <= c.add_row < self.pass_vectors.rows:
                     raise ValueError(f"the schedule names pass vector {c.add_row}, the model has "
                                      f"{self.pass_vectors.rows if self.pass_vectors else 0}")
+            if c.add_embedding and not getattr(self.blocks[c.block], "takes_embedding", False):
+                raise ValueError(f"block {c.block} ({plan.blocks[c.block].kind!r}) cannot add the embedding in front of itself")
             needs = self.blocks[c.block].cache_needs()
             if not self.slot_needs[c.cache_slot]:
                 self.slot_needs[c.cache_slot] = needs

@@ -94,8 +94,9 @@ class LayerNorm(Norm):
     def weight_and_bias(self):
         return self.p(self.param), (self.p(self.bias) if self.bias is not None else None)
 
-    def _sum_and_norm(self, residual, delta, ctx, rows, out_name, out_dtype, vectors=(), also=None):
-        """One pass of ``parallel_norm``: everything pending joins the stream, then this norm (and ``also``'s)."""
+    def _sum_and_norm(self, residual, delta, ctx, rows, out_name, out_dtype, vectors=(), also=None, embedding=None):
+        """One pass of ``parallel_norm``: everything pending joins the stream (and, with ``embedding``, a ``TokenEmbedding``, the
+        step's embedding rows), then this norm (and ``also``'s)."""
         outputs, vectors = [], list(vectors)
         if isinstance(delta, PendingSum):
             outputs, vectors = list(delta.outputs), list(delta.vectors) + vectors
@@ -108,7 +109,8 @@ class LayerNorm(Norm):
         out = ctx.buffer(out_name, (n, self.size), dtype)
         out2 = ctx.buffer(also[1], (n, self.size), dtype) if also is not None else None
         ops.parallel_norm(residual, outputs, vectors, self.eps, self.weight_and_bias(), out,
-                          also[0].weight_and_bias() if also is not None else None, out2, rows=rows)
+                          also[0].weight_and_bias() if also is not None else None, out2, rows=rows,
+                          embedding=embedding.rows_of_step(ctx) if embedding is not None else None)
         return out if also is None else (out, out2)
 
     def forward(self, residual, delta, ctx, rows: Optional[torch.Tensor] = None, lazy: bool = False, *,

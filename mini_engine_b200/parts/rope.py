@@ -37,6 +37,24 @@ class RotaryEmbedding(PositionEncoding):
         self.cos_sin = torch.cat((freqs.cos(), freqs.sin()), dim=-1).contiguous().to(device)
 
 
+def _angles_of_step(rope, freq: torch.Tensor, ctx, T: int):
+    """The cosines and sines of a step's positions ([T, frequencies, 2] float32), or None for a step so short that the kernels form
+    them themselves.  One table for all layers that share the rotation, made anew in every pass over the layers (a pass that
+    is being recorded into a graph must launch it too, or the replay would rotate by the positions of the recording)."""
+    from .. import ops
+    if T < ops.ROPE_TABLE_MIN_TOKENS:
+        return None
+    cache = getattr(ctx, "_rope_tables", None)
+    if cache is None or cache[0] != ctx.forward_serial:
+        cache = ctx._rope_tables = (ctx.forward_serial, {})
+    tables = cache[1]
+    angles = tables.get(id(rope))
+    if angles is None:
+        angles = tables[id(rope)] = ctx.buffer(f"rope_table_{id(rope)}", (T, freq.numel(), 2), torch.float32)
+        ops.rope_table(ctx.positions, freq, angles)
+    return angles
+
+
 class InterleavedRotary(PositionEncoding):
     """Rotary positions on pairs of neighbouring elements: (x[2i], x[2i+1]) at position p becomes
     (u cos a - v sin a, v cos a + u sin a) with a = p * theta^(-2i / rotary_dim), on the first ``rotary_dim`` elements.
@@ -58,6 +76,9 @@ class InterleavedRotary(PositionEncoding):
         d = self.rotary_dim
         i = torch.arange(0, d, 2, dtype=torch.float64)
         self.inv_freq = (self.theta ** (-i / d) if d else i).contiguous().to(device)
+
+    def angles_of_step(self, ctx, T: int):
+        return _angles_of_step(self, self.inv_freq, ctx, T)
 
 
 class FrequencyRotary(PositionEncoding):
@@ -103,6 +124,9 @@ class FrequencyRotary(PositionEncoding):
 
     def finalize(self, dtype, device):
         self.freq = torch.tensor(self.frequencies(), dtype=torch.float64).contiguous().to(device)
+
+    def angles_of_step(self, ctx, T: int):
+        return _angles_of_step(self, self.freq, ctx, T)
 
 
 register_position_encoding("rope", RotaryEmbedding)

@@ -97,19 +97,7 @@ class SinkAttention(Mixer):
         kv = ctx.kv_cache(call.cache_slot if self.own_kv else call.kv_slot)
         q = ctx.buffer("attn_q", (T, H * D), ctx.act_dtype)
         inv_freq = self.rope.inv_freq if self.rope is not None else self._no_freq
-        angles = None
-        if self.rope is not None and T >= ops.ROPE_TABLE_MIN_TOKENS:
-            # One table for all layers that share the rotation, made anew in every pass over the layers (a pass that is being
-            # recorded into a graph must launch it too, or the replay would rotate by the positions of the recording).
-            cache = getattr(ctx, "_rope_tables", None)
-            if cache is None or cache[0] != ctx.forward_serial:
-                cache = ctx._rope_tables = (ctx.forward_serial, {})
-            tables = cache[1]
-            angles = tables.get(id(self.rope))
-            if angles is None:
-                angles = tables[id(self.rope)] = ctx.buffer(f"rope_table_{self.rope.rotary_dim}_{self.rope.theta!r}",
-                                                            (T, inv_freq.numel(), 2), torch.float32)
-                ops.rope_table(ctx.positions, inv_freq, angles)
+        angles = self.rope.angles_of_step(ctx, T) if self.rope is not None else None
         ops.conv_rope_kv(proj, self.p("in_bias") if self.has_bias else None, self.p("in_conv") if self.taps >= 1 else None,
                          ctx.state(call.cache_slot, "conv") if self.taps > 1 else None, inv_freq, inv_freq.numel() * 2, ctx,
                          kv.slot_mapping if self.own_kv and call.writes_cache else None, q, kv.pool, kv.page_size, H, G, D, V,

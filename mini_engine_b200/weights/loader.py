@@ -54,6 +54,7 @@ class _Expected:
     row_start: int
     shape: tuple[int, ...]
     optional: bool = False
+    col_start: int = 0
 
 
 def iter_param_decls(model: Part) -> Iterator[tuple[str, Part, ParamDecl]]:
@@ -71,7 +72,8 @@ def expected_disk_tensors(model: Part) -> dict[str, _Expected]:
         full = prefix + decl.name
         if decl.sources:
             for src in decl.sources:
-                exp[prefix + src.disk_name] = _Expected(full, src.row_start, (src.rows, *decl.shape[1:]), decl.optional)
+                tail = decl.shape[1:] if src.cols is None else (src.cols, *decl.shape[2:])
+                exp[prefix + src.disk_name] = _Expected(full, src.row_start, (src.rows, *tail), decl.optional, src.col_start)
         else:
             exp[full] = _Expected(full, 0, tuple(decl.shape), decl.optional)
     return exp
@@ -132,7 +134,11 @@ def load_weights(model: Part, folder: str, dtype: torch.dtype, device) -> dict[s
                 e = expected[name]
                 dest = params[e.param]
                 piece = f.get_tensor(name)
-                dest.narrow(0, e.row_start, e.shape[0]).copy_(piece.to(dest.dtype)) if dest.dim() else dest.copy_(piece)
+                if dest.dim():
+                    dest = dest.narrow(0, e.row_start, e.shape[0])
+                    if dest.dim() > 1:
+                        dest = dest.narrow(1, e.col_start, e.shape[1])
+                dest.copy_(piece.to(dest.dtype))
 
     for full, (part, decl) in decl_of.items():
         if decl.tied_to is not None:
