@@ -28,7 +28,7 @@ GPU: for ``--gpus N`` with N > 1 one line says so and the exit code is 2.
 Modes: ``step`` (the line above), ``offline`` (the reference's own bench.py:38-66 with its options ``--num-seqs
 --budget --chunked --threshold --out --label --expect-gpu``; a JSON row like the reference's is appended to
 ``--out``), ``mixed`` (the 8B workload above, at any shape), ``decode`` (decode at batches ``--batches`` after
-``--prompt-len`` prompts), ``prefill`` (one prompt of ``--prompt-len`` tokens in portions of ``--budget``), ``logozen``, ``pugadra``, ``gevulorn`` and ``galupel``
+``--prompt-len`` prompts), ``prefill`` (one prompt of ``--prompt-len`` tokens in portions of ``--budget``), ``logozen``, ``pugadra``, ``gevulorn``, ``galupel`` and ``tidenex``
 (prefill and decode of that design at the layer sizes ``--sizes``, beside the Qwen3 of equal size (Gevulorn and Galupel: the Pugadra of equal
 size), with the time of every kernel).
 """
@@ -173,8 +173,40 @@ GALUPEL_SIZES = {   # width, layers, the twin's dense ff, heads / kv heads / hea
     "m": _galupel(2048, 8, 8192, 16, 4, 128, 1024, 32, 32, 2, 2048, (4, 2), 64, 64, 128, 256),
     "l": _galupel(4096, 6, 12288, 32, 8, 128, 1024, 32, 32, 4, 2048, (8, 4), 64, 64, 128, 512),
 }
-DESIGN_SIZES = {"logozen": LOGOZEN_SIZES, "pugadra": PUGADRA_SIZES, "gevulorn": GEVULORN_SIZES, "galupel": GALUPEL_SIZES}
-DESIGN_TWINS = {"logozen": "qwen3", "pugadra": "qwen3", "gevulorn": "pugadra", "galupel": "pugadra"}      # the model set beside each design
+def _tidenex(width, layers, ff, heads, kv_heads, dim, map_dim, g_heads, g_dim, g_vdim, vocab=32768):
+    """A Tidenex of ``layers`` layers: differential attention on the even layers (as many query columns as ``heads`` heads of ``dim``),
+    attention with a distance bias beside the HGRN2 recurrence on the odd ones, dense feed-forwards everywhere, no loop.  And a Gevulorn
+    of the same width, depth, heads, head size, recurrence, feed-forward and vocabulary to set beside it: attention without a
+    mask on the even layers, gated linear attention on the odd ones, dense feed-forwards."""
+    dense = {"kind": "dense", "ff": ff}
+    d_heads, d_kv = heads * dim // (2 * map_dim), max(1, kv_heads * dim // (2 * map_dim))
+
+    def layer(i):
+        if i % 2 == 0:
+            return {"type": "attention", "mlp": dense, "mixer": {"heads": d_heads, "kv_heads": d_kv, "dim": map_dim, "vdim": 2 * map_dim,
+                                                                 "scale": map_dim ** -0.5, "diff": 0.5, "rot": {"base": 10000.0, "dims": map_dim}}}
+        return {"type": "parallel", "mlp": dense, "mixer": {
+            "left": {"heads": heads, "kv_heads": kv_heads, "dim": dim, "vdim": dim, "scale": dim ** -0.5, "q_temp": {"coef": 0.1, "every": 256}},
+            "right": {"heads": g_heads, "dim": g_dim, "vdim": g_vdim}, "left_scale": 0.8, "right_scale": 1.2}}
+
+    def twin_layer(i):
+        if i % 2 == 0:
+            return {"type": "attention", "mlp": dense, "mixer": {"heads": heads, "kv_heads": kv_heads, "dim": dim, "vdim": dim, "scale": dim ** -0.5,
+                                                                 "rot": {"base": 10000.0, "dims": dim}}}
+        return {"type": "gla", "mixer": {"heads": g_heads, "dim": g_dim, "vdim": g_vdim, "tau": 16.0, "decay_rank": 16}, "mlp": dense}
+    cfg = {"architecture": "Tidenex", "vocab": vocab, "width": width, "norm": {"eps": 1e-5}, "layers": [layer(i) for i in range(layers)]}
+    twin = {"architecture": "Gevulorn", "vocab": vocab, "width": width, "norm": {"eps": 1e-5}, "layers": [twin_layer(i) for i in range(layers)]}
+    return cfg, twin
+
+
+TIDENEX_SIZES = {   # width, layers, ff, heads / kv heads / head size, a map's size, the recurrence's heads / channels / value size
+    "s": _tidenex(1024, 8, 3072, 16, 4, 64, 64, 8, 64, 128),
+    "m": _tidenex(2048, 8, 8192, 16, 4, 128, 64, 8, 128, 256),
+    "l": _tidenex(4096, 6, 12288, 32, 8, 128, 64, 16, 128, 256),
+}
+DESIGN_SIZES = {"logozen": LOGOZEN_SIZES, "pugadra": PUGADRA_SIZES, "gevulorn": GEVULORN_SIZES, "galupel": GALUPEL_SIZES, "tidenex": TIDENEX_SIZES}
+DESIGN_TWINS = {"logozen": "qwen3", "pugadra": "qwen3", "gevulorn": "pugadra", "galupel": "pugadra",
+                "tidenex": "gevulorn"}                                                                    # the model set beside each design
 FALLBACK_PEAKS = {"hbm_gbs": 6650.0, "bf16_tflops": 1590.0, "bf16_tflops_sustained": 1400.0, "source": "fallback"}
 
 
@@ -184,8 +216,8 @@ def parse_args():
     p.add_argument("--steps", type=int, default=200)
     p.add_argument("--warmup", type=int, default=10)
     p.add_argument("--impl", choices=["ours", "reference"], default="ours")
-    p.add_argument("--mode", choices=["step", "offline", "mixed", "decode", "prefill", "logozen", "pugadra", "gevulorn", "galupel"], default="step")
-    p.add_argument("--sizes", default="s,m", help="logozen, pugadra, gevulorn and galupel modes: which of the layer sizes " + ",".join(sorted(LOGOZEN_SIZES)))
+    p.add_argument("--mode", choices=["step", "offline", "mixed", "decode", "prefill", "logozen", "pugadra", "gevulorn", "galupel", "tidenex"], default="step")
+    p.add_argument("--sizes", default="s,m", help="logozen, pugadra, gevulorn, galupel and tidenex modes: which of the layer sizes " + ",".join(sorted(LOGOZEN_SIZES)))
     p.add_argument("--shape", choices=sorted(SHAPES), default="0.6b", help="layer sizes, when no --model is given")
     p.add_argument("--extras", type=int, default=1,
                    help="step mode: also run the offline workload, the 8B mixed workload and the 32B decode points")
@@ -899,6 +931,35 @@ def _galupel_roofline(cfg: dict, T: int, item: int, pk: dict, times: dict) -> di
                       times, pk)
 
 
+def _tidenex_roofline(cfg: dict, T: int, item: int, pk: dict, times: dict) -> dict:
+    """What Tidenex's own kernels have to move or do in a prefill step of T tokens and the fraction of the measured peak that
+    their summed time makes: bytes for the element-wise kernels, multiply-adds for attention and recurrence."""
+    W = cfg["width"]
+    need = {k: 0.0 for k in ("me_parallel_norm", "me_attn_prep", "me_sink_attn", "me_attn_prefill_tcgen05", "me_diff_combine", "me_gla_scan",
+                             "me_mlstm_out", "me_activation")}
+    pairs = T * (T + 1) / 2
+    for layer in cfg["layers"]:
+        m = layer["mixer"]
+        need["me_parallel_norm"] += (1 + (layer["mlp"] is not None)) * T * W * (8 + 2 * item)      # stream in and out, y in, h out
+        if layer["type"] == "attention":
+            H, G, D, V = m["heads"], m["kv_heads"], m["dim"], m["vdim"]
+            need["me_attn_prep"] += T * (2 * H * D + G * (2 * D + V)) * (4 + item)
+            need["me_diff_combine"] += T * H * V * 3 * item
+            att = 4.0 * H * (D + V) * pairs                            # two maps, each against the keys and over the values
+        else:
+            a, r = m["left"], m["right"]
+            H, G, D, V = a["heads"], a["kv_heads"], a["dim"], a["vdim"]
+            need["me_attn_prep"] += T * (H * D + G * (D + V)) * (4 + item)
+            att = 2.0 * H * (D + V) * pairs
+            need["me_gla_scan"] += 4.0 * r["heads"] * r["dim"] * r["vdim"] * T
+            need["me_mlstm_out"] += T * r["heads"] * r["vdim"] * (4 + item)
+        need["me_sink_attn"] += att
+        need["me_attn_prefill_tcgen05"] += att
+        if layer["mlp"] is not None:
+            need["me_activation"] += T * layer["mlp"]["ff"] * 2 * item
+    return _fractions(need, ("me_sink_attn", "me_attn_prefill_tcgen05", "me_gla_scan"), times, pk)
+
+
 def _qwen3_roofline(cfg: dict, T: int, item: int, pk: dict, times: dict) -> dict:
     """The like kernels of the Qwen3 beside a design: its norm, its q/k preparation and its prompt attention."""
     W, L = cfg["hidden_size"], cfg["num_hidden_layers"]
@@ -923,7 +984,7 @@ def run_design_mode(args, design: str) -> int:
     import torch
     sizes_of = DESIGN_SIZES[design]
     rooflines = {"logozen": _logozen_roofline, "pugadra": _pugadra_roofline, "gevulorn": _gevulorn_roofline, "galupel": _galupel_roofline,
-                 "qwen3": _qwen3_roofline}
+                 "tidenex": _tidenex_roofline, "qwen3": _qwen3_roofline}
     twin_label = DESIGN_TWINS[design]
     pk = peaks()
     item = 2 if args.dtype in ("bfloat16", "bf16") else 4

@@ -13,7 +13,7 @@ activation_kernel(const TI* __restrict__ in, int64_t in_stride, TO* __restrict__
   pdl_launch_dependents();
   const int t = blockIdx.x;
   for (int i = blockIdx.y * blockDim.x + threadIdx.x; i < F; i += gridDim.y * blockDim.x)
-    out[(int64_t)t * out_stride + i] = from_f<TO>(act_apply(to_f<TI>(in[(int64_t)t * in_stride + i]), kind));
+    out[(int64_t)t * out_stride + i] = from_f<TO>(act_apply<TO>(to_f<TI>(in[(int64_t)t * in_stride + i]), kind));
 }
 
 __global__ void __launch_bounds__(256) soft_cap_kernel(float* __restrict__ x, int64_t n, float cap, float scale) {

@@ -377,8 +377,13 @@ attn_prefill_tcgen05_kernel(const __grid_constant__ CUtensorMap q_map, const __g
 // Parities: a wait names a phase of its barrier by parity, which is only right while the phase before it is
 // over.  Every wait below stands where that is known (the comment beside it says why).
 // EXTRA: kept first keys, chunks, capped scores, learned sinks and pooled blocks are compiled in (the plain kernel keeps its
-// registers).  BIASED (without EXTRA): a distance bias is.
-template <int HD, bool EXTRA, bool BIASED>
+// registers).  BIASED (without EXTRA): a distance bias is.  PAIRS (without either): query heads 2h and 2h + 1 are two maps over the
+// same values, and what leaves is a = a_0 - lambda a_1, divided by its root mean square over the head's out_hd values and times gain.
+struct PairArgs {
+  float lambda, gain, eps;
+};
+
+template <int HD, bool EXTRA, bool BIASED, bool PAIRS>
 __global__ void __launch_bounds__(TA_THREADS)
 attn_prefill_tcgen05_two_groups_kernel(const __grid_constant__ CUtensorMap q_map, const __grid_constant__ CUtensorMap kv_map,
                                        bf16* __restrict__ out, int64_t out_row_stride, const int* __restrict__ block_tables,
@@ -388,7 +393,7 @@ attn_prefill_tcgen05_two_groups_kernel(const __grid_constant__ CUtensorMap q_map
                                        int* __restrict__ err, int keep_first_arg, int chunk_arg, float softcap_arg,
                                        const float* __restrict__ sinks_arg, const __grid_constant__ CUtensorMap pool_map,
                                        const int* __restrict__ pooled_tables, int pbt_stride, int pool_p_arg,
-                                       const float* __restrict__ bias_r1, const float* __restrict__ bias_r2, int out_hd) {
+                                       const float* __restrict__ bias_r1, const float* __restrict__ bias_r2, int out_hd, PairArgs pair) {
   const int keep_first = EXTRA ? keep_first_arg : 0, chunk = EXTRA ? chunk_arg : 0;
   const int pool_p = EXTRA ? pool_p_arg : 0;
   const float softcap = EXTRA ? softcap_arg : 0.f;
@@ -751,6 +756,48 @@ attn_prefill_tcgen05_two_groups_kernel(const __grid_constant__ CUtensorMap q_map
     if (ok && n_tiles > 1) ok = tma::mbar_wait(&o_ready[(n_tiles - 2) & 1], ((n_tiles - 2) >> 1) & 1);
     if (ok) ok = tma::mbar_wait(&o_ready[(n_tiles - 1) & 1], ((n_tiles - 1) >> 1) & 1);
     ok = __all_sync(0xffffffffu, ok);
+    if constexpr (PAIRS) {
+      // O / l goes through V's place in shared memory in float32 (every product is over), 16-byte pieces swizzled by the row; then HD / 4
+      // lanes take a pair of rows.  (A block holds whole pairs: the heads of a pack are an even number of neighbours.)
+      constexpr int OC2 = HD / 2, LANES = HD / 4;
+      if (ok) {
+        tc5::fence_after_sync();
+        const float inv = l > 0.f ? 1.f / l : 0.f;
+#pragma unroll
+        for (int c0 = 0; c0 < OC2; c0 += 32) {
+          float o_acc[32];
+          tc5::ld_32cols(tmem_o + t_row + g * OC2 + c0, o_acc);
+          tc5::wait_ld();
+#pragma unroll
+          for (int q = 0; q < 8; ++q) {
+            const int piece = (g * OC2 + c0) / 4 + q;
+            *reinterpret_cast<float4*>(v_s + r * (HD * 4) + ((piece ^ (r & 7)) << 4)) =
+                make_float4(o_acc[q * 4] * inv, o_acc[q * 4 + 1] * inv, o_acc[q * 4 + 2] * inv, o_acc[q * 4 + 3] * inv);
+          }
+        }
+      }
+      asm volatile("bar.sync 1, 256;\n" ::: "memory");
+      if (ok) {
+        const int piece = lane % LANES;
+        for (int i = (warp - 2) * 8 + lane / LANES; i < (warp - 1) * 8; i += 32 / LANES) {      // 64 pairs of rows, eight a warp
+          const int hp = i / tq, tok = i % tq, r0 = 2 * hp * tq + tok, r1 = r0 + tq;
+          const float4 x = *reinterpret_cast<const float4*>(v_s + r0 * (HD * 4) + ((piece ^ (r0 & 7)) << 4));
+          const float4 y = *reinterpret_cast<const float4*>(v_s + r1 * (HD * 4) + ((piece ^ (r1 & 7)) << 4));
+          const bool mine = piece * 4 < out_hd;
+          const float d0 = mine ? fmaf(-pair.lambda, y.x, x.x) : 0.f, d1 = mine ? fmaf(-pair.lambda, y.y, x.y) : 0.f;
+          const float d2 = mine ? fmaf(-pair.lambda, y.z, x.z) : 0.f, d3 = mine ? fmaf(-pair.lambda, y.w, x.w) : 0.f;
+          float ss = fmaf(d0, d0, d1 * d1) + fmaf(d2, d2, d3 * d3);
+#pragma unroll
+          for (int o = LANES / 2; o > 0; o >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, o);
+          const float f = pair.gain / sqrtf(ss / (float)out_hd + pair.eps);
+          if (mine && tok < n_tok) {
+            const __nv_bfloat162 lo2 = __floats2bfloat162_rn(d0 * f, d1 * f), hi2 = __floats2bfloat162_rn(d2 * f, d3 * f);
+            *reinterpret_cast<uint2*>(out + (int64_t)(tok0 + q0 + tok) * out_row_stride + (int64_t)(head0 / 2 + hp) * out_hd + piece * 4) =
+                make_uint2(*reinterpret_cast<const unsigned*>(&lo2), *reinterpret_cast<const unsigned*>(&hi2));
+          }
+        }
+      }
+    } else {
     // O / l goes through Q's place in shared memory (every Q K^T is over) so that it leaves in whole rows: a thread
     // holds one row of 128 lanes, and 32 threads storing 32 different rows would be 32 separate lines a store.
     constexpr int OC = HD / 2, PIECES = HD / 8;              // group 0 takes the first half of the row's columns, group 1 the other
@@ -796,6 +843,7 @@ attn_prefill_tcgen05_two_groups_kernel(const __grid_constant__ CUtensorMap q_map
         }
       }
     }
+    }
   }
   if (!ok) atomicOr(err + 1, 1);
   pdl_launch_dependents();
@@ -809,17 +857,19 @@ int launch_ta(const void* q_map, const void* kv_map, void* out, int64_t out_row_
               const int* cu_seqlens, const int* context_lens, const int* tiles, int num_tiles, int nh, int nkv, int gp,
               int page_size, float scale, int window, int sink, const float* gate, int64_t gate_stride, int* err,
               int keep_first, int chunk, float softcap, const float* sinks, const void* pool_map, const int* pooled_tables,
-              int pbt_stride, int pool_p, const float* bias_r1, const float* bias_r2, int out_hd, cudaStream_t stream) {
+              int pbt_stride, int pool_p, const float* bias_r1, const float* bias_r2, int out_hd, bool pairs, PairArgs pair, cudaStream_t stream) {
   const size_t smem = TWO_GROUPS ? (size_t)TA_ROWS * HD * 2 + 6 * (size_t)KT * HD * 2 + 1024
                                  : (size_t)TA_ROWS * HD * 2 + 4 * (size_t)KT * HD * 2 + 2 * (size_t)TA_ROWS * KT * 2 + 1024;
   static bool attr_set = false;
   if (!attr_set) {
-    cudaError_t e = TWO_GROUPS ? cudaFuncSetAttribute(attn_prefill_tcgen05_two_groups_kernel<HD, false, false>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem)
+    cudaError_t e = TWO_GROUPS ? cudaFuncSetAttribute(attn_prefill_tcgen05_two_groups_kernel<HD, false, false, false>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem)
                                : cudaFuncSetAttribute(attn_prefill_tcgen05_kernel<HD, KT>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
     if (TWO_GROUPS && e == cudaSuccess)
-      e = cudaFuncSetAttribute(attn_prefill_tcgen05_two_groups_kernel<HD, true, false>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+      e = cudaFuncSetAttribute(attn_prefill_tcgen05_two_groups_kernel<HD, true, false, false>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
     if (TWO_GROUPS && e == cudaSuccess)
-      e = cudaFuncSetAttribute(attn_prefill_tcgen05_two_groups_kernel<HD, false, true>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+      e = cudaFuncSetAttribute(attn_prefill_tcgen05_two_groups_kernel<HD, false, true, false>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+    if (TWO_GROUPS && e == cudaSuccess)
+      e = cudaFuncSetAttribute(attn_prefill_tcgen05_two_groups_kernel<HD, false, false, true>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
     ME_REQUIRE(e == cudaSuccess, "me_attn_prefill_tcgen05: cannot raise shared memory: %s", cudaGetErrorString(e));
     attr_set = true;
   }
@@ -828,14 +878,15 @@ int launch_ta(const void* q_map, const void* kv_map, void* out, int64_t out_row_
   // and 16% slower at 2,048, where the last round then holds long tiles.)
   dim3 grid(nkv * (nh / nkv / gp), num_tiles);
   if constexpr (TWO_GROUPS) {
-    auto kernel = bias_r1 ? attn_prefill_tcgen05_two_groups_kernel<HD, false, true>
-                : (keep_first > 0 || chunk > 0 || softcap > 0.f || sinks || pool_p > 0) ? attn_prefill_tcgen05_two_groups_kernel<HD, true, false>
-                                                                                        : attn_prefill_tcgen05_two_groups_kernel<HD, false, false>;
+    auto kernel = pairs ? attn_prefill_tcgen05_two_groups_kernel<HD, false, false, true>
+                : bias_r1 ? attn_prefill_tcgen05_two_groups_kernel<HD, false, true, false>
+                : (keep_first > 0 || chunk > 0 || softcap > 0.f || sinks || pool_p > 0) ? attn_prefill_tcgen05_two_groups_kernel<HD, true, false, false>
+                                                                                        : attn_prefill_tcgen05_two_groups_kernel<HD, false, false, false>;
     me_launch(kernel, grid, dim3(TA_THREADS), smem, stream, *reinterpret_cast<const CUtensorMap*>(q_map),
               *reinterpret_cast<const CUtensorMap*>(kv_map), (bf16*)out, out_row_stride, block_tables, bt_stride, cu_seqlens,
               context_lens, tiles, nh, nkv, gp, page_size, scale * 1.4426950408889634f, window, sink, gate, gate_stride, err,
               keep_first, chunk, softcap, sinks, *reinterpret_cast<const CUtensorMap*>(pool_p > 0 ? pool_map : kv_map), pooled_tables,
-              pbt_stride, pool_p, bias_r1, bias_r2, out_hd);
+              pbt_stride, pool_p, bias_r1, bias_r2, out_hd, pair);
   } else
     me_launch(attn_prefill_tcgen05_kernel<HD, KT>, grid, dim3(TA_THREADS), smem, stream, *reinterpret_cast<const CUtensorMap*>(q_map),
               *reinterpret_cast<const CUtensorMap*>(kv_map), (bf16*)out, out_row_stride, block_tables, bt_stride, cu_seqlens,
@@ -866,14 +917,15 @@ ME_API int me_attn_prefill_tcgen05_heads_per_block(int nh, int nkv, int hd, int 
 // block of pool_p tokens and its block tables; with a window a query at p also sees the blocks b with (b + 1) pool_p <=
 // p - window + 1 (0: none).  ``bias_r1``, ``bias_r2`` (float32 [nh], both or neither): r1 ln(1 + r2 (p - j)) is taken off the
 // scaled score of a key at j.  ``out_hd``: how many elements of a head leave (a multiple of 8; the cache's rows may be longer than the values);
-// rows of ``out`` hold nh * out_hd of them.  These seven are the kernel with two groups' alone.
+// rows of ``out`` hold nh * out_hd of them.  ``pairs``: heads 2h and 2h + 1 are joined into one output head (PAIRS above), and rows of
+// ``out`` hold nh / 2 * out_hd values.  These eight are the kernel with two groups' alone.
 ME_API int me_attn_prefill_tcgen05(const void* q_map, const void* kv_map, void* out, int64_t out_row_stride,
                                    const int* block_tables, int bt_stride, const int* cu_seqlens, const int* context_lens,
                                    const int* tiles, int num_tiles, int nh, int nkv, int hd, int page_size, float scale,
                                    int window, int key_tile, int sink, const float* gate, int64_t gate_stride, int* err,
                                    int keep_first, int chunk, float softcap, const float* sinks, const void* pool_map,
                                    const int* pooled_tables, int pbt_stride, int pool_p, const float* bias_r1, const float* bias_r2,
-                                   int out_hd, cudaStream_t stream) {
+                                   int out_hd, int pairs, float pair_lambda, float pair_gain, float pair_eps, cudaStream_t stream) {
   if (num_tiles == 0) return 0;
   const int gp = me_attn_prefill_tcgen05_heads_per_block(nh, nkv, hd, page_size);
   ME_REQUIRE(gp > 0, "me_attn_prefill_tcgen05: head_dim %d, %d/%d heads, pages of %d are not taken", hd, nh, nkv, page_size);
@@ -887,6 +939,9 @@ ME_API int me_attn_prefill_tcgen05(const void* q_map, const void* kv_map, void* 
   ME_REQUIRE(key_tile == 128 || (keep_first == 0 && chunk == 0 && softcap == 0.f && sinks == nullptr && pool_p == 0 && !bias_r1 && out_hd == hd),
              "me_attn_prefill_tcgen05: kept first keys, chunks, capped scores, learned sinks, pooled blocks, biases and short outputs need the key tile of 128");
   ME_REQUIRE(out_hd > 0 && out_hd <= hd && out_hd % 8 == 0 && !(gate && out_hd != hd), "me_attn_prefill_tcgen05: %d of %d output elements", out_hd, hd);
+  ME_REQUIRE(!pairs || (gp % 2 == 0 && key_tile == 128 && !gate && !sink && !sinks && softcap == 0.f && keep_first == 0 && chunk == 0 && pool_p == 0 && !bias_r1),
+             "me_attn_prefill_tcgen05: pairs of heads need an even group and go with a plain window at most");
+  const PairArgs pair = {pair_lambda, pair_gain, pair_eps};
   ME_REQUIRE((bias_r1 == nullptr) == (bias_r2 == nullptr) && !(bias_r1 && (softcap > 0.f || sinks || sink || pool_p > 0 || keep_first > 0 || chunk > 0)),
              "me_attn_prefill_tcgen05: a distance bias has two numbers a head and goes with a plain window at most");
   ME_REQUIRE(pool_p == 0 || (pool_p > 0 && pool_map && pooled_tables && window > 0 && keep_first == 0 && chunk == 0),
@@ -898,7 +953,7 @@ ME_API int me_attn_prefill_tcgen05(const void* q_map, const void* kv_map, void* 
   int rc;
 #define ME_TA_ARGS q_map, kv_map, out, out_row_stride, block_tables, bt_stride, cu_seqlens, context_lens, tiles, num_tiles, nh, nkv, gp, \
                    page_size, scale, window, sink, gate, gate_stride, err, keep_first, chunk, softcap, sinks, pool_map, pooled_tables, \
-                   pbt_stride, pool_p, bias_r1, bias_r2, out_hd, stream
+                   pbt_stride, pool_p, bias_r1, bias_r2, out_hd, pairs != 0, pair, stream
   if (hd == 64) rc = key_tile == 64 ? launch_ta<64, 64, false>(ME_TA_ARGS) : launch_ta<64, 128, true>(ME_TA_ARGS);
   else rc = key_tile == 64 ? launch_ta<128, 64, false>(ME_TA_ARGS) : launch_ta<128, 128, true>(ME_TA_ARGS);
 #undef ME_TA_ARGS

@@ -30,7 +30,7 @@ __device__ __forceinline__ bf16* dl_ptr(bf16* base, int row, int piece) {
 
 // X is bfloat16 [M][ldx].  With ``sumsq_in`` ([sumsq_parts][M], the sums of squares of the rows that X was made
 // from, over ``K`` columns) the results are multiplied by rsqrt(sum / K + eps) of their row.
-// EPI 0: Y[m][n] (bfloat16 or float32).  EPI 1: SiLU(gate) * up, bfloat16.
+// EPI 0: Y[m][n] (bfloat16 or float32), through activation ``act`` of common.cuh when that is not negative.  EPI 1: SiLU(gate) * up, bfloat16.
 // EPI 2: residual_out[m][n] += v, sumsq_out, and with ``next_w`` also xw_out[m][n] = residual_out[m][n] * next_w[n].
 template <int EPI, typename TO, int R /* weight rows of a strip: 16, or 8 with the upper half of the tile idle */>
 __global__ void __launch_bounds__(DL_MAX_WARPS * 32)
@@ -38,7 +38,7 @@ gemm_decode_kernel(const bf16* __restrict__ X, int64_t ldx, const float* __restr
                    const bf16* __restrict__ W, TO* __restrict__ Y, int64_t ldy, float* __restrict__ res_out,
                    float* __restrict__ sumsq_out, const float* __restrict__ next_w, bf16* __restrict__ xw_out, int M,
                    int N, int K, const unsigned char* __restrict__ ahead, unsigned long long ahead_bytes, float glu_limit,
-                   float glu_alpha, float glu_shift) {
+                   float glu_alpha, float glu_shift, int act) {
   extern __shared__ __align__(128) unsigned char dl_smem[];
   // The weights of the product that runs after this one are asked into L2 now: a decode step is a chain of
   // short dependent kernels, and without this the memory system idles while each waits for the one before.
@@ -205,7 +205,8 @@ gemm_decode_kernel(const bf16* __restrict__ X, int64_t ldx, const float* __restr
       const int m = idx / R, r = idx % R;
       const int n = strip * R + r;
       if (m >= M || n >= N) continue;
-      Y[(int64_t)m * ldy + n] = from_f<TO>(total(r, m) * row_scale[m]);
+      const float v = total(r, m) * row_scale[m];
+      Y[(int64_t)m * ldy + n] = from_f<TO>(act >= 0 ? act_apply<TO>(v, act) : v);
     }
   }
 }
@@ -214,7 +215,7 @@ template <int EPI, typename TO, int R>
 int launch_dl(int strips, int warps, cudaStream_t stream, const void* X, int64_t ldx, const float* sumsq_in, int sumsq_parts,
               float eps, const void* W, void* Y, int64_t ldy, float* res_out, float* sumsq_out, const float* next_w,
               void* xw_out, int M, int N, int K, const void* ahead, unsigned long long ahead_bytes, float glu_limit, float glu_alpha,
-              float glu_shift) {
+              float glu_shift, int act) {
   const size_t smem = (size_t)warps * (2 * 16 * DL_KW * sizeof(bf16) + 16 * 17 * sizeof(float));
   static size_t attr = 0;
   if (smem > attr) {
@@ -224,7 +225,7 @@ int launch_dl(int strips, int warps, cudaStream_t stream, const void* X, int64_t
   }
   me_launch(gemm_decode_kernel<EPI, TO, R>, dim3(strips), dim3(warps * 32), smem, stream, (const bf16*)X, ldx, sumsq_in,
             sumsq_parts, eps, (const bf16*)W, (TO*)Y, ldy, res_out, sumsq_out, next_w, (bf16*)xw_out, M, N, K,
-            (const unsigned char*)ahead, ahead_bytes, glu_limit, glu_alpha, glu_shift);
+            (const unsigned char*)ahead, ahead_bytes, glu_limit, glu_alpha, glu_shift, act);
   return 0;
 }
 }  // namespace
@@ -242,7 +243,7 @@ ME_API int me_gemm_decode_sumsq_parts(int N) { const int r = strip_rows(N); retu
 // epi 0: Y (y_dtype) [M][ldy]; epi 1: the gated epilogue g sigmoid(alpha g) (u + shift), g and u clamped by glu_limit when that
 // is positive (weight rows gate | up, N = columns of Y; SiLU-and-multiply is limit 0, alpha 1, shift 0);
 // epi 2: res_out [M][N] += X W^T, sumsq_out [me_gemm_decode_sumsq_parts(N)][M] and, with next_w [N], xw_out
-// bfloat16 [M][N] = res_out * next_w.
+// bfloat16 [M][N] = res_out * next_w; epi 3 + k: Y through activation k of common.cuh.
 // ahead (or null), ahead_bytes: memory that a later kernel will read (the next product's weights), asked into
 // L2 by this one; 16-byte aligned.
 ME_API int me_gemm_decode(int epi, const void* X, int64_t ldx, const float* sumsq_in, int sumsq_parts, float eps,
@@ -256,6 +257,8 @@ ME_API int me_gemm_decode(int epi, const void* X, int64_t ldx, const float* sums
   ME_REQUIRE(X != nullptr && (ldx * 2) % 16 == 0, "me_gemm_decode: X is missing or its rows are not 16-byte aligned");
   ME_REQUIRE(sumsq_in == nullptr || (sumsq_parts > 0 && sumsq_parts <= 192), "me_gemm_decode: sums of squares in %d parts (1..192)",
              sumsq_parts);
+  const int act = epi >= 3 && epi <= 3 + ACT_GELU_ERF ? epi - 3 : -1;
+  if (act >= 0) epi = 0;
   ME_REQUIRE(epi == 0 || epi == 1 || (epi == 2 && res_out != nullptr && sumsq_out != nullptr), "me_gemm_decode: epilogue %d", epi);
   ME_REQUIRE((next_w == nullptr) == (xw_out == nullptr) && (next_w == nullptr || epi == 2),
              "me_gemm_decode: the pre-weighted copy needs the residual epilogue, a weight and an output");
@@ -266,7 +269,7 @@ ME_API int me_gemm_decode(int epi, const void* X, int64_t ldx, const float* sums
   int rc = 1;
 #define ME_DL(EPI_, TO_, R_)                                                                                        \
   rc = launch_dl<EPI_, TO_, R_>(strips, warps, stream, X, ldx, sumsq_in, sumsq_parts, eps, W, Y, ldy, res_out, sumsq_out, \
-                                next_w, xw_out, M, N, K, ahead, ahead_bytes, glu_limit, glu_alpha, glu_shift)
+                                next_w, xw_out, M, N, K, ahead, ahead_bytes, glu_limit, glu_alpha, glu_shift, act)
   if (epi == 2) {
     if (rows == 8) ME_DL(2, float, 8); else ME_DL(2, float, 16);
   } else if (epi == 1) {

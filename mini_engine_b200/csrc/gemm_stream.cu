@@ -45,7 +45,7 @@ template <int XR> constexpr int gs_stages() { return XR == 8 ? 6 : 5; }
 __host__ __device__ __forceinline__ long long gs_first_stage(long long total, int nb, int b) { return total * b / nb; }
 __device__ __forceinline__ void consumers_sync() { asm volatile("bar.sync 1, %0;\n" ::"n"(GS_CONSUMERS) : "memory"); }
 
-// EPI 0: Y[m][n] (bfloat16 or float32).  EPI 1: SiLU(gate) * up, bfloat16 (a group is 64 gate rows and their 64 up
+// EPI 0: Y[m][n] (bfloat16 or float32), through activation ``act`` of common.cuh when that is not negative.  EPI 1: SiLU(gate) * up, bfloat16 (a group is 64 gate rows and their 64 up
 // rows).  EPI 2: residual_out[m][n] += v; sumsq_out[block][m] = the block's share of the new residual's sums of
 // squares; with ``next_w`` also xw_out[m][n] = residual_out[m][n] * next_w[n].
 // XR: rows of the X tile and of map_x's boxes (8 for up to 8 rows of X: the upper n8 tile then reads one chunk of zeros).
@@ -57,7 +57,7 @@ gemm_stream_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_const
                    const float* __restrict__ sumsq_in, int sumsq_parts, float eps, TO* __restrict__ Y, int64_t ldy,
                    float* __restrict__ res_out, float* __restrict__ sumsq_out, const float* __restrict__ next_w,
                    bf16* __restrict__ xw_out, int M, int N, int K, int groups, float* __restrict__ partials,
-                   int* __restrict__ flags, int* __restrict__ err, float glu_limit, float glu_alpha, float glu_shift) {
+                   int* __restrict__ flags, int* __restrict__ err, float glu_limit, float glu_alpha, float glu_shift, int act) {
   constexpr int STAGES = gs_stages<XR>(), STAGE_BYTES = gs_stage_bytes<XR>();
   constexpr int COLS = EPI == 1 ? GS_ROWS / 2 : GS_ROWS;         // output columns of a group
   extern __shared__ unsigned char gs_smem_raw[];
@@ -274,7 +274,7 @@ gemm_stream_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_const
                 sq += val * val;
                 if (xw_out != nullptr) xw_out[(int64_t)m * N + n] = __float2bfloat16(val * next_w[n]);
               } else {
-                Y[(int64_t)m * ldy + n] = from_f<TO>(val);
+                Y[(int64_t)m * ldy + n] = from_f<TO>(act >= 0 ? act_apply<TO>(val, act) : val);
               }
             }
           }
@@ -299,7 +299,7 @@ int gs_blocks(int groups, int n_its) {
 template <int EPI, typename TO, int XR>
 int launch_gs(cudaStream_t stream, const void* map_w, const void* map_x, const float* sumsq_in, int sumsq_parts, float eps, void* Y,
               int64_t ldy, float* res_out, float* sumsq_out, const float* next_w, void* xw_out, int M, int N, int K,
-              float* partials, int* flags, int* err, float glu_limit, float glu_alpha, float glu_shift) {
+              float* partials, int* flags, int* err, float glu_limit, float glu_alpha, float glu_shift, int act) {
   const size_t smem = (size_t)gs_stages<XR>() * gs_stage_bytes<XR>() + 1024;
   static bool attr_set = false;
   if (!attr_set) {
@@ -311,7 +311,7 @@ int launch_gs(cudaStream_t stream, const void* map_w, const void* map_x, const f
   me_launch(gemm_stream_kernel<EPI, TO, XR>, dim3(gs_blocks(groups, n_its)), dim3(GS_THREADS), smem, stream,
             *reinterpret_cast<const CUtensorMap*>(map_w), *reinterpret_cast<const CUtensorMap*>(map_x), sumsq_in, sumsq_parts, eps,
             (TO*)Y, ldy, res_out, sumsq_out, next_w, (bf16*)xw_out, M, N, K, groups, partials, flags, err, glu_limit, glu_alpha,
-            glu_shift);
+            glu_shift, act);
   return 0;
 }
 }  // namespace
@@ -342,15 +342,17 @@ ME_API int me_gemm_stream(int epi, const void* map_x, const float* sumsq_in, int
   ME_REQUIRE(map_x != nullptr && map_w != nullptr && err != nullptr && partials != nullptr && flags != nullptr,
              "me_gemm_stream: tensor maps, work buffers and the error word are required");
   ME_REQUIRE(sumsq_in == nullptr || sumsq_parts > 0, "me_gemm_stream: sums of squares in %d parts", sumsq_parts);
+  const int act = epi >= 3 && epi <= 3 + ACT_GELU_ERF ? epi - 3 : -1;
+  if (act >= 0) epi = 0;
   ME_REQUIRE(epi == 0 || epi == 1 || (epi == 2 && res_out != nullptr && sumsq_out != nullptr), "me_gemm_stream: epilogue %d", epi);
   ME_REQUIRE((next_w == nullptr) == (xw_out == nullptr) && (next_w == nullptr || epi == 2),
              "me_gemm_stream: the pre-weighted copy needs the residual epilogue, a weight and an output");
   int rc = 1;
 #define ME_GS(EPI_, TO_)                                                                                                      \
   rc = M <= 8 ? launch_gs<EPI_, TO_, 8>(stream, map_w, map_x, sumsq_in, sumsq_parts, eps, Y, ldy, res_out, sumsq_out, next_w,  \
-                                        xw_out, M, N, K, partials, flags, err, glu_limit, glu_alpha, glu_shift)                \
+                                        xw_out, M, N, K, partials, flags, err, glu_limit, glu_alpha, glu_shift, act)           \
               : launch_gs<EPI_, TO_, 16>(stream, map_w, map_x, sumsq_in, sumsq_parts, eps, Y, ldy, res_out, sumsq_out, next_w, \
-                                         xw_out, M, N, K, partials, flags, err, glu_limit, glu_alpha, glu_shift)
+                                         xw_out, M, N, K, partials, flags, err, glu_limit, glu_alpha, glu_shift, act)
   if (epi == 2) {
     ME_GS(2, float);
   } else if (epi == 1) {

@@ -86,7 +86,7 @@ __device__ __forceinline__ void write_rows(Load&& load, Fix&& fix, unsigned char
       fix(c, g);
       if (glu.act >= 0) {
 #pragma unroll
-        for (int j = 0; j < 32; ++j) g[j] = act_apply(g[j], glu.act);
+        for (int j = 0; j < 32; ++j) g[j] = act_apply<TO>(g[j], glu.act);
       }
     }
   };
@@ -864,15 +864,16 @@ ME_API int me_gemm_tcgen05_persistent(const void* map_a, const void* map_w, void
   if (M == 0 || N == 0) return 0;
   ME_REQUIRE(M > 0 && N > 0 && K > 0 && K % 8 == 0, "me_gemm_tcgen05_persistent: bad sizes M=%d N=%d K=%d (K must be a multiple of 8)", M, N, K);
   ME_REQUIRE(map_a != nullptr && map_w != nullptr && err != nullptr, "me_gemm_tcgen05_persistent: tensor maps and the error word are required");
-  ME_REQUIRE(epi == 0 || (epi == 1 && c_dtype == ME_BF16), "me_gemm_tcgen05_persistent: epilogue %d", epi);
+  ME_REQUIRE(epi == 0 || ((epi == 1 || (epi >= 2 && epi <= 2 + ACT_GELU_ERF)) && c_dtype == ME_BF16), "me_gemm_tcgen05_persistent: epilogue %d", epi);
   ME_REQUIRE(bn == 128 || bn == 256, "me_gemm_tcgen05_persistent: tile width %d is not 128 or 256", bn);
   GluParams glu;
   glu.limit = glu_limit, glu.alpha = glu_alpha, glu.shift = glu_shift;
+  glu.act = epi >= 2 ? epi - 2 : -1;
   int rc = 1;
 #define ME_TP_CASE(BN_)                                                                                  \
   if (bn == BN_) {                                                                                       \
     if (epi == 1) rc = launch_tp<BN_, 1, bf16>(map_a, map_w, C, ldc, M, N, K, err, stream, glu);         \
-    else if (c_dtype == ME_BF16) rc = launch_tp<BN_, 0, bf16>(map_a, map_w, C, ldc, M, N, K, err, stream); \
+    else if (c_dtype == ME_BF16) rc = launch_tp<BN_, 0, bf16>(map_a, map_w, C, ldc, M, N, K, err, stream, glu); \
     else rc = launch_tp<BN_, 0, float>(map_a, map_w, C, ldc, M, N, K, err, stream);                      \
   }
   ME_TP_CASE(128) ME_TP_CASE(256)
@@ -912,7 +913,7 @@ ME_API int me_gemm_tcgen05_shared(const void* map_a, const void* map_w, void* C,
 // map_a: X as [M][K], boxes 128 x 64, 128-byte swizzle; map_w: W as [rows][K], boxes
 // me_gemm_tcgen05_w_box_rows(bn, epi) x 64.  N counts output columns (epi 1: W has 2N rows, gate rows then up rows, and the
 // result is g sigmoid(alpha g) (u + shift) with g and u clamped by ``glu_limit`` when that is positive; SiLU-and-multiply is
-// limit 0, alpha 1, shift 0).
+// limit 0, alpha 1, shift 0; epi 2 + k: activation k of common.cuh on bfloat16 results).
 // bn is the accumulator's width: 64, 128 or 256.  ``splits`` > 1: the K range is shared out over that many blocks a tile, whose
 // float32 partial results lie ``split_stride`` elements apart (me_gemm_tcgen05_splits says how many there will be).
 ME_API int me_gemm_tcgen05(const void* map_a, const void* map_w, void* C, int c_dtype, int64_t ldc, int M, int N,
@@ -921,7 +922,7 @@ ME_API int me_gemm_tcgen05(const void* map_a, const void* map_w, void* C, int c_
   if (M == 0 || N == 0) return 0;
   ME_REQUIRE(M > 0 && N > 0 && K > 0 && K % 8 == 0, "me_gemm_tcgen05: bad sizes M=%d N=%d K=%d (K must be a multiple of 8)", M, N, K);
   ME_REQUIRE(map_a != nullptr && map_w != nullptr && err != nullptr, "me_gemm_tcgen05: tensor maps and the error word are required");
-  ME_REQUIRE(epi == 0 || (epi == 1 && c_dtype == ME_BF16), "me_gemm_tcgen05: epilogue %d", epi);
+  ME_REQUIRE(epi == 0 || ((epi == 1 || (epi >= 2 && epi <= 2 + ACT_GELU_ERF)) && c_dtype == ME_BF16), "me_gemm_tcgen05: epilogue %d", epi);
   ME_REQUIRE((M + TG_BM - 1) / TG_BM <= 65535, "me_gemm_tcgen05: M=%d is too large", M);
   ME_REQUIRE(splits >= 1 && splits <= 64 && (splits == 1 || (epi == 0 && c_dtype == ME_F32)),
              "me_gemm_tcgen05: %d splits (they need float32 results and no epilogue)", splits);
@@ -929,13 +930,14 @@ ME_API int me_gemm_tcgen05(const void* map_a, const void* map_w, void* C, int c_
   const int out_cols = epi == 1 ? bn / 2 : bn;
   GluParams glu;
   glu.limit = glu_limit, glu.alpha = glu_alpha, glu.shift = glu_shift;
+  glu.act = epi >= 2 ? epi - 2 : -1;
   const bool deep = (int64_t)((N + out_cols - 1) / out_cols) * ((M + TG_BM - 1) / TG_BM) * me_gemm_tcgen05_splits(K, splits) <= me_sm_count();
   int rc = 1;
 #define ME_TG_CASE(BN_)                                                                                              \
   if (bn == BN_) {                                                                                                   \
     if (epi == 1) rc = launch_tg<BN_, 1, bf16, false>(map_a, map_w, C, ldc, M, N, K, 1, 0, err, stream, glu);        \
-    else if (c_dtype == ME_BF16) rc = deep ? launch_tg<BN_, 0, bf16, true>(map_a, map_w, C, ldc, M, N, K, 1, 0, err, stream)   \
-                                           : launch_tg<BN_, 0, bf16, false>(map_a, map_w, C, ldc, M, N, K, 1, 0, err, stream); \
+    else if (c_dtype == ME_BF16) rc = deep ? launch_tg<BN_, 0, bf16, true>(map_a, map_w, C, ldc, M, N, K, 1, 0, err, stream, glu)   \
+                                           : launch_tg<BN_, 0, bf16, false>(map_a, map_w, C, ldc, M, N, K, 1, 0, err, stream, glu); \
     else rc = deep ? launch_tg<BN_, 0, float, true>(map_a, map_w, C, ldc, M, N, K, splits, split_stride, err, stream)          \
                    : launch_tg<BN_, 0, float, false>(map_a, map_w, C, ldc, M, N, K, splits, split_stride, err, stream);        \
   }

@@ -44,7 +44,7 @@ def tidenex_plan(cfg: TidenexConfig) -> ModelPlan:
                     "out_scale": m["right_scale"]}))]})
         ffn = None
         if layer["mlp"] is not None:
-            ffn = PartSpec("activation_mlp", {"hidden_size": W, "intermediate_size": layer["mlp"]["ff"], "activation": "gelu"})
+            ffn = PartSpec("activation_mlp", {"hidden_size": W, "intermediate_size": layer["mlp"]["ff"], "activation": "gelu", "in_product": True})
         blocks.append(BlockSpec(mixer=mixer, feed_forward=ffn, kind="pre_norm", mixer_norm=norm("norm1"), feed_forward_norm=norm("norm2"),
                                 mixer_prefix="mix.", feed_forward_prefix="mlp.", mixer_norm_prefix="", feed_forward_norm_prefix=""))
     # every run of a layer has a cache slot of its own: a looped layer keeps one cache or state per pass

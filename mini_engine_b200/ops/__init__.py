@@ -47,7 +47,7 @@ _PROTOS = {
     "me_gemm_tcgen05": [_P, _P, _P, _I, _L, _I, _I, _I, _I, _I, _I, _L, _F, _F, _F, _P, _P],
     "me_gemm_tcgen05_persistent": [_P, _P, _P, _I, _L, _I, _I, _I, _I, _I, _F, _F, _F, _P, _P],
     "me_gemm_tcgen05_shared": [_P, _P, _P, _I, _L, _I, _I, _I, _I, _I, _P, _P, _P, _P],
-    "me_attn_prefill_tcgen05": [_P, _P, _P, _L, _P, _I, _P, _P, _P, _I, _I, _I, _I, _I, _F, _I, _I, _I, _P, _L, _P, _I, _I, _F, _P, _P, _P, _I, _I, _P, _P, _I, _P],
+    "me_attn_prefill_tcgen05": [_P, _P, _P, _L, _P, _I, _P, _P, _P, _I, _I, _I, _I, _I, _F, _I, _I, _I, _P, _L, _P, _I, _I, _F, _P, _P, _P, _I, _I, _P, _P, _I, _I, _F, _F, _F, _P],
     "me_tma_encode_2d": [_P, _P, ctypes.c_uint64, ctypes.c_uint64, ctypes.c_uint64, ctypes.c_uint32, ctypes.c_uint32, _I],
     "me_attn_prefill": [_P, _L, _P, _L, _P, _P, _I, _P, _P, _P, _I, _I, _I, _I, _I, _F, _I, _P],
     "me_sample": [_P, _L, _P, _P, _P, _P, _I, _I, _P, _P, _P],
@@ -58,7 +58,7 @@ _PROTOS = {
     "me_rope_table": [_P, _P, _I, _I, _P, _P],
     "me_sink_attn": [_P, _I, _L, _P, _L, _P, _L, _P, _P, _I, _P, _P, _P, _I, _I, _I, _I, _I, _I, _I, _I, _F, _I, _I, _P, _F, _I, _I, _P, _P, _I, _I, _P, _P, _P],
     "me_parallel_norm": [_P, _P, _P, _I, _P, _P, _P, _P, _P, _P, _P, _P, _I, _P, _I, _I, _F, _P, _P, _I, _I, _P, _I, _F, _P],
-    "me_attn_prep": [_P, _L, _P, _P, _P, _I, _F, _P, _I, _P, _P, _P, _P, _I, _P, _I, _I, _I, _I, _I, _I, _I, _I, _I, _P, _I, _F, _F, _F, _P],
+    "me_attn_prep": [_P, _L, _P, _P, _P, _I, _F, _P, _I, _P, _P, _P, _I, _P, _I, _I, _I, _I, _I, _I, _I, _I, _I, _P, _I, _F, _F, _F, _P],
     "me_diff_combine": [_P, _I, _L, _P, _I, _L, _I, _I, _I, _I, _F, _F, _F, _P],
     "me_gla_decay": [_P, _L, _I, _I, _P, _I, _P, _F, _P, _I, _I, _P],
     "me_gla_scan": [_P, _L, _I, _I, _I, _P, _P, _P, _P, _P, _P, _I, _I, _I, _I, _F, _P, _I, _I, _P, _P, _P, _P, _P],
@@ -448,9 +448,9 @@ def decode_linear(weight: torch.Tensor, x: torch.Tensor, *, out: Optional[torch.
     "residual": residual_out += x W^T; ``sumsq_out`` [decode_linear_sumsq_parts(N), M] gets the new residual's sums
     of squares per strip of columns, and with ``next_norm`` = (weight float32 [N], xw bfloat16 [M, N]) xw gets the new
     residual times that weight).  ``fetch_ahead``: a tensor that a later kernel reads (the next product's weight);
-    this kernel asks it into L2.  ``glu`` = (limit, alpha, shift) with "silu_mul": the gated epilogue in its general form,
+    this kernel asks it into L2.  ``epilogue`` may also be a key of ``ACTIVATIONS``: that function of the results.  ``glu`` = (limit, alpha, shift) with "silu_mul": the gated epilogue in its general form,
     g sigmoid(alpha g) (u + shift) with g = min(gate, limit), u = clamp(up, -limit, limit) when limit > 0."""
-    epi = {"none": 0, "silu_mul": 1, "residual": 2}[epilogue]
+    epi = 3 + ACTIVATIONS[epilogue] if epilogue in ACTIVATIONS else {"none": 0, "silu_mul": 1, "residual": 2}[epilogue]
     _need(glu is None or epi == 1, "decode_linear: the gate's parameters go with the gated epilogue")
     glu_params = tuple(float(v) for v in (glu or (0.0, 1.0, 0.0)))
     M, K = x.shape
@@ -585,19 +585,22 @@ def linear_tcgen05(x: torch.Tensor, weight: torch.Tensor, out: torch.Tensor, epi
     """The tcgen05 product of csrc/gemm_tcgen05.cu: TMA -> swizzled shared memory -> tcgen05.mma -> tensor memory.
 
     ``glu`` = (limit, alpha, shift) with the "silu_mul" epilogue: the gated epilogue in its general form,
-    g sigmoid(alpha g) (u + shift) with g = min(gate, limit), u = clamp(up, -limit, limit) when limit > 0.
+    g sigmoid(alpha g) (u + shift) with g = min(gate, limit), u = clamp(up, -limit, limit) when limit > 0.  ``epilogue`` may also
+    be a key of ``ACTIVATIONS``: that function of the results (bfloat16).
 
     With ``splits`` > 1 ``out`` is float32 [tcgen05_splits(K, splits), M, N]: partial results over parts of K.
     ``share``: the form that cuts the stages of all tiles into one equal range an SM (``tile_n`` 128 or 256)."""
     M, K = x.shape
-    epi = {"none": 0, "silu_mul": 1}[epilogue]
+    act = 2 + ACTIVATIONS[epilogue] if epilogue in ACTIVATIONS else 0       # (as for no epilogue, but for the call itself)
+    epi = 0 if act else {"none": 0, "silu_mul": 1}[epilogue]
+    _need(not act or (splits == 1 and out.dtype == torch.bfloat16), "linear_tcgen05: an activation goes with whole sums and bfloat16 results")
     _need(glu is None or epi == 1, "linear_tcgen05: the gate's parameters go with the gated epilogue")
     glu_params = tuple(float(v) for v in (glu or (0.0, 1.0, 0.0)))
     N = weight.shape[0] // 2 if epi else weight.shape[0]
     if share is None and tile_n is None and persistent is None and splits == 1 and tcgen05_share == "auto" and tcgen05_takes(x, weight):
         share = tcgen05_share_pays(M, N, K, epi)
-    if share and glu is not None:
-        share = False                 # (the work-sharing form has no gated epilogue)
+    if share and (glu is not None or act):
+        share = False                 # (the work-sharing form has no gated epilogue in its general form and no activation)
     if share:
         bn = tile_n or 256
         _need(tcgen05_takes(x, weight) and splits == 1 and bn in (128, 256), "linear_tcgen05: operands not taken by the work-sharing form")
@@ -640,10 +643,10 @@ def linear_tcgen05(x: torch.Tensor, weight: torch.Tensor, out: torch.Tensor, epi
         persistent = False
     if persistent and splits == 1 and bn >= 128:
         _call("me_gemm_tcgen05_persistent", matrix_tensor_map(x, 128).ptr, matrix_tensor_map(weight, box_w).ptr, out.data_ptr(),
-              _dt(out), ldc, M, N, K, epi, bn, *glu_params, err.data_ptr(), _stream())
+              _dt(out), ldc, M, N, K, act or epi, bn, *glu_params, err.data_ptr(), _stream())
         return
     _call("me_gemm_tcgen05", matrix_tensor_map(x, 128).ptr, matrix_tensor_map(weight, box_w).ptr, out.data_ptr(), _dt(out),
-          ldc, M, N, K, epi, bn, splits, split_stride, *glu_params, err.data_ptr(), _stream())
+          ldc, M, N, K, act or epi, bn, splits, split_stride, *glu_params, err.data_ptr(), _stream())
 
 
 def tcgen05_splits(K: int, splits: int) -> int:
@@ -668,6 +671,12 @@ def tcgen05_split_plan(M: int, N: int, K: int) -> tuple[int, int]:
     want = max(1, min(4, 256 // max(tiles, 1), K // 512))
     parts = tcgen05_splits(K, want)
     return (bn, parts) if parts >= 2 and tcgen05_splits(K, parts) == parts else (0, 1)
+
+
+def linear_activation_takes(x: torch.Tensor, weight: torch.Tensor, out: Optional[torch.Tensor], err: Optional[torch.Tensor]) -> bool:
+    """Whether ``linear`` takes a key of ``ACTIVATIONS`` as epilogue for these operands: the tcgen05 kernels do."""
+    return (err is not None and use_tcgen05_gemm and skinny_splits(x.shape[0], x.shape[1], x, weight) == 0 and tcgen05_takes(x, weight)
+            and (out is None or out.dtype == torch.bfloat16))
 
 
 def linear(x: torch.Tensor, weight: torch.Tensor, out: torch.Tensor, epilogue: str = "none",
@@ -696,6 +705,11 @@ def linear(x: torch.Tensor, weight: torch.Tensor, out: torch.Tensor, epilogue: s
     M, K = x.shape
     _need(weight.dim() == 2 and weight.shape[1] == K and weight.is_contiguous(), "linear: weight shape")
     _need(x.stride(1) == 1 and out.stride(1) == 1, "linear: rows must be contiguous")
+    if epilogue in ACTIVATIONS:
+        _need(linear_activation_takes(x, weight, out, err), "linear: no kernel of this shape applies an activation to its results")
+        linear_tcgen05(x, weight, out, epilogue, err)
+        _remember(key, sig, before)
+        return
     epi = {"none": 0, "silu_mul": 1}[epilogue]
     N = weight.shape[0] // 2 if epi else weight.shape[0]
     _need(tuple(out.shape) == (M, N), f"linear: output is {tuple(out.shape)}, expected {(M, N)}")
@@ -851,7 +865,7 @@ def attention_prefill_tcgen05(qkv, out, num_heads, num_kv_heads, head_dim, pool,
                               scale, window, tiles=None, num_tiles=None, key_tile: int = 0, sink: bool = False,
                               gate: Optional[torch.Tensor] = None, keep_first: int = 0, chunk: int = 0, softcap: float = 0.0,
                               sinks: Optional[torch.Tensor] = None, pooled: Optional[tuple] = None, bias: Optional[tuple] = None,
-                              out_dim: int = 0) -> None:
+                              out_dim: int = 0, pairs: Optional[tuple[float, float, float]] = None) -> None:
     """The tcgen05 / tensor-memory prefill kernel (bfloat16, head_dim 64 or 128, page sizes dividing 128) over
     tiles of 128 / heads-per-block tokens; Q, K and V arrive by tensor-map loads.  ``sink``: one more term, exp(0), in
     the softmax's denominator; ``gate``: float32 rows of pre-activations whose sigmoid multiplies the output.
@@ -860,7 +874,7 @@ def attention_prefill_tcgen05(qkv, out, num_heads, num_kv_heads, head_dim, pool,
     exp(sinks[head]); ``pooled`` = (cache, block tables, P): the blocks of P tokens in front of the window, one row each in a
     second cache of the same layout; ``bias`` = (r1, r2), float32 [heads] each: r1 ln(1 + r2 (p - j)) is taken off the scaled score
     of a key at distance p - j; ``out_dim`` (0: all): how many elements of every head leave, ``out`` then holds
-    heads * out_dim columns (all of these in the kernel with the key tile of 128 only)."""
+    heads * out_dim columns; ``pairs`` = (lambda, gain, eps): heads 2h and 2h + 1 leave joined as ``diff_combine`` joins them (all of these in the kernel with the key tile of 128 only)."""
     gp = prefill_tcgen05_heads_per_block(num_heads, num_kv_heads, head_dim, page_size)
     _need(gp > 0 and qkv.dtype == torch.bfloat16 and qkv.is_contiguous() and qkv.data_ptr() % 16 == 0,
           "attention_prefill_tcgen05: shape or dtype not taken by the kernel")
@@ -874,7 +888,7 @@ def attention_prefill_tcgen05(qkv, out, num_heads, num_kv_heads, head_dim, pool,
           meta.error_flag.data_ptr(), int(keep_first or 0), int(chunk or 0), float(softcap or 0.0), _ptr(sinks),
           kv_tensor_map(pooled[0], page_size).ptr if pooled else 0, pooled[1].data_ptr() if pooled else 0,
           pooled[1].stride(0) if pooled else 0, int(pooled[2]) if pooled else 0, _ptr(bias[0]) if bias else 0, _ptr(bias[1]) if bias else 0,
-          int(out_dim), _stream())
+          int(out_dim), 1 if pairs else 0, *(float(v) for v in (pairs or (0.0, 0.0, 0.0))), _stream())
 
 
 use_tcgen05_attention = True   # False: portions of prompts use the mma.sync kernel instead (a switch for comparisons)
@@ -1425,12 +1439,12 @@ def attn_prep(proj: torch.Tensor, bias: Optional[torch.Tensor], q_norm: Optional
               norm: Optional[str], eps: float, freq: Optional[torch.Tensor], positions: torch.Tensor,
               slot_mapping: Optional[torch.Tensor], q_out: torch.Tensor, pool: Optional[torch.Tensor], page_size: int,
               num_heads: int, num_kv_heads: int, dim: int, vdim: int, q_scale: Optional[torch.Tensor] = None,
-              own_kv: bool = True, maps: int = 1, angles: Optional[torch.Tensor] = None,
+              own_kv: bool = True, maps: int = 1,
               temperature: Optional[tuple[float, float]] = None, v_scale: float = 1.0) -> None:
     """From the packed float32 projections q|k|v (the leading columns of ``proj``; q alone with ``own_kv`` False): bias, a weighted RMS norm of every q and k
     head in front of the rotation (``norm`` "before"), one over the whole q and the whole k of a token ("row", with a weight for every value)
     or a plain one behind it ("after"), the rotation of element i with
-    element i + len(freq) by position x ``freq`` (float64 frequencies; ``angles``: the step's cosines and sines, ``rope_table``), queries to ``q_out`` and keys and values into the
+    element i + len(freq) by position x ``freq`` (float64 frequencies), queries to ``q_out`` and keys and values into the
     cache rows that ``slot_mapping`` names (see csrc/attn_prep.cu).  ``q_scale`` (float32 [heads]): every query head is
     multiplied by its number at the end.  ``temperature`` = (coef, every): q is multiplied by 1 + coef ln(floor((p + 1) / every) + 1).
     ``v_scale`` multiplies the values.  ``maps`` 2: every q and k head has two maps of ``dim`` elements; ``q_out`` then has a row for
@@ -1449,8 +1463,6 @@ def attn_prep(proj: torch.Tensor, bias: Optional[torch.Tensor], q_norm: Optional
                   for w, n in list(zip((q_norm, k_norm), sizes))[:2 if own_kv else 1]),
               "attn_prep: a weighted norm needs float32 weights, [dim] in front of the rotation or one for every value of the row")
     _need(freq is None or (freq.dtype == torch.float64 and freq.is_contiguous() and 2 * freq.numel() <= dim), "attn_prep: freq must be float64 [<= dim / 2]")
-    _need(angles is None or (freq is not None and angles.dtype == torch.float32 and angles.is_contiguous() and angles.numel() == 2 * T * freq.numel()),
-          "attn_prep: angles must be float32 [T, len(freq), 2]")
     rows = num_heads * maps
     _need(q_out.is_contiguous() and q_out.shape[0] == T and q_out.shape[1] % rows == 0 and q_out.shape[1] // rows >= maps * dim,
           "attn_prep: query output shape")
@@ -1461,7 +1473,7 @@ def attn_prep(proj: torch.Tensor, bias: Optional[torch.Tensor], q_norm: Optional
     rot = 2 * freq.numel() if freq is not None else 0
     coef, every = temperature if temperature is not None else (0.0, 0.0)
     _call("me_attn_prep", proj.data_ptr(), proj.stride(0), _ptr(bias), _ptr(q_norm), _ptr(k_norm), {None: 0, "before": 1, "after": 2, "row": 3}[norm],
-          float(eps), _ptr(freq) if rot else 0, rot, _ptr(angles) if rot else 0, positions.data_ptr(), _ptr(slot_mapping), q_out.data_ptr(),
+          float(eps), _ptr(freq) if rot else 0, rot, positions.data_ptr(), _ptr(slot_mapping), q_out.data_ptr(),
           q_out.shape[1] // rows, _ptr(pool), _dt(q_out), pool.shape[-1] if pool is not None else 0, page_size, num_heads, num_kv_heads, dim, vdim,
           maps, T, _ptr(q_scale), 1 if own_kv else 0, float(coef), float(every), float(v_scale), _stream())
 
@@ -1587,31 +1599,31 @@ def sink_attention(q: torch.Tensor, gate: Optional[torch.Tensor], out: torch.Ten
     fast = (use_sink_attention_mma and q.dtype == torch.bfloat16 and (dim == vdim == HD or padded) and HD in (64, 128)
             and meta.error_flag is not None and q.is_contiguous() and q.data_ptr() % 16 == 0)
     extras = dict(keep_first=keep_first, chunk=chunk or 0, softcap=softcap or 0.0, sinks=sinks, bias=bias, out_dim=vdim)
-    joined = out                                        # with pairs: what the two maps are joined into, from row joined_from on
-    joined_from = 0
+    joined_from = 0                                     # with pairs: the rows from here on that diff_combine joins
     if fast and decodes and (not (masked or pooled) or (page_size >= 8 and DECODE_PARTITION % page_size == 0)):
         attention_decode(q, out, num_heads, num_kv_heads, HD, pool, page_size, block_tables, meta, scale, window, sink=sink, gate=gate,
                          pooled=pooled, pairs=pairs, **extras)
         joined_from, decodes = decodes, 0
-    if pairs and (decodes or meta.num_tiles > 0):
-        out = meta.workspace("attn_maps", (T, num_heads * vdim), q.dtype)
     if (fast and meta.num_tiles > 0 and use_tcgen05_attention and prefill_tcgen05_heads_per_block(num_heads, num_kv_heads, HD, page_size) > 0
             and vdim % 8 == 0 and out.stride(0) % 8 == 0 and out.data_ptr() % 16 == 0):
         attention_prefill_tcgen05(q, out, num_heads, num_kv_heads, HD, pool, page_size, block_tables, meta, scale, window,
-                                  sink=sink, gate=gate, pooled=pooled, **extras)
+                                  sink=sink, gate=gate, pooled=pooled, pairs=pairs, **extras)
         tiles_left = False
     tiles, n_tiles = meta.tile_lists[SINK_ATTN_TILE_Q]
     if not tiles_left:
         n_tiles = 0
     if decodes or n_tiles:
+        joined = out
+        if pairs:
+            out = meta.workspace("attn_maps", (T, num_heads * vdim), q.dtype)
         _call("me_sink_attn", q.data_ptr(), _dt(q), q.stride(0), _ptr(gate), gate.stride(0) if gate is not None else 0, out.data_ptr(),
               out.stride(0), pool.data_ptr(), block_tables.data_ptr(), block_tables.stride(0), meta.cu_seqlens.data_ptr(),
               meta.context_lens.data_ptr(), tiles.data_ptr(), n_tiles, decodes, num_heads, num_kv_heads, dim, vdim, HD, page_size,
               float(scale), int(window or 0), 1 if sink else 0, _ptr(sinks), float(softcap or 0.0), int(keep_first or 0),
               int(chunk or 0), pooled[0].data_ptr() if pool_p else 0, pooled[1].data_ptr() if pool_p else 0,
               pooled[1].stride(0) if pool_p else 0, pool_p, _ptr(bias[0]) if bias else 0, _ptr(bias[1]) if bias else 0, _stream())
-    if pairs and out is not joined:
-        diff_combine(out, joined, num_heads // 2, vdim, *pairs, first=joined_from)
+        if pairs:
+            diff_combine(out, joined, num_heads // 2, vdim, *pairs, first=joined_from)
 
 
 def moe_route(logits: torch.Tensor, bias: Optional[torch.Tensor], top: int, idx: torch.Tensor, weights: torch.Tensor) -> None:

@@ -77,8 +77,7 @@ class DifferentialAttention(Mixer):
         q = ctx.buffer("attn_q", (T, 2 * H * self.row), ctx.act_dtype)
         rotated = self.rope is not None and self.rope.rotary_dim > 0
         ops.attn_prep(proj, None, None, None, None, self.norm_eps, self.rope.freq if rotated else None, ctx.positions,
-                      kv.slot_mapping if call.writes_cache else None, q, kv.pool, kv.page_size, H, G, D, V, maps=2,
-                      angles=self.rope.angles_of_step(ctx, T) if rotated else None)
+                      kv.slot_mapping if call.writes_cache else None, q, kv.pool, kv.page_size, H, G, D, V, maps=2)
         out = ctx.buffer("attn_out", (T, H * V), ctx.act_dtype)
         ops.sink_attention(q, None, out, kv.pool, kv.page_size, kv.block_tables, ctx.attn_meta, 2 * H, G, self.row, V, self.scale,
                            self.window, False, padded=True, pairs=(self.lam, 1.0 - self.diff, self.norm_eps))

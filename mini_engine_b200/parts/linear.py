@@ -50,8 +50,13 @@ class Linear(Part):
         return self.weight
 
     def fuses(self, x, ctx, activation: str) -> bool:
-        """Whether this product's kernel for a step of this shape applies ``activation`` to its results itself."""
-        return False
+        """Whether this product's kernel for a step of this shape applies ``activation`` (a key of ``ops.ACTIVATIONS``) to its
+        results itself: the decode products and the tcgen05 kernels do, in bfloat16."""
+        if isinstance(x, PendingNorm) or activation not in ops.ACTIVATIONS or ctx.act_dtype != torch.bfloat16 or x.dtype != torch.bfloat16:
+            return False
+        if ops.decode_linear_takes(x.shape[0], self.in_features, self.weight, False):
+            return x.stride(0) % 8 == 0 and x.data_ptr() % 16 == 0
+        return ops.linear_activation_takes(x, self.weight, None, ctx.error_flag)
 
     def forward(self, x, ctx, out_name: str, *, out_dtype: Optional[torch.dtype] = None,
                 epilogue: str = "none", may_split: bool = False, residual: Optional[torch.Tensor] = None,

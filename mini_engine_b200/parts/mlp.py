@@ -42,12 +42,16 @@ class SwiGLU(FeedForward):
 
 
 class ActivationMLP(FeedForward):
-    """``down(act(up(x)))`` with an element-wise activation (a key of ``ops.ACTIVATIONS``; "relu_squared" is max(z, 0)^2)."""
+    """``down(act(up(x)))`` with an element-wise activation (a key of ``ops.ACTIVATIONS``; "relu_squared" is max(z, 0)^2).
+    ``in_product``: where a kernel of the first product can, it applies the activation to its float32 sums itself; else (and by
+    default) the activation is a pass of its own over the product's results in the working dtype."""
     capturable = True
 
-    def __init__(self, hidden_size: int, intermediate_size: int, activation: str = "relu_squared", up: str = "up", down: str = "down"):
+    def __init__(self, hidden_size: int, intermediate_size: int, activation: str = "relu_squared", up: str = "up", down: str = "down",
+                 in_product: bool = False):
         super().__init__()
         from .. import ops
+        self.in_product = in_product
         if activation not in ops.ACTIVATIONS:
             raise ValueError(f"unknown activation {activation!r}; known: {sorted(ops.ACTIVATIONS)}")
         self.hidden_size, self.intermediate_size, self.activation = hidden_size, intermediate_size, activation
@@ -62,8 +66,9 @@ class ActivationMLP(FeedForward):
 
     def forward(self, x, ctx, out_name: str = "ffn_out"):
         from .. import ops
-        z = self.up.forward(x, ctx, out_name + "_up", epilogue=self.activation if self.up.fuses(x, ctx, self.activation) else "none")
-        if not self.up.fuses(x, ctx, self.activation):
+        fused = self.in_product and self.up.fuses(x, ctx, self.activation)
+        z = self.up.forward(x, ctx, out_name + "_up", epilogue=self.activation if fused else "none", fetch_ahead=self.down.weight)
+        if not fused:
             act = ctx.buffer(out_name + "_act", tuple(z.shape), ctx.act_dtype)
             ops.activation(z, act, self.activation)
             z = act

@@ -125,9 +125,6 @@ class FrequencyRotary(PositionEncoding):
     def finalize(self, dtype, device):
         self.freq = torch.tensor(self.frequencies(), dtype=torch.float64).contiguous().to(device)
 
-    def angles_of_step(self, ctx, T: int):
-        return _angles_of_step(self, self.freq, ctx, T)
-
 
 register_position_encoding("rope", RotaryEmbedding)
 register_position_encoding("rope_frequencies", FrequencyRotary)

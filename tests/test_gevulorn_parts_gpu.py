@@ -307,12 +307,13 @@ def test_a_large_sink_takes_the_weight_and_is_neither_scaled_nor_capped(dtype, D
     (4, 2, 16, 24, 8, "after", False, None), (3, 1, 10, 9, 10, "before", True, (4.0, 1.0, 4.0, 64)),
     (2, 2, 64, 64, 32, "before", True, (8.0, 1.0, 4.0, 512)), (6, 2, 40, 40, 40, "after", False, None),
     (2, 1, 12, 20, 0, None, True, None), (1, 1, 8, 8, 8, None, False, None)])
-def test_bias_norms_rotation_and_cache_write(dtype, H, G, D, V, rot, norm, bias, scaling):
+@pytest.mark.parametrize("T", [37, 150])
+def test_bias_norms_rotation_and_cache_write(dtype, H, G, D, V, rot, norm, bias, scaling, T):
     """Far positions (the angle is reduced before its sine), rows written to shuffled cache places, values untouched."""
     ops = _ops()
-    dt, T, ps, eps = DT[dtype], 37, 8, 1e-5
+    dt, ps, eps = DT[dtype], 8, 1e-5
     C = H * D + G * (D + V)
-    proj = torch.randn(T, C + 5, generator=g(1)) * 2                       # columns beyond q|k|v belong to someone else
+    proj = torch.randn(T, C + (5 if T < 100 else 4), generator=g(1)) * 2   # columns beyond q|k|v belong to someone else
     b = torch.randn(C, generator=g(2)) if bias else None
     qw, kw = torch.rand(D, generator=g(3)) + 0.5, torch.rand(D, generator=g(4)) + 0.5
     positions = torch.tensor([0, 1, 2, 3, 70001, 1 << 20] + list(range(500, 500 + T - 6)), dtype=torch.int32)
@@ -326,8 +327,8 @@ def test_bias_norms_rotation_and_cache_write(dtype, H, G, D, V, rot, norm, bias,
     if norm == "after":
         q, k = plain.unit_rms(q, eps), plain.unit_rms(k, eps)
     HD = max(D, V)
-    pool = torch.zeros(8, 2, G, ps, HD, dtype=dt, device=DEV)
-    slots = torch.randperm(8 * ps, generator=g(5))[:T].to(torch.int32)
+    pool = torch.zeros(20, 2, G, ps, HD, dtype=dt, device=DEV)
+    slots = torch.randperm(20 * ps, generator=g(5))[:T].to(torch.int32)
     q_out = torch.empty(T, H * D, dtype=dt, device=DEV)
     ops.attn_prep(proj.to(DEV), b.to(DEV) if bias else None, qw.to(DEV) if norm == "before" else None,
                   kw.to(DEV) if norm == "before" else None, norm, eps,

@@ -278,13 +278,15 @@ def test_bias_at_long_distances():
 
 # ---- between the projection and the attention -----------------------------------------------------------
 @pytest.mark.parametrize("dtype", ["float32", "bfloat16"])
-@pytest.mark.parametrize("H, G, D, V", [(4, 2, 16, 24), (3, 1, 10, 9), (2, 2, 64, 64), (5, 5, 40, 72), (1, 1, 200, 8)])
-def test_norm_over_the_whole_projection_temperature_and_scaled_values(dtype, H, G, D, V):
-    """Heads of very different size (a norm by head would make them equal), positions at and around the temperature's steps, rows
+@pytest.mark.parametrize("H, G, D, V", [(4, 2, 16, 24), (3, 1, 10, 9), (2, 2, 64, 64), (5, 5, 40, 72), (1, 1, 200, 8),
+                                         (32, 8, 128, 128), (6, 2, 100, 132), (20, 10, 36, 8), (48, 48, 4, 8)])
+@pytest.mark.parametrize("extra", [5, 8])
+def test_norm_over_the_whole_projection_temperature_and_scaled_values(dtype, H, G, D, V, extra):
+    """Heads of very different size (a norm by head would make them equal), rows that can be read four values at a time and rows that cannot, positions at and around the temperature's steps, rows
     filled with zeros up to their width."""
     ops, dt, T, ps, eps = _ops(), DT[dtype], 41, 8, 1e-5
     C = H * D + G * (D + V)
-    proj = torch.randn(T, C + 5, generator=g(1)) * 2                       # columns beyond q|k|v belong to someone else
+    proj = torch.randn(T, C + extra, generator=g(1)) * 2                       # columns beyond q|k|v belong to someone else
     for h in range(H):
         proj[:, h * D:(h + 1) * D] *= 3.0 ** -h
     b = torch.randn(C, generator=g(2))
@@ -310,26 +312,24 @@ def test_norm_over_the_whole_projection_temperature_and_scaled_values(dtype, H, 
 
 
 @pytest.mark.parametrize("dtype", ["float32", "bfloat16"])
-@pytest.mark.parametrize("table", [False, True])
-@pytest.mark.parametrize("H, G, D, V, rot", [(4, 2, 8, 24, 6), (3, 3, 10, 9, 10), (4, 1, 64, 128, 32), (2, 1, 24, 20, 0), (1, 1, 80, 96, 2)])
-def test_two_maps_a_head_are_rotated_each_by_itself(dtype, table, H, G, D, V, rot):
-    ops, dt, T, ps = _ops(), DT[dtype], 37, 8
+@pytest.mark.parametrize("H, G, D, V, rot", [(4, 2, 8, 24, 6), (3, 3, 10, 9, 10), (4, 1, 64, 128, 32), (2, 1, 24, 20, 0), (1, 1, 80, 96, 2),
+                                             (32, 8, 64, 128, 64), (5, 5, 20, 100, 16), (2, 2, 12, 256, 8), (40, 8, 120, 40, 120)])
+@pytest.mark.parametrize("T", [37, 139])
+def test_two_maps_a_head_are_rotated_each_by_itself(dtype, H, G, D, V, rot, T):
+    """Short and long steps run different kernels (a warp a map, a block a token)."""
+    ops, dt, ps = _ops(), DT[dtype], 8
     C = 2 * H * D + G * (2 * D + V)
     proj = torch.randn(T, C, generator=g(1)) * 2
     positions = torch.tensor([0, 1, 2, 3, 70001, 1 << 20] + list(range(500, 500 + T - 6)), dtype=torch.int32)
     q, k = proj[:, :2 * H * D].double().view(T, H, 2, D), proj[:, 2 * H * D:2 * (H + G) * D].double().view(T, G, 2, D)
     q, k = plain.rotate(q, positions, rot, 3000.0), plain.rotate(k, positions, rot, 3000.0)
     freq = torch.tensor([3000.0 ** (-2.0 * i / rot) for i in range(rot // 2)], dtype=torch.float64, device=DEV) if rot else None
-    angles = None
-    if table and rot:
-        angles = torch.empty(T, rot // 2, 2, device=DEV)
-        ops.rope_table(positions.to(DEV), freq, angles)
     row = ops.padded_head(max(2 * D, V))
-    pool = torch.full((8, 2, G, ps, row), float("nan"), dtype=dt, device=DEV)
-    slots = torch.randperm(8 * ps, generator=g(5))[:T].to(torch.int32)
+    pool = torch.full((20, 2, G, ps, row), float("nan"), dtype=dt, device=DEV)
+    slots = torch.randperm(20 * ps, generator=g(5))[:T].to(torch.int32)
     slots[7] = -1                                                          # not written
     q_out = torch.full((T, 2 * H * row), float("nan"), dtype=dt, device=DEV)
-    ops.attn_prep(proj.to(DEV), None, None, None, None, 1e-5, freq, positions.to(DEV), slots.to(DEV), q_out, pool, ps, H, G, D, V, maps=2, angles=angles)
+    ops.attn_prep(proj.to(DEV), None, None, None, None, 1e-5, freq, positions.to(DEV), slots.to(DEV), q_out, pool, ps, H, G, D, V, maps=2)
     tol = dict(atol=2e-5, rtol=1e-5) if dtype == "float32" else dict(atol=2e-2, rtol=1e-2)
     got = q_out.float().cpu().double().view(T, H, 2, row)
     for m in (0, 1):
@@ -369,14 +369,15 @@ def test_residual_sum_with_the_embedding(dtype, W):
 # ---- the feed-forward --------------------------------------------------------------------------------------
 @pytest.mark.parametrize("dtype", ["float32", "bfloat16"])
 @pytest.mark.parametrize("T, W, F", [(1, 64, 96), (5, 52, 70), (40, 128, 200), (300, 128, 264), (1100, 256, 520), (1500, 512, 6144)])
-def test_gelu_feed_forward_in_every_kernel_of_its_product(dtype, T, W, F):
+@pytest.mark.parametrize("in_product", [True, False])
+def test_gelu_feed_forward_in_every_kernel_of_its_product(dtype, T, W, F, in_product):
     """One row to many: the products and their activation run different kernels, with the activation as a pass of its own or in the
     product's epilogue."""
     from mini_engine_b200.parts import ActivationMLP
     if dtype == "float32" and T > 500:
         T = 130
     dt = DT[dtype]
-    mlp = ActivationMLP(W, F, "gelu")
+    mlp = ActivationMLP(W, F, "gelu", in_product=in_product)
     up, down = (torch.randn(F, W, generator=g(1)) * (2.0 / W ** 0.5)).to(dt), (torch.randn(W, F, generator=g(2)) / F ** 0.5).to(dt)
     mlp.up.params["up"], mlp.down.params["down"] = up.to(DEV), down.to(DEV)
     x = torch.randn(T, W, generator=g(3)).to(dt)
