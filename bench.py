@@ -755,7 +755,8 @@ def _kernel_times(runner, cache, prompt, batch_prompts) -> dict:
         steps = {"prefill": [StepItem(h, prompt, 0, [len(prompt) - 1])],
                  "decode": [StepItem(x, [5], len(p), [0], (0.6, i)) for i, (x, p) in enumerate(zip(holders, batch_prompts))]}
         for what, items in steps.items():
-            runner.step(items, sample=True)                       # once untimed
+            for _ in range(2):
+                runner.step(items, sample=True)                   # untimed
             torch.cuda.synchronize()
             ops.timeline = []
             runner.step(items, sample=True)

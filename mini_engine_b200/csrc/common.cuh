@@ -90,17 +90,35 @@ __device__ __forceinline__ float erf_rounded(float x) {
   return copysignf(fmaf(-p * t, __expf(-a * a), 1.0f), x);
 }
 
-// TO: the type the result is stored in.
+// TO: the type the result is stored in (bfloat16: short forms with the fast exponential and division).
 template <typename TO = float>
 __device__ __forceinline__ float act_apply(float z, int kind) {
   if (kind == ACT_RELU2) {
     const float r = fmaxf(z, 0.f);
     return r * r;
   }
+  if (sizeof(TO) == 2) {
+    if (kind == ACT_GELU_ERF) return 0.5f * z * (1.f + erf_rounded(z * 0.7071067811865476f));
+    // z sigmoid(u): silu with u = z, and gelu's tanh form, whose (1 + tanh(w)) / 2 is sigmoid(2 w)
+    const float u = kind == ACT_GELU_TANH ? 1.5957691216057308f * (z + 0.044715f * z * z * z) : z;
+    return __fdividef(z, 1.f + __expf(-u));
+  }
   if (kind == ACT_GELU_TANH) return 0.5f * z * (1.f + tanhf(0.7978845608028654f * (z + 0.044715f * z * z * z)));
-  if (kind == ACT_GELU_ERF && sizeof(TO) == 2) return 0.5f * z * (1.f + erf_rounded(z * 0.7071067811865476f));
   if (kind == ACT_GELU_ERF) return 0.5f * z * (1.f + erff(z * 0.7071067811865476f));
   return z / (1.f + expf(-z));
+}
+
+// The same for a thread's registers, one branch for all of them.
+template <typename TO, int N>
+__device__ __forceinline__ void act_apply_all(float (&g)[N], int kind) {
+  auto all = [&](int k) {
+#pragma unroll
+    for (int j = 0; j < N; ++j) g[j] = act_apply<TO>(g[j], k);
+  };
+  if (kind == ACT_RELU2) all(ACT_RELU2);
+  else if (kind == ACT_GELU_TANH) all(ACT_GELU_TANH);
+  else if (kind == ACT_GELU_ERF) all(ACT_GELU_ERF);
+  else all(ACT_SILU);
 }
 
 __device__ __forceinline__ void pdl_wait() { asm volatile("griddepcontrol.wait;\n" ::: "memory"); }

@@ -84,10 +84,7 @@ __device__ __forceinline__ void write_rows(Load&& load, Fix&& fix, unsigned char
       load(c, g);
       tc5::wait_ld();
       fix(c, g);
-      if (glu.act >= 0) {
-#pragma unroll
-        for (int j = 0; j < 32; ++j) g[j] = act_apply<TO>(g[j], glu.act);
-      }
+      if (glu.act >= 0) act_apply_all<TO>(g, glu.act);
     }
   };
   if (!vec) {

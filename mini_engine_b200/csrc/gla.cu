@@ -146,21 +146,62 @@ gla_scan_kernel(const float* __restrict__ proj, int64_t ld, int off_q, int off_k
 constexpr int GLA_LC = 64;
 constexpr float GLA_LOG2E = 1.4426950408889634f;
 
+// Four floats at once where everything allows it (VEC = 4), else one by one.
+template <int VEC> struct GlaVec;
+template <> struct GlaVec<4> { using type = float4; };
+template <> struct GlaVec<1> { using type = float; };
+
+__device__ __forceinline__ void gla_cp_async16(float* dst, const float* src, bool ok) {      // zeros when not ok
+  const unsigned d = (unsigned)__cvta_generic_to_shared(dst);
+  asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;\n" ::"r"(d), "l"(src), "r"(ok ? 16 : 0) : "memory");
+}
+__device__ __forceinline__ void gla_cp_async_wait() { asm volatile("cp.async.wait_all;\n" ::: "memory"); }
+
+// ``rows`` x ``cols`` floats (cols a multiple of VEC) from a matrix in global memory into shared memory, zeros beyond n_rows and n_cols:
+// VEC 4 by asynchronous copies (the caller waits for them), VEC 1 loads from clamped places and selects afterwards, so that the
+// loads of several turns are in flight together.
+template <int VEC>
+__device__ __forceinline__ void gla_fill(float* dst, int ld_dst, int rows, int cols, const float* src, int64_t ld_src, int n_rows, int n_cols,
+                                         int tid) {
+  if constexpr (VEC == 4) {
+    const int per = cols / 4;
+    for (int i = tid; i < rows * per; i += 256) {
+      const int r = i / per, c = (i - r * per) * 4;
+      const bool ok = r < n_rows && c < n_cols;
+      gla_cp_async16(dst + r * ld_dst + c, ok ? src + (int64_t)r * ld_src + c : src, ok);
+    }
+  } else {
+#pragma unroll 8
+    for (int i = tid; i < rows * cols; i += 256) {
+      const int r = i / cols, c = i - r * cols;
+      const float x = src[(int64_t)min(r, n_rows - 1) * ld_src + min(c, n_cols - 1)];
+      dst[r * ld_dst + c] = (r < n_rows && c < n_cols) ? x : 0.f;
+    }
+  }
+}
+
 // tiles: (request, first token of the chunk within the request's tokens of this step) pairs.  la: in, the log decays
 // [T, H*D]; out, the chunk's inclusive sums B * log2(e).  A: [T, H, GLA_LC], row t holds A[t][s] for the chunk's tokens s
 // (zero for s > t).  GATED: la is no input; q and k are formed from the projection (see the top of this file) and written back
 // to it, each by the one block that holds their chunk and head.
-template <bool GATED>
+//
+// A is taken in blocks of 16 x 16.  On the diagonal every (query, key, channel) has an exponential of its own.  Below it, with r_i the
+// sum up to the last token in front of query block i, exp(B_t - B_s) = exp(B_t - r_i) exp(r_i - B_s): both exponents are <= 0, the
+// factors go into q and k once, and the block is a plain product.  From one query block to the next the keys behind take one more
+// factor a channel, exp(r_(i+1) - r_i).  All of these exponents are sums inside one block of 16 tokens, so none is a small difference
+// of large sums.
+template <bool GATED, int VEC>
 __global__ void __launch_bounds__(256)
 gla_intra_kernel(typename std::conditional<GATED, float, const float>::type* proj, int64_t ld, int off_q, int off_k, float* __restrict__ la,
                  const int* __restrict__ cu_seqlens, const int* __restrict__ tiles, float* __restrict__ A, int H, int D,
                  float q_scale, ForgetGate fg) {
   extern __shared__ __align__(16) float smem[];
-  constexpr int LC = GLA_LC;
-  const int ldq = D + 1;
-  float* Qc = smem;                             // [LC][D + 1]
-  float* Kc = Qc + LC * ldq;                    // [LC][D + 1]
-  float* Bc = Kc + LC * ldq;                    // [LC][D + 1]
+  constexpr int LC = GLA_LC, NB = LC / 16;
+  using vec_t = typename GlaVec<VEC>::type;
+  const int D4 = (D + 3) / 4 * 4, ldq = D4 + 4;
+  float* Qc = smem;                             // [LC][ldq]; elements from D on are zero
+  float* Kc = Qc + LC * ldq;
+  float* Bc = Kc + LC * ldq;
   const int tid = threadIdx.x, hd = blockIdx.y;
   pdl_wait();
   pdl_launch_dependents();
@@ -168,72 +209,113 @@ gla_intra_kernel(typename std::conditional<GATED, float, const float>::type* pro
   const int tok0 = cu_seqlens[b] + q0;
   const int L = min(LC, cu_seqlens[b + 1] - tok0);
   if (L <= 0) return;
-  // the fill loads from clamped places and selects afterwards, so that the loads of several turns are in flight together
+  const int per = D4 / VEC;
 #pragma unroll 4
-  for (int idx = tid; idx < LC * D; idx += 256) {
-    const int t = idx / D, d = idx - t * D;
-    auto* row = proj + (int64_t)(tok0 + min(t, L - 1)) * ld;
-    float qv = row[off_q + hd * D + d], kv = row[off_k + hd * D + d], bv;
-    if constexpr (GATED) {
-      if (t >= L) {
-        qv = kv = bv = 0.f;
+  for (int idx = tid; idx < LC * per; idx += 256) {
+    const int t = idx / per, d = (idx - t * per) * VEC, c = hd * D + d;
+    __align__(16) float qv[VEC] = {}, kv[VEC] = {}, bv[VEC] = {};
+    if (t < L && d < D) {
+      auto* row = proj + (int64_t)(tok0 + t) * ld;
+      *reinterpret_cast<vec_t*>(qv) = *reinterpret_cast<const vec_t*>(row + off_q + c);
+      *reinterpret_cast<vec_t*>(kv) = *reinterpret_cast<const vec_t*>(row + off_k + c);
+      if constexpr (GATED) {
+        __align__(16) float fb[VEC], lo[VEC];
+        *reinterpret_cast<vec_t*>(fb) = *reinterpret_cast<const vec_t*>(fg.bias + c);
+        *reinterpret_cast<vec_t*>(lo) = *reinterpret_cast<const vec_t*>(fg.lower + c);
+#pragma unroll
+        for (int j = 0; j < VEC; ++j) {
+          float log_a;
+          forget_gate(kv[j] + fb[j], lo[j], kv[j], log_a);
+          qv[j] = gla_silu(qv[j]);
+          bv[j] = log_a * GLA_LOG2E;
+        }
+        *reinterpret_cast<vec_t*>(row + off_q + c) = *reinterpret_cast<const vec_t*>(qv);
+        *reinterpret_cast<vec_t*>(row + off_k + c) = *reinterpret_cast<const vec_t*>(kv);
       } else {
-        const int c = hd * D + d;
-        float log_a;
-        forget_gate(kv + fg.bias[c], fg.lower[c], kv, log_a);
-        qv = gla_silu(qv);
-        bv = log_a * GLA_LOG2E;
-        row[off_q + c] = qv;
-        row[off_k + c] = kv;
+        *reinterpret_cast<vec_t*>(bv) = *reinterpret_cast<const vec_t*>(la + (int64_t)(tok0 + t) * H * D + c);
+#pragma unroll
+        for (int j = 0; j < VEC; ++j) bv[j] *= GLA_LOG2E;
       }
-    } else {
-      bv = la[(int64_t)(tok0 + min(t, L - 1)) * H * D + hd * D + d] * GLA_LOG2E;
+#pragma unroll
+      for (int j = 0; j < VEC; ++j) qv[j] *= q_scale;
     }
-    qv *= q_scale;
-    Qc[t * ldq + d] = t < L ? qv : 0.f;
-    Kc[t * ldq + d] = t < L ? kv : 0.f;
-    Bc[t * ldq + d] = t < L ? bv : 0.f;
+    *reinterpret_cast<vec_t*>(Qc + t * ldq + d) = *reinterpret_cast<const vec_t*>(qv);
+    *reinterpret_cast<vec_t*>(Kc + t * ldq + d) = *reinterpret_cast<const vec_t*>(kv);
+    *reinterpret_cast<vec_t*>(Bc + t * ldq + d) = *reinterpret_cast<const vec_t*>(bv);
   }
   __syncthreads();
-  for (int d = tid; d < D; d += 256) {          // the inclusive sums, a channel a thread
+  // the inclusive sums inside each block of 16 tokens: a channel of a block a thread
+  for (int i = tid; i < NB * D; i += 256) {
+    const int n = i / D, d = i - n * D;
     float run = 0.f;
-    for (int t = 0; t < LC; ++t) {
-      run += Bc[t * ldq + d];
-      Bc[t * ldq + d] = run;
-      if (t < L) la[(int64_t)(tok0 + t) * H * D + hd * D + d] = run;
+#pragma unroll
+    for (int t = 0; t < 16; ++t) {
+      run += Bc[(16 * n + t) * ldq + d];
+      Bc[(16 * n + t) * ldq + d] = run;
     }
   }
   __syncthreads();
-  // A in blocks of 32 x 32 (the three on and below the diagonal); a thread takes rows ty, ty + 16 and columns tx, tx + 16
+  for (int i = tid; i < LC * D; i += 256) {     // those of the whole chunk go out: the totals of the blocks in front, then the block's own
+    const int t = i / D, d = i - t * D;
+    float base = 0.f;
+    for (int n = 0; n < t / 16; ++n) base += Bc[(16 * n + 15) * ldq + d];
+    if (t < L) la[(int64_t)(tok0 + t) * H * D + hd * D + d] = base + Bc[t * ldq + d];
+  }
   const int ty = tid / 16, tx = tid % 16;
-  for (int blk = 0; blk < 4; ++blk) {
-    const int bi = blk >> 1, bj = blk & 1;
-    const int t0 = 32 * bi + ty, t1 = t0 + 16, s0 = 32 * bj + tx, s1 = s0 + 16;
-    float a00 = 0.f, a01 = 0.f, a10 = 0.f, a11 = 0.f;
-    if (bj <= bi && 32 * bi < L) {
-      const bool diag = bi == bj;               // on the diagonal (t0, s1) is never seen: s1 >= 16 > ty
-      const float *q0p = Qc + t0 * ldq, *q1p = Qc + t1 * ldq, *k0p = Kc + s0 * ldq, *k1p = Kc + s1 * ldq;
-      const float *bt0 = Bc + t0 * ldq, *bt1 = Bc + t1 * ldq, *bs0 = Bc + s0 * ldq, *bs1 = Bc + s1 * ldq;
-      const bool on00 = s0 <= t0, on10 = s0 <= t1, on11 = s1 <= t1;
-      for (int d = 0; d < D; ++d) {
-        const float qa = q0p[d], qb = q1p[d], ka = k0p[d], kb = k1p[d];
-        const float ba = bt0[d], bb = bt1[d], ca = bs0[d], cb = bs1[d];
-        if (on00) a00 = fmaf(qa * ka, exp2f(ba - ca), a00);
-        if (on10) a10 = fmaf(qb * ka, exp2f(bb - ca), a10);
-        if (on11) a11 = fmaf(qb * kb, exp2f(bb - cb), a11);
-        if (!diag) a01 = fmaf(qa * kb, exp2f(ba - cb), a01);
+  auto put = [&](int t, int s, float a) {
+    if (t < L) A[((int64_t)(tok0 + t) * H + hd) * LC + s] = a;
+  };
+  for (int i = 0; i < NB; ++i)
+    for (int j = i + 1; j < NB; ++j) put(16 * i + ty, 16 * j + tx, 0.f);
+  for (int n = 0; n < NB && 16 * n < L; ++n) {
+    const float *q = Qc + (16 * n + ty) * ldq, *k = Kc + (16 * n + tx) * ldq, *bt = Bc + (16 * n + ty) * ldq, *bs = Bc + (16 * n + tx) * ldq;
+    float a = 0.f;
+    if (tx <= ty) {
+      for (int d = 0; d < D4; d += 4) {
+        const float4 q4 = *reinterpret_cast<const float4*>(q + d), k4 = *reinterpret_cast<const float4*>(k + d);
+        const float4 t4 = *reinterpret_cast<const float4*>(bt + d), s4 = *reinterpret_cast<const float4*>(bs + d);
+        a = fmaf(q4.x * k4.x, exp2f(t4.x - s4.x), a);
+        a = fmaf(q4.y * k4.y, exp2f(t4.y - s4.y), a);
+        a = fmaf(q4.z * k4.z, exp2f(t4.z - s4.z), a);
+        a = fmaf(q4.w * k4.w, exp2f(t4.w - s4.w), a);
       }
     }
-    if (t0 < L) {
-      float* ar = A + ((int64_t)(tok0 + t0) * H + hd) * LC;
-      ar[s0] = a00;
-      ar[s1] = a01;
+    put(16 * n + ty, 16 * n + tx, a);
+  }
+  __syncthreads();
+  // q of the blocks from the second on, from the base in front of its block; k of all blocks but the last, to the base behind its block
+  for (int i = tid; i < (LC - 16) * D; i += 256) {
+    const int t = i / D, d = i - t * D;
+    Qc[(t + 16) * ldq + d] *= exp2f(Bc[(t + 16) * ldq + d]);
+    Kc[t * ldq + d] *= exp2f(Bc[(t / 16 * 16 + 15) * ldq + d] - Bc[t * ldq + d]);
+  }
+  for (int n = 1; n < NB && 16 * n < L; ++n) {
+    __syncthreads();
+    if (n > 1) {                                // the keys of the blocks before the last one: from the base before to this one
+      for (int i = tid; i < 16 * (n - 1) * D; i += 256) {
+        const int t = i / D, d = i - t * D;
+        Kc[t * ldq + d] *= exp2f(Bc[(16 * n - 1) * ldq + d]);
+      }
+      __syncthreads();
     }
-    if (t1 < L) {
-      float* ar = A + ((int64_t)(tok0 + t1) * H + hd) * LC;
-      ar[s0] = a10;
-      ar[s1] = a11;
+    const float* q = Qc + (16 * n + ty) * ldq;
+    float a[NB - 1] = {};
+    for (int d = 0; d < D4; d += 4) {
+      const float4 q4 = *reinterpret_cast<const float4*>(q + d);
+#pragma unroll
+      for (int j = 0; j < NB - 1; ++j) {
+        if (j < n) {
+          const float4 k4 = *reinterpret_cast<const float4*>(Kc + (16 * j + tx) * ldq + d);
+          a[j] = fmaf(q4.x, k4.x, a[j]);
+          a[j] = fmaf(q4.y, k4.y, a[j]);
+          a[j] = fmaf(q4.z, k4.z, a[j]);
+          a[j] = fmaf(q4.w, k4.w, a[j]);
+        }
+      }
     }
+#pragma unroll
+    for (int j = 0; j < NB - 1; ++j)
+      if (j < n) put(16 * n + ty, 16 * j + tx, a[j]);
   }
 }
 
@@ -248,6 +330,7 @@ gla_intra_kernel(typename std::conditional<GATED, float, const float>::type* pro
 constexpr int GLA_VT = 64;
 
 // One block = one chunk x one head x GLA_VT columns.  bsum: gla_intra_kernel's inclusive sums (units of log 2).
+template <int VEC>
 __global__ void __launch_bounds__(256)
 gla_chunk_state_kernel(const float* __restrict__ proj, int64_t ld, int off_k, int off_v, const float* __restrict__ bsum,
                        const int* __restrict__ cu_seqlens, const int* __restrict__ tiles, float* __restrict__ states, int H, int D,
@@ -265,28 +348,30 @@ gla_chunk_state_kernel(const float* __restrict__ proj, int64_t ld, int off_k, in
   const int L = min(LC, cu_seqlens[b + 1] - tok0);
   if (L <= 0) return;
   const float* bl = bsum + (int64_t)(tok0 + L - 1) * H * D + hd * D;
-  // the fills load from clamped places and select afterwards, so that the loads of several turns are in flight together
-#pragma unroll 8
-  for (int idx = tid; idx < LC * Dp; idx += 256) {
-    const int t = idx / Dp, d = idx - t * Dp;
-    const int tc = min(t, L - 1), dc = min(d, D - 1);
-    const float kv = proj[(int64_t)(tok0 + tc) * ld + off_k + hd * D + dc] *
-                     exp2f(bl[dc] - bsum[(int64_t)(tok0 + tc) * H * D + hd * D + dc]);
-    Kt[t * ldk + d] = (t < L && d < D) ? kv : 0.f;
+  gla_fill<VEC>(Vc, VT, LC, VT, proj + (int64_t)tok0 * ld + off_v + hd * V + v0, ld, L, V - v0, tid);
+  using vec_t = typename GlaVec<VEC>::type;
+  const int per = Dp / VEC;
+#pragma unroll 4
+  for (int idx = tid; idx < LC * per; idx += 256) {
+    const int t = idx / per, d = (idx - t * per) * VEC;
+    const int tc = min(t, L - 1), dc = min(d, D - VEC);
+    __align__(16) float kv[VEC], bv[VEC], be[VEC];
+    *reinterpret_cast<vec_t*>(kv) = *reinterpret_cast<const vec_t*>(proj + (int64_t)(tok0 + tc) * ld + off_k + hd * D + dc);
+    *reinterpret_cast<vec_t*>(bv) = *reinterpret_cast<const vec_t*>(bsum + (int64_t)(tok0 + tc) * H * D + hd * D + dc);
+    *reinterpret_cast<vec_t*>(be) = *reinterpret_cast<const vec_t*>(bl + dc);
+#pragma unroll
+    for (int j = 0; j < VEC; ++j) kv[j] = (t < L && d < D) ? kv[j] * exp2f(be[j] - bv[j]) : 0.f;
+    *reinterpret_cast<vec_t*>(Kt + t * ldk + d) = *reinterpret_cast<const vec_t*>(kv);
   }
-#pragma unroll 8
-  for (int idx = tid; idx < LC * VT; idx += 256) {
-    const int t = idx / VT, v = idx - t * VT;
-    const float x = proj[(int64_t)(tok0 + min(t, L - 1)) * ld + off_v + hd * V + min(v0 + v, V - 1)];
-    Vc[idx] = (t < L && v0 + v < V) ? x : 0.f;
-  }
+  if (VEC == 4) gla_cp_async_wait();
   __syncthreads();
   // a thread: rows d0 + 4 ty .. + 3 and columns 4 tx .. + 3; one 16-byte load of each operand a token
   const int ty = tid / 16, tx = tid % 16;
   float* out = states + ((int64_t)blockIdx.x * H + hd) * D * V;
   for (int d0 = 0; d0 < D; d0 += 64) {
     float acc[4][4] = {};
-    for (int s = 0; s < L; ++s) {
+#pragma unroll 8
+    for (int s = 0; s < LC; ++s) {              // (rows beyond L are zero)
       const float4 k4 = *reinterpret_cast<const float4*>(Kt + s * ldk + d0 + 4 * ty);
       const float4 v4 = *reinterpret_cast<const float4*>(Vc + s * VT + 4 * tx);
       const float kk[4] = {k4.x, k4.y, k4.z, k4.w}, vv[4] = {v4.x, v4.y, v4.z, v4.w};
@@ -299,10 +384,14 @@ gla_chunk_state_kernel(const float* __restrict__ proj, int64_t ld, int off_k, in
     for (int i = 0; i < 4; ++i) {
       const int d = d0 + 4 * ty + i;
       if (d >= D) continue;
+      if constexpr (VEC == 4) {
+        if (v0 + 4 * tx < V) *reinterpret_cast<float4*>(out + (int64_t)d * V + v0 + 4 * tx) = make_float4(acc[i][0], acc[i][1], acc[i][2], acc[i][3]);
+      } else {
 #pragma unroll
-      for (int j = 0; j < 4; ++j) {
-        const int v = v0 + 4 * tx + j;
-        if (v < V) out[(int64_t)d * V + v] = acc[i][j];
+        for (int j = 0; j < 4; ++j) {
+          const int v = v0 + 4 * tx + j;
+          if (v < V) out[(int64_t)d * V + v] = acc[i][j];
+        }
       }
     }
   }
@@ -341,7 +430,7 @@ gla_state_walk_kernel(const float* __restrict__ bsum, float* __restrict__ states
   const int64_t step = (int64_t)H * D * V;
   float* st = states + ((int64_t)c0 * H + hd) * D * V + e;
   const float* bd = bsum + (int64_t)tok0 * H * D + hd * D + d;
-  constexpr int AHEAD = VEC == 4 ? 4 : 8;       // chunks whose loads are in flight together
+  constexpr int AHEAD = 8;                      // chunks whose loads are in flight together
   for (int c1 = 0; c1 < n_chunks; c1 += AHEAD) {
     __align__(16) float u[AHEAD][VEC];
     float dec[AHEAD];
@@ -365,6 +454,7 @@ gla_state_walk_kernel(const float* __restrict__ bsum, float* __restrict__ states
 }
 
 // One block = one chunk x one head x GLA_VT columns.  states[c] holds the state in front of the chunk.
+template <int VEC>
 __global__ void __launch_bounds__(256)
 gla_chunk_out_kernel(const float* __restrict__ proj, int64_t ld, int off_q, int off_v, const float* __restrict__ bsum,
                      const float* __restrict__ A, const float* __restrict__ states, const int* __restrict__ cu_seqlens,
@@ -381,34 +471,23 @@ gla_chunk_out_kernel(const float* __restrict__ proj, int64_t ld, int off_q, int 
   const int tok0 = cu_seqlens[b] + q0;
   const int L = min(LC, cu_seqlens[b + 1] - tok0);
   if (L <= 0) return;
-  // the fills load from clamped places and select afterwards, so that the loads of several turns are in flight together
-#pragma unroll 8
-  for (int idx = tid; idx < LC * Dq; idx += 256) {
-    const int t = idx / Dq, c = idx - t * Dq;
-    const int tc = min(t, L - 1), cc = min(c, D - 1);
-    const float x = proj[(int64_t)(tok0 + tc) * ld + off_q + hd * D + cc] * q_scale *
-                    exp2f(bsum[(int64_t)(tok0 + tc) * H * D + hd * D + cc]);
-    X[t * ldx + c] = (t < L && c < D) ? x : 0.f;
+  gla_fill<VEC>(Y, VT, Dq, VT, states + ((int64_t)blockIdx.x * H + hd) * D * V + v0, V, D, V - v0, tid);
+  gla_fill<VEC>(Y + Dq * VT, VT, LC, VT, proj + (int64_t)tok0 * ld + off_v + hd * V + v0, ld, L, V - v0, tid);
+  gla_fill<VEC>(X + Dq, ldx, LC, LC, A + ((int64_t)tok0 * H + hd) * LC, (int64_t)H * LC, L, LC, tid);
+  using vec_t = typename GlaVec<VEC>::type;
+  const int per = Dq / VEC;
+#pragma unroll 4
+  for (int idx = tid; idx < LC * per; idx += 256) {
+    const int t = idx / per, c = (idx - t * per) * VEC;
+    const int tc = min(t, L - 1), cc = min(c, D - VEC);
+    __align__(16) float x[VEC], bv[VEC];
+    *reinterpret_cast<vec_t*>(x) = *reinterpret_cast<const vec_t*>(proj + (int64_t)(tok0 + tc) * ld + off_q + hd * D + cc);
+    *reinterpret_cast<vec_t*>(bv) = *reinterpret_cast<const vec_t*>(bsum + (int64_t)(tok0 + tc) * H * D + hd * D + cc);
+#pragma unroll
+    for (int j = 0; j < VEC; ++j) x[j] = (t < L && c < D) ? x[j] * q_scale * exp2f(bv[j]) : 0.f;
+    *reinterpret_cast<vec_t*>(X + t * ldx + c) = *reinterpret_cast<const vec_t*>(x);
   }
-#pragma unroll 8
-  for (int idx = tid; idx < LC * LC; idx += 256) {
-    const int t = idx / LC, c = idx - t * LC;
-    const float x = A[((int64_t)(tok0 + min(t, L - 1)) * H + hd) * LC + c];
-    X[t * ldx + Dq + c] = t < L ? x : 0.f;
-  }
-  const float* st = states + ((int64_t)blockIdx.x * H + hd) * D * V;
-#pragma unroll 8
-  for (int idx = tid; idx < Dq * VT; idx += 256) {
-    const int r = idx / VT, v = idx - r * VT;
-    const float y = st[(int64_t)min(r, D - 1) * V + min(v0 + v, V - 1)];
-    Y[idx] = (r < D && v0 + v < V) ? y : 0.f;
-  }
-#pragma unroll 8
-  for (int idx = tid; idx < LC * VT; idx += 256) {
-    const int r = idx / VT, v = idx - r * VT;
-    const float y = proj[(int64_t)(tok0 + min(r, L - 1)) * ld + off_v + hd * V + min(v0 + v, V - 1)];
-    Y[Dq * VT + idx] = (r < L && v0 + v < V) ? y : 0.f;
-  }
+  if (VEC == 4) gla_cp_async_wait();
   __syncthreads();
   // a thread: rows ty + 16 i and columns 4 tx .. + 3; four terms a turn with 16-byte loads of both operands
   const int ty = tid / 16, tx = tid % 16;
@@ -436,10 +515,15 @@ gla_chunk_out_kernel(const float* __restrict__ proj, int64_t ld, int off_q, int 
   for (int i = 0; i < 4; ++i) {
     const int t = ty + 16 * i;
     if (t >= L) continue;
+    if constexpr (VEC == 4) {
+      if (v0 + 4 * tx < V)
+        *reinterpret_cast<float4*>(o + (int64_t)(tok0 + t) * H * V + hd * V + v0 + 4 * tx) = make_float4(acc[i][0], acc[i][1], acc[i][2], acc[i][3]);
+    } else {
 #pragma unroll
-    for (int j = 0; j < 4; ++j) {
-      const int v = v0 + 4 * tx + j;
-      if (v < V) o[(int64_t)(tok0 + t) * H * V + hd * V + v] = acc[i][j];
+      for (int j = 0; j < 4; ++j) {
+        const int v = v0 + 4 * tx + j;
+        if (v < V) o[(int64_t)(tok0 + t) * H * V + hd * V + v] = acc[i][j];
+      }
     }
   }
 }
@@ -487,8 +571,8 @@ ME_API int me_gla_scan(float* proj, int64_t ld, int off_q, int off_k, int off_v,
   const ForgetGate fg = {gate_bias, gate_lower};
   const bool gated = gate_bias != nullptr;
   const int Dp = (D + 63) / 64 * 64, v_tiles = (V + GLA_VT - 1) / GLA_VT;
-  const size_t smem_intra = sizeof(float) * 3 * GLA_LC * ((size_t)D + 1);
   const int Dq = (D + 3) / 4 * 4;
+  const size_t smem_intra = sizeof(float) * 3 * GLA_LC * ((size_t)Dq + 4);
   const size_t smem_state = sizeof(float) * (GLA_LC * ((size_t)Dp + 4) + GLA_LC * GLA_VT);
   const size_t smem_out = sizeof(float) * (GLA_LC * ((size_t)Dq + GLA_LC + 4) + ((size_t)Dq + GLA_LC) * GLA_VT);
   const bool chunks = tiles && A_ws && states_ws && n_tiles > 0 && num_decodes < B && D <= 256 && v_tiles <= 65535 &&
@@ -505,18 +589,22 @@ ME_API int me_gla_scan(float* proj, int64_t ld, int off_q, int off_k, int off_v,
     ME_LAUNCH_CHECK("me_gla_scan");
   }
   if (chunks) {
-    if (gated) {
-      if (gla_raise_smem(gla_intra_kernel<true>, smem_intra, "me_gla_scan (intra)")) return 1;
-      me_launch(gla_intra_kernel<true>, dim3(n_tiles, H), dim3(256), smem_intra, stream, proj, ld, off_q, off_k, la, cu_seqlens, tiles,
-                A_ws, H, D, q_scale, fg);
-    } else {
-      if (gla_raise_smem(gla_intra_kernel<false>, smem_intra, "me_gla_scan (intra)")) return 1;
-      me_launch(gla_intra_kernel<false>, dim3(n_tiles, H), dim3(256), smem_intra, stream, (const float*)proj, ld, off_q, off_k, la, cu_seqlens,
-                tiles, A_ws, H, D, q_scale, fg);
-    }
+    auto off16 = [](const void* p) { return ((uintptr_t)p % 16) != 0; };
+    const bool vec = D % 4 == 0 && V % 4 == 0 && ld % 4 == 0 && off_q % 4 == 0 && off_k % 4 == 0 && off_v % 4 == 0 && !off16(proj) && !off16(la) &&
+                     !off16(A_ws) && !off16(states_ws) && !off16(o) && !off16(gate_bias) && !off16(gate_lower);
+#define GLA_INTRA(GATED_, VEC_, PROJ_)                                                                                              \
+  do {                                                                                                                              \
+    if (gla_raise_smem(gla_intra_kernel<GATED_, VEC_>, smem_intra, "me_gla_scan (intra)")) return 1;                               \
+    me_launch(gla_intra_kernel<GATED_, VEC_>, dim3(n_tiles, H), dim3(256), smem_intra, stream, PROJ_, ld, off_q, off_k, la, cu_seqlens, tiles, \
+              A_ws, H, D, q_scale, fg);                                                                                             \
+  } while (0)
+    if (gated) { if (vec) GLA_INTRA(true, 4, proj); else GLA_INTRA(true, 1, proj); }
+    else { if (vec) GLA_INTRA(false, 4, (const float*)proj); else GLA_INTRA(false, 1, (const float*)proj); }
+#undef GLA_INTRA
     ME_LAUNCH_CHECK("me_gla_scan (intra)");
-    if (gla_raise_smem(gla_chunk_state_kernel, smem_state, "me_gla_scan (chunk states)")) return 1;
-    me_launch(gla_chunk_state_kernel, dim3(n_tiles, H, v_tiles), dim3(256), smem_state, stream, (const float*)proj, ld, off_k, off_v, (const float*)la,
+    auto chunk_state = vec ? gla_chunk_state_kernel<4> : gla_chunk_state_kernel<1>;
+    if (gla_raise_smem(chunk_state, smem_state, "me_gla_scan (chunk states)")) return 1;
+    me_launch(chunk_state, dim3(n_tiles, H, v_tiles), dim3(256), smem_state, stream, (const float*)proj, ld, off_k, off_v, (const float*)la,
               cu_seqlens, tiles, states_ws, H, D, V);
     ME_LAUNCH_CHECK("me_gla_scan (chunk states)");
     const bool walk4 = V % 4 == 0 && ((uintptr_t)states_ws % 16) == 0 && ((uintptr_t)S_state % 16) == 0;
@@ -529,8 +617,9 @@ ME_API int me_gla_scan(float* proj, int64_t ld, int off_q, int off_k, int off_v,
       me_launch(gla_state_walk_kernel<1>, walk_grid, dim3(256), 0, stream, (const float*)la, states_ws, S_state, cu_seqlens,
                 context_lens, state_slots, tiles, n_tiles, num_decodes, H, D, V);
     ME_LAUNCH_CHECK("me_gla_scan (state walk)");
-    if (gla_raise_smem(gla_chunk_out_kernel, smem_out, "me_gla_scan (chunk outputs)")) return 1;
-    me_launch(gla_chunk_out_kernel, dim3(n_tiles, H, v_tiles), dim3(256), smem_out, stream, (const float*)proj, ld, off_q, off_v, (const float*)la,
+    auto chunk_out = vec ? gla_chunk_out_kernel<4> : gla_chunk_out_kernel<1>;
+    if (gla_raise_smem(chunk_out, smem_out, "me_gla_scan (chunk outputs)")) return 1;
+    me_launch(chunk_out, dim3(n_tiles, H, v_tiles), dim3(256), smem_out, stream, (const float*)proj, ld, off_q, off_v, (const float*)la,
               (const float*)A_ws, (const float*)states_ws, cu_seqlens, tiles, o, H, D, V, q_scale);
     ME_LAUNCH_CHECK("me_gla_scan (chunk outputs)");
   }
