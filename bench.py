@@ -758,9 +758,12 @@ def _kernel_times(runner, cache, prompt, batch_prompts) -> dict:
             for _ in range(2):
                 runner.step(items, sample=True)                   # untimed
             torch.cuda.synchronize()
+            gc.collect()
+            gc.disable()                                          # (a pause between two events would count as the kernel's)
             ops.timeline = []
             runner.step(items, sample=True)
             torch.cuda.synchronize()
+            gc.enable()
             tl, ops.timeline = ops.timeline, None
             acc = {}
             for _tag, name, e0, e1 in tl:
@@ -771,6 +774,7 @@ def _kernel_times(runner, cache, prompt, batch_prompts) -> dict:
         for x in holders + [h]:
             cache.free(x)
     finally:
+        gc.enable()
         ops.timeline = None
         runner.use_cuda_graphs = graphs
     return out
