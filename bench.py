@@ -29,8 +29,8 @@ Modes: ``step`` (the line above), ``offline`` (the reference's own bench.py:38-6
 --budget --chunked --threshold --out --label --expect-gpu``; a JSON row like the reference's is appended to
 ``--out``), ``mixed`` (the 8B workload above, at any shape), ``decode`` (decode at batches ``--batches`` after
 ``--prompt-len`` prompts), ``prefill`` (one prompt of ``--prompt-len`` tokens in portions of ``--budget``), ``logozen``, ``pugadra``, ``gevulorn``, ``galupel`` and ``tidenex``
-(prefill and decode of that design at the layer sizes ``--sizes``, beside the Qwen3 of equal size (Gevulorn and Galupel: the Pugadra of equal
-size), with the time of every kernel).
+(prefill and decode of that design at the layer sizes ``--sizes``, beside the Qwen3 of equal size (Gevulorn and Galupel: the Pugadra, Tidenex: the
+Gevulorn of equal size), with the time of every kernel).
 """
 from __future__ import annotations
 
@@ -984,8 +984,7 @@ def _qwen3_roofline(cfg: dict, T: int, item: int, pk: dict, times: dict) -> dict
 
 
 def run_design_mode(args, design: str) -> int:
-    """Prefill and decode throughput of a design at layer sizes that resemble real models', beside the Qwen3 (for Gevulorn the
-    Pugadra) of the same width, depth, heads, feed-forward width and vocabulary; random weights drawn on the device."""
+    """Prefill and decode throughput of a design at layer sizes that resemble real models', beside the Qwen3 (or ``DESIGN_TWINS``) of the same width, depth, heads, feed-forward width and vocabulary; random weights drawn on the device."""
     import torch
     sizes_of = DESIGN_SIZES[design]
     rooflines = {"logozen": _logozen_roofline, "pugadra": _pugadra_roofline, "gevulorn": _gevulorn_roofline, "galupel": _galupel_roofline,

@@ -30,7 +30,7 @@ __device__ __forceinline__ bf16* dl_ptr(bf16* base, int row, int piece) {
 
 // X is bfloat16 [M][ldx].  With ``sumsq_in`` ([sumsq_parts][M], the sums of squares of the rows that X was made
 // from, over ``K`` columns) the results are multiplied by rsqrt(sum / K + eps) of their row.
-// EPI 0: Y[m][n] (bfloat16 or float32), through activation ``act`` of common.cuh when that is not negative.  EPI 1: SiLU(gate) * up, bfloat16.
+// EPI 0: Y[m][n] (bfloat16 or float32); EPI 3: through activation ``act`` of common.cuh, bfloat16.  EPI 1: SiLU(gate) * up, bfloat16.
 // EPI 2: residual_out[m][n] += v, sumsq_out, and with ``next_w`` also xw_out[m][n] = residual_out[m][n] * next_w[n].
 template <int EPI, typename TO, int R /* weight rows of a strip: 16, or 8 with the upper half of the tile idle */>
 __global__ void __launch_bounds__(DL_MAX_WARPS * 32)
@@ -206,7 +206,7 @@ gemm_decode_kernel(const bf16* __restrict__ X, int64_t ldx, const float* __restr
       const int n = strip * R + r;
       if (m >= M || n >= N) continue;
       const float v = total(r, m) * row_scale[m];
-      Y[(int64_t)m * ldy + n] = from_f<TO>(act >= 0 ? act_apply<TO>(v, act) : v);
+      Y[(int64_t)m * ldy + n] = from_f<TO>(EPI == 3 ? act_apply<TO>(v, act) : v);
     }
   }
 }
@@ -243,7 +243,7 @@ ME_API int me_gemm_decode_sumsq_parts(int N) { const int r = strip_rows(N); retu
 // epi 0: Y (y_dtype) [M][ldy]; epi 1: the gated epilogue g sigmoid(alpha g) (u + shift), g and u clamped by glu_limit when that
 // is positive (weight rows gate | up, N = columns of Y; SiLU-and-multiply is limit 0, alpha 1, shift 0);
 // epi 2: res_out [M][N] += X W^T, sumsq_out [me_gemm_decode_sumsq_parts(N)][M] and, with next_w [N], xw_out
-// bfloat16 [M][N] = res_out * next_w; epi 3 + k: Y through activation k of common.cuh.
+// bfloat16 [M][N] = res_out * next_w; epi 3 + k: Y (bfloat16) through activation k of common.cuh.
 // ahead (or null), ahead_bytes: memory that a later kernel will read (the next product's weights), asked into
 // L2 by this one; 16-byte aligned.
 ME_API int me_gemm_decode(int epi, const void* X, int64_t ldx, const float* sumsq_in, int sumsq_parts, float eps,
@@ -258,8 +258,8 @@ ME_API int me_gemm_decode(int epi, const void* X, int64_t ldx, const float* sums
   ME_REQUIRE(sumsq_in == nullptr || (sumsq_parts > 0 && sumsq_parts <= 192), "me_gemm_decode: sums of squares in %d parts (1..192)",
              sumsq_parts);
   const int act = epi >= 3 && epi <= 3 + ACT_GELU_ERF ? epi - 3 : -1;
-  if (act >= 0) epi = 0;
-  ME_REQUIRE(epi == 0 || epi == 1 || (epi == 2 && res_out != nullptr && sumsq_out != nullptr), "me_gemm_decode: epilogue %d", epi);
+  if (act >= 0) epi = 3;
+  ME_REQUIRE(epi == 0 || epi == 1 || (epi == 3 && act >= 0 && y_dtype == ME_BF16) || (epi == 2 && res_out != nullptr && sumsq_out != nullptr), "me_gemm_decode: epilogue %d", epi);
   ME_REQUIRE((next_w == nullptr) == (xw_out == nullptr) && (next_w == nullptr || epi == 2),
              "me_gemm_decode: the pre-weighted copy needs the residual epilogue, a weight and an output");
   ME_REQUIRE(ahead == nullptr || ((uintptr_t)ahead & 15) == 0, "me_gemm_decode: memory to fetch ahead must be 16-byte aligned");
@@ -275,6 +275,8 @@ ME_API int me_gemm_decode(int epi, const void* X, int64_t ldx, const float* sums
   } else if (epi == 1) {
     ME_REQUIRE(y_dtype == ME_BF16, "me_gemm_decode: the SiLU epilogue writes bfloat16");
     ME_DL(1, bf16, 16);
+  } else if (epi == 3) {
+    if (rows == 8) ME_DL(3, bf16, 8); else ME_DL(3, bf16, 16);
   } else if (y_dtype == ME_BF16) {
     if (rows == 8) ME_DL(0, bf16, 8); else ME_DL(0, bf16, 16);
   } else {

@@ -45,7 +45,7 @@ template <int XR> constexpr int gs_stages() { return XR == 8 ? 6 : 5; }
 __host__ __device__ __forceinline__ long long gs_first_stage(long long total, int nb, int b) { return total * b / nb; }
 __device__ __forceinline__ void consumers_sync() { asm volatile("bar.sync 1, %0;\n" ::"n"(GS_CONSUMERS) : "memory"); }
 
-// EPI 0: Y[m][n] (bfloat16 or float32), through activation ``act`` of common.cuh when that is not negative.  EPI 1: SiLU(gate) * up, bfloat16 (a group is 64 gate rows and their 64 up
+// EPI 0: Y[m][n] (bfloat16 or float32); EPI 3: through activation ``act`` of common.cuh, bfloat16.  EPI 1: SiLU(gate) * up, bfloat16 (a group is 64 gate rows and their 64 up
 // rows).  EPI 2: residual_out[m][n] += v; sumsq_out[block][m] = the block's share of the new residual's sums of
 // squares; with ``next_w`` also xw_out[m][n] = residual_out[m][n] * next_w[n].
 // XR: rows of the X tile and of map_x's boxes (8 for up to 8 rows of X: the upper n8 tile then reads one chunk of zeros).
@@ -274,7 +274,7 @@ gemm_stream_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_const
                 sq += val * val;
                 if (xw_out != nullptr) xw_out[(int64_t)m * N + n] = __float2bfloat16(val * next_w[n]);
               } else {
-                Y[(int64_t)m * ldy + n] = from_f<TO>(act >= 0 ? act_apply<TO>(val, act) : val);
+                Y[(int64_t)m * ldy + n] = from_f<TO>(EPI == 3 ? act_apply<TO>(val, act) : val);
               }
             }
           }
@@ -343,8 +343,8 @@ ME_API int me_gemm_stream(int epi, const void* map_x, const float* sumsq_in, int
              "me_gemm_stream: tensor maps, work buffers and the error word are required");
   ME_REQUIRE(sumsq_in == nullptr || sumsq_parts > 0, "me_gemm_stream: sums of squares in %d parts", sumsq_parts);
   const int act = epi >= 3 && epi <= 3 + ACT_GELU_ERF ? epi - 3 : -1;
-  if (act >= 0) epi = 0;
-  ME_REQUIRE(epi == 0 || epi == 1 || (epi == 2 && res_out != nullptr && sumsq_out != nullptr), "me_gemm_stream: epilogue %d", epi);
+  if (act >= 0) epi = 3;
+  ME_REQUIRE(epi == 0 || epi == 1 || (epi == 3 && act >= 0 && y_dtype == ME_BF16) || (epi == 2 && res_out != nullptr && sumsq_out != nullptr), "me_gemm_stream: epilogue %d", epi);
   ME_REQUIRE((next_w == nullptr) == (xw_out == nullptr) && (next_w == nullptr || epi == 2),
              "me_gemm_stream: the pre-weighted copy needs the residual epilogue, a weight and an output");
   int rc = 1;
@@ -358,6 +358,8 @@ ME_API int me_gemm_stream(int epi, const void* map_x, const float* sumsq_in, int
   } else if (epi == 1) {
     ME_REQUIRE(y_dtype == ME_BF16, "me_gemm_stream: the SiLU epilogue writes bfloat16");
     ME_GS(1, bf16);
+  } else if (epi == 3) {
+    ME_GS(3, bf16);
   } else if (y_dtype == ME_BF16) {
     ME_GS(0, bf16);
   } else {
