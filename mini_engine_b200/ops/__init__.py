@@ -1196,7 +1196,7 @@ def gla_scan(proj: torch.Tensor, offsets: dict, la: torch.Tensor, S: torch.Tenso
     (heads * dim * vdim values for every run of GLA_CHUNK tokens: ``gla_chunk_count``) the requests that bring several tokens
     take GLA_CHUNK tokens at a time, all runs of the step side by side (``gla_chunks``); ``la`` is overwritten on the way.
 
-    ``gate`` = (bias, lower), float32 [heads * dim] each: the recurrence whose forget gate also says what is written.  The columns
+    ``gate`` = (bias, lower), float32 [heads * dim] each: the recurrence with one gate a channel for keeping and writing (HGRN2).  The columns
     ``offsets["k"]`` then hold the gate's pre-activations z, and a = lower + (1 - lower) sigmoid(z + bias), k = 1 - a, q <- silu(q);
     ``la`` is a work buffer, and the q and k columns of ``proj`` are written on the way."""
     T = proj.shape[0]

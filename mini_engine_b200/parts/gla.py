@@ -71,7 +71,7 @@ class GatedLinearAttention(Mixer):
 
 
 class HGRN2(Mixer):
-    """Linear attention whose forget gate also decides what is written, with a state slot per request.
+    """A recurrence with a matrix state in which one gate a channel is both the decay and, as 1 - gate, the key; a state slot per request.
 
     Per head: q = silu(W_q h) and a gate per channel f = l + (1 - l) sigmoid(W_f h + b), ``dim`` values each, with a learned
     lower bound l; v = W_v h (``vdim`` values); then

@@ -142,7 +142,7 @@ def gated_recurrence(q, f, v, state=None):
 
 
 def hgrn2(h, w, p, m, eps, state=None):
-    """Linear attention whose forget gate also says what is written; returns (output, last state)."""
+    """A matrix state with the gate as decay and 1 - gate as key; returns (output, last state)."""
     T, H, D, Dv = h.shape[0], m["heads"], m["dim"], m["vdim"]
     q = silu(h @ w[p + "q"].T).view(T, H, D)
     f = forget_gate(h @ w[p + "f"].T + w[p + "f.b"], w[p + "lower"]).view(T, H, D)
