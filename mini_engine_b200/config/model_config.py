@@ -756,3 +756,121 @@ class TidenexConfig(ModelConfig):
         if self.loop:
             d["loop"] = self.loop
         return d
+
+
+def _sub_object(raw: dict, key: str, where: str) -> dict:
+    v = raw.get(key)
+    if not isinstance(v, dict):
+        raise ConfigError(f"{where}: lacks the object {key!r}")
+    return v
+
+
+@dataclass
+class KuteraxConfig(ModelConfig):
+    """Kuterax: a decoder whose layers run mixer and feed-forward side by side behind ONE norm, each scaled element by element before it
+    joins the stream, with learned position vectors on the embedding; mixers are windowed attention beside a Mamba-2 recurrence, each
+    behind an output norm of its own, or retention; feed-forwards are routed squared-relu experts with a gated shared one.  A range
+    of layers may run several times in a row with the same weights, each pass starting from a product of the stream and the embedding
+    output.  config.json keys: ``vocab``, ``width``, ``max_positions``, ``norm.eps``, ``loop`` {start, stop, times} (absent: every layer once) and
+    ``layers``: a list of ``{"type", "mixer", "mlp"}`` with
+
+    * type ``parallel``: mixer {left {heads, kv_heads, dim, vdim, scale, rot {base, dims, scaling {factor, original, fast, slow}}, mask {size}},
+      right {heads, vdim, state, groups, conv (taps), norm_groups}} (``rot``, ``scaling`` and ``mask`` may be absent);
+    * type ``retention``: mixer {heads, dim, vdim, decay [a number a head]};
+    * mlp: null or moe {router {experts, top, scale, groups {count, keep}}, expert {ff}, shared {ff}} (``scale``, ``groups`` and ``shared`` may be
+      absent)."""
+
+    norm_eps: float = 0.0
+    loop: dict[str, int] | None = None
+    layers: list[dict[str, Any]] = field(default_factory=list)
+
+    @classmethod
+    def from_dict(cls, raw: dict[str, Any]) -> "KuteraxConfig":
+        layers = _need(raw, "layers", list)
+        if not isinstance(layers, list) or not layers:
+            raise ConfigError("config.json key 'layers' must be a list with at least one layer")
+        checked = [cls._layer(layer, f"layer {i}") for i, layer in enumerate(layers)]
+        loop = _opt_object(raw, "loop", "config.json")
+        if loop is not None:
+            loop = {k: _need(loop, k, int) for k in ("start", "stop", "times")}
+            if not 0 <= loop["start"] < loop["stop"] <= len(checked) or loop["times"] < 1:
+                raise ConfigError(f"loop must name a range of layers and a positive number of passes: {loop}")
+        eos = raw.get("eos_token_id", -1)
+        cfg = cls(architecture=architecture_name(raw), vocab_size=_need(raw, "vocab", int), hidden_size=_need(raw, "width", int),
+                  num_hidden_layers=len(checked), max_position_embeddings=_need(raw, "max_positions", int),
+                  eos_token_id=-1 if eos is None else int(eos), norm_eps=_need(_sub_object(raw, "norm", "config.json"), "eps", float),
+                  loop=loop, layers=checked)
+        if cfg.vocab_size < 1 or cfg.hidden_size < 1 or cfg.max_position_embeddings < 1:
+            raise ConfigError("vocab, width and max_positions must be positive")
+        if not cfg.norm_eps > 0:
+            raise ConfigError("norm.eps must be positive")
+        return cfg
+
+    @staticmethod
+    def _layer(layer: Any, where: str) -> dict[str, Any]:
+        kind = layer.get("type") if isinstance(layer, dict) else None
+        if kind not in ("parallel", "retention"):
+            raise ConfigError(f"{where}: 'type' must be 'parallel' or 'retention', got {kind!r}")
+        mixer = _sub_object(layer, "mixer", where)
+        if kind == "parallel":
+            raw, at = _sub_object(mixer, "left", where), where + " left"
+            left: dict[str, Any] = _positive_ints(raw, ("heads", "kv_heads", "dim", "vdim"), at)
+            if left["heads"] % left["kv_heads"]:
+                raise ConfigError(f"{at}: heads must be a multiple of kv_heads: {left}")
+            left["scale"] = _need(raw, "scale", float)
+            rot = _opt_object(raw, "rot", at)
+            if rot is not None:
+                left["rot"] = r = {"base": _need(rot, "base", float), "dims": _need(rot, "dims", int)}
+                if r["dims"] % 2 or not 0 <= r["dims"] <= left["dim"] or not r["base"] > 0:
+                    raise ConfigError(f"{at}: rot.dims must be even and at most dim, rot.base positive: {r}")
+                sc = _opt_object(rot, "scaling", at)
+                if sc is not None:
+                    r["scaling"] = {k: _need(sc, k, float) for k in ("factor", "original", "fast", "slow")}
+                    if not all(v > 0 for v in r["scaling"].values()) or r["base"] == 1.0:
+                        raise ConfigError(f"{at}: rot.scaling needs positive numbers and a base other than 1: {r}")
+            mask = _opt_object(raw, "mask", at)
+            if mask is not None and mask.get("size") is not None:
+                left["mask"] = _positive_ints(mask, ("size",), at + " mask")
+            right = _positive_ints(_sub_object(mixer, "right", where), ("heads", "vdim", "state", "groups", "conv", "norm_groups"), where + " right")
+            if right["heads"] % right["groups"] or (right["heads"] * right["vdim"]) % right["norm_groups"]:
+                raise ConfigError(f"{where} right: groups must divide heads, and norm_groups heads * vdim: {right}")
+            m: dict[str, Any] = {"left": left, "right": right}
+        else:
+            m = _positive_ints(mixer, ("heads", "dim", "vdim"), where)
+            decay = _need(mixer, "decay", list)
+            if (not isinstance(decay, list) or len(decay) != m["heads"]
+                    or not all(isinstance(d, (int, float)) and not isinstance(d, bool) and 0 < d <= 1 for d in decay)):
+                raise ConfigError(f"{where}: decay must list a number above 0 and up to 1 for each of the {m['heads']} heads")
+            m["decay"] = [float(d) for d in decay]
+        mlp = layer.get("mlp")
+        if mlp is not None:
+            if not isinstance(mlp, dict) or mlp.get("kind") != "moe":
+                raise ConfigError(f"{where}: 'mlp' must be null or of kind 'moe', got {mlp!r}")
+            router = _sub_object(mlp, "router", where + " mlp")
+            r = _positive_ints(router, ("experts", "top"), where + " mlp.router")
+            r["scale"] = _need(router, "scale", float) if router.get("scale") is not None else 1.0
+            groups = _opt_object(router, "groups", where + " mlp.router")
+            r["groups"] = g = _positive_ints(groups, ("count", "keep"), where + " mlp.router.groups") if groups else {"count": 1, "keep": 1}
+            if r["experts"] % g["count"] or g["keep"] > g["count"] or g["keep"] * (r["experts"] // g["count"]) < r["top"]:
+                raise ConfigError(f"{where}: {g['keep']} of {g['count']} groups over {r['experts']} experts cannot give {r['top']} choices")
+            out = {"kind": "moe", "router": r, "expert": _positive_ints(_sub_object(mlp, "expert", where + " mlp"), ("ff",), where + " mlp.expert")}
+            shared = _opt_object(mlp, "shared", where)
+            if shared is not None:
+                out["shared"] = _positive_ints(shared, ("ff",), where + " mlp.shared")
+            mlp = out
+        return {"type": kind, "mixer": m, "mlp": mlp}
+
+    def layer_runs(self) -> list[tuple[int, int | None]]:
+        """The order in which layers run as (layer, pass) pairs; ``pass``: the number of the pass that starts right before the layer (its
+        first layer's), else None."""
+        n = len(self.layers)
+        a, b, times = (self.loop["start"], self.loop["stop"], self.loop["times"]) if self.loop else (0, 0, 0)
+        passes = [(i, t if i == a else None) for t in range(times) for i in range(a, b)]
+        return [(i, None) for i in range(a)] + passes + [(i, None) for i in range(b, n)]
+
+    def to_json_dict(self) -> dict[str, Any]:
+        d = {"architecture": self.architecture, "vocab": self.vocab_size, "width": self.hidden_size, "max_positions": self.max_position_embeddings,
+             "norm": {"eps": self.norm_eps}, "layers": self.layers}
+        if self.loop:
+            d["loop"] = self.loop
+        return d

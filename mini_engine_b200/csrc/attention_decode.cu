@@ -873,7 +873,7 @@ __global__ void decode_merge_kernel(T* __restrict__ out, int64_t out_row_stride,
                                     const float* __restrict__ tmp_l, int nh, int hd, int max_parts, int part_keys,
                                     int sink, const float* __restrict__ gate, int64_t gate_stride,
                                     const float* __restrict__ sinks, int pool_base, int pool_parts, int pool_p, int pool_window,
-                                    int out_hd) {
+                                    int out_hd, int gate_heads) {
   constexpr int CHUNK = 128;                         // partitions whose factors are held in shared memory at a time
   __shared__ float f_s[CHUNK], red[32];
   const int b = blockIdx.x, h = blockIdx.y;
@@ -913,7 +913,7 @@ __global__ void decode_merge_kernel(T* __restrict__ out, int64_t out_row_stride,
     }
     if (tid < out_hd) {
       float v = lt > 0.f ? acc / lt : 0.f;
-      if (gate) v = v / (1.f + expf(-gate[tok * gate_stride + (int64_t)h * hd + tid]));
+      if (gate) v = v / (1.f + expf(-gate[tok * gate_stride + (gate_heads ? h : (int64_t)h * hd + tid)]));
       out[tok * out_row_stride + (int64_t)h * out_hd + tid] = from_f<T>(v);
     }
     return;
@@ -986,7 +986,7 @@ __global__ void decode_merge_kernel(T* __restrict__ out, int64_t out_row_stride,
     const int d = tid + c * (int)blockDim.x;
     if (d < out_hd) {
       float v = lt > 0.f ? acc[c] / lt : 0.f;
-      if (gate) v = v / (1.f + expf(-gate[tok * gate_stride + (int64_t)h * hd + d]));
+      if (gate) v = v / (1.f + expf(-gate[tok * gate_stride + (gate_heads ? h : (int64_t)h * hd + d)]));
       o[d] = from_f<T>(v);
     }
   }
@@ -1065,13 +1065,15 @@ ME_API int me_attn_decode(const void* qkv, int dtype, int64_t q_row_stride, void
                           int* err, int kind, const void* kv_map, int sink, const float* gate, int64_t gate_stride,
                           int keep_first, int chunk, float softcap, const float* sinks, const void* pool_map,
                           const int* pooled_tables, int pbt_stride, int pool_p, int pool_parts, const float* bias_r1,
-                      const float* bias_r2, int out_hd, int pairs, float pair_lambda, float pair_gain, float pair_eps, cudaStream_t stream) {
+                      const float* bias_r2, int out_hd, int pairs, float pair_lambda, float pair_gain, float pair_eps, int gate_heads,
+                      cudaStream_t stream) {
   if (num_reqs == 0) return 0;
   // out_hd: how many elements of a head leave (0: all; rows of the cache may be longer than the values).  bias_r1, bias_r2
   // (float32 [nh], both or neither; the tensor-map kernel's alone): r1 ln(1 + r2 distance) is taken off the scaled scores.
+  // gate_heads: the gate has one pre-activation a head instead of one an output element.
   // pairs: query heads come in pairs whose difference is normed and written (decode_merge_pairs_kernel).
   if (out_hd == 0) out_hd = hd;
-  ME_REQUIRE(out_hd > 0 && out_hd <= hd && !(gate && out_hd != hd), "me_attn_decode: %d of %d output elements", out_hd, hd);
+  ME_REQUIRE(out_hd > 0 && out_hd <= hd && !(gate && !gate_heads && out_hd != hd), "me_attn_decode: %d of %d output elements", out_hd, hd);
   ME_REQUIRE((bias_r1 == nullptr) == (bias_r2 == nullptr) && !(bias_r1 && (softcap > 0.f || sinks || sink || pool_p > 0)),
              "me_attn_decode: a distance bias has two numbers a head and goes without caps, sinks and pooled blocks");
   ME_REQUIRE(!pairs || (nh % 2 == 0 && hd <= 128 && !gate && !sinks && !sink && pool_p == 0), "me_attn_decode: pairs of heads go without gates, sinks and pooled blocks");
@@ -1166,7 +1168,7 @@ ME_API int me_attn_decode(const void* qkv, int dtype, int64_t q_row_stride, void
   const int mthreads = hd >= 128 ? 128 : (hd >= 64 ? 64 : 32);
   ME_DISPATCH_DTYPE(dtype, T, (me_launch(decode_merge_kernel<T>, mgrid, dim3(mthreads), 0, stream,
       (T*)out, out_row_stride, cu_seqlens, context_lens, tmp_out, tmp_m, tmp_l, nh, hd, max_parts, DEC_PART, sink, gate,
-      gate_stride, sinks, tok_parts, pool_parts, pool_p, window, out_hd)));
+      gate_stride, sinks, tok_parts, pool_parts, pool_p, window, out_hd, gate_heads)));
   ME_LAUNCH_CHECK("me_attn_decode (merge)");
   return 0;
 }
@@ -1236,7 +1238,7 @@ ME_API int me_attn_decode_fused(const void* qkv, int64_t q_row_stride, void* out
   dim3 mgrid(num_reqs, nh);
   me_launch(decode_merge_kernel<bf16>, mgrid, dim3(hd >= 128 ? 128 : 64), 0, stream, (bf16*)out, out_row_stride, cu_seqlens,
             context_lens, tmp_out, tmp_m, tmp_l, nh, hd, max_parts, DEC_PART * tiles, 0, (const float*)nullptr, (int64_t)0,
-            (const float*)nullptr, 0, 0, 0, 0, hd);
+            (const float*)nullptr, 0, 0, 0, 0, hd, 0);
   ME_LAUNCH_CHECK("me_attn_decode_fused (merge)");
   return 0;
 }

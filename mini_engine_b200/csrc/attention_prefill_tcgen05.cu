@@ -393,7 +393,8 @@ attn_prefill_tcgen05_two_groups_kernel(const __grid_constant__ CUtensorMap q_map
                                        int* __restrict__ err, int keep_first_arg, int chunk_arg, float softcap_arg,
                                        const float* __restrict__ sinks_arg, const __grid_constant__ CUtensorMap pool_map,
                                        const int* __restrict__ pooled_tables, int pbt_stride, int pool_p_arg,
-                                       const float* __restrict__ bias_r1, const float* __restrict__ bias_r2, int out_hd, PairArgs pair) {
+                                       const float* __restrict__ bias_r1, const float* __restrict__ bias_r2, int out_hd, int gate_heads,
+                                       PairArgs pair) {
   const int keep_first = EXTRA ? keep_first_arg : 0, chunk = EXTRA ? chunk_arg : 0;
   const int pool_p = EXTRA ? pool_p_arg : 0;
   const float softcap = EXTRA ? softcap_arg : 0.f;
@@ -803,7 +804,9 @@ attn_prefill_tcgen05_two_groups_kernel(const __grid_constant__ CUtensorMap q_map
     constexpr int OC = HD / 2, PIECES = HD / 8;              // group 0 takes the first half of the row's columns, group 1 the other
     if (ok) {
       tc5::fence_after_sync();
-      const float inv = l > 0.f ? 1.f / l : 0.f;
+      float inv = l > 0.f ? 1.f / l : 0.f;
+      if (gate && gate_heads && row_ok)                      // one number a head: a factor of the whole row
+        inv = __fdividef(inv, 1.f + __expf(-gate[(int64_t)(tok0 + q0 + tk) * gate_stride + head0 + r / tq]));
 #pragma unroll
       for (int c0 = 0; c0 < OC; c0 += 32) {
         float o_acc[32];
@@ -828,7 +831,7 @@ attn_prefill_tcgen05_two_groups_kernel(const __grid_constant__ CUtensorMap q_map
         const int tok = row % tq;
         if (tok < n_tok && piece * 8 < out_hd) {
           uint4 pk = *reinterpret_cast<const uint4*>(q_s + row * (HD * 2) + ((piece ^ (row & 7)) << 4));
-          if (gate) {
+          if (gate && !gate_heads) {
             // The output times the sigmoid of the gate's pre-activation, here where the lanes of a row read the gate's row
             // side by side (a lane a row, at the read-out from tensor memory, took 32 lines a load).
             const float* gr = gate + (int64_t)(tok0 + q0 + tok) * gate_stride + (int64_t)(head0 + row / tq) * HD + piece * 8;
@@ -857,7 +860,7 @@ int launch_ta(const void* q_map, const void* kv_map, void* out, int64_t out_row_
               const int* cu_seqlens, const int* context_lens, const int* tiles, int num_tiles, int nh, int nkv, int gp,
               int page_size, float scale, int window, int sink, const float* gate, int64_t gate_stride, int* err,
               int keep_first, int chunk, float softcap, const float* sinks, const void* pool_map, const int* pooled_tables,
-              int pbt_stride, int pool_p, const float* bias_r1, const float* bias_r2, int out_hd, bool pairs, PairArgs pair, cudaStream_t stream) {
+              int pbt_stride, int pool_p, const float* bias_r1, const float* bias_r2, int out_hd, bool pairs, PairArgs pair, int gate_heads, cudaStream_t stream) {
   const size_t smem = TWO_GROUPS ? (size_t)TA_ROWS * HD * 2 + 6 * (size_t)KT * HD * 2 + 1024
                                  : (size_t)TA_ROWS * HD * 2 + 4 * (size_t)KT * HD * 2 + 2 * (size_t)TA_ROWS * KT * 2 + 1024;
   static bool attr_set = false;
@@ -886,7 +889,7 @@ int launch_ta(const void* q_map, const void* kv_map, void* out, int64_t out_row_
               *reinterpret_cast<const CUtensorMap*>(kv_map), (bf16*)out, out_row_stride, block_tables, bt_stride, cu_seqlens,
               context_lens, tiles, nh, nkv, gp, page_size, scale * 1.4426950408889634f, window, sink, gate, gate_stride, err,
               keep_first, chunk, softcap, sinks, *reinterpret_cast<const CUtensorMap*>(pool_p > 0 ? pool_map : kv_map), pooled_tables,
-              pbt_stride, pool_p, bias_r1, bias_r2, out_hd, pair);
+              pbt_stride, pool_p, bias_r1, bias_r2, out_hd, gate_heads, pair);
   } else
     me_launch(attn_prefill_tcgen05_kernel<HD, KT>, grid, dim3(TA_THREADS), smem, stream, *reinterpret_cast<const CUtensorMap*>(q_map),
               *reinterpret_cast<const CUtensorMap*>(kv_map), (bf16*)out, out_row_stride, block_tables, bt_stride, cu_seqlens,
@@ -925,7 +928,8 @@ ME_API int me_attn_prefill_tcgen05(const void* q_map, const void* kv_map, void* 
                                    int window, int key_tile, int sink, const float* gate, int64_t gate_stride, int* err,
                                    int keep_first, int chunk, float softcap, const float* sinks, const void* pool_map,
                                    const int* pooled_tables, int pbt_stride, int pool_p, const float* bias_r1, const float* bias_r2,
-                                   int out_hd, int pairs, float pair_lambda, float pair_gain, float pair_eps, cudaStream_t stream) {
+                                   int out_hd, int pairs, float pair_lambda, float pair_gain, float pair_eps, int gate_heads,
+                                   cudaStream_t stream) {
   if (num_tiles == 0) return 0;
   const int gp = me_attn_prefill_tcgen05_heads_per_block(nh, nkv, hd, page_size);
   ME_REQUIRE(gp > 0, "me_attn_prefill_tcgen05: head_dim %d, %d/%d heads, pages of %d are not taken", hd, nh, nkv, page_size);
@@ -936,9 +940,9 @@ ME_API int me_attn_prefill_tcgen05(const void* q_map, const void* kv_map, void* 
   // faster one; 64: the kernel with one group and P in shared memory, which needs less of both memories.
   if (key_tile == 0) key_tile = 128;
   if (out_hd == 0) out_hd = hd;
-  ME_REQUIRE(key_tile == 128 || (keep_first == 0 && chunk == 0 && softcap == 0.f && sinks == nullptr && pool_p == 0 && !bias_r1 && out_hd == hd),
-             "me_attn_prefill_tcgen05: kept first keys, chunks, capped scores, learned sinks, pooled blocks, biases and short outputs need the key tile of 128");
-  ME_REQUIRE(out_hd > 0 && out_hd <= hd && out_hd % 8 == 0 && !(gate && out_hd != hd), "me_attn_prefill_tcgen05: %d of %d output elements", out_hd, hd);
+  ME_REQUIRE(key_tile == 128 || (keep_first == 0 && chunk == 0 && softcap == 0.f && sinks == nullptr && pool_p == 0 && !bias_r1 && out_hd == hd && !gate_heads),
+             "me_attn_prefill_tcgen05: kept first keys, chunks, capped scores, learned sinks, pooled blocks, biases, short outputs and gates a head need the key tile of 128");
+  ME_REQUIRE(out_hd > 0 && out_hd <= hd && out_hd % 8 == 0 && !(gate && !gate_heads && out_hd != hd), "me_attn_prefill_tcgen05: %d of %d output elements", out_hd, hd);
   ME_REQUIRE(!pairs || (gp % 2 == 0 && key_tile == 128 && !gate && !sink && !sinks && softcap == 0.f && keep_first == 0 && chunk == 0 && pool_p == 0 && !bias_r1),
              "me_attn_prefill_tcgen05: pairs of heads need an even group and go with a plain window at most");
   const PairArgs pair = {pair_lambda, pair_gain, pair_eps};
@@ -953,7 +957,7 @@ ME_API int me_attn_prefill_tcgen05(const void* q_map, const void* kv_map, void* 
   int rc;
 #define ME_TA_ARGS q_map, kv_map, out, out_row_stride, block_tables, bt_stride, cu_seqlens, context_lens, tiles, num_tiles, nh, nkv, gp, \
                    page_size, scale, window, sink, gate, gate_stride, err, keep_first, chunk, softcap, sinks, pool_map, pooled_tables, \
-                   pbt_stride, pool_p, bias_r1, bias_r2, out_hd, pairs != 0, pair, stream
+                   pbt_stride, pool_p, bias_r1, bias_r2, out_hd, pairs != 0, pair, gate_heads, stream
   if (hd == 64) rc = key_tile == 64 ? launch_ta<64, 64, false>(ME_TA_ARGS) : launch_ta<64, 128, true>(ME_TA_ARGS);
   else rc = key_tile == 64 ? launch_ta<128, 64, false>(ME_TA_ARGS) : launch_ta<128, 128, true>(ME_TA_ARGS);
 #undef ME_TA_ARGS

@@ -8,7 +8,7 @@
 //   q, k: rotary positions on the first ``rot`` elements of a head, element i paired with element i + rot/2:
 //         (a, b) -> (a cos t - b sin t, b cos t + a sin t), t = position * freq[i]; the angle is formed in double precision
 //         from the int32 position and a table of rot/2 frequencies (so any scaling of the frequencies is the table's
-//         business), brought into [-pi, pi] there, then float32 sine and cosine
+//         business), brought into [-pi, pi] there, then float32 sine and cosine, both times rot_mag
 //   q, k: u <- u / rms(u)       (NORM_AFTER, no weight)
 //   q: u <- u * q_scale[head]   (a learned number per query head that multiplies the head's scores; optional)
 //   q: u <- u * (1 + temp_coef ln(floor((position + 1) / temp_every) + 1))      (a temperature that grows with the position)
@@ -46,7 +46,7 @@ struct PrepArgs {
   int HD, page_size, H, G, D, Dv, M, q_row, n_tok;
   const float* q_scale;
   int own_kv;
-  float temp_coef, temp_every, v_scale;
+  float temp_coef, temp_every, v_scale, rot_mag;
 };
 
 // One unit of a token's row: hs counts the query maps, then the key maps, then the value heads.  inv_q, inv_k: 1 / rms of the
@@ -98,6 +98,8 @@ __device__ __forceinline__ void prep_unit(const PrepArgs& a, T* __restrict__ q_o
           double x = pos * a.freq[f];
           x -= 6.283185307179586476925 * rint(x * 0.15915494309189533577);
           sincosf((float)x, &sn, &cs);
+          sn *= a.rot_mag;
+          cs *= a.rot_mag;
           u[i] = d < half ? st[d] * cs - st[d + half] * sn : st[d] * cs + st[d - half] * sn;
         }
       }
@@ -220,7 +222,10 @@ __global__ void __launch_bounds__(256) attn_prep_vec_kernel(PrepArgs a, T* __res
   if (tid < half) {
     double x = (double)pos * a.freq[tid];
     x -= 6.283185307179586476925 * rint(x * 0.15915494309189533577);
-    sincosf((float)x, &sn_s[tid], &cs_s[tid]);
+    float sn, cs;
+    sincosf((float)x, &sn, &cs);
+    sn_s[tid] = sn * a.rot_mag;
+    cs_s[tid] = cs * a.rot_mag;
   }
   pdl_wait();
   pdl_launch_dependents();
@@ -352,7 +357,8 @@ static int prep_vec_passes(const PrepArgs& a, const void* q_out, const void* poo
 ME_API int me_attn_prep(const float* proj, int64_t ld, const float* bias, const float* q_w, const float* k_w, int norm_mode,
                         float eps, const double* freq, int rot, const int* positions, const int* slot_mapping,
                         void* q_out, int q_row, void* pool, int dtype, int HD, int page_size, int H, int G, int D, int Dv, int maps, int T,
-                        const float* q_scale, int own_kv, float temp_coef, float temp_every, float v_scale, cudaStream_t stream) {
+                        const float* q_scale, int own_kv, float temp_coef, float temp_every, float v_scale, float rot_mag,
+                        cudaStream_t stream) {
   if (T == 0) return 0;
   ME_REQUIRE(T > 0 && H > 0 && G > 0 && D >= 1 && D <= AP_MAX && Dv >= 1 && Dv <= AP_MAX && (maps == 1 || maps == 2),
              "me_attn_prep: bad sizes H=%d G=%d D=%d Dv=%d maps=%d", H, G, D, Dv, maps);
@@ -362,7 +368,7 @@ ME_API int me_attn_prep(const float* proj, int64_t ld, const float* bias, const 
   ME_REQUIRE(!slot_mapping || (pool && HD >= maps * D && HD >= Dv), "me_attn_prep: cache rows of %d elements are too short", HD);
   ME_REQUIRE(temp_every >= 0.f, "me_attn_prep: the temperature's step must not be negative");
   const PrepArgs a = {proj, ld, bias, q_w, k_w, norm_mode, eps, freq, rot, positions, slot_mapping, HD, page_size, H, G, D, Dv, maps,
-                      q_row, T, q_scale, own_kv, temp_coef, temp_every, v_scale};
+                      q_row, T, q_scale, own_kv, temp_coef, temp_every, v_scale, rot_mag};
   const int64_t units = (int64_t)T * (H * maps + (own_kv ? G * (maps + 1) : 0));
   int lanes = 0;
   const int passes = prep_vec_passes(a, q_out, pool, dtype, lanes);

@@ -8,36 +8,45 @@
 // A negative id ~j stands for ``feedback[j]``: the token that the step before drew for row j, still on the
 // device.  That lets the host launch a decode step before it has read the step before it.
 // The row is multiplied by ``scale`` and written ``copies`` times, ``copy_stride`` elements apart (a model that
-// keeps several residual streams starts them all from the embedding).
-template <typename TW>
+// keeps several residual streams starts them all from the embedding).  With ``pos_table`` [P, H] a row of it, that of the token's
+// position, is added (not scaled).  ``out2``: the same row once more in a second type, rows out2_ld elements apart.
+template <typename TW, typename T2>
 __global__ void embed_kernel(const int* __restrict__ ids, const TW* __restrict__ table,
                              float* __restrict__ out, int H, int V, int* __restrict__ err,
                              const int* __restrict__ feedback, int n_feedback, float scale, int copies,
-                             int64_t copy_stride) {
+                             int64_t copy_stride, const TW* __restrict__ pos_table, const int* __restrict__ positions, int P,
+                             T2* __restrict__ out2, int64_t out2_ld) {
   pdl_wait();
   pdl_launch_dependents();
   const int t = blockIdx.x;
   int id = ids[t];
   if (id < 0 && feedback != nullptr && ~id < n_feedback) id = feedback[~id];
-  const bool ok = id >= 0 && id < V;
+  const int pos = pos_table ? positions[t] : 0;
+  const bool ok = id >= 0 && id < V && (!pos_table || (pos >= 0 && pos < P));
   if (!ok && threadIdx.x == 0) atomicOr(err, 1);
   const TW* row = table + (int64_t)(ok ? id : 0) * H;
+  const TW* prow = pos_table ? pos_table + (int64_t)(ok ? pos : 0) * H : nullptr;
   float* o = out + (int64_t)t * H;
   for (int h = threadIdx.x; h < H; h += blockDim.x) {
-    const float v = ok ? to_f<TW>(row[h]) * scale : 0.f;
+    float v = ok ? to_f<TW>(row[h]) * scale : 0.f;
+    if (ok && prow) v += to_f<TW>(prow[h]);
     for (int c = 0; c < copies; ++c) o[c * copy_stride + h] = v;
+    if (out2) out2[(int64_t)t * out2_ld + h] = from_f<T2>(v);
   }
 }
 
 ME_API int me_embed(const int* ids, const void* table, int table_dtype, float* out, int T, int H,
                     int V, int* err, const int* feedback, int n_feedback, float scale, int copies,
-                    int64_t copy_stride, cudaStream_t stream) {
+                    int64_t copy_stride, const void* pos_table, const int* positions, int P, void* out2, int out2_dtype,
+                    int64_t out2_ld, cudaStream_t stream) {
   if (T == 0) return 0;
+  ME_REQUIRE(!pos_table || (positions && P > 0), "me_embed: a table over positions needs the positions");
+  ME_REQUIRE(!out2 || out2_ld >= H, "me_embed: rows of the second output %lld elements apart", (long long)out2_ld);
   ME_REQUIRE(T > 0 && H > 0 && V > 0 && copies >= 1, "me_embed: bad sizes T=%d H=%d V=%d copies=%d", T, H, V, copies);
   const int threads = H >= 1024 ? 256 : (H >= 256 ? 128 : 64);
-  ME_DISPATCH_DTYPE(table_dtype, TW,
-                    me_launch(embed_kernel<TW>, dim3(T), dim3(threads), 0, stream, ids, (const TW*)table, out, H, V, err,
-                              feedback, n_feedback, scale, copies, copy_stride));
+  ME_DISPATCH_DTYPE(table_dtype, TW, ME_DISPATCH_DTYPE(out2 ? out2_dtype : ME_F32, T2,
+                    me_launch(embed_kernel<TW, T2>, dim3(T), dim3(threads), 0, stream, ids, (const TW*)table, out, H, V, err,
+                              feedback, n_feedback, scale, copies, copy_stride, (const TW*)pos_table, positions, P, (T2*)out2, out2_ld)));
   ME_LAUNCH_CHECK("me_embed");
   return 0;
 }

@@ -117,3 +117,78 @@ ME_API int me_group_norm(float* residual, const void* y, int y_dtype, int64_t y_
   ME_LAUNCH_CHECK("me_group_norm");
   return 0;
 }
+
+// The norm behind a recurrence: a row of y is cut into ``groups`` equal parts, each divided by its own sqrt(mean^2 + eps), with the gate
+// silu(z) in front of the norm or behind it and an optional weight:
+//   first:  u = y silu(z),  out = u / rms_g(u) * w          else:  out = y / rms_g(y) * w * silu(z)
+// LANES threads a (row, group) pair: a warp for short groups (several pairs a block), a block for long ones; values are read twice (the
+// second time from the cache close by).
+template <typename TZ, typename TO, int LANES, bool VEC>
+__global__ void __launch_bounds__(256)
+gated_group_norm_kernel(const float* __restrict__ y, int64_t y_ld, const TZ* __restrict__ z, int64_t z_ld, const float* __restrict__ w, int gate_first,
+                        float eps, TO* __restrict__ out, int64_t out_ld, int64_t pairs, int groups, int n) {
+  __shared__ float red[32];
+  constexpr int V = VEC ? 4 : 1;
+  pdl_wait();
+  pdl_launch_dependents();
+  const int lane = threadIdx.x % LANES;
+  const int64_t pair = (int64_t)blockIdx.x * (blockDim.x / LANES) + threadIdx.x / LANES;
+  if (LANES == 32 && pair >= pairs) return;
+  const int64_t t = pair / groups;
+  const int c0 = (int)(pair - t * groups) * n;
+  const float* yr = y + t * y_ld + c0;
+  const TZ* zr = z + t * z_ld + c0;
+  auto gated = [&](int i, float (&u)[4], float (&s)[4]) {      // u: what is normed; s: silu(z)
+    load4<float, VEC>(yr + i, u);
+    load4<TZ, VEC>(zr + i, s);
+#pragma unroll
+    for (int j = 0; j < V; ++j) {
+      s[j] = s[j] / (1.f + expf(-s[j]));
+      if (gate_first) u[j] *= s[j];
+    }
+  };
+  float ss = 0.f;
+  for (int i = lane * V; i < n; i += LANES * V) {
+    float u[4], s[4];
+    if (gate_first) gated(i, u, s);
+    else load4<float, VEC>(yr + i, u);
+#pragma unroll
+    for (int j = 0; j < V; ++j) ss = fmaf(u[j], u[j], ss);
+  }
+  ss = LANES == 32 ? warp_sum(ss) : block_sum(ss, red);
+  const float r = 1.0f / sqrtf(ss / (float)n + eps);
+  for (int i = lane * V; i < n; i += LANES * V) {
+    float u[4], s[4], f[4];
+    gated(i, u, s);
+    if (w) load4<float, VEC>(w + c0 + i, f);
+#pragma unroll
+    for (int j = 0; j < V; ++j) u[j] = u[j] * r * (w ? f[j] : 1.f) * (gate_first ? 1.f : s[j]);
+    store4<TO, VEC>(out + t * out_ld + c0 + i, u);
+  }
+}
+
+// y: [T, W] float32 rows; z: [T, W] of z_dtype; w: [W] float32 or null; out: [T, W] of out_dtype.  Rows lie *_ld elements apart.
+ME_API int me_gated_group_norm(const float* y, int64_t y_ld, const void* z, int z_dtype, int64_t z_ld, const float* w, int gate_first, float eps,
+                               void* out, int out_dtype, int64_t out_ld, int T, int W, int groups, cudaStream_t stream) {
+  if (T == 0) return 0;
+  ME_REQUIRE(T > 0 && W > 0 && groups > 0 && W % groups == 0, "me_gated_group_norm: %d groups of %d values", groups, W);
+  const int n = W / groups;
+  auto off = [](const void* p, size_t to) { return p && ((uintptr_t)p % to) != 0; };
+  const bool vec = n % 4 == 0 && y_ld % 4 == 0 && z_ld % 4 == 0 && out_ld % 4 == 0 && !off(y, 16) && !off(z, z_dtype == ME_F32 ? 16 : 8) && !off(w, 16) &&
+                   !off(out, out_dtype == ME_F32 ? 16 : 8);
+  const bool warps = n <= (vec ? 512 : 128);
+  const int64_t pairs = (int64_t)T * groups;
+  const int threads = warps ? (pairs >= 4096 ? 256 : 64) : 256;
+  const int64_t blocks = warps ? (pairs + threads / 32 - 1) / (threads / 32) : pairs;
+  ME_REQUIRE(blocks < (1ll << 31), "me_gated_group_norm: too many rows");
+#define GGN_CASE(LANES_, VEC_)                                                                                                              \
+  me_launch(gated_group_norm_kernel<TZ, TO, LANES_, VEC_>, dim3((unsigned)blocks), dim3(threads), 0, stream, y, y_ld, (const TZ*)z, z_ld, w, \
+            gate_first, eps, (TO*)out, out_ld, pairs, groups, n)
+  ME_DISPATCH_DTYPE(z_dtype, TZ, ME_DISPATCH_DTYPE(out_dtype, TO, {
+    if (warps) { if (vec) GGN_CASE(32, true); else GGN_CASE(32, false); }
+    else { if (vec) GGN_CASE(256, true); else GGN_CASE(256, false); }
+  }));
+#undef GGN_CASE
+  ME_LAUNCH_CHECK("me_gated_group_norm");
+  return 0;
+}

@@ -5,14 +5,16 @@
 //   me_moe_route_grouped   the other routing rule: scores s = sigmoid(z); an expert is chosen by s + correction (a learned number per
 //                   expert that steers the choice and nothing else); the experts form ``groups`` equal groups of neighbours, a
 //                   group's score is the sum of its two largest choice scores, and only experts of the ``keep`` best groups can be
-//                   chosen; the weights are the chosen experts' s themselves, not renormalised;
+//                   chosen; the weights are the chosen experts' s themselves, not renormalised.  ``softmax``: s is the softmax over all
+//                   experts instead, and a group's score is its largest.  The weights are multiplied by ``weight_scale``;
 //   me_moe_sort     the T * top (token, choice) pairs grouped by expert, in token order inside an expert: offsets [E + 1],
 //                   ``sorted`` (pair ids in expert order) and ``place`` (where each pair went);
 //   me_moe_gemm     one product per expert over its rows: rows of A are gathered through ``sorted`` (pair id / top = token)
 //                   or are already in expert order; with ``glu`` 1 the expert's weight holds gate rows then up rows and the
 //                   result is the clamped gated activation of the two products; ``glu`` 2 + k: activation k of common.cuh on
 //                   the plain product;
-//   me_moe_combine  y_t = sum_k weight[t, k] * rows[place[t * top + k]] (+ a shared expert's output), k in a fixed order.
+//   me_moe_combine  y_t = sum_k weight[t, k] * rows[place[t * top + k]] (+ a shared expert's output, times the sigmoid of one number a
+//                   token where it has a gate), k in a fixed order.
 //
 // The products here run on the CUDA cores with float32 accumulation in a fixed order (any dtypes, any sizes); bfloat16
 // operands whose sizes allow it take the tensor-core kernel of moe_mma.cu.
@@ -50,13 +52,31 @@ __device__ __forceinline__ void route_token(float* mine, int E, int top, int lan
 
 // The grouped rule for one token: ``mine`` [E] holds the logits and becomes the choice scores, ``score`` [E] the sigmoids,
 // ``gs`` [groups] the groups' scores.  Ties go to the lower index, among groups and among experts.
+struct GroupRule {
+  int groups, keep, softmax;      // softmax: scores by softmax over all experts and groups by their largest; else sigmoids, two largest
+  float weight_scale;
+};
 __device__ __forceinline__ void route_token_grouped(float* mine, float* score, float* gs, const float* __restrict__ correction, int E,
-                                                    int top, int groups, int keep, int lane, int* __restrict__ idx,
+                                                    int top, const GroupRule& rule, int lane, int* __restrict__ idx,
                                                     float* __restrict__ wgt) {
-  for (int e = lane; e < E; e += 32) {
-    const float sg = 1.0f / (1.0f + expf(-mine[e]));
-    score[e] = sg;
-    mine[e] = sg + (correction ? correction[e] : 0.f);
+  const int groups = rule.groups, keep = rule.keep;
+  if (rule.softmax) {
+    float m = -INFINITY, sum = 0.f;
+    for (int e = lane; e < E; e += 32) m = fmaxf(m, mine[e]);
+    m = warp_max(m);
+    for (int e = lane; e < E; e += 32) sum += score[e] = expf(mine[e] - m);
+    const float inv = 1.0f / warp_sum(sum);
+    for (int e = lane; e < E; e += 32) {
+      const float s = score[e] * inv;
+      score[e] = s;
+      mine[e] = s + (correction ? correction[e] : 0.f);
+    }
+  } else {
+    for (int e = lane; e < E; e += 32) {
+      const float sg = 1.0f / (1.0f + expf(-mine[e]));
+      score[e] = sg;
+      mine[e] = sg + (correction ? correction[e] : 0.f);
+    }
   }
   __syncwarp();
   if (groups > 1 && keep < groups) {
@@ -68,7 +88,7 @@ __device__ __forceinline__ void route_token_grouped(float* mine, float* score, f
         if (v > a) { b = a; a = v; }
         else if (v > b) b = v;
       }
-      gs[g] = n > 1 ? a + b : a;
+      gs[g] = n > 1 && !rule.softmax ? a + b : a;
     }
     __syncwarp();
     for (int k = 0; k < keep; ++k) {             // the best group still unmarked gets +inf, so that it is never taken twice
@@ -107,7 +127,7 @@ __device__ __forceinline__ void route_token_grouped(float* mine, float* score, f
     if (at == 0x7fffffff) at = k;                // nothing left to choose from: keep going with a valid index
     if (lane == 0) {
       idx[k] = at;
-      wgt[k] = best == -INFINITY ? 0.f : score[at];
+      wgt[k] = best == -INFINITY ? 0.f : score[at] * rule.weight_scale;
       mine[at] = -INFINITY;
     }
     __syncwarp();
@@ -115,7 +135,7 @@ __device__ __forceinline__ void route_token_grouped(float* mine, float* score, f
 }
 
 __global__ void __launch_bounds__(128)
-moe_route_grouped_kernel(const float* __restrict__ z, const float* __restrict__ correction, int E, int top, int groups, int keep,
+moe_route_grouped_kernel(const float* __restrict__ z, int64_t z_ld, const float* __restrict__ correction, int E, int top, GroupRule rule,
                          int* __restrict__ idx, float* __restrict__ wgt, int T) {
   extern __shared__ float zs[];               // [warps][2 E + groups]
   pdl_wait();
@@ -123,10 +143,10 @@ moe_route_grouped_kernel(const float* __restrict__ z, const float* __restrict__ 
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const int t = blockIdx.x * (blockDim.x >> 5) + warp;
   if (t >= T) return;
-  float* mine = zs + warp * (2 * E + groups);
-  for (int e = lane; e < E; e += 32) mine[e] = z[(int64_t)t * E + e];
+  float* mine = zs + warp * (2 * E + rule.groups);
+  for (int e = lane; e < E; e += 32) mine[e] = z[(int64_t)t * z_ld + e];
   __syncwarp();
-  route_token_grouped(mine, mine + E, mine + 2 * E, correction, E, top, groups, keep, lane, idx + (int64_t)t * top, wgt + (int64_t)t * top);
+  route_token_grouped(mine, mine + E, mine + 2 * E, correction, E, top, rule, lane, idx + (int64_t)t * top, wgt + (int64_t)t * top);
 }
 
 __global__ void __launch_bounds__(128)
@@ -195,20 +215,20 @@ moe_route_sort_small_kernel(const float* __restrict__ z, const float* __restrict
 
 // The same for the grouped rule (sigmoid scores, a correction, groups of experts).
 __global__ void __launch_bounds__(256)
-moe_route_grouped_sort_small_kernel(const float* __restrict__ z, const float* __restrict__ correction, int E, int top, int groups, int keep,
-                                    int T, int* __restrict__ idx, float* __restrict__ wgt, int* __restrict__ offsets,
+moe_route_grouped_sort_small_kernel(const float* __restrict__ z, int64_t z_ld, const float* __restrict__ correction, int E, int top,
+                                    GroupRule rule, int T, int* __restrict__ idx, float* __restrict__ wgt, int* __restrict__ offsets,
                                     int* __restrict__ sorted, int* __restrict__ place) {
   extern __shared__ float zs[];               // [8][2 E + groups] a warp's scores, then [T * top] chosen experts, then [E + 1] offsets
   pdl_wait();
   pdl_launch_dependents();
-  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, A = T * top, per = 2 * E + groups;
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, A = T * top, per = 2 * E + rule.groups;
   int* chosen = reinterpret_cast<int*>(zs + 8 * per);
   int* off = chosen + A;
   float* mine = zs + warp * per;
   for (int t = warp; t < T; t += 8) {
-    for (int e = lane; e < E; e += 32) mine[e] = z[(int64_t)t * E + e];
+    for (int e = lane; e < E; e += 32) mine[e] = z[(int64_t)t * z_ld + e];
     __syncwarp();
-    route_token_grouped(mine, mine + E, mine + 2 * E, correction, E, top, groups, keep, lane, idx + (int64_t)t * top, wgt + (int64_t)t * top);
+    route_token_grouped(mine, mine + E, mine + 2 * E, correction, E, top, rule, lane, idx + (int64_t)t * top, wgt + (int64_t)t * top);
     __syncwarp();
     for (int k = lane; k < top; k += 32) chosen[t * top + k] = idx[(int64_t)t * top + k];
     __syncwarp();
@@ -341,15 +361,17 @@ moe_gemm_kernel(const TA* __restrict__ a, int64_t a_stride, const int* __restric
 template <typename TS, typename TO>
 __global__ void __launch_bounds__(256)
 moe_combine_kernel(const float* __restrict__ rows, int64_t rows_stride, const int* __restrict__ place, const float* __restrict__ wgt,
-                   int top, const TS* __restrict__ shared, int64_t shared_stride, TO* __restrict__ out, int64_t out_stride, int W) {
+                   int top, const TS* __restrict__ shared, int64_t shared_stride, const float* __restrict__ shared_gate, int64_t gate_stride,
+                   TO* __restrict__ out, int64_t out_stride, int W) {
   pdl_wait();
   pdl_launch_dependents();
   const int t = blockIdx.x;
+  const float share = shared_gate ? 1.f / (1.f + expf(-shared_gate[(int64_t)t * gate_stride])) : 1.f;
   for (int i = blockIdx.y * blockDim.x + threadIdx.x; i < W; i += gridDim.y * blockDim.x) {
     float acc = 0.f;
     for (int k = 0; k < top; ++k)
       acc = fmaf(wgt[(int64_t)t * top + k], rows[(int64_t)place[(int64_t)t * top + k] * rows_stride + i], acc);
-    if (shared) acc += to_f<TS>(shared[(int64_t)t * shared_stride + i]);
+    if (shared) acc = fmaf(share, to_f<TS>(shared[(int64_t)t * shared_stride + i]), acc);
     out[(int64_t)t * out_stride + i] = from_f<TO>(acc);
   }
 }
@@ -413,21 +435,22 @@ ME_API int me_moe_route_sort(const float* z, const float* bias, int T, int E, in
   return rc ? rc : me_moe_sort(idx, T, top, E, counts, offsets, sorted, place, stream);
 }
 
-ME_API int me_moe_route_grouped(const float* z, const float* correction, int T, int E, int top, int groups, int keep, int* idx,
-                                float* wgt, cudaStream_t stream) {
+// z: [T, E] float32, rows z_ld elements apart.
+ME_API int me_moe_route_grouped(const float* z, int64_t z_ld, const float* correction, int T, int E, int top, int groups, int keep, int softmax,
+                                float weight_scale, int* idx, float* wgt, cudaStream_t stream) {
   if (T == 0) return 0;
   ME_REQUIRE(E >= 1 && top >= 1 && top <= E && E <= 2048, "me_moe_route_grouped: %d experts, %d chosen", E, top);
   ME_REQUIRE(groups >= 1 && E % groups == 0 && keep >= 1 && keep <= groups && keep * (E / groups) >= top,
              "me_moe_route_grouped: %d of %d groups of %d experts cannot give %d choices", keep, groups, E / (groups > 0 ? groups : 1), top);
-  me_launch(moe_route_grouped_kernel, dim3((T + 3) / 4), dim3(128), sizeof(float) * 4 * (2 * E + groups), stream, z, correction, E, top,
-            groups, keep, idx, wgt, T);
+  me_launch(moe_route_grouped_kernel, dim3((T + 3) / 4), dim3(128), sizeof(float) * 4 * (2 * E + groups), stream, z, z_ld, correction, E, top,
+            GroupRule{groups, keep, softmax, weight_scale}, idx, wgt, T);
   ME_LAUNCH_CHECK("me_moe_route_grouped");
   return 0;
 }
 
 // Grouped routing and grouping together: one kernel for a step of few tokens, else routing and the sort's two kernels.
-ME_API int me_moe_route_grouped_sort(const float* z, const float* correction, int T, int E, int top, int groups, int keep, int* idx,
-                                     float* wgt, int* counts, int* offsets, int* sorted, int* place, cudaStream_t stream) {
+ME_API int me_moe_route_grouped_sort(const float* z, int64_t z_ld, const float* correction, int T, int E, int top, int groups, int keep,
+                                     int softmax, float weight_scale, int* idx, float* wgt, int* counts, int* offsets, int* sorted, int* place, cudaStream_t stream) {
   if (T == 0) return 0;
   const size_t small = sizeof(float) * 8 * (2 * (size_t)E + groups) + sizeof(int) * ((size_t)T * top + E + 1);
   // (a warp routes a token at a time, and this rule takes longer a token than a plain top-k: beyond four tokens a warp the
@@ -435,12 +458,12 @@ ME_API int me_moe_route_grouped_sort(const float* z, const float* correction, in
   if (T <= 32 && (int64_t)T * top <= 1024 && E <= 256 && small <= 40 * 1024) {
     ME_REQUIRE(E >= 1 && top >= 1 && top <= E && groups >= 1 && E % groups == 0 && keep >= 1 && keep <= groups && keep * (E / groups) >= top,
                "me_moe_route_grouped_sort: %d of %d groups over %d experts cannot give %d choices", keep, groups, E, top);
-    me_launch(moe_route_grouped_sort_small_kernel, dim3(1), dim3(256), small, stream, z, correction, E, top, groups, keep, T, idx, wgt,
-              offsets, sorted, place);
+    me_launch(moe_route_grouped_sort_small_kernel, dim3(1), dim3(256), small, stream, z, z_ld, correction, E, top,
+              GroupRule{groups, keep, softmax, weight_scale}, T, idx, wgt, offsets, sorted, place);
     ME_LAUNCH_CHECK("me_moe_route_grouped_sort");
     return 0;
   }
-  int rc = me_moe_route_grouped(z, correction, T, E, top, groups, keep, idx, wgt, stream);
+  int rc = me_moe_route_grouped(z, z_ld, correction, T, E, top, groups, keep, softmax, weight_scale, idx, wgt, stream);
   return rc ? rc : me_moe_sort(idx, T, top, E, counts, offsets, sorted, place, stream);
 }
 
@@ -473,13 +496,13 @@ ME_API int me_moe_gemm(const void* a, int a_dtype, int64_t a_stride, const int* 
 }
 
 ME_API int me_moe_combine(const float* rows, int64_t rows_stride, const int* place, const float* wgt, int top, const void* shared,
-                          int shared_dtype, int64_t shared_stride, void* out, int out_dtype, int64_t out_stride, int T, int W,
-                          cudaStream_t stream) {
+                          int shared_dtype, int64_t shared_stride, const float* shared_gate, int64_t gate_stride, void* out, int out_dtype,
+                          int64_t out_stride, int T, int W, cudaStream_t stream) {
   if (T == 0) return 0;
   dim3 grid(T, (W + 1023) / 1024);
   ME_DISPATCH_DTYPE(shared ? shared_dtype : ME_F32, TS, ME_DISPATCH_DTYPE(out_dtype, TO,
       me_launch(moe_combine_kernel<TS, TO>, grid, dim3(256), 0, stream, rows, rows_stride, place, wgt, top, (const TS*)shared,
-                shared_stride, (TO*)out, out_stride, W)));
+                shared_stride, shared_gate, gate_stride, (TO*)out, out_stride, W)));
   ME_LAUNCH_CHECK("me_moe_combine");
   return 0;
 }

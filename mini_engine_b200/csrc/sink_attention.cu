@@ -1,6 +1,6 @@
 // Paged attention with an optional mask (a sliding window that may also keep the sequence's first tokens, or chunks), an
 // optional sink in the softmax's denominator (of score 0, or a learned score per head), optionally capped scores, key and
-// value sizes of their own and an optional sigmoid gate on the output, on the CUDA cores: any sizes up to 256, float32 or
+// value sizes of their own and an optional sigmoid gate on the output (a number an element, or one a head), on the CUDA cores: any sizes up to 256, float32 or
 // bfloat16 storage, float32 arithmetic.  It serves portions of prompts (query tiles from the step's tile list) and
 // single tokens (one block per request and head) alike.
 //
@@ -36,7 +36,7 @@ sink_attn_kernel(const T* __restrict__ q, int64_t q_stride, const float* __restr
                  const int* __restrict__ tiles, int nh, int nkv, int D, int Dv, int HD, int page_size, float scale, int window,
                  int sink, const float* __restrict__ sinks, float softcap, int keep_first, int chunk,
                  const T* __restrict__ pooled, const int* __restrict__ pooled_tables, int pbt_stride, int pool_p,
-                 const float* __restrict__ r1, const float* __restrict__ r2) {
+                 const float* __restrict__ r1, const float* __restrict__ r2, int gate_heads) {
   extern __shared__ float smem[];
   pdl_wait();
   pdl_launch_dependents();
@@ -153,13 +153,13 @@ sink_attn_kernel(const T* __restrict__ q, int64_t q_stride, const float* __restr
     const float inv = l > 0.f ? 1.0f / l : 0.f;
     const int64_t t = tok0 + q0 + r;
     T* o = out + t * out_stride + (int64_t)head * Dv;
-    const float* g = gate ? gate + t * gate_stride + (int64_t)head * Dv : nullptr;
+    const float* g = gate ? gate + t * gate_stride + (gate_heads ? head : (int64_t)head * Dv) : nullptr;
 #pragma unroll
     for (int k = 0; k < SA_MAX / 8; ++k) {
       const int d = c + 8 * k;
       if (d < Dv) {
         float v = acc[k] * inv;
-        if (g) v = v / (1.f + expf(-g[d]));
+        if (g) v = v / (1.f + expf(-g[gate_heads ? 0 : d]));
         o[d] = from_f<T>(v);
       }
     }
@@ -168,7 +168,7 @@ sink_attn_kernel(const T* __restrict__ q, int64_t q_stride, const float* __restr
 
 ME_API int me_sink_attn_tile_q() { return SA_BQ; }
 
-// q: [T, nh*D]; gate: float32 [T, >= nh*Dv] pre-activations or null; out: [T, nh*Dv]; pool: [pages][2][nkv][page_size][HD].
+// q: [T, nh*D]; gate: float32 [T, >= nh*Dv] pre-activations (>= nh with gate_heads: one a head) or null; out: [T, nh*Dv]; pool: [pages][2][nkv][page_size][HD].
 // tiles: [num_tiles, 2] (request, first local query) for requests that bring several tokens; the first num_decodes
 // requests bring one token each and get one block per head.  sinks: [nh] float32 or null; softcap, keep_first, chunk: 0 = none.
 // pooled, pooled_tables: the cache of pooled blocks (same layout and dtype) and its block tables, with pool_p tokens a block; null and 0: none.
@@ -178,7 +178,7 @@ ME_API int me_sink_attn(const void* q, int dtype, int64_t q_stride, const float*
                         const int* context_lens, const int* tiles, int num_tiles, int num_decodes, int nh, int nkv, int D, int Dv,
                         int HD, int page_size, float scale, int window, int sink, const float* sinks, float softcap,
                         int keep_first, int chunk, const void* pooled, const int* pooled_tables, int pbt_stride, int pool_p,
-                        const float* r1, const float* r2, cudaStream_t stream) {
+                        const float* r1, const float* r2, int gate_heads, cudaStream_t stream) {
   ME_REQUIRE(D >= 1 && D <= SA_MAX && Dv >= 1 && Dv <= SA_MAX, "me_sink_attn: key size %d / value size %d beyond %d", D, Dv, SA_MAX);
   ME_REQUIRE(HD >= D && HD >= Dv, "me_sink_attn: cache rows of %d elements are too short", HD);
   ME_REQUIRE(nh > 0 && nkv > 0 && nh % nkv == 0 && nh <= 65535, "me_sink_attn: %d heads, %d kv heads", nh, nkv);
@@ -196,11 +196,11 @@ ME_API int me_sink_attn(const void* q, int dtype, int64_t q_stride, const float*
     if (num_decodes > 0)
       me_launch(sink_attn_kernel<T>, dim3(num_decodes, nh), dim3(SA_THREADS), smem, stream, (const T*)q, q_stride, gate, gate_stride,
                 (T*)out, out_stride, (const T*)pool, block_tables, bt_stride, cu_seqlens, context_lens, (const int*)nullptr, nh, nkv,
-                D, Dv, HD, page_size, scale, window, sink, sinks, softcap, keep_first, chunk, (const T*)pooled, pooled_tables, pbt_stride, pool_p, r1, r2);
+                D, Dv, HD, page_size, scale, window, sink, sinks, softcap, keep_first, chunk, (const T*)pooled, pooled_tables, pbt_stride, pool_p, r1, r2, gate_heads);
     if (num_tiles > 0)
       me_launch(sink_attn_kernel<T>, dim3(num_tiles, nh), dim3(SA_THREADS), smem, stream, (const T*)q, q_stride, gate, gate_stride,
                 (T*)out, out_stride, (const T*)pool, block_tables, bt_stride, cu_seqlens, context_lens, tiles, nh, nkv, D, Dv,
-                HD, page_size, scale, window, sink, sinks, softcap, keep_first, chunk, (const T*)pooled, pooled_tables, pbt_stride, pool_p, r1, r2);
+                HD, page_size, scale, window, sink, sinks, softcap, keep_first, chunk, (const T*)pooled, pooled_tables, pbt_stride, pool_p, r1, r2, gate_heads);
   });
   ME_LAUNCH_CHECK("me_sink_attn");
   return 0;

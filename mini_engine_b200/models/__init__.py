@@ -1,2 +1,2 @@
 """Built-in architectures; importing this package registers them."""
-from . import galupel, gevulorn, logozen, pugadra, qwen3, tidenex  # noqa: F401
+from . import galupel, gevulorn, kuterax, logozen, pugadra, qwen3, tidenex  # noqa: F401

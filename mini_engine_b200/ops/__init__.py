@@ -22,7 +22,7 @@ MAX_HEAD_DIM = 256
 
 _P, _I, _L, _F = ctypes.c_void_p, ctypes.c_int, ctypes.c_int64, ctypes.c_float
 _PROTOS = {
-    "me_embed": [_P, _P, _I, _P, _I, _I, _I, _P, _P, _I, _F, _I, _L, _P],
+    "me_embed": [_P, _P, _I, _P, _I, _I, _I, _P, _P, _I, _F, _I, _L, _P, _P, _I, _P, _I, _L, _P],
     "me_hc_norm": [_P, _L, _I, _P, _I, _P, _P, _P, _P, _F, _P, _I, _P, _I, _I, _P, _P, _P, _P, _I, _P],
     "me_short_conv": [_P, _P, _P, _P, _P, _P, _P, _P, _I, _I, _I, _I, _I, _I, _I, _P],
     "me_polynorm": [_P, _I, _L, _P, _F, _P, _I, _L, _I, _I, _P],
@@ -39,7 +39,7 @@ _PROTOS = {
     "me_gemm_simt": [_P, _I, _L, _P, _I, _P, _I, _L, _I, _I, _I, _I, _P],
     "me_qk_norm_rope_kv_write": [_P, _I, _L, _I, _I, _I, _I, _P, _P, _F, _P, _I, _P, _P, _P, _I, _P],
     "me_attn_chunk": [_P, _I, _L, _P, _L, _P, _P, _I, _P, _P, _P, _I, _I, _I, _I, _I, _F, _I, _P],
-    "me_attn_decode": [_P, _I, _L, _P, _L, _P, _P, _I, _P, _P, _I, _I, _I, _I, _I, _F, _I, _P, _P, _P, _I, _P, _I, _P, _I, _P, _L, _I, _I, _F, _P, _P, _P, _I, _I, _I, _P, _P, _I, _I, _F, _F, _F, _P],
+    "me_attn_decode": [_P, _I, _L, _P, _L, _P, _P, _I, _P, _P, _I, _I, _I, _I, _I, _F, _I, _P, _P, _P, _I, _P, _I, _P, _I, _P, _L, _I, _I, _F, _P, _P, _P, _I, _I, _I, _P, _P, _I, _I, _F, _F, _F, _I, _P],
     "me_attn_decode_fused": [_P, _L, _P, _L, _P, _P, _P, _I, _P, _P, _I, _I, _I, _I, _I, _F, _I, _P, _P, _F, _P, _P, _P, _P, _P,
                              _I, _I, _I, _P, _P],
     "me_gemm_decode": [_I, _P, _L, _P, _I, _F, _P, _P, _I, _L, _P, _P, _P, _P, _I, _I, _I, _P, ctypes.c_uint64, _F, _F, _F, _P],
@@ -47,7 +47,7 @@ _PROTOS = {
     "me_gemm_tcgen05": [_P, _P, _P, _I, _L, _I, _I, _I, _I, _I, _I, _L, _F, _F, _F, _P, _P],
     "me_gemm_tcgen05_persistent": [_P, _P, _P, _I, _L, _I, _I, _I, _I, _I, _F, _F, _F, _P, _P],
     "me_gemm_tcgen05_shared": [_P, _P, _P, _I, _L, _I, _I, _I, _I, _I, _P, _P, _P, _P],
-    "me_attn_prefill_tcgen05": [_P, _P, _P, _L, _P, _I, _P, _P, _P, _I, _I, _I, _I, _I, _F, _I, _I, _I, _P, _L, _P, _I, _I, _F, _P, _P, _P, _I, _I, _P, _P, _I, _I, _F, _F, _F, _P],
+    "me_attn_prefill_tcgen05": [_P, _P, _P, _L, _P, _I, _P, _P, _P, _I, _I, _I, _I, _I, _F, _I, _I, _I, _P, _L, _P, _I, _I, _F, _P, _P, _P, _I, _I, _P, _P, _I, _I, _F, _F, _F, _I, _P],
     "me_tma_encode_2d": [_P, _P, ctypes.c_uint64, ctypes.c_uint64, ctypes.c_uint64, ctypes.c_uint32, ctypes.c_uint32, _I],
     "me_attn_prefill": [_P, _L, _P, _L, _P, _P, _I, _P, _P, _P, _I, _I, _I, _I, _I, _F, _I, _P],
     "me_sample": [_P, _L, _P, _P, _P, _P, _I, _I, _P, _P, _P],
@@ -56,18 +56,22 @@ _PROTOS = {
     "me_clamped_glu": [_P, _I, _L, _P, _I, _L, _I, _I, _F, _F, _F, _P],
     "me_conv_rope_kv": [_P, _L, _P, _P, _P, _I, _P, _I, _P, _P, _P, _P, _P, _P, _P, _P, _I, _I, _I, _I, _I, _I, _I, _I, _I, _I, _I, _P, _P],
     "me_rope_table": [_P, _P, _I, _I, _P, _P],
-    "me_sink_attn": [_P, _I, _L, _P, _L, _P, _L, _P, _P, _I, _P, _P, _P, _I, _I, _I, _I, _I, _I, _I, _I, _F, _I, _I, _P, _F, _I, _I, _P, _P, _I, _I, _P, _P, _P],
+    "me_sink_attn": [_P, _I, _L, _P, _L, _P, _L, _P, _P, _I, _P, _P, _P, _I, _I, _I, _I, _I, _I, _I, _I, _F, _I, _I, _P, _F, _I, _I, _P, _P, _I, _I, _P, _P, _I, _P],
     "me_parallel_norm": [_P, _P, _P, _I, _P, _P, _P, _P, _P, _P, _P, _P, _I, _P, _I, _I, _F, _P, _P, _I, _I, _P, _I, _F, _P],
-    "me_attn_prep": [_P, _L, _P, _P, _P, _I, _F, _P, _I, _P, _P, _P, _I, _P, _I, _I, _I, _I, _I, _I, _I, _I, _I, _P, _I, _F, _F, _F, _P],
+    "me_attn_prep": [_P, _L, _P, _P, _P, _I, _F, _P, _I, _P, _P, _P, _I, _P, _I, _I, _I, _I, _I, _I, _I, _I, _I, _P, _I, _F, _F, _F, _F, _P],
     "me_diff_combine": [_P, _I, _L, _P, _I, _L, _I, _I, _I, _I, _F, _F, _F, _P],
     "me_gla_decay": [_P, _L, _I, _I, _P, _I, _P, _F, _P, _I, _I, _P],
     "me_gla_scan": [_P, _L, _I, _I, _I, _P, _P, _P, _P, _P, _P, _I, _I, _I, _I, _F, _P, _I, _I, _P, _P, _P, _P, _P],
+    "me_stream_norm": [_P, _P, _P, _P, _I, _P, _P, _P, _F, _F, _F, _P, _P, _P, _F, _P, _I, _L, _P, _I, _I, _P],
+    "me_conv_silu": [_P, _L, _P, _P, _P, _P, _I, _I, _P, _P, _P, _P, _I, _I, _I, _I, _P],
+    "me_head_decay_scan": [_P, _P, _P, _I, _L, _L, _L, _I, _I, _I, _I, _F, _P, _L, _P, _P, _P, _P, _P, _P, _P, _P, _P, _I, _I, _P, _I, _P, _P, _P],
+    "me_gated_group_norm": [_P, _L, _P, _I, _L, _P, _I, _F, _P, _I, _L, _I, _I, _I, _P],
     "me_activation": [_P, _I, _L, _P, _I, _L, _I, _I, _I, _P],
     "me_soft_cap": [_P, _L, _F, _F, _P],
     "me_add_row_vector": [_P, _I, _I, _I, _P, _P],
     "me_moe_route": [_P, _P, _I, _I, _I, _P, _P, _P],
-    "me_moe_route_grouped": [_P, _P, _I, _I, _I, _I, _I, _P, _P, _P],
-    "me_moe_route_grouped_sort": [_P, _P, _I, _I, _I, _I, _I, _P, _P, _P, _P, _P, _P, _P],
+    "me_moe_route_grouped": [_P, _L, _P, _I, _I, _I, _I, _I, _I, _F, _P, _P, _P],
+    "me_moe_route_grouped_sort": [_P, _L, _P, _I, _I, _I, _I, _I, _I, _F, _P, _P, _P, _P, _P, _P, _P],
     "me_group_norm": [_P, _P, _I, _L, _P, _I, _F, _P, _I, _P, _I, _I, _P],
     "me_pool_kv": [_P, _P, _I, _P, _P, _I, _P, _P, _P, _P, _I, _I, _I, _I, _I, _I, _I, _I, _I, _I, _P],
     "me_moe_sort": [_P, _I, _I, _I, _P, _P, _P, _P, _P],
@@ -75,7 +79,7 @@ _PROTOS = {
     "me_moe_gemm": [_P, _I, _L, _P, _I, _P, _I, _L, _P, _I, _P, _I, _L, _I, _I, _I, _I, _F, _F, _F, _I, _P],
     "me_moe_gather": [_P, _I, _L, _P, _I, _P, _I, _I, _P],
     "me_gemm_tcgen05_grouped": [_P, _P, _P, _I, _L, _P, _I, _I, _I, _I, _I, _I, _F, _F, _F, _I, _P, _P],
-    "me_moe_combine": [_P, _L, _P, _P, _I, _P, _I, _L, _P, _I, _L, _I, _I, _P],
+    "me_moe_combine": [_P, _L, _P, _P, _I, _P, _I, _L, _P, _L, _P, _I, _L, _I, _I, _P],
     "me_token_side_gate": [_P, _I, _L, _P, _P, _P, _I, _L, _I, _I, _I, _P, _I, _I, _P],
 }
 _DT = {torch.float32: 0, torch.bfloat16: 1}
@@ -268,8 +272,11 @@ def check_attention_sizes(head_dim: int, num_heads: int, num_kv_heads: int) -> N
 
 # ---- element-wise and normalisation ----------------------------------------------------
 def embed(ids: torch.Tensor, table: torch.Tensor, out: torch.Tensor, err: torch.Tensor,
-          feedback: Optional[torch.Tensor] = None, scale: float = 1.0) -> None:
+          feedback: Optional[torch.Tensor] = None, scale: float = 1.0, position_rows: Optional[tuple] = None,
+          copy: Optional[torch.Tensor] = None) -> None:
     """Rows of ``table`` times ``scale`` into the float32 ``out`` [T, H], or into every stream of ``out`` [S, T, H].
+    ``position_rows`` = (table [P, H] of the same dtype, int32 positions [T]): the row of a token's position is added.  ``copy`` [T, H]
+    (any dtype, rows may lie apart) takes the same rows once more.
     An id ~j (negative) stands for ``feedback[j]`` (int32 on the device: the tokens the step before drew); ids
     outside the vocabulary set flag 0 of ``err``."""
     _need(ids.dtype == torch.int32 and ids.is_contiguous(), "embed: token ids must be contiguous int32")
@@ -278,8 +285,15 @@ def embed(ids: torch.Tensor, table: torch.Tensor, out: torch.Tensor, err: torch.
     T, (V, H) = ids.shape[0], table.shape
     copies = out.shape[0] if out.dim() == 3 else 1
     _need(tuple(out.shape[-2:]) == (T, H) and out.dim() in (2, 3), "embed: output shape")
+    ptable, positions = position_rows if position_rows is not None else (None, None)
+    _need(ptable is None or (ptable.is_contiguous() and ptable.dtype == table.dtype and ptable.dim() == 2 and ptable.shape[1] == H
+                             and positions.dtype == torch.int32 and positions.is_contiguous() and positions.numel() == T),
+          "embed: the table over positions is [positions, H] of the table's dtype, with an int32 position a token")
+    _need(copy is None or (tuple(copy.shape) == (T, H) and copy.stride(1) == 1), "embed: the copy is [T, H]")
     _call("me_embed", ids.data_ptr(), table.data_ptr(), _dt(table), out.data_ptr(), T, H, V, err.data_ptr(), _ptr(feedback),
-          feedback.numel() if feedback is not None else 0, float(scale), copies, T * H, _stream())
+          feedback.numel() if feedback is not None else 0, float(scale), copies, T * H, _ptr(ptable), _ptr(positions),
+          ptable.shape[0] if ptable is not None else 0, _ptr(copy), _dt(copy) if copy is not None else 0,
+          copy.stride(0) if copy is not None else H, _stream())
 
 
 def add_rmsnorm(residual: torch.Tensor, delta: Optional[torch.Tensor], weight: torch.Tensor, eps: float,
@@ -865,7 +879,7 @@ def attention_prefill_tcgen05(qkv, out, num_heads, num_kv_heads, head_dim, pool,
                               scale, window, tiles=None, num_tiles=None, key_tile: int = 0, sink: bool = False,
                               gate: Optional[torch.Tensor] = None, keep_first: int = 0, chunk: int = 0, softcap: float = 0.0,
                               sinks: Optional[torch.Tensor] = None, pooled: Optional[tuple] = None, bias: Optional[tuple] = None,
-                              out_dim: int = 0, pairs: Optional[tuple[float, float, float]] = None) -> None:
+                              out_dim: int = 0, pairs: Optional[tuple[float, float, float]] = None, gate_heads: bool = False) -> None:
     """The tcgen05 / tensor-memory prefill kernel (bfloat16, head_dim 64 or 128, page sizes dividing 128) over
     tiles of 128 / heads-per-block tokens; Q, K and V arrive by tensor-map loads.  ``sink``: one more term, exp(0), in
     the softmax's denominator; ``gate``: float32 rows of pre-activations whose sigmoid multiplies the output.
@@ -874,7 +888,8 @@ def attention_prefill_tcgen05(qkv, out, num_heads, num_kv_heads, head_dim, pool,
     exp(sinks[head]); ``pooled`` = (cache, block tables, P): the blocks of P tokens in front of the window, one row each in a
     second cache of the same layout; ``bias`` = (r1, r2), float32 [heads] each: r1 ln(1 + r2 (p - j)) is taken off the scaled score
     of a key at distance p - j; ``out_dim`` (0: all): how many elements of every head leave, ``out`` then holds
-    heads * out_dim columns; ``pairs`` = (lambda, gain, eps): heads 2h and 2h + 1 leave joined as ``diff_combine`` joins them (all of these in the kernel with the key tile of 128 only)."""
+    heads * out_dim columns; ``pairs`` = (lambda, gain, eps): heads 2h and 2h + 1 leave joined as ``diff_combine`` joins them;
+    ``gate_heads``: the gate has one pre-activation a head (all of these in the kernel with the key tile of 128 only)."""
     gp = prefill_tcgen05_heads_per_block(num_heads, num_kv_heads, head_dim, page_size)
     _need(gp > 0 and qkv.dtype == torch.bfloat16 and qkv.is_contiguous() and qkv.data_ptr() % 16 == 0,
           "attention_prefill_tcgen05: shape or dtype not taken by the kernel")
@@ -888,7 +903,7 @@ def attention_prefill_tcgen05(qkv, out, num_heads, num_kv_heads, head_dim, pool,
           meta.error_flag.data_ptr(), int(keep_first or 0), int(chunk or 0), float(softcap or 0.0), _ptr(sinks),
           kv_tensor_map(pooled[0], page_size).ptr if pooled else 0, pooled[1].data_ptr() if pooled else 0,
           pooled[1].stride(0) if pooled else 0, int(pooled[2]) if pooled else 0, _ptr(bias[0]) if bias else 0, _ptr(bias[1]) if bias else 0,
-          int(out_dim), 1 if pairs else 0, *(float(v) for v in (pairs or (0.0, 0.0, 0.0))), _stream())
+          int(out_dim), 1 if pairs else 0, *(float(v) for v in (pairs or (0.0, 0.0, 0.0))), 1 if gate_heads else 0, _stream())
 
 
 use_tcgen05_attention = True   # False: portions of prompts use the mma.sync kernel instead (a switch for comparisons)
@@ -898,12 +913,13 @@ def attention_decode(qkv, out, num_heads, num_kv_heads, head_dim, pool, page_siz
                      scale, window, kind: str = "auto", sink: bool = False, gate: Optional[torch.Tensor] = None,
                      keep_first: int = 0, chunk: int = 0, softcap: float = 0.0, sinks: Optional[torch.Tensor] = None,
                      pooled: Optional[tuple] = None, bias: Optional[tuple] = None, out_dim: int = 0,
-                     pairs: Optional[tuple[float, float, float]] = None) -> None:
+                     pairs: Optional[tuple[float, float, float]] = None, gate_heads: bool = False) -> None:
     """The split-K decode kernel and its merge over requests [0, meta.num_decodes).  ``sink``: one more term, exp(0), in
     the softmax's denominator (added once, in the merge); ``gate``: float32 rows of pre-activations whose sigmoid
     multiplies the output.  ``sinks`` (float32 [heads]): the term is exp(sinks[head]).  ``keep_first``, ``chunk`` and
     ``softcap``, ``bias`` and ``out_dim`` as for ``attention_prefill_tcgen05`` (the partition kernel fed by tensor-map loads only).
     ``pairs`` = (lambda, gain, eps): the merge joins heads 2h and 2h + 1 as ``diff_combine`` does and ``out`` holds half as many heads.
+    ``gate_heads``: the gate has one pre-activation a head.
 
     ``kind`` picks the partition kernel: "auto" (for bfloat16 with head_dim 64 or 128 the tensor cores, fed by
     tensor-map loads where the page size divides 128, else by cp.async; otherwise the CUDA cores), or one
@@ -928,7 +944,8 @@ def attention_decode(qkv, out, num_heads, num_kv_heads, head_dim, pool, page_siz
           gate.stride(0) if gate is not None else 0, int(keep_first or 0), int(chunk or 0), float(softcap or 0.0), _ptr(sinks),
           kv_tensor_map(pooled[0], page_size).ptr if pooled else 0, pooled[1].data_ptr() if pooled else 0,
           pooled[1].stride(0) if pooled else 0, int(pooled[2]) if pooled else 0, pool_parts, _ptr(bias[0]) if bias else 0,
-          _ptr(bias[1]) if bias else 0, int(out_dim), 1 if pairs else 0, *(float(v) for v in (pairs or (0.0, 0.0, 0.0))), _stream())
+          _ptr(bias[1]) if bias else 0, int(out_dim), 1 if pairs else 0, *(float(v) for v in (pairs or (0.0, 0.0, 0.0))), 1 if gate_heads else 0,
+          _stream())
     global launches
     launches += 2 if pooled else 1          # partition kernel(s) + merge kernel
 
@@ -1411,6 +1428,115 @@ def parallel_norm(residual: torch.Tensor, adds: Sequence[torch.Tensor], vectors:
           feedback.numel() if feedback is not None else 0, float(scale), _stream())
 
 
+# ---- the stream with everything pending, and its RMS norm -----------------------------------------------
+def stream_norm(residual: torch.Tensor, terms: Sequence[tuple], vectors: Sequence[torch.Tensor], weight: Optional[torch.Tensor], eps: float,
+                out: torch.Tensor, rows: Optional[torch.Tensor] = None) -> None:
+    """``residual += sum of terms + sum of vectors`` (float32, in place), then ``out = residual / rms(residual) * weight``, or without a weight
+    a copy of the stream (``out`` may be columns of wider rows).  A term is (y [T, W], scale, eps_y): scale * y with a float32 [W]
+    scale or None, or, with eps_y not None, scale * y / sqrt(mean(y^2) + eps_y).  Up to three terms of one dtype and two float32 [W]
+    vectors.  With ``rows`` only those rows are computed and ``residual`` is not written."""
+    T, W = residual.shape
+    terms, vectors = list(terms), list(vectors)
+    _need(residual.dtype == torch.float32 and residual.is_contiguous(), "stream_norm: the residual must be float32 [T, W]")
+    _need(len(terms) <= 3 and len(vectors) <= 2, "stream_norm: at most three outputs and two vectors can be added")
+    _need(all(tuple(y.shape) == (T, W) and y.is_contiguous() and y.dtype == terms[0][0].dtype for y, _, _ in terms), "stream_norm: outputs must be [T, W]")
+    floats = [s for _, s, _ in terms if s is not None] + vectors + ([weight] if weight is not None else [])
+    _need(all(v.dtype == torch.float32 and v.numel() == W and v.is_contiguous() for v in floats), "stream_norm: scales, vectors and the weight are float32 [W]")
+    n = T if rows is None else rows.shape[0]
+    _need(tuple(out.shape) == (n, W) and out.stride(1) == 1, "stream_norm: output shape")
+    _need(rows is None or (rows.dtype == torch.int32 and rows.is_contiguous()), "stream_norm: rows must be int32")
+    terms += [(None, None, None)] * (3 - len(terms))
+    vectors += [None] * (2 - len(vectors))
+    _call("me_stream_norm", residual.data_ptr(), *(_ptr(y) for y, _, _ in terms), _dt(terms[0][0]) if terms[0][0] is not None else 0,
+          *(_ptr(s) for _, s, _ in terms), *(-1.0 if e is None else float(e) for _, _, e in terms), _ptr(vectors[0]), _ptr(vectors[1]), _ptr(weight),
+          float(eps), out.data_ptr(), _dt(out), out.stride(0), _ptr(rows), n, W, _stream())
+
+
+# ---- recurrences whose state decays by one number a head ----------------------------------------------------
+CONV_TILE = 16            # tokens per block of the convolution (csrc/short_conv.cu)
+
+
+def conv_silu(u: torch.Tensor, weight: torch.Tensor, bias: Optional[torch.Tensor], state: Optional[torch.Tensor], meta, state_slots: torch.Tensor,
+              out: torch.Tensor) -> None:
+    """``out_t = silu(bias + sum_j weight[:, j] u_(t - taps + 1 + j))`` per channel over each request's tokens, zeros before its first
+    token; inputs from before this step come from ``state`` [slots, taps - 1, C], which then takes the step's last inputs.  ``u`` float32
+    [T, C], possibly columns of wider rows; ``weight`` [C, taps], ``bias`` [C] and ``state`` float32; ``out`` [T, C] of any dtype."""
+    T, C = u.shape
+    taps = weight.shape[1]
+    _need(u.dtype == torch.float32 and u.stride(1) == 1 and weight.dtype == torch.float32 and weight.is_contiguous() and weight.shape[0] == C,
+          "conv_silu: u [T, C] and weight [C, taps] must be float32")
+    _need(bias is None or (bias.dtype == torch.float32 and bias.numel() == C and bias.is_contiguous()), "conv_silu: bias must be float32 [C]")
+    _need(taps == 1 or (state is not None and state.dtype == torch.float32 and state.is_contiguous() and tuple(state.shape[1:]) == (taps - 1, C)),
+          "conv_silu: state must be float32 [slots, taps - 1, C]")
+    _need(out.is_contiguous() and tuple(out.shape) == (T, C), "conv_silu: output shape")
+    tiles, n_tiles = meta.tile_lists[CONV_TILE]
+    _call("me_conv_silu", u.data_ptr(), u.stride(0), weight.data_ptr(), _ptr(bias), _ptr(state) if taps > 1 else 0, tiles.data_ptr(), n_tiles,
+          meta.num_decodes, meta.cu_seqlens.data_ptr(), meta.context_lens.data_ptr(), state_slots.data_ptr(), out.data_ptr(), _dt(out),
+          meta.num_reqs, C, taps, _stream())
+    global launches
+    launches += 1 if taps > 1 and meta.num_decodes < meta.num_reqs else 0
+
+
+HEAD_DECAY_CHUNK = 64     # tokens per run of the recurrence's prompt kernels (csrc/head_decay.cu)
+head_decay_chunks = True  # portions of prompts by runs of tokens (False: token by token, always); a switch for comparisons
+
+
+def head_decay_chunk_count(meta) -> int:
+    """An upper bound of the runs of HEAD_DECAY_CHUNK tokens that the step's requests with several tokens are cut into (it depends
+    on the step's shape only, so that a recorded step keeps its workspace)."""
+    multi = meta.num_reqs - meta.num_decodes
+    return 0 if multi <= 0 else (meta.num_tokens - meta.num_decodes) // HEAD_DECAY_CHUNK + multi
+
+
+def head_decay_scan(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, S: torch.Tensor, meta, state_slots: torch.Tensor, o: torch.Tensor,
+                    num_heads: int, num_groups: int, dim: int, vdim: int, *, k_scale: float = 1.0, dt: Optional[tuple] = None,
+                    log2_decay: Optional[torch.Tensor] = None, skip: Optional[torch.Tensor] = None, chunk_states: Optional[torch.Tensor] = None,
+                    totals: Optional[torch.Tensor] = None) -> None:
+    """Walks every request's tokens of this step through S_t = a_t S_(t-1) + g_t k_t v_t^T, o_t = S_t^T q_t + skip v_t from the state in
+    its slot, per head, with one decay a and one factor g a head and token (see csrc/head_decay.cu).  ``q``, ``k`` [T, groups * dim]
+    and ``v`` [T, heads * vdim]: columns of rows of one dtype; head h reads group h // (heads / groups) of q and k.
+
+    ``dt`` = (pre-activations [T, heads] float32 (columns of wider rows), bias [heads], a_log [heads]): g = softplus(dt + bias), a =
+    exp(-exp(a_log) g).  Or ``log2_decay`` float32 [heads]: a = 2^log2_decay, g = ``k_scale``.  With the float32 workspaces ``chunk_states``
+    (heads * dim * vdim values a run of HEAD_DECAY_CHUNK tokens: ``head_decay_chunk_count``) and ``totals`` (heads values a run) the
+    requests that bring several tokens take a run at a time, all runs of the step side by side."""
+    T = o.shape[0]
+    _need(num_heads % num_groups == 0, "head_decay_scan: heads must be a multiple of the groups")
+    _need(q.dtype == k.dtype == v.dtype and all(t.stride(1) == 1 for t in (q, k, v)), "head_decay_scan: q, k and v are rows of one dtype")
+    _need(tuple(q.shape) == tuple(k.shape) == (T, num_groups * dim) and tuple(v.shape) == (T, num_heads * vdim), "head_decay_scan: shapes of q, k, v")
+    _need(S.dtype == torch.float32 and S.is_contiguous() and tuple(S.shape[1:]) == (num_heads, dim, vdim), "head_decay_scan: state shape")
+    _need(o.dtype == torch.float32 and o.is_contiguous() and tuple(o.shape) == (T, num_heads * vdim), "head_decay_scan: output shape")
+    _need((dt is None) != (log2_decay is None), "head_decay_scan: decays from dt or constants")
+    per_head = [t for t in ((*dt[1:],) if dt is not None else (log2_decay,)) + ((skip,) if skip is not None else ())]
+    _need(all(t.dtype == torch.float32 and t.is_contiguous() and t.numel() == num_heads for t in per_head), "head_decay_scan: float32 numbers a head")
+    _need(dt is None or (dt[0].dtype == torch.float32 and dt[0].stride(1) == 1 and tuple(dt[0].shape) == (T, num_heads)), "head_decay_scan: dt is float32 [T, heads]")
+    tiles, n_tiles = meta.tile_lists[HEAD_DECAY_CHUNK]
+    chunked = head_decay_chunks and chunk_states is not None and totals is not None and n_tiles > 0 and dim <= 256
+    if chunked:
+        _need(all(t.dtype == torch.float32 and t.is_contiguous() for t in (chunk_states, totals))
+              and chunk_states.numel() >= n_tiles * num_heads * dim * vdim and totals.numel() >= n_tiles * num_heads, "head_decay_scan: workspaces")
+    _call("me_head_decay_scan", q.data_ptr(), k.data_ptr(), v.data_ptr(), _dt(q), q.stride(0), k.stride(0), v.stride(0), num_heads, num_groups,
+          dim, vdim, float(k_scale), _ptr(dt[0]) if dt else 0, dt[0].stride(0) if dt else 0, _ptr(dt[1]) if dt else 0, _ptr(dt[2]) if dt else 0,
+          _ptr(log2_decay), _ptr(skip), S.data_ptr(), meta.cu_seqlens.data_ptr(), meta.context_lens.data_ptr(), state_slots.data_ptr(),
+          o.data_ptr(), meta.num_reqs, meta.num_decodes, tiles.data_ptr() if chunked else 0, n_tiles if chunked else 0,
+          chunk_states.data_ptr() if chunked else 0, totals.data_ptr() if chunked else 0, _stream())
+    global launches
+    launches += (2 + (1 if meta.num_decodes else 0)) if chunked else 0
+
+
+def gated_group_norm(y: torch.Tensor, z: torch.Tensor, weight: Optional[torch.Tensor], groups: int, eps: float, out: torch.Tensor,
+                     gate_first: bool) -> None:
+    """Rows of ``y`` (float32 [T, W]) normed in ``groups`` equal parts, each by its own root mean square, with the gate silu(``z``) in front of
+    the norm (``gate_first``) or behind it, and a float32 [W] weight or None.  All rows may be columns of wider ones."""
+    T, W = y.shape
+    _need(y.dtype == torch.float32 and y.stride(1) == 1 and tuple(z.shape) == tuple(out.shape) == (T, W) and z.stride(1) == out.stride(1) == 1,
+          "gated_group_norm: shapes")
+    _need(weight is None or (weight.dtype == torch.float32 and weight.is_contiguous() and weight.numel() == W), "gated_group_norm: weight must be float32 [W]")
+    _need(groups >= 1 and W % groups == 0, "gated_group_norm: groups must divide the row")
+    _call("me_gated_group_norm", y.data_ptr(), y.stride(0), z.data_ptr(), _dt(z), z.stride(0), _ptr(weight), 1 if gate_first else 0, float(eps),
+          out.data_ptr(), _dt(out), out.stride(0), T, W, groups, _stream())
+
+
 ACTIVATIONS = {"relu_squared": 0, "gelu_tanh": 1, "silu": 2, "gelu": 3}     # "gelu": the exact form, z Phi(z)
 
 
@@ -1440,14 +1566,14 @@ def attn_prep(proj: torch.Tensor, bias: Optional[torch.Tensor], q_norm: Optional
               slot_mapping: Optional[torch.Tensor], q_out: torch.Tensor, pool: Optional[torch.Tensor], page_size: int,
               num_heads: int, num_kv_heads: int, dim: int, vdim: int, q_scale: Optional[torch.Tensor] = None,
               own_kv: bool = True, maps: int = 1,
-              temperature: Optional[tuple[float, float]] = None, v_scale: float = 1.0) -> None:
+              temperature: Optional[tuple[float, float]] = None, v_scale: float = 1.0, magnitude: float = 1.0) -> None:
     """From the packed float32 projections q|k|v (the leading columns of ``proj``; q alone with ``own_kv`` False): bias, a weighted RMS norm of every q and k
     head in front of the rotation (``norm`` "before"), one over the whole q and the whole k of a token ("row", with a weight for every value)
     or a plain one behind it ("after"), the rotation of element i with
     element i + len(freq) by position x ``freq`` (float64 frequencies), queries to ``q_out`` and keys and values into the
     cache rows that ``slot_mapping`` names (see csrc/attn_prep.cu).  ``q_scale`` (float32 [heads]): every query head is
     multiplied by its number at the end.  ``temperature`` = (coef, every): q is multiplied by 1 + coef ln(floor((p + 1) / every) + 1).
-    ``v_scale`` multiplies the values.  ``maps`` 2: every q and k head has two maps of ``dim`` elements; ``q_out`` then has a row for
+    ``v_scale`` multiplies the values, ``magnitude`` the rotation's cosines and sines.  ``maps`` 2: every q and k head has two maps of ``dim`` elements; ``q_out`` then has a row for
     every map of every head.  ``q_out`` [T, rows * width]: rows wider than what they hold are filled with zeros (cache rows too)."""
     T = proj.shape[0]
     C = num_heads * maps * dim + (num_kv_heads * (maps * dim + vdim) if own_kv else 0)
@@ -1475,7 +1601,7 @@ def attn_prep(proj: torch.Tensor, bias: Optional[torch.Tensor], q_norm: Optional
     _call("me_attn_prep", proj.data_ptr(), proj.stride(0), _ptr(bias), _ptr(q_norm), _ptr(k_norm), {None: 0, "before": 1, "after": 2, "row": 3}[norm],
           float(eps), _ptr(freq) if rot else 0, rot, positions.data_ptr(), _ptr(slot_mapping), q_out.data_ptr(),
           q_out.shape[1] // rows, _ptr(pool), _dt(q_out), pool.shape[-1] if pool is not None else 0, page_size, num_heads, num_kv_heads, dim, vdim,
-          maps, T, _ptr(q_scale), 1 if own_kv else 0, float(coef), float(every), float(v_scale), _stream())
+          maps, T, _ptr(q_scale), 1 if own_kv else 0, float(coef), float(every), float(v_scale), float(magnitude), _stream())
 
 
 def padded_head(width: int) -> int:
@@ -1552,10 +1678,11 @@ def sink_attention(q: torch.Tensor, gate: Optional[torch.Tensor], out: torch.Ten
                    block_tables: torch.Tensor, meta, num_heads: int, num_kv_heads: int, dim: int, vdim: int, scale: float,
                    window: Optional[int], sink: bool, sinks: Optional[torch.Tensor] = None, softcap: Optional[float] = None,
                    keep_first: int = 0, chunk: Optional[int] = None, pooled: Optional[tuple] = None, bias: Optional[tuple] = None,
-                   pairs: Optional[tuple[float, float, float]] = None, padded: bool = False) -> None:
+                   pairs: Optional[tuple[float, float, float]] = None, padded: bool = False, gate_heads: bool = False) -> None:
     """Attention over the paged cache with keys of ``dim`` and values of ``vdim`` elements: ``q`` [T, heads * dim] -> ``out``
     [T, heads * vdim]; a query at position p sees keys p - window < j <= p; with ``sink`` the softmax's denominator has one
-    more term, exp(0); ``gate`` (float32 rows of pre-activations, heads * vdim wide) multiplies the output by its sigmoid.
+    more term, exp(0); ``gate`` (float32 rows of pre-activations, heads * vdim wide; with ``gate_heads`` one a head) multiplies the
+    output by its sigmoid.
     ``sinks`` (float32 [heads]): the term is exp(sinks[head]) instead; ``softcap`` c: scores become c tanh(s / c) after the
     scale; ``keep_first``: the window also shows keys j < keep_first; ``chunk`` (instead of a window): a query sees the keys
     j <= p with floor(j / chunk) = floor(p / chunk).  ``pooled`` = (cache, block tables, P): a second cache of the same layout
@@ -1574,14 +1701,15 @@ def sink_attention(q: torch.Tensor, gate: Optional[torch.Tensor], out: torch.Ten
     HD = pool.shape[-1]
     _need(q.stride(1) == 1 and out.stride(1) == 1 and q.shape[1] == num_heads * dim
           and tuple(out.shape) == (T, num_heads // (2 if pairs else 1) * vdim) and (not pairs or num_heads % 2 == 0), "sink_attention: shapes")
-    _need(not padded or (dim == HD and gate is None), "sink_attention: padded rows of q are as wide as the cache's, and go without a gate")
+    _need(not padded or (dim == HD and (gate is None or gate_heads)),
+          "sink_attention: padded rows of q are as wide as the cache's, and go without a gate an element")
     _need(bias is None or (all(b.dtype == torch.float32 and b.numel() == num_heads and b.is_contiguous() for b in bias)
                            and not (softcap or sink or sinks is not None or pooled or keep_first or chunk)),
           "sink_attention: a distance bias is two float32 numbers a head and goes with a plain window at most")
     _need(pairs is None or not (gate is not None or sink or sinks is not None or pooled), "sink_attention: pairs go without gates, sinks and pooled blocks")
     _need(pool.dtype == q.dtype == out.dtype and pool.is_contiguous() and pool.dim() == 5 and pool.shape[1] == 2 and HD >= max(dim, vdim),
           "sink_attention: the cache must be [pages, 2, kv heads, page, >= max(dim, vdim)] of the activations' dtype")
-    _need(gate is None or (gate.dtype == torch.float32 and gate.stride(1) == 1 and gate.shape[1] == num_heads * vdim),
+    _need(gate is None or (gate.dtype == torch.float32 and gate.stride(1) == 1 and gate.shape[1] == num_heads * (1 if gate_heads else vdim)),
           "sink_attention: the gate must be float32 rows")
     _need(block_tables.dtype == torch.int32 and block_tables.stride(1) == 1, "sink_attention: block tables")
     _need(sinks is None or (sinks.dtype == torch.float32 and sinks.numel() == num_heads and sinks.is_contiguous()),
@@ -1598,7 +1726,7 @@ def sink_attention(q: torch.Tensor, gate: Optional[torch.Tensor], out: torch.Ten
     decodes, tiles_left = meta.num_decodes, True
     fast = (use_sink_attention_mma and q.dtype == torch.bfloat16 and (dim == vdim == HD or padded) and HD in (64, 128)
             and meta.error_flag is not None and q.is_contiguous() and q.data_ptr() % 16 == 0)
-    extras = dict(keep_first=keep_first, chunk=chunk or 0, softcap=softcap or 0.0, sinks=sinks, bias=bias, out_dim=vdim)
+    extras = dict(keep_first=keep_first, chunk=chunk or 0, softcap=softcap or 0.0, sinks=sinks, bias=bias, out_dim=vdim, gate_heads=gate_heads)
     joined_from = 0                                     # with pairs: the rows from here on that diff_combine joins
     if fast and decodes and (not (masked or pooled) or (page_size >= 8 and DECODE_PARTITION % page_size == 0)):
         attention_decode(q, out, num_heads, num_kv_heads, HD, pool, page_size, block_tables, meta, scale, window, sink=sink, gate=gate,
@@ -1621,7 +1749,7 @@ def sink_attention(q: torch.Tensor, gate: Optional[torch.Tensor], out: torch.Ten
               meta.context_lens.data_ptr(), tiles.data_ptr(), n_tiles, decodes, num_heads, num_kv_heads, dim, vdim, HD, page_size,
               float(scale), int(window or 0), 1 if sink else 0, _ptr(sinks), float(softcap or 0.0), int(keep_first or 0),
               int(chunk or 0), pooled[0].data_ptr() if pool_p else 0, pooled[1].data_ptr() if pool_p else 0,
-              pooled[1].stride(0) if pool_p else 0, pool_p, _ptr(bias[0]) if bias else 0, _ptr(bias[1]) if bias else 0, _stream())
+              pooled[1].stride(0) if pool_p else 0, pool_p, _ptr(bias[0]) if bias else 0, _ptr(bias[1]) if bias else 0, 1 if gate_heads else 0, _stream())
         if pairs:
             diff_combine(out, joined, num_heads // 2, vdim, *pairs, first=joined_from)
 
@@ -1637,31 +1765,34 @@ def moe_route(logits: torch.Tensor, bias: Optional[torch.Tensor], top: int, idx:
 
 
 def moe_route_grouped(logits: torch.Tensor, correction: Optional[torch.Tensor], top: int, groups: int, keep: int, idx: torch.Tensor,
-                      weights: torch.Tensor) -> None:
+                      weights: torch.Tensor, softmax: bool = False, scale: float = 1.0) -> None:
     """Routing by sigmoid scores with a correction that only steers the choice, over groups of neighbouring experts: s =
     sigmoid(``logits``) [T, E]; choice scores s + ``correction``; a group's score is the sum of its two largest choice scores;
-    the ``top`` best experts of the ``keep`` best groups are chosen (ties: the lower index); ``weights`` are their s."""
+    the ``top`` best experts of the ``keep`` best groups are chosen (ties: the lower index); ``weights`` are their s times ``scale``.
+    ``softmax``: s is the softmax over all experts, and a group's score is its largest choice score.  ``logits`` may be columns of
+    wider rows."""
     T, E = logits.shape
-    _need(logits.dtype == torch.float32 and logits.is_contiguous(), "moe_route_grouped: logits must be float32")
+    _need(logits.dtype == torch.float32 and logits.stride(1) == 1, "moe_route_grouped: logits must be float32")
     _need(correction is None or (correction.dtype == torch.float32 and correction.numel() == E), "moe_route_grouped: correction must be float32 [E]")
     _need(idx.dtype == torch.int32 and weights.dtype == torch.float32 and tuple(idx.shape) == tuple(weights.shape) == (T, top)
           and idx.is_contiguous() and weights.is_contiguous(), "moe_route_grouped: outputs are [T, top]")
-    _call("me_moe_route_grouped", logits.data_ptr(), _ptr(correction), T, E, top, int(groups), int(keep), idx.data_ptr(), weights.data_ptr(),
-          _stream())
+    _call("me_moe_route_grouped", logits.data_ptr(), logits.stride(0), _ptr(correction), T, E, top, int(groups), int(keep),
+          1 if softmax else 0, float(scale), idx.data_ptr(), weights.data_ptr(), _stream())
 
 
 def moe_route_grouped_sort(logits: torch.Tensor, correction: Optional[torch.Tensor], top: int, groups: int, keep: int, idx: torch.Tensor,
-                           weights: torch.Tensor, counts: torch.Tensor, offsets: torch.Tensor, order: torch.Tensor, place: torch.Tensor) -> None:
+                           weights: torch.Tensor, counts: torch.Tensor, offsets: torch.Tensor, order: torch.Tensor, place: torch.Tensor,
+                           softmax: bool = False, scale: float = 1.0) -> None:
     """``moe_route_grouped`` and ``moe_sort`` together; a step of few tokens does both in one kernel."""
     T, E = logits.shape
-    _need(logits.dtype == torch.float32 and logits.is_contiguous() and (correction is None or (correction.dtype == torch.float32 and correction.numel() == E)),
+    _need(logits.dtype == torch.float32 and logits.stride(1) == 1 and (correction is None or (correction.dtype == torch.float32 and correction.numel() == E)),
           "moe_route_grouped_sort: logits and correction must be float32")
     _need(idx.dtype == torch.int32 and weights.dtype == torch.float32 and tuple(idx.shape) == tuple(weights.shape) == (T, top)
           and idx.is_contiguous() and weights.is_contiguous(), "moe_route_grouped_sort: outputs are [T, top]")
     _need(all(t.dtype == torch.int32 and t.is_contiguous() for t in (counts, offsets, order, place)) and counts.numel() >= E
           and offsets.numel() >= E + 1 and order.numel() >= T * top and place.numel() >= T * top, "moe_route_grouped_sort: output sizes")
-    _call("me_moe_route_grouped_sort", logits.data_ptr(), _ptr(correction), T, E, top, int(groups), int(keep), idx.data_ptr(),
-          weights.data_ptr(), counts.data_ptr(), offsets.data_ptr(), order.data_ptr(), place.data_ptr(), _stream())
+    _call("me_moe_route_grouped_sort", logits.data_ptr(), logits.stride(0), _ptr(correction), T, E, top, int(groups), int(keep),
+          1 if softmax else 0, float(scale), idx.data_ptr(), weights.data_ptr(), counts.data_ptr(), offsets.data_ptr(), order.data_ptr(), place.data_ptr(), _stream())
 
 
 def moe_sort(idx: torch.Tensor, num_experts: int, counts: torch.Tensor, offsets: torch.Tensor, order: torch.Tensor,
@@ -1734,15 +1865,18 @@ def moe_gemm(a: torch.Tensor, order: Optional[torch.Tensor], top: int, weight: t
           float(shift), 1 if use_moe_mma else 0, _stream())
 
 
-def moe_combine(rows: torch.Tensor, place: torch.Tensor, weights: torch.Tensor, shared: Optional[torch.Tensor], out: torch.Tensor) -> None:
-    """``out[t] = sum_k weights[t, k] * rows[place[t, k]]`` (+ ``shared[t]``); ``rows`` float32 in expert order."""
+def moe_combine(rows: torch.Tensor, place: torch.Tensor, weights: torch.Tensor, shared: Optional[torch.Tensor], out: torch.Tensor,
+                shared_gate: Optional[torch.Tensor] = None) -> None:
+    """``out[t] = sum_k weights[t, k] * rows[place[t, k]]`` (+ ``shared[t]``); ``rows`` float32 in expert order.  ``shared_gate`` (float32,
+    one number a token, possibly a column of wider rows): its sigmoid multiplies ``shared[t]``."""
     T, top = weights.shape
     W = rows.shape[1]
     _need(rows.dtype == torch.float32 and rows.stride(1) == 1 and tuple(out.shape) == (T, W) and out.stride(1) == 1, "moe_combine: shapes")
     _need(shared is None or (tuple(shared.shape) == (T, W) and shared.stride(1) == 1), "moe_combine: the shared expert's output")
+    _need(shared_gate is None or (shared_gate.dtype == torch.float32 and shared_gate.shape[0] == T), "moe_combine: the shared expert's gate is float32 [T]")
     _call("me_moe_combine", rows.data_ptr(), rows.stride(0), place.data_ptr(), weights.data_ptr(), top, _ptr(shared),
-          _dt(shared) if shared is not None else 0, shared.stride(0) if shared is not None else 0, out.data_ptr(), _dt(out),
-          out.stride(0), T, W, _stream())
+          _dt(shared) if shared is not None else 0, shared.stride(0) if shared is not None else 0, _ptr(shared_gate),
+          shared_gate.stride(0) if shared_gate is not None else 0, out.data_ptr(), _dt(out), out.stride(0), T, W, _stream())
 
 
 def token_side_gate(z: torch.Tensor, token_ids: torch.Tensor, feedback: Optional[torch.Tensor], table: torch.Tensor, first: int,

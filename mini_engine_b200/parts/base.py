@@ -104,12 +104,33 @@ class StreamCopy:
 
 
 @dataclass
+class PendingTerm:
+    """An output that joins the residual stream changed: x += scale * y with a float32 [width] ``scale`` (None: ones), or, with
+    ``eps`` given, x += scale * y / sqrt(mean(y^2) + eps) (an output that passes an RMS norm of its own)."""
+    y: "torch.Tensor"
+    scale: "Optional[torch.Tensor]" = None
+    eps: Optional[float] = None
+
+
+@dataclass
 class PendingSum:
     """What a block whose sub-layers run side by side returns instead of a plain output: the ``outputs`` ([T, width] each, at
-    most two) and ``vectors`` (float32 [width] each, e.g. a projection's bias left to be added) have not joined the residual
-    stream yet; the next kernel that reads the stream (the next norm, or the model's last) adds them all first."""
+    most two; tensors, or, for norms that take them, up to three tensors and ``PendingTerm``s) and ``vectors`` (float32 [width]
+    each, e.g. a projection's bias left to be added) have not joined the residual stream yet; the next kernel that reads the
+    stream (the next norm, or the model's last) adds them all first."""
     outputs: list
     vectors: list = field(default_factory=list)
+
+
+def pending_terms(delta) -> tuple[list[tuple], list]:
+    """Whatever a block left pending as (terms (y, scale, eps), vectors) of ``ops.stream_norm``."""
+    if delta is None or isinstance(delta, (AddedToResidual, StreamCopy)):
+        return [], []
+    if isinstance(delta, PendingSum):
+        return [(o.y, o.scale, o.eps) if isinstance(o, PendingTerm) else (o, None, None) for o in delta.outputs], list(delta.vectors)
+    if isinstance(delta, torch.Tensor) and delta.dim() == 2:
+        return [(delta, None, None)], []
+    raise TypeError(f"a pending {type(delta).__name__} cannot join the stream term by term")
 
 
 @dataclass

@@ -10,7 +10,7 @@ from __future__ import annotations
 from dataclasses import dataclass, field
 from typing import Any, Optional
 
-from .base import NormedUpdate, ParamDecl, Part, PendingSum, StreamCopy, StreamUpdate, Upcoming
+from .base import NormedUpdate, ParamDecl, Part, PendingSum, PendingTerm, StreamCopy, StreamUpdate, Upcoming
 from .registry import PartSpec, build_part, register_block
 
 
@@ -57,25 +57,27 @@ class Block(Part):
         mixer_spec = spec.mixer
         if shared:
             # Objects that several layers share (one rotary table for all of them).
-            args = {k: shared.get(v.key, v) if isinstance(v, SharedRef) else v
-                    for k, v in mixer_spec.args.items()}
-            mixer_spec = PartSpec(mixer_spec.kind, args)
+            mixer_spec = _with_shared(mixer_spec, shared)
         self.mixer = build_part("mixer", mixer_spec)
         self.mixer_norm = build_part("norm", spec.norm_of("mixer_norm"))
         self.feed_forward = self.feed_forward_norm = None
         if spec.feed_forward is not None:
             self.feed_forward = build_part("feed_forward", spec.feed_forward)
-            self.feed_forward_norm = build_part("norm", spec.norm_of("feed_forward_norm"))
+            if not self.one_norm:
+                self.feed_forward_norm = build_part("norm", spec.norm_of("feed_forward_norm"))
         elif not self.feed_forward_optional:
             raise ValueError(f"a {spec.kind!r} block needs a feed-forward")
 
     feed_forward_optional = False
+    one_norm = False                      # both sub-layers read the mixer's norm (there is no second one)
 
     def sub_parts(self):
         s = self.spec
         parts = [(s.mixer_norm_prefix, self.mixer_norm), (s.mixer_prefix, self.mixer)]
+        if self.feed_forward_norm is not None:
+            parts.append((s.feed_forward_norm_prefix, self.feed_forward_norm))
         if self.feed_forward is not None:
-            parts += [(s.feed_forward_norm_prefix, self.feed_forward_norm), (s.feed_forward_prefix, self.feed_forward)]
+            parts.append((s.feed_forward_prefix, self.feed_forward))
         return parts
 
     def _unused_second_norm(self) -> list:
@@ -272,36 +274,63 @@ class ParallelBlock(Block):
     (``PendingSum``) and join the stream in the kernel that reads it next, which also computes both norms of the new rows in
     one pass; a mixer's output bias (``output_bias()``) is deferred the same way.  A ``LayerCall`` may name a pass vector
     (``add_row``) that joins the stream right before the block's norms.  The norms must be of a kind that takes a
-    ``PendingSum`` (a layer norm with a bias)."""
+    ``PendingSum`` (kinds ``layernorm`` and ``rmsnorm``).
+
+    ``BlockSpec.args``: ``one_norm``: there is one norm and both sub-layers read its output; ``scales`` = {"mixer": name,
+    "feed_forward": name, "width": size}: each sub-layer's output is multiplied element by element by the vector of that name before
+    it joins the stream (the norm's kind must take ``PendingTerm``s: ``rmsnorm``)."""
     capturable = True
     feed_forward_optional = True
     takes_pass_vector = True
 
     def __init__(self, spec: BlockSpec, shared: Optional[dict] = None):
+        self.one_norm = bool(spec.args.get("one_norm"))
+        self.scales = dict(spec.args.get("scales") or {})
         super().__init__(spec, shared)
         self.pass_vectors = (shared or {}).get("pass_vectors")
         for norm in (self.mixer_norm, self.feed_forward_norm):
             if norm is not None and not hasattr(norm, "_sum_and_norm"):
-                raise ValueError("a 'parallel' block needs norms that can add a pending sum (kind 'layernorm')")
+                raise ValueError("a 'parallel' block needs norms that can add a pending sum (kinds 'layernorm' and 'rmsnorm')")
         if hasattr(self.mixer, "defer_output_bias"):
             self.mixer.defer_output_bias = True
+        self._scaled: dict = {}
 
     def param_decls(self):
-        return self._unused_second_norm()
+        if not self.scales:
+            return self._unused_second_norm()
+        size = (int(self.scales["width"]),)
+        return [ParamDecl(self.scales["mixer"], size, init="norm", role="vector"),
+                ParamDecl(self.scales["feed_forward"], size, init="norm", role="vector", optional=self.feed_forward is None)]
+
+    def _terms(self, output, place: str) -> list:
+        """A sub-layer's output (a tensor, or a ``PendingSum`` of terms) as terms with the place's scale."""
+        outputs = output.outputs if isinstance(output, PendingSum) else [output]
+        if not self.scales:
+            return list(outputs)
+        scale, terms = self.p(self.scales[place]), []
+        for o in outputs:
+            if isinstance(o, PendingTerm):
+                own = self._scaled.get(id(o.scale)) if o.scale is not None else (None, scale)
+                if own is None:                   # both factors in one vector, once
+                    own = self._scaled[id(o.scale)] = (o.scale, (o.scale * scale).contiguous())
+                terms.append(PendingTerm(o.y, own[1], o.eps))
+            else:
+                terms.append(PendingTerm(o, scale))
+        return terms
 
     def forward(self, residual, delta, ctx, call, upcoming=None):
         vectors = []
         if call.add_row is not None:
             vectors.append(self.pass_vectors.row(call.add_row))
-        also = (self.feed_forward_norm, "norm_out2") if self.feed_forward is not None else None
+        also = (self.feed_forward_norm, "norm_out2") if self.feed_forward_norm is not None else None
         h = self.mixer_norm._sum_and_norm(residual, delta, ctx, None, "norm_out", None, vectors=vectors, also=also)
-        h1, h2 = h if also is not None else (h, None)
-        pending = PendingSum([self.mixer.forward(h1, ctx, call)])
+        h1, h2 = h if also is not None else (h, h)
+        pending = PendingSum(self._terms(self.mixer.forward(h1, ctx, call), "mixer"))
         bias = self.mixer.output_bias() if hasattr(self.mixer, "output_bias") else None
         if bias is not None:
             pending.vectors.append(bias)
         if self.feed_forward is not None:
-            pending.outputs.append(self.feed_forward.forward(h2, ctx))
+            pending.outputs += self._terms(self.feed_forward.forward(h2, ctx), "feed_forward")
         return pending
 
 
@@ -339,6 +368,19 @@ class PostNormBlock(Block):
 class SharedRef:
     """Stands in a PartSpec's args for an object that the model builds once and shares."""
     key: str
+
+
+def _with_shared(value, shared: dict):
+    """``value`` with every ``SharedRef`` in it replaced by the object it stands for (also in the arguments of inner parts)."""
+    if isinstance(value, SharedRef):
+        return shared.get(value.key, value)
+    if isinstance(value, PartSpec):
+        return PartSpec(value.kind, _with_shared(value.args, shared))
+    if isinstance(value, dict):
+        return {k: _with_shared(v, shared) for k, v in value.items()}
+    if isinstance(value, (list, tuple)):
+        return type(value)(_with_shared(v, shared) for v in value)
+    return value
 
 
 register_block("pre_norm", PreNormBlock)

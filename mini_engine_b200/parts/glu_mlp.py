@@ -13,7 +13,10 @@ Two more choices.  ``routing`` "sigmoid_groups" (instead of "softmax_top"): scor
 s + ``correction`` (a learned number per expert that only steers the choice); the experts form ``groups`` = (count, keep)
 equal groups of neighbours, a group's score is the sum of its two largest choice scores, and only experts of the ``keep``
 best groups can be chosen; the weights are the chosen experts' s, not renormalised.  ``activation`` (a key of
-``ops.ACTIVATIONS``, instead of the gate): an expert is W_down act(W_up h) and has no gate matrix.
+``ops.ACTIVATIONS``, instead of the gate): an expert is W_down act(W_up h) and has no gate matrix (a ``shared`` expert with an
+``activation`` of its own likewise).  ``routing`` "softmax_groups": as "sigmoid_groups" with s the softmax over all experts' logits and a
+group's score its largest choice score.  ``weight_scale`` multiplies the weights of either grouped rule.  ``shared_gate`` (a tensor's
+name): the shared expert's output is multiplied by sigmoid(W_sg h), one number a token, whose row is packed with the router's.
 """
 from __future__ import annotations
 
@@ -24,6 +27,7 @@ import torch
 from .. import ops
 from .base import DiskSource, FeedForward, ParamDecl
 from .linear import Linear
+from .mlp import ActivationMLP
 from .registry import register_feed_forward
 
 
@@ -72,20 +76,26 @@ class RoutedExperts(FeedForward):
     def __init__(self, hidden_size: int, num_experts: int, top: int, expert_size: int, limit: Optional[float] = None,
                  alpha: float = 1.702, shift: float = 1.0, router_bias: bool = True, shared: Optional[dict] = None,
                  routing: str = "softmax_top", groups: Optional[tuple] = None, correction: bool = False,
-                 activation: Optional[str] = None, out_dtype: Optional[str] = None):
+                 activation: Optional[str] = None, out_dtype: Optional[str] = None, weight_scale: float = 1.0, shared_gate: Optional[str] = None):
         super().__init__()
         if not 1 <= top <= num_experts:
             raise ValueError(f"{top} of {num_experts} experts cannot be chosen")
-        if routing not in ("softmax_top", "sigmoid_groups"):
-            raise ValueError(f"routing must be 'softmax_top' or 'sigmoid_groups', got {routing!r}")
+        if routing not in ("softmax_top", "sigmoid_groups", "softmax_groups"):
+            raise ValueError(f"routing must be 'softmax_top', 'sigmoid_groups' or 'softmax_groups', got {routing!r}")
+        grouped = routing != "softmax_top"
+        if shared_gate and not shared:
+            raise ValueError("a shared expert's gate needs the shared expert")
+        if not grouped and (weight_scale != 1.0 or shared_gate):
+            raise ValueError("a factor on the weights and a gate on the shared expert go with the grouped routings")
         if activation is not None and activation not in ops.ACTIVATIONS:
             raise ValueError(f"unknown activation {activation!r}; known: {sorted(ops.ACTIVATIONS)}")
         count, keep = (int(groups[0]), int(groups[1])) if groups else (1, 1)
-        if routing == "sigmoid_groups" and (count < 1 or num_experts % count or not 1 <= keep <= count
+        if grouped and (count < 1 or num_experts % count or not 1 <= keep <= count
                                             or keep * (num_experts // count) < top):
             raise ValueError(f"{keep} of {count} groups over {num_experts} experts cannot give {top} choices")
         if routing == "softmax_top" and (groups or correction):
-            raise ValueError("groups and a correction go with routing 'sigmoid_groups'")
+            raise ValueError("groups and a correction go with the grouped routings")
+        self.grouped, self.weight_scale, self.shared_gate = grouped, float(weight_scale), shared_gate
         self.routing, self.groups, self.has_correction, self.activation = routing, (count, keep), correction, activation
         self.out_dtype = getattr(torch, out_dtype) if out_dtype else None    # what the weighted sum is written as (None: the working dtype)
         self.hidden_size, self.num_experts, self.top, self.expert_size = hidden_size, num_experts, top, expert_size
@@ -93,8 +103,10 @@ class RoutedExperts(FeedForward):
         self.alpha = float(alpha)
         self.shift = float(shift)
         self.has_router_bias = router_bias and routing == "softmax_top"
-        self.router = Linear(hidden_size, [("router", num_experts)], name="router")
-        self.shared = ClampedGLU(hidden_size, **shared) if shared else None
+        self.router = Linear(hidden_size, [("router", num_experts)] + ([(shared_gate, 1)] if shared_gate else []), name="router")
+        self.shared = None
+        if shared:
+            self.shared = ActivationMLP(hidden_size, in_product=True, **shared) if shared.get("activation") else ClampedGLU(hidden_size, **shared)
         self._gate_up = self._down = None
 
     def sub_parts(self):
@@ -129,15 +141,16 @@ class RoutedExperts(FeedForward):
         E, F, W, top = self.num_experts, self.expert_size, self.hidden_size, self.top
         T = x.shape[0]
         z = self.router.forward(x, ctx, "moe_logits", out_dtype=torch.float32)
+        gate = z[:, E] if self.shared_gate else None
         idx = ctx.buffer("moe_idx", (T, top), torch.int32)
         wgt = ctx.buffer("moe_weights", (T, top), torch.float32)
         counts = ctx.buffer("moe_counts", (E,), torch.int32)
         offsets = ctx.buffer("moe_offsets", (E + 1,), torch.int32)
         order = ctx.buffer("moe_order", (T * top,), torch.int32)
         place = ctx.buffer("moe_place", (T * top,), torch.int32)
-        if self.routing == "sigmoid_groups":
-            ops.moe_route_grouped_sort(z, self.p("correction") if self.has_correction else None, top, *self.groups, idx, wgt, counts,
-                                       offsets, order, place)
+        if self.grouped:
+            ops.moe_route_grouped_sort(z[:, :E], self.p("correction") if self.has_correction else None, top, *self.groups, idx, wgt, counts,
+                                       offsets, order, place, softmax=self.routing == "softmax_groups", scale=self.weight_scale)
         else:
             ops.moe_route_sort(z, self.p("router.b") if self.has_router_bias else None, top, idx, wgt, counts, offsets, order, place)
         act = ctx.buffer("moe_act", (T * top, F), ctx.act_dtype)
@@ -150,7 +163,7 @@ class RoutedExperts(FeedForward):
         ops.moe_gemm(act, None, top, self._down, offsets, rows, workspace=ctx.buffer, err=ctx.error_flag)
         shared = self.shared.forward(x, ctx, out_name="moe_shared") if self.shared is not None else None
         out = ctx.buffer("ffn_out", (T, W), self.out_dtype or ctx.act_dtype)
-        ops.moe_combine(rows, place, wgt, shared, out)
+        ops.moe_combine(rows, place, wgt, shared, out, shared_gate=gate)
         return out
 
 

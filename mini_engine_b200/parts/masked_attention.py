@@ -1,6 +1,7 @@
-"""Grouped-query attention with a mask, a learned sink in the softmax, and choices around scores and rotation.
+"""Grouped-query attention with a mask, a sink in the softmax, and choices around scores, rotation and output.
 
-q = W_q h, k = W_k h, v = W_v h, each with a bias when ``bias`` is set (then the output projection has one too).  Every q
+q = W_q h, k = W_k h, v = W_v h, each with a bias when ``bias`` is set (then the output projection has one too, unless
+``output_bias`` is False).  Every q
 and k head may be RMS-normed: ``qk_norm`` "before" (with a weight of ``dim`` values for q and one for k, shared by the
 heads, in front of the rotation) or "after" (no weight, behind the rotation); "row" takes the root mean square over ALL of a
 token's q (and of its k), with a weight for every value.  The rotation pairs element i with element
@@ -10,7 +11,8 @@ score = q . k * scale, then, with ``softcap`` c, c tanh(score / c), or, with ``d
 learned numbers a head (``r1``, ``r2``).  ``mask``: None (every key j <= p),
 ("window", size, keep_first): keys with p - j < size or j < keep_first, or ("chunk", size): keys of the query's own
 chunk, floor(j / size) = floor(p / size).  The weights are exp(s_j) / (exp(sink_h) + sum exp(s_j)) with a learned number
-per head when ``sink`` is set: a term without key or value that is neither scaled nor capped.  ``out_scale`` multiplies the
+per head when ``sink`` is set: a term without key or value that is neither scaled nor capped (``sink`` "one": the term is 1, a
+sink whose score is 0).  ``head_gate``: head h's output is multiplied by sigmoid(W_g x)_h, one number a head.  ``out_scale`` multiplies the
 mixer's output (the values carry it, and the output bias).  Keys have ``dim`` elements
 and values ``vdim``; the cache is the engine's usual one (pages of keys and of values) with rows of max(dim, vdim)
 elements, or with ``pad_rows`` of the next size the tensor-core kernels take (zeros behind keys and values), and it keeps
@@ -36,10 +38,12 @@ class MaskedSinkAttention(Mixer):
 
     def __init__(self, hidden_size: int, num_heads: int, num_kv_heads: int, dim: int, vdim: int, scale: float, norm_eps: float,
                  position_encoding: Optional[PartSpec | object] = None, qk_norm: Optional[str] = None, bias: bool = False,
-                 softcap: Optional[float] = None, mask: Optional[tuple] = None, sink: bool = True,
+                 softcap: Optional[float] = None, mask: Optional[tuple] = None, sink: "bool | str" = True,
                  temperature: Optional[tuple[float, float]] = None, distance_bias: bool = False, out_scale: float = 1.0,
-                 pad_rows: bool = False, hosted: bool = False):
+                 pad_rows: bool = False, hosted: bool = False, output_bias: bool = True, head_gate: bool = False):
         super().__init__()
+        if sink not in (True, False, "one"):
+            raise ValueError(f"sink must be True, False or 'one', got {sink!r}")
         if num_heads < 1 or num_kv_heads < 1 or num_heads % num_kv_heads:
             raise ValueError(f"{num_heads} heads are no multiple of {num_kv_heads} kv heads")
         if qk_norm not in (None, "before", "after", "row"):
@@ -51,7 +55,8 @@ class MaskedSinkAttention(Mixer):
         self.hidden_size, self.num_heads, self.num_kv_heads = hidden_size, num_heads, num_kv_heads
         self.dim, self.vdim = dim, vdim
         self.scale, self.norm_eps = float(scale), float(norm_eps)
-        self.qk_norm, self.has_bias, self.has_sink = qk_norm, bias, sink
+        self.qk_norm, self.has_bias, self.has_sink, self.unit_sink = qk_norm, bias, sink is True, sink == "one"
+        self.has_output_bias, self.head_gate = bias and output_bias, head_gate
         self.softcap = float(softcap) if softcap else None
         self.temperature = (float(temperature[0]), float(temperature[1])) if temperature is not None else None
         self.distance_bias, self.out_scale, self.pad_rows = bool(distance_bias), float(out_scale), bool(pad_rows)
@@ -73,7 +78,10 @@ class MaskedSinkAttention(Mixer):
                              f"(got layout {self.rope.layout!r}, {self.rope.rotary_dim} of {dim})")
         H, G = num_heads, num_kv_heads
         self.pieces = [("q", H * dim), ("k", G * dim), ("v", G * vdim)]
-        self.channels = sum(n for _, n in self.pieces)
+        self.channels = sum(n for _, n in self.pieces)          # what passes through biases, norms and the rotation
+        self.biased = list(self.pieces)
+        if head_gate:
+            self.pieces.append(("g", H))
         self.heads_width = H * vdim
         self.in_proj = None if hosted else Linear(hidden_size, self.pieces, name="in_proj")
         self.o_proj = None if hosted else Linear(self.heads_width, [("o", hidden_size)], name="o")
@@ -90,11 +98,12 @@ class MaskedSinkAttention(Mixer):
         decls = []
         if self.has_bias:
             sources, start = [], 0
-            for piece, n in self.pieces:
+            for piece, n in self.biased:
                 sources.append(DiskSource(piece + ".b", start, n))
                 start += n
-            decls += [ParamDecl("in_bias", (self.channels,), sources=sources, role="vector"),
-                      ParamDecl("o.b", (self.hidden_size,), role="vector")]
+            decls.append(ParamDecl("in_bias", (self.channels,), sources=sources, role="vector"))
+        if self.has_output_bias:
+            decls.append(ParamDecl("o.b", (self.hidden_size,), role="vector"))
         if self.qk_norm == "before":
             decls += [ParamDecl("q.norm", (self.dim,), init="norm", role="vector"), ParamDecl("k.norm", (self.dim,), init="norm", role="vector")]
         if self.qk_norm == "row":
@@ -107,7 +116,7 @@ class MaskedSinkAttention(Mixer):
         return decls
 
     def finalize(self, dtype, device):
-        if self.has_bias:
+        if self.has_output_bias:
             self._o_bias = (self.p("o.b") * self.out_scale).contiguous() if self.out_scale != 1.0 else self.p("o.b")
 
     def cache_needs(self):
@@ -118,7 +127,7 @@ class MaskedSinkAttention(Mixer):
 
     def output_bias(self):
         """The output projection's bias when the caller has asked to add it itself (``defer_output_bias``), else None."""
-        return self._o_bias if self.has_bias and self.defer_output_bias else None
+        return self._o_bias if self.has_output_bias and self.defer_output_bias else None
 
     def heads_of(self, proj, ctx, call, out) -> None:
         """``proj`` [T, columns of ``pieces``] float32 -> the joined heads in ``out`` [T, heads_width]."""
@@ -131,18 +140,19 @@ class MaskedSinkAttention(Mixer):
                       self.p("k.norm") if weighted else None, self.qk_norm, self.norm_eps,
                       self.rope.freq if self.rope is not None and self.rope.rotary_dim else None, ctx.positions,
                       kv.slot_mapping if call.writes_cache else None, q, kv.pool, kv.page_size, H, G, D, V,
-                      temperature=self.temperature, v_scale=self.out_scale)
-        ops.sink_attention(q, None, out, kv.pool, kv.page_size, kv.block_tables, ctx.attn_meta, H, G, self.q_row, V, self.scale,
-                           self.window, False, sinks=self.p("sink") if self.has_sink else None, softcap=self.softcap,
+                      temperature=self.temperature, v_scale=self.out_scale, magnitude=self.rope.magnitude if self.rope is not None else 1.0)
+        gate = proj[:, self.channels:self.channels + H] if self.head_gate else None
+        ops.sink_attention(q, gate, out, kv.pool, kv.page_size, kv.block_tables, ctx.attn_meta, H, G, self.q_row, V, self.scale,
+                           self.window, self.unit_sink, sinks=self.p("sink") if self.has_sink else None, softcap=self.softcap,
                            keep_first=self.keep_first, chunk=self.chunk, padded=self.pad_rows,
-                           bias=(self.p("r1"), self.p("r2")) if self.distance_bias else None)
+                           bias=(self.p("r1"), self.p("r2")) if self.distance_bias else None, gate_heads=self.head_gate)
 
     def forward(self, x, ctx, call):
         proj = self.in_proj.forward(x, ctx, "attn_proj", out_dtype=torch.float32)
         out = ctx.buffer("attn_out", (proj.shape[0], self.heads_width), ctx.act_dtype)
         self.heads_of(proj, ctx, call, out)
         y = self.o_proj.forward(out, ctx, "mixer_out")
-        if self.has_bias and not self.defer_output_bias:
+        if self.has_output_bias and not self.defer_output_bias:
             ops.add_row_vector(y, self._o_bias)
         return y
 

@@ -15,9 +15,11 @@ from typing import Any, Iterator, Optional
 
 import torch
 
-from .base import Part, ParamDecl
+from .. import ops
+from .base import Part, ParamDecl, pending_terms
 from .block import BlockSpec, SharedRef
 from .embed import LMHead, TokenEmbedding
+from .linear import Linear
 from .registry import PartSpec, build_block, build_part
 
 
@@ -29,6 +31,7 @@ class LayerCall:
     kv_slot: "Optional[int]" = None    # a mixer that reads ANOTHER call's keys and values: the cache slot that holds them
     add_row: "Optional[int]" = None    # the row of the model's pass vectors that joins the stream right before this call
     add_embedding: bool = False        # the step's embedding rows join the stream once more right before this call
+    join_embedding: bool = False       # the stream becomes W [x; embedding output] right before this call (ModelPlan.pass_input)
 
 
 @dataclass
@@ -58,6 +61,9 @@ class ModelPlan:
     embed_norm_prefix: str = ""
     pass_vectors: "Optional[tuple[str, int]]" = None   # (tensor name, rows): vectors of ``hidden_size`` values of which a
                                        # ``LayerCall.add_row`` names one (what each pass over looped layers adds to the stream)
+    pass_input: "Optional[str]" = None         # name of a matrix [hidden, 2 hidden] that maps [stream; embedding output] to the stream in
+                                       # front of every ``LayerCall`` with ``join_embedding``
+    position_table: "Optional[tuple[str, int]]" = None   # (tensor name, rows): learned vectors, one a position, added to the embedding
 
 
 class PassVectors(Part):
@@ -76,6 +82,33 @@ class PassVectors(Part):
         return self.p(self.name)[i]
 
 
+class PassInput(Part):
+    """x <- W [x; x0] in front of a pass over looped layers, x0 being the embedding output: the stream and the embedding output lie side
+    by side in one work buffer in the working dtype, whose second half the embedding's kernel fills once a step and whose first half
+    takes the stream with everything pending right before the product, which writes the float32 stream itself."""
+    capturable = True
+
+    def __init__(self, name: str, width: int):
+        super().__init__()
+        self.width = width
+        self.map = Linear(2 * width, [(name, width)], name=name)
+
+    def sub_parts(self):
+        return [("", self.map)]
+
+    def _rows(self, ctx, T: int) -> torch.Tensor:
+        return ctx.buffer("pass_input", (T, 2 * self.width), ctx.act_dtype)
+
+    def embedding_half(self, ctx, T: int) -> torch.Tensor:
+        return self._rows(ctx, T)[:, self.width:]
+
+    def forward(self, residual, delta, ctx) -> None:
+        rows = self._rows(ctx, residual.shape[0])
+        terms, vectors = pending_terms(delta)
+        ops.stream_norm(residual, terms, vectors, None, 0.0, rows[:, :self.width])
+        self.map.forward(rows, ctx, "residual", out_dtype=torch.float32)      # (the stream's own buffer)
+
+
 class DecoderModel(Part):
     capturable = True
 
@@ -84,7 +117,7 @@ class DecoderModel(Part):
         self.plan = plan
         self.shared = {k: build_part("position_encoding", s) for k, s in plan.shared.items()}
         self.embed = TokenEmbedding(plan.vocab_size, plan.hidden_size, scale=plan.embedding_scale, streams=plan.streams,
-                                    param=plan.embed_param)
+                                    param=plan.embed_param, positions=plan.position_table)
         self.embed_norm = build_part("norm", plan.embed_norm) if plan.embed_norm is not None else None
         if self.embed_norm is not None and not hasattr(self.embed_norm, "normalize_stream"):
             raise ValueError(f"norm kind {plan.embed_norm.kind!r} cannot normalise the stream in place (ModelPlan.embed_norm)")
@@ -94,6 +127,7 @@ class DecoderModel(Part):
         self.pass_vectors = None
         if plan.pass_vectors is not None:
             self.pass_vectors = self.shared["pass_vectors"] = PassVectors(plan.pass_vectors[0], plan.pass_vectors[1], plan.hidden_size)
+        self.pass_input = PassInput(plan.pass_input, plan.hidden_size) if plan.pass_input is not None else None
         self.blocks = [build_block(s, self.shared) for s in plan.blocks]
         self.final_norm = build_part("norm", plan.final_norm)
         tied = plan.embed_prefix + plan.embed_param if plan.tie_word_embeddings else None
@@ -115,6 +149,8 @@ class DecoderModel(Part):
                                      f"{self.pass_vectors.rows if self.pass_vectors else 0}")
             if c.add_embedding and not getattr(self.blocks[c.block], "takes_embedding", False):
                 raise ValueError(f"block {c.block} ({plan.blocks[c.block].kind!r}) cannot add the embedding in front of itself")
+            if c.join_embedding and (self.pass_input is None or plan.streams != 1):
+                raise ValueError("the schedule joins the embedding output in front of a call, but the plan names no matrix for it (pass_input)")
             needs = self.blocks[c.block].cache_needs()
             if not self.slot_needs[c.cache_slot]:
                 self.slot_needs[c.cache_slot] = needs
@@ -135,6 +171,8 @@ class DecoderModel(Part):
         parts += [("", t) for t in self.tables.values()]
         if self.pass_vectors is not None:
             parts.append(("", self.pass_vectors))
+        if self.pass_input is not None:
+            parts.append(("", self.pass_input))
         parts += [(self.plan.block_prefix.format(i=i), b) for i, b in enumerate(self.blocks)]
         parts += [(self.plan.final_norm_prefix, self.final_norm), (self.plan.head_prefix, self.head)]
         return parts
@@ -162,11 +200,15 @@ class DecoderModel(Part):
         """Hidden states of the wanted rows, normalised: ``[len(ctx.logits_rows), hidden]``."""
         ctx.token_ids = token_ids
         ctx.forward_serial = getattr(ctx, "forward_serial", 0) + 1      # what parts cache for ONE pass over the layers is keyed by this
-        residual = self.embed.forward(token_ids, ctx)
+        copy = self.pass_input.embedding_half(ctx, token_ids.shape[0]) if self.pass_input is not None else None
+        residual = self.embed.forward(token_ids, ctx, copy=copy)
         delta = self.embed_norm.normalize_stream(residual, ctx) if self.embed_norm is not None else None
         for i, call in enumerate(self.schedule):
             # the block learns what runs after it, so that its last kernel can prepare for it
             after = self.blocks[self.schedule[i + 1].block].upcoming() if i + 1 < len(self.schedule) else None
+            if call.join_embedding:
+                self.pass_input.forward(residual, delta, ctx)
+                delta = None
             delta = self.blocks[call.block].forward(residual, delta, ctx, call, upcoming=after)
         return self.final_norm.forward(residual, delta, ctx, rows=ctx.logits_rows)
 

@@ -13,7 +13,8 @@ from typing import Optional
 import torch
 
 from .. import ops
-from .base import AddedToResidual, Norm, NormedUpdate, ParamDecl, PendingNorm, PendingSum, StreamCopy, StreamUpdate
+from .base import (AddedToResidual, Norm, NormedUpdate, ParamDecl, PendingNorm, PendingSum, PendingTerm, StreamCopy, StreamUpdate,
+                   pending_terms)
 from .registry import register_norm
 
 
@@ -21,7 +22,8 @@ class RMSNorm(Norm):
     """``param``: the weight's name on disk, for models that do not call it ``weight``.  ``unit_offset``: the weight is
     stored as its distance from one (y = x / rms(x) * (1 + w)); the sum is formed once, in float32, when the weights
     are in place.  A pending ``NormedUpdate`` (a sub-layer's output that is itself normalised, weighted and scaled before
-    it joins the stream) goes into the residual in the same pass."""
+    it joins the stream) or ``PendingSum`` (several outputs, each with a scale or a norm of its own where it has one, and vectors)
+    goes into the residual in the same pass."""
     capturable = True
 
     def __init__(self, size: int, eps: float, param: str = "weight", unit_offset: bool = False):
@@ -48,7 +50,19 @@ class RMSNorm(Norm):
         in front may write x * w itself."""
         return self.weight
 
+    def _sum_and_norm(self, residual, delta, ctx, rows, out_name, out_dtype, vectors=(), also=None, embedding=None):
+        """One pass of ``stream_norm``: everything pending and ``vectors`` join the stream, then this norm."""
+        if also is not None or embedding is not None:
+            raise ValueError("RMSNorm takes neither a second norm nor the embedding in the same pass")
+        terms, pending = pending_terms(delta)
+        n = residual.shape[0] if rows is None else rows.shape[0]
+        out = ctx.buffer(out_name, (n, self.size), out_dtype or ctx.act_dtype)
+        ops.stream_norm(residual, terms, pending + list(vectors), self.weight, self.eps, out, rows=rows)
+        return out
+
     def forward(self, residual, delta, ctx, rows: Optional[torch.Tensor] = None, lazy: bool = False):
+        if isinstance(delta, PendingSum):
+            return self._sum_and_norm(residual, delta, ctx, rows, "norm_out", None)
         n = residual.shape[0] if rows is None else rows.shape[0]
         if isinstance(delta, NormedUpdate):
             out = ctx.buffer("norm_out", (n, self.size), ctx.act_dtype)
@@ -100,6 +114,8 @@ class LayerNorm(Norm):
         outputs, vectors = [], list(vectors)
         if isinstance(delta, PendingSum):
             outputs, vectors = list(delta.outputs), list(delta.vectors) + vectors
+            if any(isinstance(o, PendingTerm) for o in outputs):
+                raise TypeError("LayerNorm cannot add an output that joins the stream with a scale or a norm of its own")
         elif isinstance(delta, torch.Tensor):
             outputs = [delta]
         elif delta is not None and not isinstance(delta, AddedToResidual):

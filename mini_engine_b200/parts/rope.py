@@ -86,8 +86,12 @@ class FrequencyRotary(PositionEncoding):
     elements, from a table of frequencies instead of a table over positions: f_i = theta^(-2i / rotary_dim), optionally
     rescaled by wavelength (``scaling`` = {factor, low, high, original}, the rule Llama 3.1 uses for long contexts: with
     l = 2 pi / f, a frequency with l < original / high stays, one with l > original / low is divided by factor, and between
-    the two (1 - s) f / factor + s f with s = (original / l - low) / (high - low)).  The kernels form each angle from the
-    position and ``freq`` (float64, so that the angle is rounded once), which leaves the longest position open."""
+    the two (1 - s) f / factor + s f with s = (original / l - low) / (high - low)), or by index (``scaling`` = {factor, fast,
+    slow, original}, YaRN: with d(n) = rotary_dim ln(original / (2 pi n)) / (2 ln theta), the index whose wavelength fits n times
+    into ``original`` positions, a ramp r_i rises from 0 at lo = max(floor d(fast), 0) to 1 at hi = min(ceil d(slow),
+    rotary_dim - 1), and the frequency is r_i f / factor + (1 - r_i) f; cosines and sines are multiplied by ``magnitude`` =
+    0.1 ln(factor) + 1).  The kernels form each angle from the position and ``freq`` (float64, so that the angle is rounded once),
+    which leaves the longest position open."""
     capturable = True
 
     layout = "half_split"
@@ -99,7 +103,15 @@ class FrequencyRotary(PositionEncoding):
         self.rotary_dim = rotary_dim
         self.theta = float(theta)
         self.scaling = dict(scaling) if scaling else None
-        if self.scaling:
+        self.magnitude = 1.0                          # a factor on the cosines and sines
+        self.yarn = bool(scaling) and "fast" in scaling
+        if self.yarn:
+            import math
+            s = self.scaling
+            if not (s["factor"] > 0 and s["original"] > 0 and s["fast"] > 0 and s["slow"] > 0 and self.theta > 0 and self.theta != 1.0):
+                raise ValueError(f"YaRN scaling needs factor, original, fast and slow > 0 and a base other than 1, got {s}, base {theta}")
+            self.magnitude = 0.1 * math.log(s["factor"]) + 1.0
+        elif self.scaling:
             s = self.scaling
             if not (s["factor"] > 0 and s["original"] > 0 and s["high"] > s["low"] > 0):
                 raise ValueError(f"rotary scaling needs factor > 0, original > 0 and high > low > 0, got {s}")
@@ -109,9 +121,18 @@ class FrequencyRotary(PositionEncoding):
         import math
         d = self.rotary_dim
         out = []
+        if self.yarn:
+            s = self.scaling
+
+            def index(turns: float) -> float:
+                return d * math.log(s["original"] / (turns * 2.0 * math.pi)) / (2.0 * math.log(self.theta))
+            lo, hi = max(math.floor(index(s["fast"])), 0), min(math.ceil(index(s["slow"])), d - 1)
         for i in range(d // 2):
             f = self.theta ** (-2.0 * i / d)
-            if self.scaling:
+            if self.yarn:
+                r = min(max((i - lo) / max(hi - lo, 0.001), 0.0), 1.0)
+                f = f / s["factor"] * r + f * (1.0 - r)
+            elif self.scaling:
                 s = self.scaling
                 wavelength = 2.0 * math.pi / f
                 if wavelength > s["original"] / s["low"]:
