@@ -28,7 +28,7 @@ GPU: for ``--gpus N`` with N > 1 one line says so and the exit code is 2.
 Modes: ``step`` (the line above), ``offline`` (the reference's own bench.py:38-66 with its options ``--num-seqs
 --budget --chunked --threshold --out --label --expect-gpu``; a JSON row like the reference's is appended to
 ``--out``), ``mixed`` (the 8B workload above, at any shape), ``decode`` (decode at batches ``--batches`` after
-``--prompt-len`` prompts), ``prefill`` (one prompt of ``--prompt-len`` tokens in portions of ``--budget``), ``logozen``, ``pugadra``, ``gevulorn``, ``galupel`` and ``tidenex``
+``--prompt-len`` prompts), ``prefill`` (one prompt of ``--prompt-len`` tokens in portions of ``--budget``), ``logozen``, ``pugadra``, ``gevulorn``, ``galupel``, ``tidenex`` and ``kuterax``
 (prefill and decode of that design at the layer sizes ``--sizes``, beside the Qwen3 of equal size (Gevulorn and Galupel: the Pugadra, Tidenex: the
 Gevulorn of equal size), with the time of every kernel).
 """
@@ -204,9 +204,38 @@ TIDENEX_SIZES = {   # width, layers, ff, heads / kv heads / head size, a map's s
     "m": _tidenex(2048, 8, 8192, 16, 4, 128, 64, 8, 128, 256),
     "l": _tidenex(4096, 6, 12288, 32, 8, 128, 64, 16, 128, 256),
 }
-DESIGN_SIZES = {"logozen": LOGOZEN_SIZES, "pugadra": PUGADRA_SIZES, "gevulorn": GEVULORN_SIZES, "galupel": GALUPEL_SIZES, "tidenex": TIDENEX_SIZES}
+def _kuterax(width, layers, heads, kv_heads, dim, window, m_heads, m_vdim, m_state, m_groups, r_heads, r_dim, r_vdim, experts, top, expert_ff, shared_ff, groups,
+             vocab=32768):
+    """A Kuterax of ``layers`` layers: windowed attention beside Mamba-2 on the even layers, retention on the odd ones, routed experts in
+    groups beside a gated shared one everywhere, no loop.  And a Gevulorn of the same width, depth, heads, head size, window, expert sizes
+    and vocabulary to set beside it: attention with a window on the even layers, gated linear attention of retention's sizes on the odd
+    ones, routed experts everywhere."""
+    moe = {"kind": "moe", "router": {"experts": experts, "top": top}, "expert": {"ff": expert_ff}, "shared": {"ff": shared_ff}}
+    grouped = dict(moe, router=dict(moe["router"], scale=1.5, groups={"count": groups[0], "keep": groups[1]}))
+    left = {"heads": heads, "kv_heads": kv_heads, "dim": dim, "vdim": dim, "scale": dim ** -0.5, "mask": {"size": window}, "rot": {
+        "base": 1000000.0, "dims": dim, "scaling": {"factor": 4.0, "original": 4096, "fast": 32.0, "slow": 1.0}}}
+    right = {"heads": m_heads, "vdim": m_vdim, "state": m_state, "groups": m_groups, "conv": 4, "norm_groups": m_groups}
+    retention = {"heads": r_heads, "dim": r_dim, "vdim": r_vdim, "decay": [1.0 - 2.0 ** (-5 - 3.0 * i / r_heads) for i in range(r_heads)]}
+    cfg = {"architecture": "Kuterax", "vocab": vocab, "width": width, "max_positions": 8192, "norm": {"eps": 1e-5},
+           "layers": [{"type": "retention", "mixer": retention, "mlp": grouped} if i % 2 else {"type": "parallel", "mixer": {"left": left, "right": right}, "mlp": grouped}
+                      for i in range(layers)]}
+    attention = {"heads": heads, "kv_heads": kv_heads, "dim": dim, "vdim": dim, "scale": dim ** -0.5, "rot": {"base": 10000.0, "dims": dim}, "mask": {"size": window}}
+    gla = {"heads": r_heads, "dim": r_dim, "vdim": r_vdim, "tau": 16.0, "decay_rank": 16}
+    twin = {"architecture": "Gevulorn", "vocab": vocab, "width": width, "norm": {"eps": 1e-5},
+            "layers": [{"type": "gla", "mixer": gla, "mlp": moe} if i % 2 else {"type": "attention", "mixer": attention, "mlp": moe} for i in range(layers)]}
+    return cfg, twin
+
+
+KUTERAX_SIZES = {   # width, layers, heads / kv heads / head size, window, Mamba-2's heads / value size / state / groups, retention's heads / key
+                    # size / value size, experts / chosen / expert ff / shared ff / (groups, kept)
+    "s": _kuterax(1024, 8, 16, 4, 64, 512, 32, 64, 64, 1, 8, 64, 128, 16, 2, 768, 768, (4, 2)),
+    "m": _kuterax(2048, 8, 16, 4, 128, 1024, 64, 64, 128, 1, 8, 128, 256, 32, 2, 2048, 2048, (4, 2)),
+    "l": _kuterax(4096, 6, 32, 8, 128, 1024, 128, 64, 128, 8, 16, 128, 256, 32, 4, 2048, 4096, (4, 2)),
+}
+DESIGN_SIZES = {"logozen": LOGOZEN_SIZES, "pugadra": PUGADRA_SIZES, "gevulorn": GEVULORN_SIZES, "galupel": GALUPEL_SIZES, "tidenex": TIDENEX_SIZES,
+                "kuterax": KUTERAX_SIZES}
 DESIGN_TWINS = {"logozen": "qwen3", "pugadra": "qwen3", "gevulorn": "pugadra", "galupel": "pugadra",
-                "tidenex": "gevulorn"}                                                                    # the model set beside each design
+                "tidenex": "gevulorn", "kuterax": "gevulorn"}                                                                    # the model set beside each design
 FALLBACK_PEAKS = {"hbm_gbs": 6650.0, "bf16_tflops": 1590.0, "bf16_tflops_sustained": 1400.0, "source": "fallback"}
 
 
@@ -216,8 +245,8 @@ def parse_args():
     p.add_argument("--steps", type=int, default=200)
     p.add_argument("--warmup", type=int, default=10)
     p.add_argument("--impl", choices=["ours", "reference"], default="ours")
-    p.add_argument("--mode", choices=["step", "offline", "mixed", "decode", "prefill", "logozen", "pugadra", "gevulorn", "galupel", "tidenex"], default="step")
-    p.add_argument("--sizes", default="s,m", help="logozen, pugadra, gevulorn, galupel and tidenex modes: which of the layer sizes " + ",".join(sorted(LOGOZEN_SIZES)))
+    p.add_argument("--mode", choices=["step", "offline", "mixed", "decode", "prefill", "logozen", "pugadra", "gevulorn", "galupel", "tidenex", "kuterax"], default="step")
+    p.add_argument("--sizes", default="s,m", help="logozen, pugadra, gevulorn, galupel, tidenex and kuterax modes: which of the layer sizes " + ",".join(sorted(LOGOZEN_SIZES)))
     p.add_argument("--shape", choices=sorted(SHAPES), default="0.6b", help="layer sizes, when no --model is given")
     p.add_argument("--extras", type=int, default=1,
                    help="step mode: also run the offline workload, the 8B mixed workload and the 32B decode points")
@@ -965,6 +994,40 @@ def _tidenex_roofline(cfg: dict, T: int, item: int, pk: dict, times: dict) -> di
     return _fractions(need, ("me_sink_attn", "me_attn_prefill_tcgen05", "me_gla_scan"), times, pk)
 
 
+def _kuterax_roofline(cfg: dict, T: int, item: int, pk: dict, times: dict) -> dict:
+    """What Kuterax's own kernels have to move or do in a prefill step of T tokens and the fraction of the measured peak that
+    their summed time makes: bytes for the element-wise kernels, multiply-adds for attention, recurrences and experts."""
+    W = cfg["width"]
+    need = {k: 0.0 for k in ("me_stream_norm", "me_attn_prep", "me_sink_attn", "me_attn_prefill_tcgen05", "me_conv_silu", "me_head_decay_scan",
+                             "me_gated_group_norm", "me_moe_gemm", "me_gemm_tcgen05_grouped", "me_moe_combine")}
+    pending = 0                                                            # outputs that the layer before left for this layer's norm
+    for layer in cfg["layers"]:
+        m, mlp = layer["mixer"], layer["mlp"]
+        need["me_stream_norm"] += T * W * (8 + (pending + 1) * item)       # stream in and out, the outputs in, h out
+        pending = (2 if layer["type"] == "parallel" else 1) + (mlp is not None)
+        if layer["type"] == "parallel":
+            a, r = m["left"], m["right"]
+            H, G, D, V = a["heads"], a["kv_heads"], a["dim"], a["vdim"]
+            need["me_attn_prep"] += T * (H * D + G * (D + V)) * (4 + item)
+            att = 2.0 * H * (D + V) * _window_pairs(T, a.get("mask", {}).get("size"))
+            need["me_sink_attn"] += att
+            need["me_attn_prefill_tcgen05"] += att
+            inner = r["heads"] * r["vdim"]
+            need["me_conv_silu"] += T * (inner + 2 * r["groups"] * r["state"]) * (4 + item)
+            need["me_head_decay_scan"] += 4.0 * inner * r["state"] * T     # k v^T into the state and the state times q, for every token
+            need["me_gated_group_norm"] += T * inner * (4 + 4 + item)
+        else:
+            inner = m["heads"] * m["vdim"]
+            need["me_head_decay_scan"] += 4.0 * inner * m["dim"] * T
+            need["me_gated_group_norm"] += T * inner * (4 + 2 * item)
+        if mlp is not None:
+            flops = 4.0 * T * mlp["router"]["top"] * mlp["expert"]["ff"] * W
+            need["me_moe_gemm"] += flops
+            need["me_gemm_tcgen05_grouped"] += flops
+            need["me_moe_combine"] += T * W * (4 * mlp["router"]["top"] + 2 * item)
+    return _fractions(need, ("me_sink_attn", "me_attn_prefill_tcgen05", "me_head_decay_scan", "me_moe_gemm", "me_gemm_tcgen05_grouped"), times, pk)
+
+
 def _qwen3_roofline(cfg: dict, T: int, item: int, pk: dict, times: dict) -> dict:
     """The like kernels of the Qwen3 beside a design: its norm, its q/k preparation and its prompt attention."""
     W, L = cfg["hidden_size"], cfg["num_hidden_layers"]
@@ -988,7 +1051,7 @@ def run_design_mode(args, design: str) -> int:
     import torch
     sizes_of = DESIGN_SIZES[design]
     rooflines = {"logozen": _logozen_roofline, "pugadra": _pugadra_roofline, "gevulorn": _gevulorn_roofline, "galupel": _galupel_roofline,
-                 "tidenex": _tidenex_roofline, "qwen3": _qwen3_roofline}
+                 "tidenex": _tidenex_roofline, "kuterax": _kuterax_roofline, "qwen3": _qwen3_roofline}
     twin_label = DESIGN_TWINS[design]
     pk = peaks()
     item = 2 if args.dtype in ("bfloat16", "bf16") else 4

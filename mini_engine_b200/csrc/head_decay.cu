@@ -5,7 +5,7 @@
 //   o_t = S_t^T q_t + skip * v_t                    (V; ``skip``: a number a head, or none)
 // q and k may be shared by groups of neighbouring heads (G groups; head h uses group h / (H / G)).  Two sources of a and g:
 //   ``dt`` (the state-space form): g_t = softplus(dt_t + bias), a_t = exp(-exp(a_log) g_t), a column of ``dt`` a head;
-//   ``log2_decay`` (a constant a head): a = 2^log2_decay, and g_t = k_scale for every token.
+//   ``decay`` (a constant a head, with its logarithm ``log2_decay`` in double precision): a = decay, and g_t = k_scale for every token.
 // S starts at zero and is float32, as are a, g, their logarithms and all sums; q, k and v are float32 or bfloat16.
 //
 //   hd_step_kernel         walks a request's tokens one by one, its state in registers: single tokens of a decode step
@@ -18,7 +18,7 @@
 #include "common.cuh"
 
 constexpr int HD_LC = 64, HD_VT = 64;
-constexpr float HD_LOG2E = 1.4426950408889634f;
+constexpr double HD_LOG2E = 1.4426950408889634074;
 
 struct HdArgs {
   const void *q, *k, *v;
@@ -27,21 +27,39 @@ struct HdArgs {
   float k_scale;
   const float* dt;            // null: the constant form
   int64_t ld_dt;
-  const float *dt_bias, *a_log, *log2_decay, *skip;
+  const float *dt_bias, *a_log, *decay;
+  const double* log2_decay;
+  const float* skip;
   float* S;
   const int *cu, *ctx, *slots;
   float* o;
 };
 
-// The factor g and log2 of the decay of token row t, head h.
-__device__ __forceinline__ void hd_token(const HdArgs& a, int64_t t, int h, float& gain, float& log2_a) {
+// The factor g of token row t, head h, and the natural logarithm of its decay (the state-space form).
+__device__ __forceinline__ void hd_step_size(const HdArgs& a, int64_t t, int h, float& gain, float& log_a) {
+  const float z = a.dt[t * a.ld_dt + h] + a.dt_bias[h];
+  gain = fmaxf(z, 0.f) + log1pf(expf(-fabsf(z)));
+  log_a = -expf(a.a_log[h]) * gain;
+}
+// The factor g and log2 of the decay; the factor g and the decay itself.
+__device__ __forceinline__ void hd_token_log2(const HdArgs& a, int64_t t, int h, float& gain, double& log2_a) {
+  gain = a.k_scale;
   if (a.dt) {
-    const float z = a.dt[t * a.ld_dt + h] + a.dt_bias[h];
-    gain = fmaxf(z, 0.f) + log1pf(expf(-fabsf(z)));
-    log2_a = -expf(a.a_log[h]) * gain * HD_LOG2E;
+    float log_a;
+    hd_step_size(a, t, h, gain, log_a);
+    log2_a = (double)log_a * HD_LOG2E;
   } else {
-    gain = a.k_scale;
     log2_a = a.log2_decay[h];
+  }
+}
+__device__ __forceinline__ void hd_token(const HdArgs& a, int64_t t, int h, float& gain, float& decay) {
+  gain = a.k_scale;
+  if (a.dt) {
+    float log_a;
+    hd_step_size(a, t, h, gain, log_a);
+    decay = expf(log_a);
+  } else {
+    decay = a.decay[h];
   }
 }
 
@@ -95,9 +113,8 @@ __global__ void __launch_bounds__(256) hd_step_kernel(HdArgs a) {
   const float skip = a.skip ? a.skip[h] : 0.f;
   for (int i = 0; i < n_tok; ++i) {
     const int64_t t = tok0 + i;
-    float gain, log2_a;
-    hd_token(a, t, h, gain, log2_a);
-    const float decay = exp2f(log2_a);
+    float gain, decay;
+    hd_token(a, t, h, gain, decay);
     const T *qr = reinterpret_cast<const T*>(a.q) + t * a.ldq + (int64_t)g * D, *kr = reinterpret_cast<const T*>(a.k) + t * a.ldk + (int64_t)g * D;
     if (i) __syncthreads();                     // the token before is done with q_s, k_s, parts
     for (int d = tid; d < D; d += 256) {
@@ -148,10 +165,11 @@ __global__ void __launch_bounds__(256) hd_step_kernel(HdArgs a) {
 __device__ __forceinline__ void hd_run_scalars(const HdArgs& a, int tok0, int L, int h, float* g_s, double* b_s) {
   if (threadIdx.x >= 32) return;
   const int lane = threadIdx.x, t0 = 2 * lane, t1 = t0 + 1;
-  float g0 = 0.f, g1 = 0.f, l0 = 0.f, l1 = 0.f;
-  if (t0 < L) hd_token(a, tok0 + t0, h, g0, l0);
-  if (t1 < L) hd_token(a, tok0 + t1, h, g1, l1);
-  const double pair = (double)l0 + (double)l1;
+  float g0 = 0.f, g1 = 0.f;
+  double l0 = 0.0, l1 = 0.0;
+  if (t0 < L) hd_token_log2(a, tok0 + t0, h, g0, l0);
+  if (t1 < L) hd_token_log2(a, tok0 + t1, h, g1, l1);
+  const double pair = l0 + l1;
   double run = pair;
 #pragma unroll
   for (int o = 1; o < 32; o <<= 1) {
@@ -160,7 +178,7 @@ __device__ __forceinline__ void hd_run_scalars(const HdArgs& a, int tok0, int L,
   }
   g_s[t0] = g0;
   g_s[t1] = g1;
-  b_s[t0] = run - pair + (double)l0;
+  b_s[t0] = run - pair + l0;
   b_s[t1] = run;
 }
 
@@ -400,20 +418,20 @@ static int hd_raise_smem(K kernel, size_t smem, const char* what) {
 ME_API int me_head_decay_chunk_len() { return HD_LC; }
 
 // q, k: rows of ``dtype`` holding the G groups' D values, ldq / ldk elements apart; v: rows of H heads' V values.  dt: float32 rows of H
-// pre-activations with dt_bias, a_log [H], or null with log2_decay [H].  skip: [H] or null.  S: [slots, H, D, V] float32; o: [T, H*V]
+// pre-activations with dt_bias, a_log [H], or null with decay [H] and log2_decay [H] (float64).  skip: [H] or null.  S: [slots, H, D, V] float32; o: [T, H*V]
 // float32.  Requests [0, num_decodes) are walked token by token.  The others too, unless ``tiles`` ([n_tiles, 2] int32: request and first
 // token of every run of HD_LC tokens of the requests from num_decodes on, a request's runs in order and side by side),
 // ``states_ws`` ([n_tiles, H, D, V] float32) and ``totals_ws`` ([n_tiles, H] float32) are given and D is at most 256.
 ME_API int me_head_decay_scan(const void* q, const void* k, const void* v, int dtype, int64_t ldq, int64_t ldk, int64_t ldv, int H, int G, int D,
                               int V, float k_scale, const float* dt, int64_t ld_dt, const float* dt_bias, const float* a_log,
-                              const float* log2_decay, const float* skip, float* S, const int* cu_seqlens, const int* context_lens,
+                              const float* decay, const double* log2_decay, const float* skip, float* S, const int* cu_seqlens, const int* context_lens,
                               const int* state_slots, float* o, int B, int num_decodes, const int* tiles, int n_tiles, float* states_ws,
                               float* totals_ws, cudaStream_t stream) {
   if (B == 0) return 0;
   ME_REQUIRE(B > 0 && H > 0 && G > 0 && H % G == 0 && D > 0 && V > 0 && H <= 65535 && D <= 1024, "me_head_decay_scan: bad sizes B=%d H=%d G=%d D=%d V=%d", B, H, G, D, V);
   ME_REQUIRE(num_decodes >= 0 && num_decodes <= B, "me_head_decay_scan: %d single-token requests of %d", num_decodes, B);
-  ME_REQUIRE(dt ? (dt_bias && a_log) : (log2_decay != nullptr), "me_head_decay_scan: decays from dt (with its bias and a_log) or constants");
-  const HdArgs a = {q, k, v, ldq, ldk, ldv, H, G, D, V, k_scale, dt, ld_dt, dt_bias, a_log, log2_decay, skip, S, cu_seqlens, context_lens, state_slots, o};
+  ME_REQUIRE(dt ? (dt_bias && a_log) : (decay && log2_decay), "me_head_decay_scan: decays from dt (with its bias and a_log) or constants");
+  const HdArgs a = {q, k, v, ldq, ldk, ldv, H, G, D, V, k_scale, dt, ld_dt, dt_bias, a_log, decay, log2_decay, skip, S, cu_seqlens, context_lens, state_slots, o};
   auto off = [](const void* p, size_t to) { return ((uintptr_t)p % to) != 0; };
   const size_t al = dtype == ME_F32 ? 16 : 8;
   const bool out4 = V % 4 == 0 && ldv % 4 == 0 && !off(v, al) && !off(S, 16) && !off(o, 16);

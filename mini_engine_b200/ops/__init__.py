@@ -64,7 +64,7 @@ _PROTOS = {
     "me_gla_scan": [_P, _L, _I, _I, _I, _P, _P, _P, _P, _P, _P, _I, _I, _I, _I, _F, _P, _I, _I, _P, _P, _P, _P, _P],
     "me_stream_norm": [_P, _P, _P, _P, _I, _P, _P, _P, _F, _F, _F, _P, _P, _P, _F, _P, _I, _L, _P, _I, _I, _P],
     "me_conv_silu": [_P, _L, _P, _P, _P, _P, _I, _I, _P, _P, _P, _P, _I, _I, _I, _I, _P],
-    "me_head_decay_scan": [_P, _P, _P, _I, _L, _L, _L, _I, _I, _I, _I, _F, _P, _L, _P, _P, _P, _P, _P, _P, _P, _P, _P, _I, _I, _P, _I, _P, _P, _P],
+    "me_head_decay_scan": [_P, _P, _P, _I, _L, _L, _L, _I, _I, _I, _I, _F, _P, _L, _P, _P, _P, _P, _P, _P, _P, _P, _P, _P, _I, _I, _P, _I, _P, _P, _P],
     "me_gated_group_norm": [_P, _L, _P, _I, _L, _P, _I, _F, _P, _I, _L, _I, _I, _I, _P],
     "me_activation": [_P, _I, _L, _P, _I, _L, _I, _I, _I, _P],
     "me_soft_cap": [_P, _L, _F, _F, _P],
@@ -1490,14 +1490,14 @@ def head_decay_chunk_count(meta) -> int:
 
 def head_decay_scan(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, S: torch.Tensor, meta, state_slots: torch.Tensor, o: torch.Tensor,
                     num_heads: int, num_groups: int, dim: int, vdim: int, *, k_scale: float = 1.0, dt: Optional[tuple] = None,
-                    log2_decay: Optional[torch.Tensor] = None, skip: Optional[torch.Tensor] = None, chunk_states: Optional[torch.Tensor] = None,
+                    decay: Optional[tuple] = None, skip: Optional[torch.Tensor] = None, chunk_states: Optional[torch.Tensor] = None,
                     totals: Optional[torch.Tensor] = None) -> None:
     """Walks every request's tokens of this step through S_t = a_t S_(t-1) + g_t k_t v_t^T, o_t = S_t^T q_t + skip v_t from the state in
     its slot, per head, with one decay a and one factor g a head and token (see csrc/head_decay.cu).  ``q``, ``k`` [T, groups * dim]
     and ``v`` [T, heads * vdim]: columns of rows of one dtype; head h reads group h // (heads / groups) of q and k.
 
     ``dt`` = (pre-activations [T, heads] float32 (columns of wider rows), bias [heads], a_log [heads]): g = softplus(dt + bias), a =
-    exp(-exp(a_log) g).  Or ``log2_decay`` float32 [heads]: a = 2^log2_decay, g = ``k_scale``.  With the float32 workspaces ``chunk_states``
+    exp(-exp(a_log) g).  Or ``decay`` = (decays float32 [heads], their log2 float64 [heads]): constants, and g = ``k_scale``.  With the float32 workspaces ``chunk_states``
     (heads * dim * vdim values a run of HEAD_DECAY_CHUNK tokens: ``head_decay_chunk_count``) and ``totals`` (heads values a run) the
     requests that bring several tokens take a run at a time, all runs of the step side by side."""
     T = o.shape[0]
@@ -1506,9 +1506,11 @@ def head_decay_scan(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, S: torch.
     _need(tuple(q.shape) == tuple(k.shape) == (T, num_groups * dim) and tuple(v.shape) == (T, num_heads * vdim), "head_decay_scan: shapes of q, k, v")
     _need(S.dtype == torch.float32 and S.is_contiguous() and tuple(S.shape[1:]) == (num_heads, dim, vdim), "head_decay_scan: state shape")
     _need(o.dtype == torch.float32 and o.is_contiguous() and tuple(o.shape) == (T, num_heads * vdim), "head_decay_scan: output shape")
-    _need((dt is None) != (log2_decay is None), "head_decay_scan: decays from dt or constants")
-    per_head = [t for t in ((*dt[1:],) if dt is not None else (log2_decay,)) + ((skip,) if skip is not None else ())]
+    _need((dt is None) != (decay is None), "head_decay_scan: decays from dt or constants")
+    per_head = [t for t in ((*dt[1:],) if dt is not None else (decay[0],)) + ((skip,) if skip is not None else ())]
     _need(all(t.dtype == torch.float32 and t.is_contiguous() and t.numel() == num_heads for t in per_head), "head_decay_scan: float32 numbers a head")
+    _need(decay is None or (decay[1].dtype == torch.float64 and decay[1].is_contiguous() and decay[1].numel() == num_heads),
+          "head_decay_scan: log2 of the decays is float64 [heads]")
     _need(dt is None or (dt[0].dtype == torch.float32 and dt[0].stride(1) == 1 and tuple(dt[0].shape) == (T, num_heads)), "head_decay_scan: dt is float32 [T, heads]")
     tiles, n_tiles = meta.tile_lists[HEAD_DECAY_CHUNK]
     chunked = head_decay_chunks and chunk_states is not None and totals is not None and n_tiles > 0 and dim <= 256
@@ -1517,7 +1519,7 @@ def head_decay_scan(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, S: torch.
               and chunk_states.numel() >= n_tiles * num_heads * dim * vdim and totals.numel() >= n_tiles * num_heads, "head_decay_scan: workspaces")
     _call("me_head_decay_scan", q.data_ptr(), k.data_ptr(), v.data_ptr(), _dt(q), q.stride(0), k.stride(0), v.stride(0), num_heads, num_groups,
           dim, vdim, float(k_scale), _ptr(dt[0]) if dt else 0, dt[0].stride(0) if dt else 0, _ptr(dt[1]) if dt else 0, _ptr(dt[2]) if dt else 0,
-          _ptr(log2_decay), _ptr(skip), S.data_ptr(), meta.cu_seqlens.data_ptr(), meta.context_lens.data_ptr(), state_slots.data_ptr(),
+          _ptr(decay[0]) if decay else 0, _ptr(decay[1]) if decay else 0, _ptr(skip), S.data_ptr(), meta.cu_seqlens.data_ptr(), meta.context_lens.data_ptr(), state_slots.data_ptr(),
           o.data_ptr(), meta.num_reqs, meta.num_decodes, tiles.data_ptr() if chunked else 0, n_tiles if chunked else 0,
           chunk_states.data_ptr() if chunked else 0, totals.data_ptr() if chunked else 0, _stream())
     global launches

@@ -42,13 +42,14 @@ class Retention(Mixer):
         H = num_heads
         self.in_proj = Linear(hidden_size, [("q", H * dim), ("k", H * dim), ("v", H * vdim), ("g", H * vdim)], name="in_proj")
         self.o_proj = Linear(H * vdim, [("o", hidden_size)], name="o")
-        self._log2_decay = None
+        self._decay = None
 
     def sub_parts(self):
         return [("", self.in_proj), ("", self.o_proj)]
 
     def finalize(self, dtype, device):
-        self._log2_decay = torch.tensor([math.log2(d) for d in self.decay], dtype=torch.float32).to(device)
+        self._decay = (torch.tensor(self.decay, dtype=torch.float32).to(device),
+                       torch.tensor([math.log2(d) for d in self.decay], dtype=torch.float64).to(device))
 
     def cache_needs(self):
         return [StateNeed((self.num_heads, self.dim, self.vdim), "float32", "S")]
@@ -63,7 +64,7 @@ class Retention(Mixer):
         q, k, v, g = proj.split([H * D, H * D, H * V, H * V], dim=1)
         o = ctx.buffer("head_decay_o", (T, H * V), torch.float32)
         ops.head_decay_scan(q, k, v, ctx.state(call.cache_slot, "S"), ctx.attn_meta, ctx.state_slots, o, H, H, D, V, k_scale=D ** -0.5,
-                            log2_decay=self._log2_decay, **_workspaces(ctx, H, D, V))
+                            decay=self._decay, **_workspaces(ctx, H, D, V))
         gated = ctx.buffer("retention_gated", (T, H * V), ctx.act_dtype)
         ops.gated_group_norm(o, g, None, H, self.norm_eps, gated, gate_first=False)
         return self.o_proj.forward(gated, ctx, "mixer_out")
