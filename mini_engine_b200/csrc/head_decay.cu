@@ -14,54 +14,9 @@
 //   hd_state_walk_kernel   per request, in order: states[c] <- the state in front of run c; S <- 2^(B_L) S + U_c
 //   hd_chunk_out_kernel    o_t = 2^(B_t) q_t^T S_in + sum_{s<=t} (q_t . k_s) g_s 2^(B_t - B_s) v_s + skip v_t
 // Every exponent is <= 0.  B is summed and its differences are taken in double precision (64 numbers a run and head), so a decay
-// close to 1 behind strong ones keeps its digits.  The results differ from the token-by-token kernel by the order of sums only.
-#include "common.cuh"
-
-constexpr int HD_LC = 64, HD_VT = 64;
-constexpr double HD_LOG2E = 1.4426950408889634074;
-
-struct HdArgs {
-  const void *q, *k, *v;
-  int64_t ldq, ldk, ldv;
-  int H, G, D, V;
-  float k_scale;
-  const float* dt;            // null: the constant form
-  int64_t ld_dt;
-  const float *dt_bias, *a_log, *decay;
-  const double* log2_decay;
-  const float* skip;
-  float* S;
-  const int *cu, *ctx, *slots;
-  float* o;
-};
-
-// The factor g of token row t, head h, and the natural logarithm of its decay (the state-space form).
-__device__ __forceinline__ void hd_step_size(const HdArgs& a, int64_t t, int h, float& gain, float& log_a) {
-  const float z = a.dt[t * a.ld_dt + h] + a.dt_bias[h];
-  gain = fmaxf(z, 0.f) + log1pf(expf(-fabsf(z)));
-  log_a = -expf(a.a_log[h]) * gain;
-}
-// The factor g and log2 of the decay; the factor g and the decay itself.
-__device__ __forceinline__ void hd_token_log2(const HdArgs& a, int64_t t, int h, float& gain, double& log2_a) {
-  gain = a.k_scale;
-  if (a.dt) {
-    float log_a;
-    hd_step_size(a, t, h, gain, log_a);
-    log2_a = (double)log_a * HD_LOG2E;
-  } else {
-    log2_a = a.log2_decay[h];
-  }
-}
-__device__ __forceinline__ void hd_token(const HdArgs& a, int64_t t, int h, float& gain, float& decay) {
-  gain = a.k_scale;
-  if (a.dt) {
-    float log_a;
-    hd_step_size(a, t, h, gain, log_a);
-    decay = expf(log_a);
-  } else {
-    decay = a.decay[h];
-  }
-}
+// close to 1 behind strong ones keeps its digits.  The first and the last of these three are those of head_decay_mma.cu where bfloat16
+// operands and their sizes allow.  The results differ from the token-by-token kernel by the order of sums only.
+#include "head_decay.cuh"
 
 template <int N> struct HdVec;
 template <> struct HdVec<4> {
@@ -160,28 +115,6 @@ __global__ void __launch_bounds__(256) hd_step_kernel(HdArgs a) {
 }
 
 // ---- runs of HD_LC tokens -------------------------------------------------------------------------------------
-// The run's factors g and inclusive sums B (double) into shared memory, zero factors and no further decay beyond its L tokens; the
-// first warp's work.
-__device__ __forceinline__ void hd_run_scalars(const HdArgs& a, int tok0, int L, int h, float* g_s, double* b_s) {
-  if (threadIdx.x >= 32) return;
-  const int lane = threadIdx.x, t0 = 2 * lane, t1 = t0 + 1;
-  float g0 = 0.f, g1 = 0.f;
-  double l0 = 0.0, l1 = 0.0;
-  if (t0 < L) hd_token_log2(a, tok0 + t0, h, g0, l0);
-  if (t1 < L) hd_token_log2(a, tok0 + t1, h, g1, l1);
-  const double pair = l0 + l1;
-  double run = pair;
-#pragma unroll
-  for (int o = 1; o < 32; o <<= 1) {
-    const double up = __shfl_up_sync(0xffffffffu, run, o);
-    if (lane >= o) run += up;
-  }
-  g_s[t0] = g0;
-  g_s[t1] = g1;
-  b_s[t0] = run - pair + l0;
-  b_s[t1] = run;
-}
-
 // rows x cols values of a matrix in global memory into shared memory as float32, zeros beyond n_rows and n_cols.
 template <typename T, int VEC>
 __device__ __forceinline__ void hd_fill(float* dst, int ld_dst, int rows, int cols, const T* src, int64_t ld_src, int n_rows, int n_cols) {
@@ -406,6 +339,10 @@ hd_chunk_out_kernel(HdArgs a, const int* __restrict__ tiles, const float* __rest
   }
 }
 
+int me_head_decay_mma_states(const HdArgs& a, const int* tiles, int n_tiles, float* states, float* totals, cudaStream_t stream);
+int me_head_decay_mma_out(const HdArgs& a, const int* tiles, int n_tiles, const float* states, cudaStream_t stream);
+bool me_head_decay_mma_takes(const HdArgs& a, int dtype);
+
 template <typename K>
 static int hd_raise_smem(K kernel, size_t smem, const char* what) {
   if (smem > 40 * 1024) {
@@ -421,12 +358,13 @@ ME_API int me_head_decay_chunk_len() { return HD_LC; }
 // pre-activations with dt_bias, a_log [H], or null with decay [H] and log2_decay [H] (float64).  skip: [H] or null.  S: [slots, H, D, V] float32; o: [T, H*V]
 // float32.  Requests [0, num_decodes) are walked token by token.  The others too, unless ``tiles`` ([n_tiles, 2] int32: request and first
 // token of every run of HD_LC tokens of the requests from num_decodes on, a request's runs in order and side by side),
-// ``states_ws`` ([n_tiles, H, D, V] float32) and ``totals_ws`` ([n_tiles, H] float32) are given and D is at most 256.
+// ``states_ws`` ([n_tiles, H, D, V] float32) and ``totals_ws`` ([n_tiles, H] float32) are given and D is at most 256.  allow_mma: the
+// products of prompts may run on the tensor cores.
 ME_API int me_head_decay_scan(const void* q, const void* k, const void* v, int dtype, int64_t ldq, int64_t ldk, int64_t ldv, int H, int G, int D,
                               int V, float k_scale, const float* dt, int64_t ld_dt, const float* dt_bias, const float* a_log,
                               const float* decay, const double* log2_decay, const float* skip, float* S, const int* cu_seqlens, const int* context_lens,
                               const int* state_slots, float* o, int B, int num_decodes, const int* tiles, int n_tiles, float* states_ws,
-                              float* totals_ws, cudaStream_t stream) {
+                              float* totals_ws, int allow_mma, cudaStream_t stream) {
   if (B == 0) return 0;
   ME_REQUIRE(B > 0 && H > 0 && G > 0 && H % G == 0 && D > 0 && V > 0 && H <= 65535 && D <= 1024, "me_head_decay_scan: bad sizes B=%d H=%d G=%d D=%d V=%d", B, H, G, D, V);
   ME_REQUIRE(num_decodes >= 0 && num_decodes <= B, "me_head_decay_scan: %d single-token requests of %d", num_decodes, B);
@@ -463,7 +401,10 @@ ME_API int me_head_decay_scan(const void* q, const void* k, const void* v, int d
     if (hd_raise_smem(KERNEL_<T, VEC_>, SMEM_, "me_head_decay_scan")) return 1;                                       \
     me_launch(KERNEL_<T, VEC_>, dim3(n_tiles, H, (unsigned)v_tiles), dim3(256), SMEM_, stream, a, tiles, __VA_ARGS__); \
   } while (0)
-    ME_DISPATCH_DTYPE(dtype, T, {
+    const bool mma = allow_mma && me_head_decay_mma_takes(a, dtype) && !off(states_ws, 16);
+    if (mma) {
+      if (me_head_decay_mma_states(a, tiles, n_tiles, states_ws, totals_ws, stream)) return 1;
+    } else ME_DISPATCH_DTYPE(dtype, T, {
       if (vec) HD_CHUNK(hd_chunk_state_kernel, 4, smem_state, states_ws, totals_ws);
       else HD_CHUNK(hd_chunk_state_kernel, 1, smem_state, states_ws, totals_ws);
     });
@@ -474,7 +415,9 @@ ME_API int me_head_decay_scan(const void* q, const void* k, const void* v, int d
     if (walk4) me_launch(hd_state_walk_kernel<4>, walk_grid, dim3(256), 0, stream, a, (const float*)totals_ws, states_ws, tiles, n_tiles, num_decodes);
     else me_launch(hd_state_walk_kernel<1>, walk_grid, dim3(256), 0, stream, a, (const float*)totals_ws, states_ws, tiles, n_tiles, num_decodes);
     ME_LAUNCH_CHECK("me_head_decay_scan (state walk)");
-    ME_DISPATCH_DTYPE(dtype, T, {
+    if (mma) {
+      if (me_head_decay_mma_out(a, tiles, n_tiles, states_ws, stream)) return 1;
+    } else ME_DISPATCH_DTYPE(dtype, T, {
       if (vec) HD_CHUNK(hd_chunk_out_kernel, 4, smem_out, (const float*)states_ws);
       else HD_CHUNK(hd_chunk_out_kernel, 1, smem_out, (const float*)states_ws);
     });

@@ -1,0 +1,277 @@
+// The prompt kernels of head_decay.cu on the tensor cores (mma.sync m16n8k16, bfloat16 in, float32 accumulate), for bfloat16 q, k and v.
+//
+// q, k and v enter the products as they are.  What is float32 (the state, the weighted scores, the weighted values) enters as the
+// sum of three bfloat16 numbers, x = hi + mid + lo, each the rounding of what the ones before left: 24 digits, float32's own.  A
+// product of such a factor with a bfloat16 one is three products added in float32, so the results are those of float32 products
+// up to the order of sums.
+//
+//   hd_mma_state_kernel   U = k^T (g_s 2^(B_L - B_s) v_s) of a run: 64 tokens x 64 columns a block, a warp a strip of 16 rows by 32 columns
+//   hd_mma_out_kernel     a warp takes 16 tokens of the run: q S_in (three parts), scaled by 2^(B_t); then, 16 keys at a time up to the
+//                         diagonal, the scores q k^T, their weights in the registers, and the product with v (three parts)
+#include "head_decay.cuh"
+#include "mma_prims.cuh"
+
+namespace {
+
+using namespace mma_prims;
+
+constexpr int HM_LDV = HD_VT + 8;             // bfloat16 elements of a row of 64 columns in shared memory (an odd number of 16-byte pieces)
+
+__device__ __forceinline__ void split3(float x, bf16& hi, bf16& mid, bf16& lo) {
+  hi = __float2bfloat16_rn(x);
+  const float r = x - __bfloat162float(hi);
+  mid = __float2bfloat16_rn(r);
+  lo = __float2bfloat16_rn(r - __bfloat162float(mid));
+}
+__device__ __forceinline__ uint32_t pack2(bf16 a, bf16 b) {
+  const __nv_bfloat162 v = __halves2bfloat162(a, b);
+  return *reinterpret_cast<const uint32_t*>(&v);
+}
+// Two floats as a pair of bfloat16 in each of the three parts.
+__device__ __forceinline__ void split3_pair(float x, float y, uint32_t (&p)[3]) {
+  bf16 a[3], b[3];
+  split3(x, a[0], a[1], a[2]);
+  split3(y, b[0], b[1], b[2]);
+#pragma unroll
+  for (int i = 0; i < 3; ++i) p[i] = pack2(a[i], b[i]);
+}
+
+// rows x cols (a multiple of 8) bfloat16 values into shared memory by asynchronous copies, zeros beyond n_rows and n_cols.
+template <int THREADS>
+__device__ __forceinline__ void hm_fill(bf16* dst, int ld_dst, int rows, int cols, const bf16* src, int64_t ld_src, int n_rows, int n_cols) {
+  const int per = cols / 8;
+  for (int i = threadIdx.x; i < rows * per; i += THREADS) {
+    const int r = i / per, c = (i - r * per) * 8;
+    const bool ok = r < n_rows && c < n_cols;
+    cp_async16(dst + r * ld_dst + c, ok ? src + (int64_t)r * ld_src + c : src, ok);
+  }
+}
+
+// One block = one run x one head x HD_VT columns of U; totals[c, h] = B of the run's last token.
+__global__ void __launch_bounds__(256)
+hd_mma_state_kernel(HdArgs a, const int* __restrict__ tiles, float* __restrict__ states, float* __restrict__ totals) {
+  extern __shared__ __align__(16) unsigned char hm_smem[];
+  __shared__ float g_s[HD_LC];
+  __shared__ double b_s[HD_LC];
+  constexpr int LC = HD_LC, VT = HD_VT, LDV = HM_LDV;
+  const int D = a.D, V = a.V, D16 = (D + 15) / 16 * 16, ldk = D16 + 8;
+  bf16* Ks = reinterpret_cast<bf16*>(hm_smem);  // [LC][ldk]
+  bf16* Ws = Ks + LC * ldk;                     // [3][LC][LDV]: g_s 2^(B_L - B_s) v_s in three parts
+  const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, h = blockIdx.y, v0 = blockIdx.z * VT;
+  const int b = tiles[2 * blockIdx.x], q0 = tiles[2 * blockIdx.x + 1];
+  const int tok0 = a.cu[b] + q0, L = min(LC, a.cu[b + 1] - tok0);
+  pdl_wait();
+  pdl_launch_dependents();
+  if (L <= 0) return;
+  const int g = h / (a.H / a.G);
+  hm_fill<256>(Ks, ldk, LC, D16, reinterpret_cast<const bf16*>(a.k) + (int64_t)tok0 * a.ldk + (int64_t)g * D, a.ldk, L, D);
+  cp_async_commit();
+  // this thread's 16 values (two rows' pieces of eight columns), on their way while the first warp sums the decays
+  const bf16* vsrc = reinterpret_cast<const bf16*>(a.v) + (int64_t)tok0 * a.ldv + (int64_t)h * V + v0;
+  uint4 raw[2];
+#pragma unroll
+  for (int i = 0; i < 2; ++i) {
+    const int r = tid / 8 + 32 * i, c = tid % 8 * 8;
+    raw[i] = r < L && v0 + c < V ? *reinterpret_cast<const uint4*>(vsrc + (int64_t)r * a.ldv + c) : make_uint4(0, 0, 0, 0);
+  }
+  hd_run_scalars(a, tok0, L, h, g_s, b_s);
+  __syncthreads();
+  const double bl = b_s[LC - 1];
+  if (tid == 0 && blockIdx.z == 0) totals[(int64_t)blockIdx.x * a.H + h] = (float)bl;
+#pragma unroll
+  for (int i = 0; i < 2; ++i) {
+    const int r = tid / 8 + 32 * i, c = tid % 8 * 8;
+    const float f = g_s[r] * exp2f((float)(bl - b_s[r]));
+    const __nv_bfloat162* x = reinterpret_cast<const __nv_bfloat162*>(&raw[i]);
+    uint32_t p[4][3];
+#pragma unroll
+    for (int j = 0; j < 4; ++j) split3_pair(__low2float(x[j]) * f, __high2float(x[j]) * f, p[j]);
+#pragma unroll
+    for (int k = 0; k < 3; ++k) *reinterpret_cast<uint4*>(Ws + (k * LC + r) * LDV + c) = make_uint4(p[0][k], p[1][k], p[2][k], p[3][k]);
+  }
+  cp_async_wait<0>();
+  __syncthreads();
+  const int mr = lane & 7, mj = lane >> 3;
+  float* out = states + ((int64_t)blockIdx.x * a.H + h) * D * V;
+  for (int u = warp; u < D16 / 8; u += 8) {     // strips of 16 rows (key channels) x 32 columns
+    const int d0 = u / 2 * 16, c0 = u % 2 * 32;
+    if (v0 + c0 >= V) continue;
+    float acc[4][4] = {};
+#pragma unroll
+    for (int ks = 0; ks < LC / 16; ++ks) {
+      if (16 * ks >= L) break;                  // (zeros from here on)
+      uint32_t ka[4];
+      ldmatrix_x4_trans(ka, Ks + (16 * ks + mr + (mj >= 2 ? 8 : 0)) * ldk + d0 + (mj & 1 ? 8 : 0));
+#pragma unroll
+      for (int p = 0; p < 3; ++p)
+#pragma unroll
+        for (int n = 0; n < 2; ++n) {
+          uint32_t vb[4];
+          ldmatrix_x4_trans(vb, Ws + (p * LC + 16 * ks + mr + (mj & 1 ? 8 : 0)) * LDV + c0 + 16 * n + (mj >= 2 ? 8 : 0));
+          mma_bf16(acc[2 * n], ka, vb[0], vb[1]);
+          mma_bf16(acc[2 * n + 1], ka, vb[2], vb[3]);
+        }
+    }
+#pragma unroll
+    for (int n = 0; n < 4; ++n) {
+      const int c = v0 + c0 + 8 * n + 2 * (lane & 3), d = d0 + (lane >> 2);
+      if (c >= V) continue;
+      if (d < D) *reinterpret_cast<float2*>(out + (int64_t)d * V + c) = make_float2(acc[n][0], acc[n][1]);
+      if (d + 8 < D) *reinterpret_cast<float2*>(out + (int64_t)(d + 8) * V + c) = make_float2(acc[n][2], acc[n][3]);
+    }
+  }
+}
+
+// One block = one run x one head x HD_VT columns; states[c] holds the state in front of the run.
+__global__ void __launch_bounds__(128)
+hd_mma_out_kernel(HdArgs a, const int* __restrict__ tiles, const float* __restrict__ states) {
+  extern __shared__ __align__(16) unsigned char hm_smem[];
+  __shared__ float g_s[HD_LC];
+  __shared__ double b_s[HD_LC];
+  constexpr int LC = HD_LC, VT = HD_VT, LDV = HM_LDV;
+  const int D = a.D, V = a.V, D16 = (D + 15) / 16 * 16, ldk = D16 + 8;
+  bf16* Qs = reinterpret_cast<bf16*>(hm_smem);  // [LC][ldk]
+  bf16* Ks = Qs + LC * ldk;                     // [LC][ldk]
+  bf16* Vs = Ks + LC * ldk;                     // [LC][LDV]
+  bf16* Ss = Vs + LC * LDV;                     // [3][D16][LDV]: the state in three parts
+  const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, h = blockIdx.y, v0 = blockIdx.z * VT;
+  const int b = tiles[2 * blockIdx.x], q0 = tiles[2 * blockIdx.x + 1];
+  const int tok0 = a.cu[b] + q0, L = min(LC, a.cu[b + 1] - tok0);
+  pdl_wait();
+  pdl_launch_dependents();
+  if (L <= 0) return;
+  const int g = h / (a.H / a.G);
+  hm_fill<128>(Qs, ldk, LC, D16, reinterpret_cast<const bf16*>(a.q) + (int64_t)tok0 * a.ldq + (int64_t)g * D, a.ldq, L, D);
+  hm_fill<128>(Ks, ldk, LC, D16, reinterpret_cast<const bf16*>(a.k) + (int64_t)tok0 * a.ldk + (int64_t)g * D, a.ldk, L, D);
+  hm_fill<128>(Vs, LDV, LC, VT, reinterpret_cast<const bf16*>(a.v) + (int64_t)tok0 * a.ldv + (int64_t)h * V + v0, a.ldv, L, V - v0);
+  cp_async_commit();
+  {
+    const float* src = states + ((int64_t)blockIdx.x * a.H + h) * D * V + v0;
+#pragma unroll 8
+    for (int i = tid; i < D16 * (VT / 4); i += 128) {
+      const int d = i / (VT / 4), c = i % (VT / 4) * 4;
+      const float4 x = d < D && v0 + c < V ? *reinterpret_cast<const float4*>(src + (int64_t)d * V + c) : make_float4(0.f, 0.f, 0.f, 0.f);
+      uint32_t p0[3], p1[3];
+      split3_pair(x.x, x.y, p0);
+      split3_pair(x.z, x.w, p1);
+#pragma unroll
+      for (int k = 0; k < 3; ++k) *reinterpret_cast<uint2*>(Ss + (k * D16 + d) * LDV + c) = make_uint2(p0[k], p1[k]);
+    }
+  }
+  hd_run_scalars(a, tok0, L, h, g_s, b_s);
+  cp_async_wait<0>();
+  __syncthreads();
+  const int r0 = 16 * warp;
+  if (r0 >= L) return;
+  const int mr = lane & 7, mj = lane >> 3, t0 = r0 + (lane >> 2), t1 = t0 + 8;
+  float acc[8][4] = {};
+  const bf16* q_at = Qs + (r0 + mr + (mj & 1 ? 8 : 0)) * ldk + (mj >= 2 ? 8 : 0);
+  for (int d0 = 0; d0 < D16; d0 += 16) {
+    uint32_t qa[4];
+    ldmatrix_x4(qa, q_at + d0);
+#pragma unroll
+    for (int p = 0; p < 3; ++p)
+#pragma unroll
+      for (int n = 0; n < 4; ++n) {
+        uint32_t sb[4];
+        ldmatrix_x4_trans(sb, Ss + (p * D16 + d0 + mr + (mj & 1 ? 8 : 0)) * LDV + 16 * n + (mj >= 2 ? 8 : 0));
+        mma_bf16(acc[2 * n], qa, sb[0], sb[1]);
+        mma_bf16(acc[2 * n + 1], qa, sb[2], sb[3]);
+      }
+  }
+  const double bt0 = b_s[t0], bt1 = b_s[t1];
+  {
+    const float f0 = exp2f((float)bt0), f1 = exp2f((float)bt1);
+#pragma unroll
+    for (int n = 0; n < 8; ++n) {
+      acc[n][0] *= f0; acc[n][1] *= f0;
+      acc[n][2] *= f1; acc[n][3] *= f1;
+    }
+  }
+  for (int s0 = 0; s0 <= r0; s0 += 16) {        // keys up to the diagonal
+    float sc[2][4] = {};
+    const bf16* k_at = Ks + (s0 + mr + (mj >= 2 ? 8 : 0)) * ldk + (mj & 1 ? 8 : 0);
+    for (int d0 = 0; d0 < D16; d0 += 16) {
+      uint32_t qa[4], kb[4];
+      ldmatrix_x4(qa, q_at + d0);
+      ldmatrix_x4(kb, k_at + d0);
+      mma_bf16(sc[0], qa, kb[0], kb[1]);
+      mma_bf16(sc[1], qa, kb[2], kb[3]);
+    }
+    uint32_t pa[3][4];
+#pragma unroll
+    for (int n = 0; n < 2; ++n) {
+      const int s = s0 + 8 * n + 2 * (lane & 3);
+      const double bs0 = b_s[s], bs1 = b_s[s + 1];
+      const float g0 = g_s[s], g1 = g_s[s + 1];
+      const float w0 = s <= t0 ? sc[n][0] * g0 * exp2f((float)(bt0 - bs0)) : 0.f, w1 = s + 1 <= t0 ? sc[n][1] * g1 * exp2f((float)(bt0 - bs1)) : 0.f;
+      const float w2 = s <= t1 ? sc[n][2] * g0 * exp2f((float)(bt1 - bs0)) : 0.f, w3 = s + 1 <= t1 ? sc[n][3] * g1 * exp2f((float)(bt1 - bs1)) : 0.f;
+      uint32_t lo[3], hi[3];
+      split3_pair(w0, w1, lo);
+      split3_pair(w2, w3, hi);
+#pragma unroll
+      for (int p = 0; p < 3; ++p) {
+        pa[p][2 * n] = lo[p];
+        pa[p][2 * n + 1] = hi[p];
+      }
+    }
+#pragma unroll
+    for (int n = 0; n < 4; ++n) {
+      uint32_t vb[4];
+      ldmatrix_x4_trans(vb, Vs + (s0 + mr + (mj & 1 ? 8 : 0)) * LDV + 16 * n + (mj >= 2 ? 8 : 0));
+#pragma unroll
+      for (int p = 0; p < 3; ++p) {
+        mma_bf16(acc[2 * n], pa[p], vb[0], vb[1]);
+        mma_bf16(acc[2 * n + 1], pa[p], vb[2], vb[3]);
+      }
+    }
+  }
+  const float skip = a.skip ? a.skip[h] : 0.f;
+  float* o0 = a.o + (int64_t)(tok0 + t0) * a.H * V + (int64_t)h * V + v0;
+  float* o1 = o0 + (int64_t)8 * a.H * V;
+#pragma unroll
+  for (int n = 0; n < 8; ++n) {
+    const int c = 8 * n + 2 * (lane & 3);
+    if (v0 + c >= V) continue;
+    if (a.skip) {
+      const __nv_bfloat162 x0 = *reinterpret_cast<const __nv_bfloat162*>(Vs + t0 * LDV + c), x1 = *reinterpret_cast<const __nv_bfloat162*>(Vs + t1 * LDV + c);
+      acc[n][0] = fmaf(skip, __low2float(x0), acc[n][0]);
+      acc[n][1] = fmaf(skip, __high2float(x0), acc[n][1]);
+      acc[n][2] = fmaf(skip, __low2float(x1), acc[n][2]);
+      acc[n][3] = fmaf(skip, __high2float(x1), acc[n][3]);
+    }
+    if (t0 < L) *reinterpret_cast<float2*>(o0 + c) = make_float2(acc[n][0], acc[n][1]);
+    if (t1 < L) *reinterpret_cast<float2*>(o1 + c) = make_float2(acc[n][2], acc[n][3]);
+  }
+}
+
+size_t state_smem(int D) { return sizeof(bf16) * ((size_t)HD_LC * ((D + 15) / 16 * 16 + 8) + 3 * HD_LC * HM_LDV); }
+size_t out_smem(int D) {
+  const size_t D16 = (D + 15) / 16 * 16;
+  return sizeof(bf16) * (2 * HD_LC * (D16 + 8) + HD_LC * HM_LDV + 3 * D16 * HM_LDV);
+}
+
+}  // namespace
+
+// bfloat16 rows that start on 16 bytes, sizes in whole pieces of eight.
+bool me_head_decay_mma_takes(const HdArgs& a, int dtype) {
+  auto ok = [](const void* p, int64_t ld) { return ((uintptr_t)p % 16) == 0 && ld % 8 == 0; };
+  return dtype == ME_BF16 && a.D % 8 == 0 && a.V % 8 == 0 && a.D <= 256 && ok(a.q, a.ldq) && ok(a.k, a.ldk) && ok(a.v, a.ldv) &&
+         ((uintptr_t)a.o % 16) == 0 && out_smem(a.D) <= 220 * 1024;
+}
+
+int me_head_decay_mma_states(const HdArgs& a, const int* tiles, int n_tiles, float* states, float* totals, cudaStream_t stream) {
+  const size_t smem = state_smem(a.D);
+  cudaError_t e = cudaFuncSetAttribute(hd_mma_state_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+  ME_REQUIRE(e == cudaSuccess, "me_head_decay_scan: cannot raise shared memory to %zu: %s", smem, cudaGetErrorString(e));
+  me_launch(hd_mma_state_kernel, dim3(n_tiles, a.H, (a.V + HD_VT - 1) / HD_VT), dim3(256), smem, stream, a, tiles, states, totals);
+  return 0;
+}
+
+int me_head_decay_mma_out(const HdArgs& a, const int* tiles, int n_tiles, const float* states, cudaStream_t stream) {
+  const size_t smem = out_smem(a.D);
+  cudaError_t e = cudaFuncSetAttribute(hd_mma_out_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+  ME_REQUIRE(e == cudaSuccess, "me_head_decay_scan: cannot raise shared memory to %zu: %s", smem, cudaGetErrorString(e));
+  me_launch(hd_mma_out_kernel, dim3(n_tiles, a.H, (a.V + HD_VT - 1) / HD_VT), dim3(128), smem, stream, a, tiles, states);
+  return 0;
+}

@@ -64,7 +64,7 @@ _PROTOS = {
     "me_gla_scan": [_P, _L, _I, _I, _I, _P, _P, _P, _P, _P, _P, _I, _I, _I, _I, _F, _P, _I, _I, _P, _P, _P, _P, _P],
     "me_stream_norm": [_P, _P, _P, _P, _I, _P, _P, _P, _F, _F, _F, _P, _P, _P, _F, _P, _I, _L, _P, _I, _I, _P],
     "me_conv_silu": [_P, _L, _P, _P, _P, _P, _I, _I, _P, _P, _P, _P, _I, _I, _I, _I, _P],
-    "me_head_decay_scan": [_P, _P, _P, _I, _L, _L, _L, _I, _I, _I, _I, _F, _P, _L, _P, _P, _P, _P, _P, _P, _P, _P, _P, _P, _I, _I, _P, _I, _P, _P, _P],
+    "me_head_decay_scan": [_P, _P, _P, _I, _L, _L, _L, _I, _I, _I, _I, _F, _P, _L, _P, _P, _P, _P, _P, _P, _P, _P, _P, _P, _I, _I, _P, _I, _P, _P, _I, _P],
     "me_gated_group_norm": [_P, _L, _P, _I, _L, _P, _I, _F, _P, _I, _L, _I, _I, _I, _P],
     "me_activation": [_P, _I, _L, _P, _I, _L, _I, _I, _I, _P],
     "me_soft_cap": [_P, _L, _F, _F, _P],
@@ -1478,6 +1478,7 @@ def conv_silu(u: torch.Tensor, weight: torch.Tensor, bias: Optional[torch.Tensor
 
 
 HEAD_DECAY_CHUNK = 64     # tokens per run of the recurrence's prompt kernels (csrc/head_decay.cu)
+use_head_decay_mma = True # bfloat16 prompts on the tensor cores where the sizes allow (csrc/head_decay_mma.cu); a switch for comparisons
 head_decay_chunks = True  # portions of prompts by runs of tokens (False: token by token, always); a switch for comparisons
 
 
@@ -1521,7 +1522,7 @@ def head_decay_scan(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, S: torch.
           dim, vdim, float(k_scale), _ptr(dt[0]) if dt else 0, dt[0].stride(0) if dt else 0, _ptr(dt[1]) if dt else 0, _ptr(dt[2]) if dt else 0,
           _ptr(decay[0]) if decay else 0, _ptr(decay[1]) if decay else 0, _ptr(skip), S.data_ptr(), meta.cu_seqlens.data_ptr(), meta.context_lens.data_ptr(), state_slots.data_ptr(),
           o.data_ptr(), meta.num_reqs, meta.num_decodes, tiles.data_ptr() if chunked else 0, n_tiles if chunked else 0,
-          chunk_states.data_ptr() if chunked else 0, totals.data_ptr() if chunked else 0, _stream())
+          chunk_states.data_ptr() if chunked else 0, totals.data_ptr() if chunked else 0, 1 if use_head_decay_mma else 0, _stream())
     global launches
     launches += (2 + (1 if meta.num_decodes else 0)) if chunked else 0
 

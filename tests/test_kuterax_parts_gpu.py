@@ -51,6 +51,7 @@ class _Scan:
         self.dt_bias = torch.randn(H, generator=g(seed + 2)) - 1.0 if dt_bias is None else torch.full((H,), float(dt_bias))
         self.skip = torch.randn(H, generator=g(seed + 3))
         self.S = torch.full((slots, H, D, V), float("nan"), device=DEV)
+        self.pad = 4                                                     # columns in front of and between q, k and v
 
     def inputs(self, T, seed):
         q, k = (torch.randn(T, self.G * self.D, generator=g(seed + i)) / self.D ** 0.25 for i in (0, 1))
@@ -71,9 +72,11 @@ class _Scan:
         ops = _ops()
         H, G, D, V = self.H, self.G, self.D, self.V
         T = x[0].shape[0]
-        wide = torch.full((T, 2 * G * D + H * V + 16), float("nan"), dtype=self.dt, device=DEV)
-        wide[:, 4:4 + G * D], wide[:, 8 + G * D:8 + 2 * G * D], wide[:, 12 + 2 * G * D:12 + 2 * G * D + H * V] = (t.to(self.dt).to(DEV) for t in x[:3])
-        q, k, v = wide[:, 4:4 + G * D], wide[:, 8 + G * D:8 + 2 * G * D], wide[:, 12 + 2 * G * D:12 + 2 * G * D + H * V]
+        p = self.pad
+        wide = torch.full((T, 2 * G * D + H * V + 4 * p), float("nan"), dtype=self.dt, device=DEV)
+        q, k, v = wide[:, p:p + G * D], wide[:, 2 * p + G * D:2 * p + 2 * G * D], wide[:, 3 * p + 2 * G * D:3 * p + 2 * G * D + H * V]
+        for dst, src in zip((q, k, v), x):
+            dst.copy_(src)
         dtw = torch.full((T, H + 5), float("nan"), device=DEV)
         dtw[:, 3:3 + H] = x[3].to(DEV)
         meta = _meta(list(lens), list(contexts))
@@ -101,14 +104,17 @@ def _close(got, ref, rel=3e-6):
     assert err <= rel * max(top, 1e-3), (err, top)
 
 
-SCANS = [(2, 2, 16, 32), (3, 1, 24, 40), (4, 2, 64, 64), (2, 1, 7, 5), (2, 2, 64, 128), (6, 3, 128, 64), (1, 1, 130, 70), (2, 2, 256, 24), (1, 1, 300, 12)]
+SCANS = [(2, 2, 16, 32), (2, 1, 8, 8), (4, 2, 72, 136), (3, 1, 24, 40), (4, 2, 64, 64), (2, 1, 7, 5), (2, 2, 64, 128), (6, 3, 128, 64), (1, 1, 130, 70), (2, 2, 256, 24), (1, 1, 300, 12)]
 
 
 @both
 @pytest.mark.parametrize("constant", [True, False])
+@pytest.mark.parametrize("pad", [4, 8])
 @pytest.mark.parametrize("H, G, D, V", SCANS)
-def test_recurrence_against_the_plain_one_and_cut_anywhere(dtype, constant, H, G, D, V):
+def test_recurrence_against_the_plain_one_and_cut_anywhere(dtype, constant, pad, H, G, D, V):
+    """Rows of bfloat16 that start on 16 bytes (``pad`` 8) run the tensor-core kernels for prompts where the sizes allow."""
     run = _Scan(H, G, D, V, dtype, constant, seed=H * 100 + D)
+    run.pad = pad
     x = run.inputs(200, H + D + V)
     ref = run.plain(x)
     whole = run.sequence(x, [200], 1)                                    # three runs of 64 tokens and a rest of 8
@@ -128,6 +134,7 @@ def test_recurrence_against_the_plain_one_and_cut_anywhere(dtype, constant, H, G
 @pytest.mark.parametrize("constant", [True, False])
 def test_recurrence_of_unequal_requests_with_slots_used_again(dtype, constant):
     run = _Scan(4, 2, 24, 40, dtype, constant, seed=77, slots=5)
+    run.pad = 8
     totals, first = [90, 31, 140, 131, 66], [89, 30, 70, 1, 64]
     xs = [run.inputs(n, 200 + 10 * i) for i, n in enumerate(totals)]
     refs, slots = [run.plain(x) for x in xs], [4, 0, 2, 3, 1]
@@ -146,20 +153,24 @@ def test_recurrence_of_unequal_requests_with_slots_used_again(dtype, constant):
     _close(out[100:], refs[0][:65])
 
 
+@both
 @pytest.mark.parametrize("a_log, dt_bias", [(6.0, 4.0), (-12.0, 2.0), (0.0, -30.0), (2.0, 60.0), (-3.0, -4.0)])
-def test_recurrence_that_forgets_at_once_or_never(a_log, dt_bias):
+def test_recurrence_that_forgets_at_once_or_never(dtype, a_log, dt_bias):
     """Decays of 0 in float32, decays so close to 1 that nothing is forgotten, steps of almost nothing and of sixty."""
-    run = _Scan(2, 1, 16, 24, "float32", False, a_log=a_log, dt_bias=dt_bias)
+    run = _Scan(2, 1, 16, 24, dtype, False, a_log=a_log, dt_bias=dt_bias)
+    run.pad = 8
     x = run.inputs(150, 9)
     ref = run.plain(x)
     for cuts, slot in (([150], 0), ([1] * 150, 1), ([70, 2, 78], 2)):
         _close(run.sequence(x, cuts, slot), ref, rel=1e-5)
 
 
-def test_recurrence_a_slow_stretch_behind_strong_decays_keeps_its_digits():
+@both
+def test_recurrence_a_slow_stretch_behind_strong_decays_keeps_its_digits(dtype):
     """Within one run of 64 tokens the first twenty decay by e^-900 each and the rest hardly at all: differences of large sums of
     logarithms would have lost the digits of the small ones."""
-    run = _Scan(1, 1, 8, 16, "float32", False, a_log=4.5, dt_bias=0.0)
+    run = _Scan(1, 1, 8, 16, dtype, False, a_log=4.5, dt_bias=0.0)
+    run.pad = 8
     x = run.inputs(64, 4)
     x[3][:20], x[3][20:] = 10.0, -13.0
     x[0][:], x[1][:] = x[0].abs(), x[1].abs()                            # no cancellation in the sums
@@ -169,10 +180,12 @@ def test_recurrence_a_slow_stretch_behind_strong_decays_keeps_its_digits():
     assert rel < 1e-6, rel
 
 
+@both
 @pytest.mark.parametrize("constant", [True, False])
-def test_recurrence_carries_the_first_token_across_many_runs(constant):
+def test_recurrence_carries_the_first_token_across_many_runs(dtype, constant):
     """One channel is written by the first token alone and read by the last one alone."""
-    run = _Scan(1, 1, 8, 16, "float32", constant, decay=[1.0], a_log=-25.0, dt_bias=0.5)
+    run = _Scan(1, 1, 8, 16, dtype, constant, decay=[1.0], a_log=-25.0, dt_bias=0.5)
+    run.pad = 8
     T = 401
     x = run.inputs(T, 22)
     x[1][1:, 3] = 0
