@@ -128,10 +128,10 @@ __device__ __forceinline__ void hd_fill(float* dst, int ld_dst, int rows, int co
   }
 }
 
-// One block = one run x one head x HD_VT columns.  totals[c, h] = B of the run's last token.
+// One block = one run x one head x HD_VT columns.  nums[c, h]: the run's numbers.
 template <typename T, int VEC>
 __global__ void __launch_bounds__(256)
-hd_chunk_state_kernel(HdArgs a, const int* __restrict__ tiles, float* __restrict__ states, float* __restrict__ totals) {
+hd_chunk_state_kernel(HdArgs a, const int* __restrict__ tiles, float* __restrict__ states, HdRun* __restrict__ nums) {
   extern __shared__ __align__(16) float smem[];
   __shared__ float g_s[HD_LC];
   __shared__ double b_s[HD_LC];
@@ -150,7 +150,11 @@ hd_chunk_state_kernel(HdArgs a, const int* __restrict__ tiles, float* __restrict
   hd_fill<T, VEC>(Kt, ldk, LC, Dp, reinterpret_cast<const T*>(a.k) + (int64_t)tok0 * a.ldk + (int64_t)g * D, a.ldk, L, D);
   __syncthreads();
   const double bl = b_s[LC - 1];
-  if (tid == 0 && blockIdx.z == 0) totals[(int64_t)blockIdx.x * a.H + h] = (float)bl;
+  if (tid < LC && blockIdx.z == 0) {
+    HdRun& run = nums[(int64_t)blockIdx.x * a.H + h];
+    run.b[tid] = b_s[tid];
+    run.g[tid] = g_s[tid];
+  }
   {
     const T* src = reinterpret_cast<const T*>(a.v) + (int64_t)tok0 * a.ldv + (int64_t)h * V + v0;
     constexpr int per = VT / VEC;
@@ -197,17 +201,19 @@ hd_chunk_state_kernel(HdArgs a, const int* __restrict__ tiles, float* __restrict
   }
 }
 
-// One block = one request (first_req + blockIdx.x) x one head x 256 VEC elements of S; a thread walks VEC neighbours.
+// One block = one request (first_req + blockIdx.x) x one head x HD_WALK VEC elements of S; a thread walks VEC neighbours.
+constexpr int HD_WALK = 128;
+
 template <int VEC>
-__global__ void __launch_bounds__(256)
-hd_state_walk_kernel(HdArgs a, const float* __restrict__ totals, float* __restrict__ states, const int* __restrict__ tiles, int n_tiles, int first_req) {
+__global__ void __launch_bounds__(HD_WALK, 8)
+hd_state_walk_kernel(HdArgs a, const HdRun* __restrict__ nums, float* __restrict__ states, const int* __restrict__ tiles, int n_tiles, int first_req) {
   __shared__ int first_tile;
   const int b = first_req + blockIdx.x, h = blockIdx.y, DV = a.D * a.V;
-  const int e = (blockIdx.z * 256 + threadIdx.x) * VEC;
+  const int e = (blockIdx.z * HD_WALK + threadIdx.x) * VEC;
   const int slot = a.slots[b], tok0 = a.cu[b], n_tok = a.cu[b + 1] - tok0;
   if (threadIdx.x == 0) first_tile = -1;
   __syncthreads();
-  for (int i = threadIdx.x; i < n_tiles; i += 256)           // a request's runs follow one another in the list
+  for (int i = threadIdx.x; i < n_tiles; i += HD_WALK)           // a request's runs follow one another in the list
     if (tiles[2 * i] == b && tiles[2 * i + 1] == 0) first_tile = i;
   __syncthreads();
   pdl_wait();
@@ -220,7 +226,7 @@ hd_state_walk_kernel(HdArgs a, const float* __restrict__ totals, float* __restri
   const int n_chunks = (n_tok + HD_LC - 1) / HD_LC;
   const int64_t step = (int64_t)a.H * DV;
   float* st = states + ((int64_t)c0 * a.H + h) * DV + e;
-  const float* tot = totals + (int64_t)c0 * a.H + h;
+  const HdRun* run = nums + (int64_t)c0 * a.H + h;
   constexpr int AHEAD = 8;                      // runs whose loads are in flight together
   for (int c1 = 0; c1 < n_chunks; c1 += AHEAD) {
     float u[AHEAD][VEC], dec[AHEAD];
@@ -228,7 +234,7 @@ hd_state_walk_kernel(HdArgs a, const float* __restrict__ totals, float* __restri
     for (int j = 0; j < AHEAD; ++j) {
       const int c = min(c1 + j, n_chunks - 1);
       HdVec<VEC>::load(st + c * step, u[j]);
-      dec[j] = tot[(int64_t)c * a.H];
+      dec[j] = (float)run[(int64_t)c * a.H].b[HD_LC - 1];
     }
 #pragma unroll
     for (int j = 0; j < AHEAD; ++j) {
@@ -246,7 +252,7 @@ hd_state_walk_kernel(HdArgs a, const float* __restrict__ totals, float* __restri
 // One block = one run x one head x HD_VT columns; states[c] holds the state in front of the run.
 template <typename T, int VEC>
 __global__ void __launch_bounds__(256)
-hd_chunk_out_kernel(HdArgs a, const int* __restrict__ tiles, const float* __restrict__ states) {
+hd_chunk_out_kernel(HdArgs a, const int* __restrict__ tiles, const float* __restrict__ states, const HdRun* __restrict__ nums) {
   extern __shared__ __align__(16) float smem[];
   __shared__ float g_s[HD_LC];
   __shared__ double b_s[HD_LC];
@@ -263,7 +269,11 @@ hd_chunk_out_kernel(HdArgs a, const int* __restrict__ tiles, const float* __rest
   pdl_launch_dependents();
   if (L <= 0) return;
   const int g = h / (a.H / a.G);
-  hd_run_scalars(a, tok0, L, h, g_s, b_s);
+  if (tid < LC) {
+    const HdRun& run = nums[(int64_t)blockIdx.x * a.H + h];
+    b_s[tid] = run.b[tid];
+    g_s[tid] = run.g[tid];
+  }
   hd_fill<T, VEC>(Q, ldq, LC, D4, reinterpret_cast<const T*>(a.q) + (int64_t)tok0 * a.ldq + (int64_t)g * D, a.ldq, L, D);
   hd_fill<T, VEC>(K, ldq, LC, D4, reinterpret_cast<const T*>(a.k) + (int64_t)tok0 * a.ldk + (int64_t)g * D, a.ldk, L, D);
   hd_fill<T, VEC>(Vs, VT, LC, VT, reinterpret_cast<const T*>(a.v) + (int64_t)tok0 * a.ldv + (int64_t)h * V + v0, a.ldv, L, V - v0);
@@ -339,8 +349,8 @@ hd_chunk_out_kernel(HdArgs a, const int* __restrict__ tiles, const float* __rest
   }
 }
 
-int me_head_decay_mma_states(const HdArgs& a, const int* tiles, int n_tiles, float* states, float* totals, cudaStream_t stream);
-int me_head_decay_mma_out(const HdArgs& a, const int* tiles, int n_tiles, const float* states, cudaStream_t stream);
+int me_head_decay_mma_states(const HdArgs& a, const int* tiles, int n_tiles, float* states, HdRun* nums, cudaStream_t stream);
+int me_head_decay_mma_out(const HdArgs& a, const int* tiles, int n_tiles, const float* states, const HdRun* nums, cudaStream_t stream);
 bool me_head_decay_mma_takes(const HdArgs& a, int dtype);
 
 template <typename K>
@@ -353,18 +363,19 @@ static int hd_raise_smem(K kernel, size_t smem, const char* what) {
 }
 
 ME_API int me_head_decay_chunk_len() { return HD_LC; }
+ME_API int me_head_decay_run_bytes() { return (int)sizeof(HdRun); }      // what a run and head takes of ``nums_ws``
 
 // q, k: rows of ``dtype`` holding the G groups' D values, ldq / ldk elements apart; v: rows of H heads' V values.  dt: float32 rows of H
 // pre-activations with dt_bias, a_log [H], or null with decay [H] and log2_decay [H] (float64).  skip: [H] or null.  S: [slots, H, D, V] float32; o: [T, H*V]
 // float32.  Requests [0, num_decodes) are walked token by token.  The others too, unless ``tiles`` ([n_tiles, 2] int32: request and first
 // token of every run of HD_LC tokens of the requests from num_decodes on, a request's runs in order and side by side),
-// ``states_ws`` ([n_tiles, H, D, V] float32) and ``totals_ws`` ([n_tiles, H] float32) are given and D is at most 256.  allow_mma: the
+// ``states_ws`` ([n_tiles, H, D, V] float32) and ``nums_ws`` (n_tiles * H times me_head_decay_run_bytes, on 16 bytes) are given and D is at most 256.  allow_mma: the
 // products of prompts may run on the tensor cores.
 ME_API int me_head_decay_scan(const void* q, const void* k, const void* v, int dtype, int64_t ldq, int64_t ldk, int64_t ldv, int H, int G, int D,
                               int V, float k_scale, const float* dt, int64_t ld_dt, const float* dt_bias, const float* a_log,
                               const float* decay, const double* log2_decay, const float* skip, float* S, const int* cu_seqlens, const int* context_lens,
                               const int* state_slots, float* o, int B, int num_decodes, const int* tiles, int n_tiles, float* states_ws,
-                              float* totals_ws, int allow_mma, cudaStream_t stream) {
+                              void* nums_ws, int allow_mma, cudaStream_t stream) {
   if (B == 0) return 0;
   ME_REQUIRE(B > 0 && H > 0 && G > 0 && H % G == 0 && D > 0 && V > 0 && H <= 65535 && D <= 1024, "me_head_decay_scan: bad sizes B=%d H=%d G=%d D=%d V=%d", B, H, G, D, V);
   ME_REQUIRE(num_decodes >= 0 && num_decodes <= B, "me_head_decay_scan: %d single-token requests of %d", num_decodes, B);
@@ -377,8 +388,8 @@ ME_API int me_head_decay_scan(const void* q, const void* k, const void* v, int d
   const size_t smem_state = sizeof(float) * (HD_LC * (Dp + 4) + HD_LC * HD_VT);
   const size_t lk = HD_LC * (D4 + 4), ls = D4 * HD_VT;
   const size_t smem_out = sizeof(float) * (lk + (lk > ls ? lk : ls) + HD_LC * (HD_LC + 4) + HD_LC * HD_VT);
-  const bool chunks = tiles && states_ws && totals_ws && n_tiles > 0 && num_decodes < B && D <= 256 && v_tiles <= 65535 &&
-                      ((int64_t)D * V + 255) / 256 <= 65535 && smem_state <= 220 * 1024 && smem_out <= 220 * 1024;
+  const bool chunks = tiles && states_ws && nums_ws && n_tiles > 0 && num_decodes < B && D <= 256 && v_tiles <= 65535 &&
+                      ((int64_t)D * V + HD_WALK - 1) / HD_WALK <= 65535 && smem_state <= 220 * 1024 && smem_out <= 220 * 1024;
   const int n_step = chunks ? num_decodes : B;
   if (n_step > 0) {
 #define HD_STEP(R_, VEC_)                                                                                                       \
@@ -395,6 +406,8 @@ ME_API int me_head_decay_scan(const void* q, const void* k, const void* v, int d
     ME_LAUNCH_CHECK("me_head_decay_scan (tokens)");
   }
   if (chunks) {
+    HdRun* nums = reinterpret_cast<HdRun*>(nums_ws);
+    ME_REQUIRE(!off(nums_ws, 16), "me_head_decay_scan: the runs' numbers must start on 16 bytes");
     const bool vec = out4 && D % 4 == 0 && ldq % 4 == 0 && ldk % 4 == 0 && !off(q, al) && !off(k, al) && !off(states_ws, 16);
 #define HD_CHUNK(KERNEL_, VEC_, SMEM_, ...)                                                                          \
   do {                                                                                                               \
@@ -403,23 +416,23 @@ ME_API int me_head_decay_scan(const void* q, const void* k, const void* v, int d
   } while (0)
     const bool mma = allow_mma && me_head_decay_mma_takes(a, dtype) && !off(states_ws, 16);
     if (mma) {
-      if (me_head_decay_mma_states(a, tiles, n_tiles, states_ws, totals_ws, stream)) return 1;
+      if (me_head_decay_mma_states(a, tiles, n_tiles, states_ws, nums, stream)) return 1;
     } else ME_DISPATCH_DTYPE(dtype, T, {
-      if (vec) HD_CHUNK(hd_chunk_state_kernel, 4, smem_state, states_ws, totals_ws);
-      else HD_CHUNK(hd_chunk_state_kernel, 1, smem_state, states_ws, totals_ws);
+      if (vec) HD_CHUNK(hd_chunk_state_kernel, 4, smem_state, states_ws, nums);
+      else HD_CHUNK(hd_chunk_state_kernel, 1, smem_state, states_ws, nums);
     });
     ME_LAUNCH_CHECK("me_head_decay_scan (run states)");
     const bool walk4 = V % 4 == 0 && !off(states_ws, 16) && !off(S, 16);
-    const int per = walk4 ? 1024 : 256;
+    const int per = walk4 ? 4 * HD_WALK : HD_WALK;
     const dim3 walk_grid(B - num_decodes, H, (unsigned)(((int64_t)D * V + per - 1) / per));
-    if (walk4) me_launch(hd_state_walk_kernel<4>, walk_grid, dim3(256), 0, stream, a, (const float*)totals_ws, states_ws, tiles, n_tiles, num_decodes);
-    else me_launch(hd_state_walk_kernel<1>, walk_grid, dim3(256), 0, stream, a, (const float*)totals_ws, states_ws, tiles, n_tiles, num_decodes);
+    if (walk4) me_launch(hd_state_walk_kernel<4>, walk_grid, dim3(HD_WALK), 0, stream, a, (const HdRun*)nums, states_ws, tiles, n_tiles, num_decodes);
+    else me_launch(hd_state_walk_kernel<1>, walk_grid, dim3(HD_WALK), 0, stream, a, (const HdRun*)nums, states_ws, tiles, n_tiles, num_decodes);
     ME_LAUNCH_CHECK("me_head_decay_scan (state walk)");
     if (mma) {
-      if (me_head_decay_mma_out(a, tiles, n_tiles, states_ws, stream)) return 1;
+      if (me_head_decay_mma_out(a, tiles, n_tiles, states_ws, nums, stream)) return 1;
     } else ME_DISPATCH_DTYPE(dtype, T, {
-      if (vec) HD_CHUNK(hd_chunk_out_kernel, 4, smem_out, (const float*)states_ws);
-      else HD_CHUNK(hd_chunk_out_kernel, 1, smem_out, (const float*)states_ws);
+      if (vec) HD_CHUNK(hd_chunk_out_kernel, 4, smem_out, (const float*)states_ws, (const HdRun*)nums);
+      else HD_CHUNK(hd_chunk_out_kernel, 1, smem_out, (const float*)states_ws, (const HdRun*)nums);
     });
 #undef HD_CHUNK
     ME_LAUNCH_CHECK("me_head_decay_scan (run outputs)");

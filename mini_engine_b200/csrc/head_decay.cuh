@@ -49,8 +49,14 @@ __device__ __forceinline__ void hd_token(const HdArgs& a, int64_t t, int h, floa
   }
 }
 
-// The run's factors g and inclusive sums B (double) into shared memory, zero factors and no further decay beyond its L tokens; the
-// first warp's work.
+// A run's numbers for one head: the inclusive sums B of log2 a and the factors g, zero factors and no further decay beyond its tokens.  The
+// kernel that makes the runs' states leaves them in global memory for the two behind it.
+struct HdRun {
+  double b[HD_LC];
+  float g[HD_LC];
+};
+
+// The first warp's work.
 __device__ __forceinline__ void hd_run_scalars(const HdArgs& a, int tok0, int L, int h, float* g_s, double* b_s) {
   if (threadIdx.x >= 32) return;
   const int lane = threadIdx.x, t0 = 2 * lane, t1 = t0 + 1;

@@ -6,7 +6,7 @@
 // up to the order of sums.
 //
 //   hd_mma_state_kernel   U = k^T (g_s 2^(B_L - B_s) v_s) of a run: 64 tokens x 64 columns a block, a warp a strip of 16 rows by 32 columns
-//   hd_mma_out_kernel     a warp takes 16 tokens of the run: q S_in (three parts), scaled by 2^(B_t); then, 16 keys at a time up to the
+//   hd_mma_out_kernel     a warp takes 16 tokens of the run and 32 columns: q S_in (three parts), scaled by 2^(B_t); then, 16 keys at a time up to the
 //                         diagonal, the scores q k^T, their weights in the registers, and the product with v (three parts)
 #include "head_decay.cuh"
 #include "mma_prims.cuh"
@@ -17,39 +17,33 @@ using namespace mma_prims;
 
 constexpr int HM_LDV = HD_VT + 8;             // bfloat16 elements of a row of 64 columns in shared memory (an odd number of 16-byte pieces)
 
-__device__ __forceinline__ void split3(float x, bf16& hi, bf16& mid, bf16& lo) {
-  hi = __float2bfloat16_rn(x);
-  const float r = x - __bfloat162float(hi);
-  mid = __float2bfloat16_rn(r);
-  lo = __float2bfloat16_rn(r - __bfloat162float(mid));
-}
-__device__ __forceinline__ uint32_t pack2(bf16 a, bf16 b) {
-  const __nv_bfloat162 v = __halves2bfloat162(a, b);
-  return *reinterpret_cast<const uint32_t*>(&v);
-}
-// Two floats as a pair of bfloat16 in each of the three parts.
+// Two floats as a pair of bfloat16 (x in the lower half) in each of the three parts.
 __device__ __forceinline__ void split3_pair(float x, float y, uint32_t (&p)[3]) {
-  bf16 a[3], b[3];
-  split3(x, a[0], a[1], a[2]);
-  split3(y, b[0], b[1], b[2]);
-#pragma unroll
-  for (int i = 0; i < 3; ++i) p[i] = pack2(a[i], b[i]);
+  p[0] = pack_bf16(x, y);
+  x -= __uint_as_float(p[0] << 16);
+  y -= __uint_as_float(p[0] & 0xffff0000u);
+  p[1] = pack_bf16(x, y);
+  p[2] = pack_bf16(x - __uint_as_float(p[1] << 16), y - __uint_as_float(p[1] & 0xffff0000u));
 }
 
-// rows x cols (a multiple of 8) bfloat16 values into shared memory by asynchronous copies, zeros beyond n_rows and n_cols.
-template <int THREADS>
-__device__ __forceinline__ void hm_fill(bf16* dst, int ld_dst, int rows, int cols, const bf16* src, int64_t ld_src, int n_rows, int n_cols) {
-  const int per = cols / 8;
-  for (int i = threadIdx.x; i < rows * per; i += THREADS) {
-    const int r = i / per, c = (i - r * per) * 8;
-    const bool ok = r < n_rows && c < n_cols;
-    cp_async16(dst + r * ld_dst + c, ok ? src + (int64_t)r * ld_src + c : src, ok);
+// HD_LC rows of cols (a multiple of 8) bfloat16 values into shared memory by asynchronous copies of a block of 256, zeros beyond n_rows and
+// n_cols.  Eight neighbouring threads take a row's pieces of 16 bytes.
+__device__ __forceinline__ void hm_fill(bf16* dst, int ld_dst, int cols, const bf16* src, int64_t ld_src, int n_rows, int n_cols) {
+  const int r0 = threadIdx.x >> 3, c0 = (threadIdx.x & 7) * 8;
+#pragma unroll
+  for (int i = 0; i < HD_LC / 32; ++i) {
+    const int r = r0 + 32 * i;
+    const bf16* s = src + (int64_t)r * ld_src;
+    for (int c = c0; c < cols; c += 64) {
+      const bool ok = r < n_rows && c < n_cols;
+      cp_async16(dst + r * ld_dst + c, ok ? s + c : src, ok);
+    }
   }
 }
 
-// One block = one run x one head x HD_VT columns of U; totals[c, h] = B of the run's last token.
+// One block = one run x one head x HD_VT columns of U; nums[c, h]: the run's numbers.
 __global__ void __launch_bounds__(256)
-hd_mma_state_kernel(HdArgs a, const int* __restrict__ tiles, float* __restrict__ states, float* __restrict__ totals) {
+hd_mma_state_kernel(HdArgs a, const int* __restrict__ tiles, float* __restrict__ states, HdRun* __restrict__ nums) {
   extern __shared__ __align__(16) unsigned char hm_smem[];
   __shared__ float g_s[HD_LC];
   __shared__ double b_s[HD_LC];
@@ -64,7 +58,7 @@ hd_mma_state_kernel(HdArgs a, const int* __restrict__ tiles, float* __restrict__
   pdl_launch_dependents();
   if (L <= 0) return;
   const int g = h / (a.H / a.G);
-  hm_fill<256>(Ks, ldk, LC, D16, reinterpret_cast<const bf16*>(a.k) + (int64_t)tok0 * a.ldk + (int64_t)g * D, a.ldk, L, D);
+  hm_fill(Ks, ldk, D16, reinterpret_cast<const bf16*>(a.k) + (int64_t)tok0 * a.ldk + (int64_t)g * D, a.ldk, L, D);
   cp_async_commit();
   // this thread's 16 values (two rows' pieces of eight columns), on their way while the first warp sums the decays
   const bf16* vsrc = reinterpret_cast<const bf16*>(a.v) + (int64_t)tok0 * a.ldv + (int64_t)h * V + v0;
@@ -77,7 +71,11 @@ hd_mma_state_kernel(HdArgs a, const int* __restrict__ tiles, float* __restrict__
   hd_run_scalars(a, tok0, L, h, g_s, b_s);
   __syncthreads();
   const double bl = b_s[LC - 1];
-  if (tid == 0 && blockIdx.z == 0) totals[(int64_t)blockIdx.x * a.H + h] = (float)bl;
+  if (tid < LC && blockIdx.z == 0) {
+    HdRun& run = nums[(int64_t)blockIdx.x * a.H + h];
+    run.b[tid] = b_s[tid];
+    run.g[tid] = g_s[tid];
+  }
 #pragma unroll
   for (int i = 0; i < 2; ++i) {
     const int r = tid / 8 + 32 * i, c = tid % 8 * 8;
@@ -123,8 +121,8 @@ hd_mma_state_kernel(HdArgs a, const int* __restrict__ tiles, float* __restrict__
 }
 
 // One block = one run x one head x HD_VT columns; states[c] holds the state in front of the run.
-__global__ void __launch_bounds__(128)
-hd_mma_out_kernel(HdArgs a, const int* __restrict__ tiles, const float* __restrict__ states) {
+__global__ void __launch_bounds__(256)
+hd_mma_out_kernel(HdArgs a, const int* __restrict__ tiles, const float* __restrict__ states, const HdRun* __restrict__ nums) {
   extern __shared__ __align__(16) unsigned char hm_smem[];
   __shared__ float g_s[HD_LC];
   __shared__ double b_s[HD_LC];
@@ -141,14 +139,14 @@ hd_mma_out_kernel(HdArgs a, const int* __restrict__ tiles, const float* __restri
   pdl_launch_dependents();
   if (L <= 0) return;
   const int g = h / (a.H / a.G);
-  hm_fill<128>(Qs, ldk, LC, D16, reinterpret_cast<const bf16*>(a.q) + (int64_t)tok0 * a.ldq + (int64_t)g * D, a.ldq, L, D);
-  hm_fill<128>(Ks, ldk, LC, D16, reinterpret_cast<const bf16*>(a.k) + (int64_t)tok0 * a.ldk + (int64_t)g * D, a.ldk, L, D);
-  hm_fill<128>(Vs, LDV, LC, VT, reinterpret_cast<const bf16*>(a.v) + (int64_t)tok0 * a.ldv + (int64_t)h * V + v0, a.ldv, L, V - v0);
+  hm_fill(Qs, ldk, D16, reinterpret_cast<const bf16*>(a.q) + (int64_t)tok0 * a.ldq + (int64_t)g * D, a.ldq, L, D);
+  hm_fill(Ks, ldk, D16, reinterpret_cast<const bf16*>(a.k) + (int64_t)tok0 * a.ldk + (int64_t)g * D, a.ldk, L, D);
+  hm_fill(Vs, LDV, VT, reinterpret_cast<const bf16*>(a.v) + (int64_t)tok0 * a.ldv + (int64_t)h * V + v0, a.ldv, L, V - v0);
   cp_async_commit();
   {
     const float* src = states + ((int64_t)blockIdx.x * a.H + h) * D * V + v0;
 #pragma unroll 8
-    for (int i = tid; i < D16 * (VT / 4); i += 128) {
+    for (int i = tid; i < D16 * (VT / 4); i += 256) {
       const int d = i / (VT / 4), c = i % (VT / 4) * 4;
       const float4 x = d < D && v0 + c < V ? *reinterpret_cast<const float4*>(src + (int64_t)d * V + c) : make_float4(0.f, 0.f, 0.f, 0.f);
       uint32_t p0[3], p1[3];
@@ -158,13 +156,17 @@ hd_mma_out_kernel(HdArgs a, const int* __restrict__ tiles, const float* __restri
       for (int k = 0; k < 3; ++k) *reinterpret_cast<uint2*>(Ss + (k * D16 + d) * LDV + c) = make_uint2(p0[k], p1[k]);
     }
   }
-  hd_run_scalars(a, tok0, L, h, g_s, b_s);
+  if (tid < LC) {
+    const HdRun& run = nums[(int64_t)blockIdx.x * a.H + h];
+    b_s[tid] = run.b[tid];
+    g_s[tid] = run.g[tid];
+  }
   cp_async_wait<0>();
   __syncthreads();
-  const int r0 = 16 * warp;
-  if (r0 >= L) return;
+  const int r0 = 16 * (warp >> 1), c0 = 32 * (warp & 1);
+  if (r0 >= L || v0 + c0 >= V) return;
   const int mr = lane & 7, mj = lane >> 3, t0 = r0 + (lane >> 2), t1 = t0 + 8;
-  float acc[8][4] = {};
+  float acc[4][4] = {};
   const bf16* q_at = Qs + (r0 + mr + (mj & 1 ? 8 : 0)) * ldk + (mj >= 2 ? 8 : 0);
   for (int d0 = 0; d0 < D16; d0 += 16) {
     uint32_t qa[4];
@@ -172,9 +174,9 @@ hd_mma_out_kernel(HdArgs a, const int* __restrict__ tiles, const float* __restri
 #pragma unroll
     for (int p = 0; p < 3; ++p)
 #pragma unroll
-      for (int n = 0; n < 4; ++n) {
+      for (int n = 0; n < 2; ++n) {
         uint32_t sb[4];
-        ldmatrix_x4_trans(sb, Ss + (p * D16 + d0 + mr + (mj & 1 ? 8 : 0)) * LDV + 16 * n + (mj >= 2 ? 8 : 0));
+        ldmatrix_x4_trans(sb, Ss + (p * D16 + d0 + mr + (mj & 1 ? 8 : 0)) * LDV + c0 + 16 * n + (mj >= 2 ? 8 : 0));
         mma_bf16(acc[2 * n], qa, sb[0], sb[1]);
         mma_bf16(acc[2 * n + 1], qa, sb[2], sb[3]);
       }
@@ -183,11 +185,15 @@ hd_mma_out_kernel(HdArgs a, const int* __restrict__ tiles, const float* __restri
   {
     const float f0 = exp2f((float)bt0), f1 = exp2f((float)bt1);
 #pragma unroll
-    for (int n = 0; n < 8; ++n) {
+    for (int n = 0; n < 4; ++n) {
       acc[n][0] *= f0; acc[n][1] *= f0;
       acc[n][2] *= f1; acc[n][3] *= f1;
     }
   }
+  // Weights of keys in front of the diagonal block: 2^(B_t - B_s) = 2^(B_t - r) 2^(r - B_s) with r the sum up to the last token in front of
+  // this warp's; both exponents are <= 0.  On the diagonal every (query, key) has an exponential of its own.
+  const double ref = r0 > 0 ? b_s[r0 - 1] : 0.0;
+  const float e0 = exp2f((float)(bt0 - ref)), e1 = exp2f((float)(bt1 - ref));
   for (int s0 = 0; s0 <= r0; s0 += 16) {        // keys up to the diagonal
     float sc[2][4] = {};
     const bf16* k_at = Ks + (s0 + mr + (mj >= 2 ? 8 : 0)) * ldk + (mj & 1 ? 8 : 0);
@@ -204,8 +210,15 @@ hd_mma_out_kernel(HdArgs a, const int* __restrict__ tiles, const float* __restri
       const int s = s0 + 8 * n + 2 * (lane & 3);
       const double bs0 = b_s[s], bs1 = b_s[s + 1];
       const float g0 = g_s[s], g1 = g_s[s + 1];
-      const float w0 = s <= t0 ? sc[n][0] * g0 * exp2f((float)(bt0 - bs0)) : 0.f, w1 = s + 1 <= t0 ? sc[n][1] * g1 * exp2f((float)(bt0 - bs1)) : 0.f;
-      const float w2 = s <= t1 ? sc[n][2] * g0 * exp2f((float)(bt1 - bs0)) : 0.f, w3 = s + 1 <= t1 ? sc[n][3] * g1 * exp2f((float)(bt1 - bs1)) : 0.f;
+      float w0, w1, w2, w3;
+      if (s0 < r0) {
+        const float f0 = g0 * exp2f((float)(ref - bs0)), f1 = g1 * exp2f((float)(ref - bs1));
+        w0 = sc[n][0] * (e0 * f0); w1 = sc[n][1] * (e0 * f1);
+        w2 = sc[n][2] * (e1 * f0); w3 = sc[n][3] * (e1 * f1);
+      } else {
+        w0 = s <= t0 ? sc[n][0] * g0 * exp2f((float)(bt0 - bs0)) : 0.f; w1 = s + 1 <= t0 ? sc[n][1] * g1 * exp2f((float)(bt0 - bs1)) : 0.f;
+        w2 = s <= t1 ? sc[n][2] * g0 * exp2f((float)(bt1 - bs0)) : 0.f; w3 = s + 1 <= t1 ? sc[n][3] * g1 * exp2f((float)(bt1 - bs1)) : 0.f;
+      }
       uint32_t lo[3], hi[3];
       split3_pair(w0, w1, lo);
       split3_pair(w2, w3, hi);
@@ -216,9 +229,9 @@ hd_mma_out_kernel(HdArgs a, const int* __restrict__ tiles, const float* __restri
       }
     }
 #pragma unroll
-    for (int n = 0; n < 4; ++n) {
+    for (int n = 0; n < 2; ++n) {
       uint32_t vb[4];
-      ldmatrix_x4_trans(vb, Vs + (s0 + mr + (mj & 1 ? 8 : 0)) * LDV + 16 * n + (mj >= 2 ? 8 : 0));
+      ldmatrix_x4_trans(vb, Vs + (s0 + mr + (mj & 1 ? 8 : 0)) * LDV + c0 + 16 * n + (mj >= 2 ? 8 : 0));
 #pragma unroll
       for (int p = 0; p < 3; ++p) {
         mma_bf16(acc[2 * n], pa[p], vb[0], vb[1]);
@@ -230,8 +243,8 @@ hd_mma_out_kernel(HdArgs a, const int* __restrict__ tiles, const float* __restri
   float* o0 = a.o + (int64_t)(tok0 + t0) * a.H * V + (int64_t)h * V + v0;
   float* o1 = o0 + (int64_t)8 * a.H * V;
 #pragma unroll
-  for (int n = 0; n < 8; ++n) {
-    const int c = 8 * n + 2 * (lane & 3);
+  for (int n = 0; n < 4; ++n) {
+    const int c = c0 + 8 * n + 2 * (lane & 3);
     if (v0 + c >= V) continue;
     if (a.skip) {
       const __nv_bfloat162 x0 = *reinterpret_cast<const __nv_bfloat162*>(Vs + t0 * LDV + c), x1 = *reinterpret_cast<const __nv_bfloat162*>(Vs + t1 * LDV + c);
@@ -260,18 +273,18 @@ bool me_head_decay_mma_takes(const HdArgs& a, int dtype) {
          ((uintptr_t)a.o % 16) == 0 && out_smem(a.D) <= 220 * 1024;
 }
 
-int me_head_decay_mma_states(const HdArgs& a, const int* tiles, int n_tiles, float* states, float* totals, cudaStream_t stream) {
+int me_head_decay_mma_states(const HdArgs& a, const int* tiles, int n_tiles, float* states, HdRun* nums, cudaStream_t stream) {
   const size_t smem = state_smem(a.D);
   cudaError_t e = cudaFuncSetAttribute(hd_mma_state_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
   ME_REQUIRE(e == cudaSuccess, "me_head_decay_scan: cannot raise shared memory to %zu: %s", smem, cudaGetErrorString(e));
-  me_launch(hd_mma_state_kernel, dim3(n_tiles, a.H, (a.V + HD_VT - 1) / HD_VT), dim3(256), smem, stream, a, tiles, states, totals);
+  me_launch(hd_mma_state_kernel, dim3(n_tiles, a.H, (a.V + HD_VT - 1) / HD_VT), dim3(256), smem, stream, a, tiles, states, nums);
   return 0;
 }
 
-int me_head_decay_mma_out(const HdArgs& a, const int* tiles, int n_tiles, const float* states, cudaStream_t stream) {
+int me_head_decay_mma_out(const HdArgs& a, const int* tiles, int n_tiles, const float* states, const HdRun* nums, cudaStream_t stream) {
   const size_t smem = out_smem(a.D);
   cudaError_t e = cudaFuncSetAttribute(hd_mma_out_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
   ME_REQUIRE(e == cudaSuccess, "me_head_decay_scan: cannot raise shared memory to %zu: %s", smem, cudaGetErrorString(e));
-  me_launch(hd_mma_out_kernel, dim3(n_tiles, a.H, (a.V + HD_VT - 1) / HD_VT), dim3(128), smem, stream, a, tiles, states);
+  me_launch(hd_mma_out_kernel, dim3(n_tiles, a.H, (a.V + HD_VT - 1) / HD_VT), dim3(256), smem, stream, a, tiles, states, nums);
   return 0;
 }

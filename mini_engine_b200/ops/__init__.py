@@ -1478,6 +1478,7 @@ def conv_silu(u: torch.Tensor, weight: torch.Tensor, bias: Optional[torch.Tensor
 
 
 HEAD_DECAY_CHUNK = 64     # tokens per run of the recurrence's prompt kernels (csrc/head_decay.cu)
+HEAD_DECAY_RUN = 3 * HEAD_DECAY_CHUNK   # float32 values that hold a run's decays and factors of one head (64 float64 and 64 float32)
 use_head_decay_mma = True # bfloat16 prompts on the tensor cores where the sizes allow (csrc/head_decay_mma.cu); a switch for comparisons
 head_decay_chunks = True  # portions of prompts by runs of tokens (False: token by token, always); a switch for comparisons
 
@@ -1492,14 +1493,14 @@ def head_decay_chunk_count(meta) -> int:
 def head_decay_scan(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, S: torch.Tensor, meta, state_slots: torch.Tensor, o: torch.Tensor,
                     num_heads: int, num_groups: int, dim: int, vdim: int, *, k_scale: float = 1.0, dt: Optional[tuple] = None,
                     decay: Optional[tuple] = None, skip: Optional[torch.Tensor] = None, chunk_states: Optional[torch.Tensor] = None,
-                    totals: Optional[torch.Tensor] = None) -> None:
+                    run_numbers: Optional[torch.Tensor] = None) -> None:
     """Walks every request's tokens of this step through S_t = a_t S_(t-1) + g_t k_t v_t^T, o_t = S_t^T q_t + skip v_t from the state in
     its slot, per head, with one decay a and one factor g a head and token (see csrc/head_decay.cu).  ``q``, ``k`` [T, groups * dim]
     and ``v`` [T, heads * vdim]: columns of rows of one dtype; head h reads group h // (heads / groups) of q and k.
 
     ``dt`` = (pre-activations [T, heads] float32 (columns of wider rows), bias [heads], a_log [heads]): g = softplus(dt + bias), a =
     exp(-exp(a_log) g).  Or ``decay`` = (decays float32 [heads], their log2 float64 [heads]): constants, and g = ``k_scale``.  With the float32 workspaces ``chunk_states``
-    (heads * dim * vdim values a run of HEAD_DECAY_CHUNK tokens: ``head_decay_chunk_count``) and ``totals`` (heads values a run) the
+    (heads * dim * vdim values a run of HEAD_DECAY_CHUNK tokens: ``head_decay_chunk_count``) and ``run_numbers`` (heads * HEAD_DECAY_RUN values a run) the
     requests that bring several tokens take a run at a time, all runs of the step side by side."""
     T = o.shape[0]
     _need(num_heads % num_groups == 0, "head_decay_scan: heads must be a multiple of the groups")
@@ -1514,15 +1515,15 @@ def head_decay_scan(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, S: torch.
           "head_decay_scan: log2 of the decays is float64 [heads]")
     _need(dt is None or (dt[0].dtype == torch.float32 and dt[0].stride(1) == 1 and tuple(dt[0].shape) == (T, num_heads)), "head_decay_scan: dt is float32 [T, heads]")
     tiles, n_tiles = meta.tile_lists[HEAD_DECAY_CHUNK]
-    chunked = head_decay_chunks and chunk_states is not None and totals is not None and n_tiles > 0 and dim <= 256
+    chunked = head_decay_chunks and chunk_states is not None and run_numbers is not None and n_tiles > 0 and dim <= 256
     if chunked:
-        _need(all(t.dtype == torch.float32 and t.is_contiguous() for t in (chunk_states, totals))
-              and chunk_states.numel() >= n_tiles * num_heads * dim * vdim and totals.numel() >= n_tiles * num_heads, "head_decay_scan: workspaces")
+        _need(all(t.dtype == torch.float32 and t.is_contiguous() for t in (chunk_states, run_numbers))
+              and chunk_states.numel() >= n_tiles * num_heads * dim * vdim and run_numbers.numel() >= n_tiles * num_heads * HEAD_DECAY_RUN, "head_decay_scan: workspaces")
     _call("me_head_decay_scan", q.data_ptr(), k.data_ptr(), v.data_ptr(), _dt(q), q.stride(0), k.stride(0), v.stride(0), num_heads, num_groups,
           dim, vdim, float(k_scale), _ptr(dt[0]) if dt else 0, dt[0].stride(0) if dt else 0, _ptr(dt[1]) if dt else 0, _ptr(dt[2]) if dt else 0,
           _ptr(decay[0]) if decay else 0, _ptr(decay[1]) if decay else 0, _ptr(skip), S.data_ptr(), meta.cu_seqlens.data_ptr(), meta.context_lens.data_ptr(), state_slots.data_ptr(),
           o.data_ptr(), meta.num_reqs, meta.num_decodes, tiles.data_ptr() if chunked else 0, n_tiles if chunked else 0,
-          chunk_states.data_ptr() if chunked else 0, totals.data_ptr() if chunked else 0, 1 if use_head_decay_mma else 0, _stream())
+          chunk_states.data_ptr() if chunked else 0, run_numbers.data_ptr() if chunked else 0, 1 if use_head_decay_mma else 0, _stream())
     global launches
     launches += (2 + (1 if meta.num_decodes else 0)) if chunked else 0
 

@@ -23,7 +23,7 @@ def _workspaces(ctx, heads: int, dim: int, vdim: int) -> dict:
     if not runs:
         return {}
     return {"chunk_states": ctx.buffer("head_decay_states", (runs, heads, dim, vdim), torch.float32),
-            "totals": ctx.buffer("head_decay_totals", (runs, heads), torch.float32)}
+            "run_numbers": ctx.buffer("head_decay_run_numbers", (runs, heads, ops.HEAD_DECAY_RUN), torch.float32)}
 
 
 class Retention(Mixer):

@@ -85,7 +85,7 @@ class _Scan:
         kw = dict(k_scale=0.6, decay=(self.decay.to(DEV), torch.log2(self.decay.double()).to(DEV))) if self.constant else \
             dict(dt=(dtw[:, 3:3 + H], self.dt_bias.to(DEV), self.a_log.to(DEV)), skip=self.skip.to(DEV))
         if runs:
-            kw.update(chunk_states=torch.full((runs, H, D, V), float("nan"), device=DEV), totals=torch.full((runs, H), float("nan"), device=DEV))
+            kw.update(chunk_states=torch.full((runs, H, D, V), float("nan"), device=DEV), run_numbers=torch.full((runs, H, ops.HEAD_DECAY_RUN), float("nan"), device=DEV))
         ops.head_decay_scan(q, k, v, self.S, meta, torch.tensor(slots, dtype=torch.int32, device=DEV), o, H, G, D, V, **kw)
         return o.cpu()
 
