@@ -358,7 +358,38 @@ moe_gemm_kernel(const TA* __restrict__ a, int64_t a_stride, const int* __restric
     }
 }
 
-template <typename TS, typename TO>
+// VEC neighbours of a row a thread (four: W and the rows' distances are multiples of four, pointers on 16 bytes, 8 for bfloat16).
+template <int VEC> __device__ __forceinline__ void combine_load(const float* p, float (&v)[VEC]) {
+  if constexpr (VEC == 4) {
+    const float4 t = *reinterpret_cast<const float4*>(p);
+    v[0] = t.x; v[1] = t.y; v[2] = t.z; v[3] = t.w;
+  } else {
+    v[0] = p[0];
+  }
+}
+template <int VEC> __device__ __forceinline__ void combine_load(const bf16* p, float (&v)[VEC]) {
+  if constexpr (VEC == 4) {
+    const uint2 t = *reinterpret_cast<const uint2*>(p);
+    const __nv_bfloat162 a = *reinterpret_cast<const __nv_bfloat162*>(&t.x), b = *reinterpret_cast<const __nv_bfloat162*>(&t.y);
+    v[0] = __low2float(a); v[1] = __high2float(a); v[2] = __low2float(b); v[3] = __high2float(b);
+  } else {
+    v[0] = to_f<bf16>(p[0]);
+  }
+}
+template <int VEC> __device__ __forceinline__ void combine_store(float* p, const float (&v)[VEC]) {
+  if constexpr (VEC == 4) *reinterpret_cast<float4*>(p) = make_float4(v[0], v[1], v[2], v[3]);
+  else p[0] = v[0];
+}
+template <int VEC> __device__ __forceinline__ void combine_store(bf16* p, const float (&v)[VEC]) {
+  if constexpr (VEC == 4) {
+    const __nv_bfloat162 a = __floats2bfloat162_rn(v[0], v[1]), b = __floats2bfloat162_rn(v[2], v[3]);
+    *reinterpret_cast<uint2*>(p) = make_uint2(*reinterpret_cast<const unsigned*>(&a), *reinterpret_cast<const unsigned*>(&b));
+  } else {
+    p[0] = from_f<bf16>(v[0]);
+  }
+}
+
+template <typename TS, typename TO, int VEC>
 __global__ void __launch_bounds__(256)
 moe_combine_kernel(const float* __restrict__ rows, int64_t rows_stride, const int* __restrict__ place, const float* __restrict__ wgt,
                    int top, const TS* __restrict__ shared, int64_t shared_stride, const float* __restrict__ shared_gate, int64_t gate_stride,
@@ -367,12 +398,21 @@ moe_combine_kernel(const float* __restrict__ rows, int64_t rows_stride, const in
   pdl_launch_dependents();
   const int t = blockIdx.x;
   const float share = shared_gate ? 1.f / (1.f + expf(-shared_gate[(int64_t)t * gate_stride])) : 1.f;
-  for (int i = blockIdx.y * blockDim.x + threadIdx.x; i < W; i += gridDim.y * blockDim.x) {
-    float acc = 0.f;
-    for (int k = 0; k < top; ++k)
-      acc = fmaf(wgt[(int64_t)t * top + k], rows[(int64_t)place[(int64_t)t * top + k] * rows_stride + i], acc);
-    if (shared) acc = fmaf(share, to_f<TS>(shared[(int64_t)t * shared_stride + i]), acc);
-    out[(int64_t)t * out_stride + i] = from_f<TO>(acc);
+  for (int i = VEC * (blockIdx.y * blockDim.x + threadIdx.x); i < W; i += VEC * gridDim.y * blockDim.x) {
+    float acc[VEC] = {}, x[VEC];
+#pragma unroll 4
+    for (int k = 0; k < top; ++k) {
+      const float w = wgt[(int64_t)t * top + k];
+      combine_load<VEC>(rows + (int64_t)place[(int64_t)t * top + k] * rows_stride + i, x);
+#pragma unroll
+      for (int j = 0; j < VEC; ++j) acc[j] = fmaf(w, x[j], acc[j]);
+    }
+    if (shared) {
+      combine_load<VEC>(shared + (int64_t)t * shared_stride + i, x);
+#pragma unroll
+      for (int j = 0; j < VEC; ++j) acc[j] = fmaf(share, x[j], acc[j]);
+    }
+    combine_store<VEC>(out + (int64_t)t * out_stride + i, acc);
   }
 }
 
@@ -499,10 +539,18 @@ ME_API int me_moe_combine(const float* rows, int64_t rows_stride, const int* pla
                           int shared_dtype, int64_t shared_stride, const float* shared_gate, int64_t gate_stride, void* out, int out_dtype,
                           int64_t out_stride, int T, int W, cudaStream_t stream) {
   if (T == 0) return 0;
-  dim3 grid(T, (W + 1023) / 1024);
-  ME_DISPATCH_DTYPE(shared ? shared_dtype : ME_F32, TS, ME_DISPATCH_DTYPE(out_dtype, TO,
-      me_launch(moe_combine_kernel<TS, TO>, grid, dim3(256), 0, stream, rows, rows_stride, place, wgt, top, (const TS*)shared,
-                shared_stride, shared_gate, gate_stride, (TO*)out, out_stride, W)));
+  auto off = [](const void* p, size_t to) { return p && ((uintptr_t)p % to) != 0; };
+  const bool vec = W % 4 == 0 && rows_stride % 4 == 0 && shared_stride % 4 == 0 && out_stride % 4 == 0 && !off(rows, 16) &&
+                   !off(shared, shared_dtype == ME_F32 ? 16 : 8) && !off(out, out_dtype == ME_F32 ? 16 : 8);
+  // four columns a thread: a row of up to 1,024 in one block
+  const dim3 grid(T, (W + 1023) / 1024);
+  const int threads = vec && W <= 512 ? 128 : 256;
+#define MC_CASE(VEC_)                                                                                                                me_launch(moe_combine_kernel<TS, TO, VEC_>, grid, dim3(threads), 0, stream, rows, rows_stride, place, wgt, top, (const TS*)shared,             shared_stride, shared_gate, gate_stride, (TO*)out, out_stride, W)
+  ME_DISPATCH_DTYPE(shared ? shared_dtype : ME_F32, TS, ME_DISPATCH_DTYPE(out_dtype, TO, {
+    if (vec) MC_CASE(4);
+    else MC_CASE(1);
+  }));
+#undef MC_CASE
   ME_LAUNCH_CHECK("me_moe_combine");
   return 0;
 }

@@ -108,10 +108,11 @@ def attention_branch(h, w, p, m, eps):
     k = (h @ w[p + "k"].T + w[p + "k.b"]).view(T, G, D)
     v = (h @ w[p + "v"].T + w[p + "v.b"]).view(T, G, Dv)
     q, k = over_rms(q, eps) * w[p + "q.norm"], over_rms(k, eps) * w[p + "k.norm"]
-    freqs, magnitude = yarn_frequencies(m["rot"]["dims"], m["rot"]["base"], m["rot"].get("scaling"))
-    at = torch.arange(T)
-    q, k = rotate_halves(q, at, freqs, magnitude), rotate_halves(k, at, freqs, magnitude)
-    o = window_attention(q, k, v, m["scale"], m["mask"]["size"])
+    if m.get("rot"):
+        freqs, magnitude = yarn_frequencies(m["rot"]["dims"], m["rot"]["base"], m["rot"].get("scaling"))
+        at = torch.arange(T)
+        q, k = rotate_halves(q, at, freqs, magnitude), rotate_halves(k, at, freqs, magnitude)
+    o = window_attention(q, k, v, m["scale"], m["mask"]["size"] if m.get("mask") else T)
     o = o * torch.sigmoid(h @ w[p + "g"].T)[:, :, None]
     return o.reshape(T, H * Dv) @ w[p + "o"].T
 
