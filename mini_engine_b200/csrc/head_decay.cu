@@ -41,10 +41,10 @@ template <> struct HdVec<1> {
 template <typename T, int R, int VEC>
 __global__ void __launch_bounds__(256) hd_step_kernel(HdArgs a) {
   extern __shared__ __align__(16) float smem[];
-  const int D = a.D, V = a.V;
-  float* q_s = smem;                            // [D]
-  float* k_s = q_s + D;                         // [D]
-  float* parts = k_s + D;                       // [8][16 VEC]
+  const int D = a.D, V = a.V, D4 = (D + 3) / 4 * 4;      // (what follows starts on 16 bytes)
+  float* q_s = smem;                            // [D4]
+  float* k_s = q_s + D4;                        // [D4]
+  float* parts = k_s + D4;                      // [8][16 VEC]
   const int b = blockIdx.x, h = blockIdx.y, tid = threadIdx.x, c = tid & 15, dy = tid >> 4, warp = tid >> 5, lane = tid & 31;
   const int v0 = (blockIdx.z * 16 + c) * VEC;
   const bool v_ok = v0 < V;                     // (V is a multiple of VEC)

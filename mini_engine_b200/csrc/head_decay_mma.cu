@@ -15,6 +15,7 @@ namespace {
 
 using namespace mma_prims;
 
+constexpr int HM_SR = 64;                     // rows of the state that hd_mma_out_kernel holds in shared memory at a time
 constexpr int HM_LDV = HD_VT + 8;             // bfloat16 elements of a row of 64 columns in shared memory (an odd number of 16-byte pieces)
 
 // Two floats as a pair of bfloat16 (x in the lower half) in each of the three parts.
@@ -121,7 +122,7 @@ hd_mma_state_kernel(HdArgs a, const int* __restrict__ tiles, float* __restrict__
 }
 
 // One block = one run x one head x HD_VT columns; states[c] holds the state in front of the run.
-__global__ void __launch_bounds__(256)
+__global__ void __launch_bounds__(256, 3)
 hd_mma_out_kernel(HdArgs a, const int* __restrict__ tiles, const float* __restrict__ states, const HdRun* __restrict__ nums) {
   extern __shared__ __align__(16) unsigned char hm_smem[];
   __shared__ float g_s[HD_LC];
@@ -131,7 +132,7 @@ hd_mma_out_kernel(HdArgs a, const int* __restrict__ tiles, const float* __restri
   bf16* Qs = reinterpret_cast<bf16*>(hm_smem);  // [LC][ldk]
   bf16* Ks = Qs + LC * ldk;                     // [LC][ldk]
   bf16* Vs = Ks + LC * ldk;                     // [LC][LDV]
-  bf16* Ss = Vs + LC * LDV;                     // [3][D16][LDV]: the state in three parts
+  bf16* Ss = Vs + LC * LDV;                     // [3][HM_SR][LDV]: rows of the state in three parts
   const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, h = blockIdx.y, v0 = blockIdx.z * VT;
   const int b = tiles[2 * blockIdx.x], q0 = tiles[2 * blockIdx.x + 1];
   const int tok0 = a.cu[b] + q0, L = min(LC, a.cu[b + 1] - tok0);
@@ -143,44 +144,69 @@ hd_mma_out_kernel(HdArgs a, const int* __restrict__ tiles, const float* __restri
   hm_fill(Ks, ldk, D16, reinterpret_cast<const bf16*>(a.k) + (int64_t)tok0 * a.ldk + (int64_t)g * D, a.ldk, L, D);
   hm_fill(Vs, LDV, VT, reinterpret_cast<const bf16*>(a.v) + (int64_t)tok0 * a.ldv + (int64_t)h * V + v0, a.ldv, L, V - v0);
   cp_async_commit();
-  {
-    const float* src = states + ((int64_t)blockIdx.x * a.H + h) * D * V + v0;
-#pragma unroll 8
-    for (int i = tid; i < D16 * (VT / 4); i += 256) {
-      const int d = i / (VT / 4), c = i % (VT / 4) * 4;
-      const float4 x = d < D && v0 + c < V ? *reinterpret_cast<const float4*>(src + (int64_t)d * V + c) : make_float4(0.f, 0.f, 0.f, 0.f);
-      uint32_t p0[3], p1[3];
-      split3_pair(x.x, x.y, p0);
-      split3_pair(x.z, x.w, p1);
+  // HM_SR rows of the state at a time: into registers (on their way while the products of the rows before run), then split into shared memory
+  const int sr = tid / 16, scol = tid % 16 * 4;
+  const float* ssrc = states + ((int64_t)blockIdx.x * a.H + h) * D * V + v0 + scol;
+  float4 sx[HM_SR / 16];
+  auto fetch_rows = [&](int d0) {
 #pragma unroll
-      for (int k = 0; k < 3; ++k) *reinterpret_cast<uint2*>(Ss + (k * D16 + d) * LDV + c) = make_uint2(p0[k], p1[k]);
+    for (int i = 0; i < HM_SR / 16; ++i) {
+      const int d = d0 + sr + 16 * i;
+      sx[i] = d < D && v0 + scol < V ? *reinterpret_cast<const float4*>(ssrc + (int64_t)d * V) : make_float4(0.f, 0.f, 0.f, 0.f);
     }
-  }
+  };
+  auto store_rows = [&]() {
+#pragma unroll
+    for (int i = 0; i < HM_SR / 16; ++i) {
+      uint32_t p0[3], p1[3];
+      split3_pair(sx[i].x, sx[i].y, p0);
+      split3_pair(sx[i].z, sx[i].w, p1);
+#pragma unroll
+      for (int k = 0; k < 3; ++k) *reinterpret_cast<uint2*>(Ss + (k * HM_SR + sr + 16 * i) * LDV + scol) = make_uint2(p0[k], p1[k]);
+    }
+  };
+  fetch_rows(0);
   if (tid < LC) {
     const HdRun& run = nums[(int64_t)blockIdx.x * a.H + h];
     b_s[tid] = run.b[tid];
     g_s[tid] = run.g[tid];
   }
+  store_rows();
   cp_async_wait<0>();
   __syncthreads();
   const int r0 = 16 * (warp >> 1), c0 = 32 * (warp & 1);
-  if (r0 >= L || v0 + c0 >= V) return;
+  const bool active = r0 < L && v0 + c0 < V;
   const int mr = lane & 7, mj = lane >> 3, t0 = r0 + (lane >> 2), t1 = t0 + 8;
   float acc[4][4] = {};
   const bf16* q_at = Qs + (r0 + mr + (mj & 1 ? 8 : 0)) * ldk + (mj >= 2 ? 8 : 0);
-  for (int d0 = 0; d0 < D16; d0 += 16) {
-    uint32_t qa[4];
-    ldmatrix_x4(qa, q_at + d0);
+  const bf16* s_at = Ss + (mr + (mj & 1 ? 8 : 0)) * LDV + c0 + (mj >= 2 ? 8 : 0);
+  for (int s0 = 0; s0 < D16; s0 += HM_SR) {
+    const bool more = s0 + HM_SR < D16;
+    if (more) fetch_rows(s0 + HM_SR);
+    if (active) {
 #pragma unroll
-    for (int p = 0; p < 3; ++p)
+      for (int j = 0; j < HM_SR / 16; ++j) {
+        if (s0 + 16 * j >= D16) break;
+        uint32_t qa[4];
+        ldmatrix_x4(qa, q_at + s0 + 16 * j);
 #pragma unroll
-      for (int n = 0; n < 2; ++n) {
-        uint32_t sb[4];
-        ldmatrix_x4_trans(sb, Ss + (p * D16 + d0 + mr + (mj & 1 ? 8 : 0)) * LDV + c0 + 16 * n + (mj >= 2 ? 8 : 0));
-        mma_bf16(acc[2 * n], qa, sb[0], sb[1]);
-        mma_bf16(acc[2 * n + 1], qa, sb[2], sb[3]);
+        for (int p = 0; p < 3; ++p)
+#pragma unroll
+          for (int n = 0; n < 2; ++n) {
+            uint32_t sb[4];
+            ldmatrix_x4_trans(sb, s_at + (p * HM_SR + 16 * j) * LDV + 16 * n);
+            mma_bf16(acc[2 * n], qa, sb[0], sb[1]);
+            mma_bf16(acc[2 * n + 1], qa, sb[2], sb[3]);
+          }
       }
+    }
+    if (more) {                                 // (the same in all threads)
+      __syncthreads();
+      store_rows();
+      __syncthreads();
+    }
   }
+  if (!active) return;
   const double bt0 = b_s[t0], bt1 = b_s[t1];
   {
     const float f0 = exp2f((float)bt0), f1 = exp2f((float)bt1);
@@ -261,7 +287,7 @@ hd_mma_out_kernel(HdArgs a, const int* __restrict__ tiles, const float* __restri
 size_t state_smem(int D) { return sizeof(bf16) * ((size_t)HD_LC * ((D + 15) / 16 * 16 + 8) + 3 * HD_LC * HM_LDV); }
 size_t out_smem(int D) {
   const size_t D16 = (D + 15) / 16 * 16;
-  return sizeof(bf16) * (2 * HD_LC * (D16 + 8) + HD_LC * HM_LDV + 3 * D16 * HM_LDV);
+  return sizeof(bf16) * (2 * HD_LC * (D16 + 8) + HD_LC * HM_LDV + 3 * HM_SR * HM_LDV);
 }
 
 }  // namespace

@@ -104,7 +104,7 @@ def _close(got, ref, rel=3e-6):
     assert err <= rel * max(top, 1e-3), (err, top)
 
 
-SCANS = [(2, 2, 16, 32), (2, 1, 8, 8), (4, 2, 72, 136), (3, 1, 24, 40), (4, 2, 64, 64), (2, 1, 7, 5), (2, 2, 64, 128), (6, 3, 128, 64), (1, 1, 130, 70), (2, 2, 256, 24), (1, 1, 300, 12)]
+SCANS = [(2, 2, 16, 32), (4, 4, 45, 68), (2, 1, 13, 20), (2, 1, 8, 8), (4, 2, 72, 136), (3, 1, 24, 40), (4, 2, 64, 64), (2, 1, 7, 5), (2, 2, 64, 128), (6, 3, 128, 64), (1, 1, 130, 70), (2, 2, 256, 24), (1, 1, 300, 12)]
 
 
 @both
