@@ -206,7 +206,7 @@ constexpr int HD_WALK = 128;
 
 template <int VEC>
 __global__ void __launch_bounds__(HD_WALK, 8)
-hd_state_walk_kernel(HdArgs a, const HdRun* __restrict__ nums, float* __restrict__ states, const int* __restrict__ tiles, int n_tiles, int first_req) {
+hd_state_walk_kernel(HdArgs a, const HdRun* __restrict__ nums, float* states, const int* __restrict__ tiles, int n_tiles, int first_req) {
   __shared__ int first_tile;
   const int b = first_req + blockIdx.x, h = blockIdx.y, DV = a.D * a.V;
   const int e = (blockIdx.z * HD_WALK + threadIdx.x) * VEC;
@@ -227,22 +227,33 @@ hd_state_walk_kernel(HdArgs a, const HdRun* __restrict__ nums, float* __restrict
   const int64_t step = (int64_t)a.H * DV;
   float* st = states + ((int64_t)c0 * a.H + h) * DV + e;
   const HdRun* run = nums + (int64_t)c0 * a.H + h;
-  constexpr int AHEAD = 8;                      // runs whose loads are in flight together
-  for (int c1 = 0; c1 < n_chunks; c1 += AHEAD) {
-    float u[AHEAD][VEC], dec[AHEAD];
+  // The loads of the next AHEAD runs are on their way while these runs' states are stored (one group of loads at a time, then its stores,
+  // took nearly twice as long: 53 against 29 us for 32 runs of 64 heads of 128 x 64).
+  constexpr int AHEAD = 4;
+  float u[2][AHEAD][VEC], dec[2][AHEAD];
+  auto fetch = [&](int into, int c1) {
 #pragma unroll
     for (int j = 0; j < AHEAD; ++j) {
       const int c = min(c1 + j, n_chunks - 1);
-      HdVec<VEC>::load(st + c * step, u[j]);
-      dec[j] = (float)run[(int64_t)c * a.H].b[HD_LC - 1];
+      HdVec<VEC>::load(st + c * step, u[into][j]);
+      dec[into][j] = (float)run[(int64_t)c * a.H].b[HD_LC - 1];
     }
+  };
+  fetch(0, 0);
+  for (int pair = 0; pair < n_chunks; pair += 2 * AHEAD) {
 #pragma unroll
-    for (int j = 0; j < AHEAD; ++j) {
-      if (c1 + j < n_chunks) {
-        HdVec<VEC>::store(st + (c1 + j) * step, S);
-        const float f = exp2f(dec[j]);
+    for (int half = 0; half < 2; ++half) {
+      const int c1 = pair + half * AHEAD;
+      if (c1 >= n_chunks) break;
+      if (c1 + AHEAD < n_chunks) fetch(half ^ 1, c1 + AHEAD);
 #pragma unroll
-        for (int k = 0; k < VEC; ++k) S[k] = fmaf(f, S[k], u[j][k]);
+      for (int j = 0; j < AHEAD; ++j) {
+        if (c1 + j < n_chunks) {
+          HdVec<VEC>::store(st + (c1 + j) * step, S);
+          const float f = exp2f(dec[half][j]);
+#pragma unroll
+          for (int k = 0; k < VEC; ++k) S[k] = fmaf(f, S[k], u[half][j][k]);
+        }
       }
     }
   }
