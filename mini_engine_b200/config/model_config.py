@@ -770,8 +770,7 @@ class KuteraxConfig(ModelConfig):
     """Kuterax: a decoder whose layers run mixer and feed-forward side by side behind ONE norm, each scaled element by element before it
     joins the stream, with learned position vectors on the embedding; mixers are windowed attention beside a Mamba-2 recurrence, each
     behind an output norm of its own, or retention; feed-forwards are routed squared-relu experts with a gated shared one.  A range
-    of layers may run several times in a row with the same weights, each pass starting from a product of the stream and the embedding
-    output.  config.json keys: ``vocab``, ``width``, ``max_positions``, ``norm.eps``, ``loop`` {start, stop, times} (absent: every layer once) and
+    of layers may be looped over, each pass starting from a product of the stream and the embedding output.  config.json keys: ``vocab``, ``width``, ``max_positions``, ``norm.eps``, ``loop`` {start, stop, times} (absent: every layer once) and
     ``layers``: a list of ``{"type", "mixer", "mlp"}`` with
 
     * type ``parallel``: mixer {left {heads, kv_heads, dim, vdim, scale, rot {base, dims, scaling {factor, original, fast, slow}}, mask {size}},

@@ -5,7 +5,7 @@ outputs.  The mixer is retention (``retention``) or two mixers side by side (``s
 averaged: windowed grouped-query attention with biased projections, a weighted norm of q and k in front of a YaRN rotation, a one in the
 softmax's denominator and a gate a head (``masked_sink_attention``), and Mamba-2 (``mamba2``).  The feed-forward is routed squared-relu experts
 chosen by a softmax over all of them within the best groups, with a gated shared expert (``routed_experts``), or absent.  A range of layers may
-run several times in a row with the same weights: every pass has cache and state slots of its own, and in front of it the stream becomes a
+be looped over: every pass has cache and state slots of its own, and in front of it the stream becomes a
 product of itself and the embedding output, plus the pass's vector.  The embedding has a learned vector for every position.  Layer i's
 tensors are ``l<i>.*``; all numbers come from the configuration.
 """

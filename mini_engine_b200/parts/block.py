@@ -276,9 +276,9 @@ class ParallelBlock(Block):
     (``add_row``) that joins the stream right before the block's norms.  The norms must be of a kind that takes a
     ``PendingSum`` (kinds ``layernorm`` and ``rmsnorm``).
 
-    ``BlockSpec.args``: ``one_norm``: there is one norm and both sub-layers read its output; ``scales`` = {"mixer": name,
-    "feed_forward": name, "width": size}: each sub-layer's output is multiplied element by element by the vector of that name before
-    it joins the stream (the norm's kind must take ``PendingTerm``s: ``rmsnorm``)."""
+    ``BlockSpec.args``: ``one_norm``: the mixer's norm serves the feed-forward too; ``scales`` = {"mixer": name,
+    "feed_forward": name, "width": size}: a vector of that name scales each sub-layer's output, value by value, as it joins the
+    stream (the norm's kind must take ``PendingTerm``s: ``rmsnorm``)."""
     capturable = True
     feed_forward_optional = True
     takes_pass_vector = True

@@ -16,7 +16,7 @@ best groups can be chosen; the weights are the chosen experts' s, not renormalis
 ``ops.ACTIVATIONS``, instead of the gate): an expert is W_down act(W_up h) and has no gate matrix (a ``shared`` expert with an
 ``activation`` of its own likewise).  ``routing`` "softmax_groups": as "sigmoid_groups" with s the softmax over all experts' logits and a
 group's score its largest choice score.  ``weight_scale`` multiplies the weights of either grouped rule.  ``shared_gate`` (a tensor's
-name): the shared expert's output is multiplied by sigmoid(W_sg h), one number a token, whose row is packed with the router's.
+name): the shared expert is weighed by the sigmoid of one number a token, whose row of weights is packed with the router's.
 """
 from __future__ import annotations
 

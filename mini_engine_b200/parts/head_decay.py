@@ -27,8 +27,8 @@ def _workspaces(ctx, heads: int, dim: int, vdim: int) -> dict:
 
 
 class Retention(Mixer):
-    """q = W_q x, k = W_k x * dim^-1/2, v = W_v x, no biases; a_t = ``decay`` of the head, a constant, and g = 1.  Every head's o is divided by
-    its root mean square (no weight), the joined heads are multiplied by silu(W_g x) and projected by W_o."""
+    """q = W_q x, k = W_k x * dim^-1/2, v = W_v x; a_t is the head's entry of ``decay``, the same for every token, and g_t = 1.  An RMS norm
+    without a weight brings each head's o to unit size, silu(W_g x) gates the joined heads, and W_o takes them back to the stream's width."""
     capturable = True
 
     def __init__(self, hidden_size: int, num_heads: int, dim: int, vdim: int, decay: Sequence[float], norm_eps: float):
@@ -71,10 +71,11 @@ class Retention(Mixer):
 
 
 class Mamba2(Mixer):
-    """W_in x is laid out as [z | x | B | C | dt] with ``heads * vdim``, as many, ``groups * state`` twice and ``heads`` rows; x, B and C pass a causal
-    convolution per channel (``taps``, with a bias) and silu together.  Per head, with its group's B and C: g_t = softplus(dt + dt_bias), a_t =
-    exp(-exp(A_log) g_t), k = B, q = C, v = x, and D x joins o.  The joined heads times silu(z) are normed in ``norm_groups`` equal parts,
-    multiplied by a weight and projected by W_o.  The convolution's last taps - 1 inputs are part of the state.
+    """One projection makes, in this order, a gate z and values x (``heads * vdim`` columns each), keys B and queries C (``groups * state`` each) and
+    a step size dt a head.  x, B and C go through one short causal convolution (``taps`` weights and a bias for every channel) and silu.
+    Per head, with its group's B and C: g_t = softplus(dt + dt_bias), a_t = exp(-exp(A_log) g_t), k = B, q = C, v = x, and D x joins o.
+    silu(z) gates the joined heads in front of an RMS norm over ``norm_groups`` equal parts of the row; then a weight and W_o.  A request's
+    slot holds S and the ``taps - 1`` inputs that the convolution still needs.
 
     Its heads can run inside a mixer that owns the projections (``heads_of``, see ``SideBySide``): ``hosted`` leaves both out."""
     capturable = True

@@ -11,8 +11,8 @@ score = q . k * scale, then, with ``softcap`` c, c tanh(score / c), or, with ``d
 learned numbers a head (``r1``, ``r2``).  ``mask``: None (every key j <= p),
 ("window", size, keep_first): keys with p - j < size or j < keep_first, or ("chunk", size): keys of the query's own
 chunk, floor(j / size) = floor(p / size).  The weights are exp(s_j) / (exp(sink_h) + sum exp(s_j)) with a learned number
-per head when ``sink`` is set: a term without key or value that is neither scaled nor capped (``sink`` "one": the term is 1, a
-sink whose score is 0).  ``head_gate``: head h's output is multiplied by sigmoid(W_g x)_h, one number a head.  ``out_scale`` multiplies the
+per head when ``sink`` is set: a term without key or value that is neither scaled nor capped (``sink`` "one": the term is 1,
+nothing learned).  ``head_gate``: the mixer's input also makes a gate a head, whose sigmoid scales that head's result.  ``out_scale`` multiplies the
 mixer's output (the values carry it, and the output bias).  Keys have ``dim`` elements
 and values ``vdim``; the cache is the engine's usual one (pages of keys and of values) with rows of max(dim, vdim)
 elements, or with ``pad_rows`` of the next size the tensor-core kernels take (zeros behind keys and values), and it keeps

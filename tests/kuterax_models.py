@@ -67,7 +67,7 @@ B = config(75, 52, [
 #    kernel of the experts' products
 C = config(130, 128, [
     par((8, 2, 64, 64), (4, 64, 64, 2, 4, 2), 100, 64, base=1e6, mlp=moe(8, 4, 64, groups=(2, 1), scale=1.5, shared=128)),
-    ret(2, 64, 128, (0.96875, 0.998), mlp=moe(4, 2, 128, groups=(2, 2), scale=1.0, shared=64)),
+    ret(2, 64, 128, (0.95, 0.998), mlp=moe(4, 2, 128, groups=(2, 2), scale=1.0, shared=64)),
     par((4, 1, 128, 128), (2, 128, 128, 1, 4, 1), 129, 32, base=1e4, scaling=(4.0, 512, 32.0, 1.0), mlp=None),
 ], max_positions=700)
 # D: rows that tensor-core kernels take only when filled up, heads too wide for them in the third layer, a window of one token and
